@@ -28,4 +28,6 @@ else:
     # The package stays importable so that `python -m onnxruntime_b200.build` can run; everything else
     # fails loudly until the native runtime exists.
     def __getattr__(name):
+        if name == "build":   # `from onnxruntime_b200 import build`: let the import system find the submodule
+            raise AttributeError(name)
         raise ImportError("onnxruntime_b200._core is not built: run `python -m onnxruntime_b200.build`")

@@ -15,6 +15,7 @@ C++ runtime).  nvcc cross-compiles without a GPU.
 from __future__ import annotations
 
 import argparse
+import fcntl
 import glob
 import os
 import subprocess
@@ -33,6 +34,11 @@ NVCC_FLAGS = [
 ]
 
 
+# Kernels whose arithmetic is specified in 32-bit (recurrences, norms, softmax of fp32 models) keep the accurate divisions,
+# square roots and transcendentals.
+ACCURATE_MATH = {"recurrent.cu", "hybrid.cu"}
+
+
 def _cuda_home() -> str:
     for cand in (os.environ.get("CUDA_HOME"), "/usr/local/cuda"):
         if cand and os.path.exists(os.path.join(cand, "bin", "nvcc")):
@@ -44,7 +50,7 @@ def core_ext_name() -> str:
     return "_core" + (sysconfig.get_config_var("EXT_SUFFIX") or ".so")
 
 
-def write_ninja(kernels_only: bool = False) -> str:
+def write_ninja(kernels_only: bool = False, c_api: bool = True) -> str:
     os.makedirs(BUILD, exist_ok=True)
     os.makedirs(LIBDIR, exist_ok=True)
     cuda = _cuda_home()
@@ -55,8 +61,12 @@ def write_ninja(kernels_only: bool = False) -> str:
         f"nvcc = {cuda}/bin/nvcc",
         "cxx = g++",
         "nvflags = " + " ".join(NVCC_FLAGS) + f" -I{CSRC}/cuda",
+        "nvflags_accurate = " + " ".join(f for f in NVCC_FLAGS if f != "--use_fast_math") + f" -I{CSRC}/cuda",
         "rule nvcc",
         "  command = $nvcc $nvflags -c $in -o $out",
+        "  description = NVCC $in",
+        "rule nvcc_accurate",
+        "  command = $nvcc $nvflags_accurate -c $in -o $out",
         "  description = NVCC $in",
         "rule nvlink",
         f"  command = $nvcc -shared -o $out $in -L{cuda}/lib64 -lcudart",
@@ -66,7 +76,8 @@ def write_ninja(kernels_only: bool = False) -> str:
     for src in cu_srcs:
         obj = os.path.join(BUILD, os.path.basename(src)[:-3] + ".o")
         objs.append(obj)
-        lines.append(f"build {obj}: nvcc {src} | " + " ".join(cu_hdrs))
+        rule = "nvcc_accurate" if os.path.basename(src) in ACCURATE_MATH else "nvcc"
+        lines.append(f"build {obj}: {rule} {src} | " + " ".join(cu_hdrs))
     kern_so = os.path.join(LIBDIR, "libortb200_kernels.so")
     lines.append(f"build {kern_so}: nvlink " + " ".join(objs))
     defaults = [kern_so]
@@ -103,6 +114,7 @@ def write_ninja(kernels_only: bool = False) -> str:
         core_so = os.path.join(HERE, core_ext_name())
         lines.append(f"build {core_so}: cxxlink " + " ".join(cobjs) + f" | {kern_so}")
         defaults.append(core_so)
+    if cpp_srcs and not kernels_only and c_api:
         # the same runtime without the Python bindings, behind the C API (ortb200_c_api.h)
         lines += [
             "rule cxxlink_c",
@@ -123,15 +135,29 @@ def write_ninja(kernels_only: bool = False) -> str:
     return path
 
 
-def build(kernels_only: bool = False, verbose: bool = False) -> None:
-    path = write_ninja(kernels_only)
+def build(kernels_only: bool = False, verbose: bool = False, c_api: bool = True, log=None) -> None:
+    path = write_ninja(kernels_only, c_api)
     cmd = ["ninja", "-f", path] + (["-v"] if verbose else [])
     jobs = os.environ.get("ORTB200_BUILD_JOBS")
     if jobs:
         cmd += ["-j", jobs]
-    res = subprocess.run(cmd, cwd=BUILD)
+    res = subprocess.run(cmd, cwd=BUILD, stdout=log)
     if res.returncode != 0:
         raise RuntimeError("native build failed")
+
+
+def ensure_built() -> bool:
+    """Compile what the Python package needs (kernel library and runtime, not the C API library) when it is missing; True
+    when something was compiled (a process that imported the package before has to start anew).  Callers that start at the same time wait for the first one; the compiler's output goes to standard error."""
+    wanted = [os.path.join(HERE, core_ext_name()), os.path.join(LIBDIR, "libortb200_kernels.so")]
+    if all(os.path.exists(w) for w in wanted):
+        return False
+    os.makedirs(BUILD, exist_ok=True)
+    with open(os.path.join(BUILD, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not all(os.path.exists(w) for w in wanted):
+            build(c_api=False, log=sys.stderr)
+    return True
 
 
 if __name__ == "__main__":

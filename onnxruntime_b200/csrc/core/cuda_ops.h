@@ -32,5 +32,6 @@ at::Tensor GemmAllReduce(OpKernelContext& ctx, const at::Tensor& partial, const 
 
 void RegisterMoreCudaKernels(KernelRegistry& r);
 void RegisterCudaKernels3(KernelRegistry& r);
+void RegisterCudaKernels4(KernelRegistry& r);
 
 }  // namespace ortb

@@ -197,6 +197,7 @@ void RegisterStringKernels(KernelRegistry& r);
 bool CastWithStrings(OpKernelContext& ctx, int32_t to);
 void RegisterControlFlowKernels(KernelRegistry& r);
 void RegisterCollectiveKernels(KernelRegistry& r);
+void RegisterHybridKernels(KernelRegistry& r);
 void RegisterCudaKernels(KernelRegistry& r);
 void EnsureKernelsRegistered();
 

@@ -98,6 +98,7 @@ void EnsureKernelsRegistered() {
     RegisterStringKernels(g);
     RegisterControlFlowKernels(g);
     RegisterCollectiveKernels(g);
+    RegisterHybridKernels(g);
     // com.microsoft operators that are early forms of ONNX operators with the same semantics (contrib_ops/cpu_contrib_kernels.cc)
     for (const char* op : {"GatherND", "GridSample", "Pad", "QLinearConv", "Range"}) g.RegisterAlias("", op, "com.microsoft");
     RegisterCudaKernels(KernelRegistry::Cuda());

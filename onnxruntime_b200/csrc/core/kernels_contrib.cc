@@ -838,7 +838,9 @@ void RegisterContribKernels(KernelRegistry& r) {
   });
   r.RegisterFn("com.ortb200", "GemmSwiGLU", 1, kMax, [normed_input](Ctx& ctx) {
     at::Tensor x = normed_input(ctx, 3);
-    ctx.SetOutput(0, at::silu(at::matmul(x, ctx.RequiredInput(1))) * at::matmul(x, ctx.RequiredInput(2)));
+    at::Tensor gate = at::matmul(x, ctx.RequiredInput(1));
+    gate = ctx.node().attr_s("activation", "swiglu") == "geglu" ? at::gelu(gate, "tanh") : at::silu(gate);
+    ctx.SetOutput(0, gate * at::matmul(x, ctx.RequiredInput(2)));
   });
 }
 

@@ -41,6 +41,7 @@ int ActCode(const std::string& a) {
   if (a == "silu") return ORTB200_ACT_SILU;
   if (a == "quickgelu") return ORTB200_ACT_QUICKGELU;
   if (a == "swiglu") return ORTB200_ACT_SWIGLU;
+  if (a == "geglu") return ORTB200_ACT_GEGLU;
   ORTB_THROW(INVALID_ARGUMENT, "unknown activation ", a);
 }
 
@@ -424,6 +425,7 @@ class GemmSwiGLUKernel final : public OpKernel {
     const at::Tensor* wu = info.constant_input(2);
     ORTB_ENFORCE(wg && wu, "GemmSwiGLU needs constant weights");
     I_ = wg->size(1);
+    gelu_ = info.node.attr_s("activation", "swiglu") == "geglu";
     w_ = at::cat({wg->t(), wu->t()}, 0).contiguous();  // [2I, K]: gate rows then up rows
     rms_eps_ = info.node.attr_f("rms_eps", 0.f);
     if (rms_eps_ > 0.f) {
@@ -442,13 +444,15 @@ class GemmSwiGLUKernel final : public OpKernel {
       // saves; one plain GEMM over the stacked gate | up rows at 256-token tiles plus a streaming SwiGLU is faster.
       at::Tensor gu = LaunchNormedGemm(ctx, x2, w_, 2 * I_, 0, at::Tensor(), at::Tensor(), ORTB200_ACT_NONE, 1.f, rms_eps_, unit_gamma_);
       at::Tensor y = at::empty({x2.size(0), I_}, x2.options());
-      CheckLaunch(ortb200_swiglu(gu.data_ptr(), y.data_ptr(), x2.size(0), static_cast<int>(I_), DtypeCode(x2.scalar_type()), ctx.cuda_stream()),
+      CheckLaunch((gelu_ ? ortb200_geglu : ortb200_swiglu)(gu.data_ptr(), y.data_ptr(), x2.size(0), static_cast<int>(I_), DtypeCode(x2.scalar_type()),
+                                                           ctx.cuda_stream()),
                   "ortb200_swiglu");
       ctx.session()->AddLaunches(1);
       ctx.SetOutput(0, y.reshape(OutShape(x, I_)));
       return;
     }
-    at::Tensor y = LaunchNormedGemm(ctx, x2, w_, I_, I_, at::Tensor(), at::Tensor(), ORTB200_ACT_SWIGLU, 1.f, rms_eps_, unit_gamma_);
+    at::Tensor y = LaunchNormedGemm(ctx, x2, w_, I_, I_, at::Tensor(), at::Tensor(), gelu_ ? ORTB200_ACT_GEGLU : ORTB200_ACT_SWIGLU, 1.f,
+                                    rms_eps_, unit_gamma_);
     ctx.SetOutput(0, y.reshape(OutShape(x, I_)));
   }
 
@@ -456,6 +460,7 @@ class GemmSwiGLUKernel final : public OpKernel {
   at::Tensor w_, unit_gamma_;
   float rms_eps_ = 0.f;
   int64_t I_ = 0;
+  bool gelu_ = false;
 };
 
 // com.ortb200.SwiGLU: [..., 2 I] -> silu(x[..., :I]) * x[..., I:], one streaming kernel (behind the stacked gate | up
@@ -504,6 +509,7 @@ void RegisterCudaKernels(KernelRegistry& r) {
   RegisterClass<SwiGLUKernel>(r, kFusedDomain, "SwiGLU");
   RegisterMoreCudaKernels(r);
   RegisterCudaKernels3(r);
+  RegisterCudaKernels4(r);
 }
 
 }  // namespace ortb

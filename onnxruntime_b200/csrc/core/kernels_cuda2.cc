@@ -139,6 +139,7 @@ class EmbeddingGatherKernel final : public WithFallback {
 
 class ArgMaxKernel final : public WithFallback {
   mutable at::Tensor ws_;  // per-row merge slots + counters, kept zero between launches
+  mutable std::vector<at::Tensor> retired_;  // smaller scratch that captured graphs still point to
 
  public:
   explicit ArgMaxKernel(const OpKernelInfo& info) : WithFallback(info) {}
@@ -157,8 +158,10 @@ class ArgMaxKernel final : public WithFallback {
     else shape.pop_back();
     at::Tensor out = at::empty(shape, x.options().dtype(at::kLong));
     const int64_t rows = xc.numel() / x.size(-1);
-    if (!ws_.defined() || ws_.numel() < rows * 16 || ws_.device() != x.device())
+    if (!ws_.defined() || ws_.numel() < rows * 16 || ws_.device() != x.device()) {
+      if (ws_.defined()) retired_.push_back(ws_);
       ws_ = at::zeros({std::max<int64_t>(rows, 64) * 16}, x.options().dtype(at::kByte));
+    }
     CheckLaunch(ortb200_argmax(xc.data_ptr(), out.data_ptr<int64_t>(), rows, x.size(-1), dt, ws_.data_ptr(), ws_.numel(),
                                ctx.cuda_stream()),
                 "ortb200_argmax");

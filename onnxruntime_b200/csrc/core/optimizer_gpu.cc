@@ -5,7 +5,8 @@
 //    one tcgen05 GEMM whose epilogue applies bias, activation and the residual
 //    add (the reference runs cuBLAS followed by separate BiasGelu / Add kernels).
 //  * SwiGLUFusion:  Mul(silu(MatMul(x, Wg)), MatMul(x, Wu)) -> com.ortb200.GemmSwiGLU(x, Wg, Wu)
-//    one kernel with two TMEM accumulators sharing the activation tile.
+//    one kernel with two TMEM accumulators sharing the activation tile; FastGelu in place of silu sets
+//    activation = "geglu".
 //  * MatMulAllReduceFusion:  AllReduce(GEMM) -> the GEMM carries all_reduce=1 and
 //    its kernel finishes the row-parallel sum over NVLink itself.
 #include "optimizer.h"
@@ -56,18 +57,21 @@ int SwiGLUFusion(PassContext& c) {
       if (!silu || !up) continue;
       std::string gate_out;
       Node* sig = nullptr;
-      if (!MatchSilu(g, silu, &gate_out, &sig)) continue;
+      const bool gelu = silu->domain == kMSDomain && silu->op_type == "FastGelu" && !silu->has_input(1);
+      if (gelu) gate_out = silu->inputs[0];
+      else if (!MatchSilu(g, silu, &gate_out, &sig)) continue;
       Node* gate = g.Producer(gate_out);
       if (!gate || gate->op_type != "MatMul" || !gate->domain.empty() || up->op_type != "MatMul" || !up->domain.empty()) continue;
       if (gate->inputs[0] != up->inputs[0]) continue;
       if (!IsHalfWeight2D(g, gate->inputs[1]) || !IsHalfWeight2D(g, up->inputs[1])) continue;
       if (g.GetConstant(gate->inputs[1])->sizes() != g.GetConstant(up->inputs[1])->sizes()) continue;
-      if (g.NumConsumers(gate_out) != 2 || g.NumConsumers(up->outputs[0]) != 1 || g.NumConsumers(silu->outputs[0]) != 1) continue;
-      g.AddNode("GemmSwiGLU", {gate->inputs[0], gate->inputs[1], up->inputs[1]}, {top->outputs[0]}, kFusedDomain,
-                g.UniqueName("GemmSwiGLU"));
+      if (g.NumConsumers(gate_out) != (gelu ? 1u : 2u) || g.NumConsumers(up->outputs[0]) != 1 || g.NumConsumers(silu->outputs[0]) != 1) continue;
+      Node* f = g.AddNode("GemmSwiGLU", {gate->inputs[0], gate->inputs[1], up->inputs[1]}, {top->outputs[0]}, kFusedDomain,
+                          g.UniqueName("GemmSwiGLU"));
+      if (gelu) f->set_attr_s("activation", "geglu");
       g.RemoveNode(top);
       g.RemoveNode(silu);
-      g.RemoveNode(sig);
+      if (sig) g.RemoveNode(sig);
       g.RemoveNode(gate);
       g.RemoveNode(up);
       ++count;

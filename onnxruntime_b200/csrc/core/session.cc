@@ -447,6 +447,7 @@ std::vector<std::tuple<std::string, std::string, std::string>> InferenceSession:
 
 at::Tensor& InferenceSession::GemmWorkspace(int64_t nbytes) {
   if (!gemm_ws_.defined() || gemm_ws_.numel() < nbytes) {
+    if (gemm_ws_.defined()) retired_ws_.push_back(gemm_ws_);
     const int64_t sz = std::max<int64_t>(nbytes, 64 << 20);
     gemm_ws_ = at::zeros({sz}, at::TensorOptions().dtype(at::kByte).device(device_));
   }
@@ -455,6 +456,7 @@ at::Tensor& InferenceSession::GemmWorkspace(int64_t nbytes) {
 
 at::Tensor& InferenceSession::AttnWorkspace(int64_t nbytes) {
   if (!attn_ws_.defined() || attn_ws_.numel() < nbytes) {
+    if (attn_ws_.defined()) retired_ws_.push_back(attn_ws_);
     const int64_t sz = std::max<int64_t>(nbytes, 8 << 20);
     attn_ws_ = at::zeros({sz}, at::TensorOptions().dtype(at::kByte).device(device_));
   }
@@ -598,6 +600,7 @@ std::vector<Value> InferenceSession::RunImpl(const RunOptions& ro, const std::ve
     }
   }
 
+  bool captured_now = false;
   if (graph_id >= 0) {
     auto& cg_ptr = cuda_graphs_[graph_id];
     if (!cg_ptr) cg_ptr = std::make_unique<CapturedGraph>();
@@ -637,8 +640,10 @@ std::vector<Value> InferenceSession::RunImpl(const RunOptions& ro, const std::ve
         }
         cg.graph.capture_end();
       }
+      // The capture itself executed nothing, and it must stay that way: the eager run above was this call's step, and a
+      // replay would advance recurrent state that the step updates in place a second time.
       cg.captured = true;
-      cg.graph.replay();  // the capture itself executed nothing
+      captured_now = true;
     } else {
       for (size_t i = 0; i < inputs.size(); ++i) {
         if (!inputs[i].t.defined()) continue;
@@ -650,15 +655,17 @@ std::vector<Value> InferenceSession::RunImpl(const RunOptions& ro, const std::ve
       }
       cg.graph.replay();
     }
-    results.clear();
-    for (auto& n : output_names) results.push_back(cg.slots[ex->SlotOf(n)]);
+    if (!captured_now) {
+      results.clear();
+      for (auto& n : output_names) results.push_back(cg.slots[ex->SlotOf(n)]);
+    }
     for (size_t i = 0; i < results.size(); ++i) {
       if (!results[i].t.defined()) continue;
       const at::Tensor b = bound_outputs ? (*bound_outputs)[i].t : at::Tensor();
       if (b.defined()) {
         if (b.data_ptr() != results[i].t.data_ptr()) const_cast<at::Tensor&>(b).copy_(results[i].t, true);
         results[i].t = b;
-      } else if (!bound_outputs || !AliasesAny(results[i].t, cg.static_in)) {
+      } else if (!captured_now && (!bound_outputs || !AliasesAny(results[i].t, cg.static_in))) {
         // the graph's own output buffer is overwritten by the next replay: hand out a copy (an output that is one of
         // the bound input buffers, such as an in-place KV cache, is returned as it is)
         results[i].t = results[i].t.clone();

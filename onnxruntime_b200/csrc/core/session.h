@@ -219,6 +219,7 @@ class InferenceSession {
   std::map<std::string, size_t> input_index_;
   std::vector<const ValueInfo*> input_info_;
   at::Tensor gemm_ws_, attn_ws_, status_word_;
+  std::vector<at::Tensor> retired_ws_;  // outgrown workspaces that captured graphs still point to
   std::mutex run_mu_;
 };
 

@@ -675,6 +675,11 @@ void RegisterBuiltinSchemas(std::map<std::string, OpSchema>& t) {
   // ---- this runtime's fused operators
   Reg(t, FUSED, "FusedGemm", 2, 5, FusedGemm);
   Reg(t, FUSED, "GemmSwiGLU", 3, 4, FusedGemm);
+  Reg(t, FUSED, "HyperConnectionNorm", 5, 7);
+  Reg(t, FUSED, "PackedGatedDelta", 11, 11);
+  Reg(t, FUSED, "PackedMLstm", 9, 9);
+  Reg(t, FUSED, "GatedPagedAttention", 6, 11);
+  Reg(t, FUSED, "SoftCap", 1, 1);
   Reg(t, FUSED, "SwiGLU", 1, 1, [](Ctx& c) {
     if (!c.HasShape(0) || c.Rank(0) < 1) return;
     Dims out = c.Dims(0);

@@ -40,9 +40,15 @@ struct AttnParams {
   float scale_log2, softcap, scale;
   int bf16;
   int* status;
+  // packed queries over a paged cache (block_table given)
+  const int* block_table;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  int block_size, max_blocks, num_blocks;
 };
 
-template <int HD>
+// SPLIT: P is held as the sum of two 16-bit tiles (leading part and remainder), both multiplied with V.
+template <int HD, bool SPLIT>
 struct AttnSmem {
   static constexpr int kBoxBytes = 128 * 128;          // [128 rows][64 elems] of 16-bit data
   static constexpr int kBoxes = HD / 64;                // boxes per Q / K / V tile
@@ -53,7 +59,7 @@ struct AttnSmem {
   static constexpr int kOffQ = 0;
   static constexpr int kOffKV = kQBytes;
   static constexpr int kOffP = kOffKV + 2 * kStageBytes;
-  static constexpr int kOffBar = kOffP + kPBytes;
+  static constexpr int kOffBar = kOffP + kPBytes * (SPLIT ? 2 : 1);
   static constexpr int kTotal = kOffBar + 128 + 1024;
   static constexpr int kTmemCols = 512;                // two score buffers (2 x 128 columns) + O (HD columns)
 };
@@ -80,19 +86,33 @@ __device__ __forceinline__ float ex2_approx(float x) {
 // barrier indices
 enum { BAR_Q = 0, BAR_KV_FULL0, BAR_KV_FULL1, BAR_KV_EMPTY0, BAR_KV_EMPTY1, BAR_S_FULL0, BAR_S_FULL1, BAR_P_READY, BAR_O_FULL, BAR_COUNT };
 
-template <int HD>
+template <int HD, bool SPLIT>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                     const __grid_constant__ CUtensorMap tm_v, const AttnParams p) {
-  using L = AttnSmem<HD>;
+  using L = AttnSmem<HD, SPLIT>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::kOffBar);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + BAR_COUNT);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int q0 = blockIdx.x * kQT;
-  const int head = blockIdx.y, b = blockIdx.z;
+  int q0 = blockIdx.x * kQT, b = blockIdx.z, q_row0 = 0, S = p.S;
+  if (p.block_table != nullptr) {
+    // query tiles of all sequences are numbered consecutively; the grid is an upper bound of their count
+    pdl_wait_prior_grids();
+    int tile = blockIdx.x;
+    for (b = 0; b < p.B; ++b) {
+      q_row0 = p.cu_seqlens[b];
+      S = p.cu_seqlens[b + 1] - q_row0;
+      const int tiles = (S + kQT - 1) / kQT;
+      if (tile < tiles) break;
+      tile -= tiles;
+    }
+    if (b == p.B) return;
+    q0 = tile * kQT;
+  }
+  const int head = blockIdx.y;
   const int kvh = head / (p.N / p.Nk);
 
   if (threadIdx.x == 0) {
@@ -114,8 +134,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   const uint32_t tmem_o = tmem_base + 256;    // O: columns [256, 256 + HD), accumulated over all key tiles
 
   pdl_wait_prior_grids();
-  const int total = p.seqlens_k ? p.seqlens_k[b] + 1 : p.kv_len;
-  const int past = p.first_prompt ? 0 : total - p.S;
+  const bool paged = p.block_table != nullptr;
+  const int total = paged ? p.past_seqlens[b] + S : (p.seqlens_k ? p.seqlens_k[b] + 1 : p.kv_len);
+  const int past = paged ? total - S : (p.first_prompt ? 0 : total - S);
   // key range needed by this query tile
   int kv_end = total;
   if (p.causal) kv_end = min(kv_end, past + q0 + kQT);
@@ -128,7 +149,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     if (lane == 0 && n_tiles > 0) {
       mbar_expect_tx(&bars[BAR_Q], L::kQBytes);
       for (int bx = 0; bx < L::kBoxes; ++bx)
-        tma_load_4d(smem + L::kOffQ + bx * L::kBoxBytes, &tm_q, &bars[BAR_Q], bx * 64, q0, head, b);
+        tma_load_4d(smem + L::kOffQ + bx * L::kBoxBytes, &tm_q, &bars[BAR_Q], bx * 64, q_row0 + q0, head, paged ? 0 : b);
       for (int t = 0; t < n_tiles; ++t) {
         const int s = t & 1;
         if (t >= 2) {
@@ -140,9 +161,16 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         uint8_t* st = smem + L::kOffKV + s * L::kStageBytes;
         mbar_expect_tx(&bars[BAR_KV_FULL0 + s], L::kStageBytes);
         const int key0 = kv_begin + t * kKT;
+        // cache coordinates behind the head entry: (position, head, batch), or (position in block, head, block)
+        int c1 = key0, c3 = b;
+        if (paged) {
+          const int bi = min(key0 / p.block_size, p.max_blocks - 1);
+          c1 = key0 % p.block_size;
+          c3 = min(max(p.block_table[static_cast<long long>(b) * p.max_blocks + bi], 0), p.num_blocks - 1);
+        }
         for (int bx = 0; bx < L::kBoxes; ++bx) {
-          tma_load_4d(st + bx * L::kBoxBytes, &tm_k, &bars[BAR_KV_FULL0 + s], bx * 64, key0, kvh, b);
-          tma_load_4d(st + L::kKVBytes + bx * L::kBoxBytes, &tm_v, &bars[BAR_KV_FULL0 + s], bx * 64, key0, kvh, b);
+          tma_load_4d(st + bx * L::kBoxBytes, &tm_k, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
+          tma_load_4d(st + L::kKVBytes + bx * L::kBoxBytes, &tm_v, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
         }
       }
     }
@@ -186,6 +214,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           const uint64_t pdesc = umma_desc_sw128(p_addr + (kk / 4) * L::kBoxBytes + (kk % 4) * 32);
           const uint64_t vdesc = umma_desc_mn_sw128(v_addr + kk * 2048, L::kBoxBytes, 1024);
           umma_f16(tmem_o, pdesc, vdesc, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
+          if (SPLIT) {
+            const uint64_t rdesc = umma_desc_sw128(p_addr + L::kPBytes + (kk / 4) * L::kBoxBytes + (kk % 4) * 32);
+            umma_f16(tmem_o, rdesc, vdesc, idesc_o, 1u);
+          }
         }
         umma_commit(&bars[BAR_O_FULL]);
         umma_commit(&bars[BAR_KV_EMPTY0 + s]);
@@ -280,7 +312,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       float row_sum = 0.f, row_sum1 = 0.f;
 #pragma unroll
       for (int c = 0; c < kKT; c += 32) {
-        uint32_t packed[16];
+        uint32_t packed[16], rest[SPLIT ? 16 : 1];
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
           const float p0 = ex2_approx(fmaf(sv[c + j], fs, neg_m));
@@ -290,9 +322,17 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           if (p.bf16) {
             __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
             packed[j / 2] = *reinterpret_cast<uint32_t*>(&h);
+            if (SPLIT) {
+              __nv_bfloat162 e = __floats2bfloat162_rn(p0 - __bfloat162float(h.x), p1 - __bfloat162float(h.y));
+              rest[SPLIT ? j / 2 : 0] = *reinterpret_cast<uint32_t*>(&e);
+            }
           } else {
             __half2 h = __floats2half2_rn(p0, p1);
             packed[j / 2] = *reinterpret_cast<uint32_t*>(&h);
+            if (SPLIT) {
+              __half2 e = __floats2half2_rn(p0 - __half2float(h.x), p1 - __half2float(h.y));
+              rest[SPLIT ? j / 2 : 0] = *reinterpret_cast<uint32_t*>(&e);
+            }
           }
         }
         // 32 keys = 4 chunks of 16 bytes; column c lives in box c / 64
@@ -302,6 +342,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           const int chunk = ((c % 64) * 2) / 16 + ch;
           uint8_t* dst = p_smem + box * L::kBoxBytes + r * 128 + ((chunk ^ (r & 7)) << 4);
           *reinterpret_cast<uint4*>(dst) = make_uint4(packed[ch * 4], packed[ch * 4 + 1], packed[ch * 4 + 2], packed[ch * 4 + 3]);
+          if (SPLIT) *reinterpret_cast<uint4*>(dst + L::kPBytes) = make_uint4(rest[SPLIT ? ch * 4 : 0], rest[SPLIT ? ch * 4 + 1 : 0], rest[SPLIT ? ch * 4 + 2 : 0], rest[SPLIT ? ch * 4 + 3 : 0]);
         }
       }
       l += row_sum + row_sum1;
@@ -324,7 +365,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       denom = l * rescale + exp2f(sink - mm);
     }
     const float inv = (denom > 0.f && n_tiles > 0) ? rescale / denom : 0.f;
-    uint8_t* orow = static_cast<uint8_t*>(p.out) + 2 * (b * p.o_strides[0] + s_idx * p.o_strides[1] + head * p.o_strides[2]);
+    uint8_t* orow = static_cast<uint8_t*>(p.out) + 2 * ((paged ? 0 : b * p.o_strides[0]) + (q_row0 + s_idx) * p.o_strides[1] + head * p.o_strides[2]);
 #pragma unroll 1
     for (int c0 = 0; c0 < HD; c0 += 32) {
       float v[32];
@@ -335,7 +376,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = 0.f;
       }
-      if (ok && s_idx < p.S) {
+      if (ok && s_idx < S) {
 #pragma unroll
         for (int c = 0; c < 32; c += 8) {
           uint32_t w[4];
@@ -363,28 +404,32 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   }
 }
 
-template <int HD>
+template <int HD, bool SPLIT>
 static int launch_attn(const ortb200_attn_prefill_args* a, cudaStream_t stream) {
-  using L = AttnSmem<HD>;
+  using L = AttnSmem<HD, SPLIT>;
   const CUtensorMapDataType dt = a->dtype == ORTB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+  const bool paged = a->block_table != nullptr;
   CUtensorMap tq, tk, tv;
   {
-    const int64_t dims[4] = {HD, a->S, a->N, a->B};
-    const int64_t strides[3] = {a->q_strides[1] * 2, a->q_strides[2] * 2, a->q_strides[0] * 2};
+    const int64_t dims[4] = {HD, paged ? a->T : a->S, a->N, paged ? 1 : a->B};
+    const int64_t strides[3] = {a->q_strides[1] * 2, a->q_strides[2] * 2, paged ? a->T * a->q_strides[1] * 2 : a->q_strides[0] * 2};
     if (make_tensor_map_4d(&tq, a->q, dt, 2, dims, strides, 64, kQT) != 0) return -6;
   }
   {
-    const int64_t dims[4] = {HD, a->kv_len, a->Nk, a->B};
-    const int64_t strides[3] = {a->kv_strides[2] * 2, a->kv_strides[1] * 2, a->kv_strides[0] * 2};
+    const int64_t row = static_cast<int64_t>(a->Nk) * HD * 2;
+    const int64_t dims[4] = {HD, paged ? a->block_size : a->kv_len, a->Nk, paged ? a->num_blocks : a->B};
+    const int64_t contiguous[3] = {a->kv_strides[2] * 2, a->kv_strides[1] * 2, a->kv_strides[0] * 2};
+    const int64_t blocks[3] = {row, HD * 2, row * a->block_size};
+    const int64_t* strides = paged ? blocks : contiguous;
     if (make_tensor_map_4d(&tk, a->k, dt, 2, dims, strides, 64, kKT) != 0) return -6;
     if (make_tensor_map_4d(&tv, a->v, dt, 2, dims, strides, 64, kKT) != 0) return -6;
   }
   AttnParams p;
   p.seqlens_k = a->seqlens_k;
-  p.key_mask = a->key_mask;
+  p.key_mask = paged ? nullptr : a->key_mask;
   p.head_sink = a->head_sink;
   p.out = a->out;
-  p.B = a->B; p.S = a->S; p.N = a->N; p.Nk = a->Nk; p.kv_len = a->kv_len;
+  p.B = a->B; p.S = a->S; p.N = a->N; p.Nk = a->Nk; p.kv_len = paged ? (1 << 30) : a->kv_len;
   for (int i = 0; i < 3; ++i) p.o_strides[i] = a->o_strides[i];
   p.first_prompt = a->first_prompt; p.causal = a->causal; p.window = a->window;
   p.scale = a->scale != 0.f ? a->scale : 1.0f / sqrtf(static_cast<float>(HD));
@@ -392,13 +437,17 @@ static int launch_attn(const ortb200_attn_prefill_args* a, cudaStream_t stream) 
   p.softcap = a->softcap;
   p.bf16 = a->dtype == ORTB200_BF16 ? 1 : 0;
   p.status = a->status;
-  auto kern = attn_prefill_kernel<HD>;
+  p.block_table = a->block_table; p.cu_seqlens = a->cu_seqlens; p.past_seqlens = a->past_seqlens;
+  p.block_size = a->block_size; p.max_blocks = a->max_blocks; p.num_blocks = a->num_blocks;
+  auto kern = attn_prefill_kernel<HD, SPLIT>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal) != cudaSuccess) return -10;
     attr_set = true;
   }
-  dim3 grid((a->S + kQT - 1) / kQT, a->N, a->B);
+  // packed form: every sequence has at most one partly filled query tile
+  const int tiles = paged ? a->T / kQT + (a->B < a->T ? a->B : a->T) : (a->S + kQT - 1) / kQT;
+  dim3 grid(tiles, a->N, paged ? 1 : a->B);
   kern<<<grid, kAttnThreads, L::kTotal, stream>>>(tq, tk, tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
@@ -410,13 +459,19 @@ using namespace ortb200;
 extern "C" int ortb200_attn_prefill(const ortb200_attn_prefill_args* a, ortb200_stream_t stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (!a || !a->q || !a->k || !a->v || !a->out) return -1;
-  if (a->B <= 0 || a->S <= 0 || a->N <= 0 || a->Nk <= 0 || a->N % a->Nk != 0 || a->kv_len <= 0) return -1;
+  const bool paged = a->block_table != nullptr;
+  if (a->B <= 0 || a->N <= 0 || a->N > 65535 || a->Nk <= 0 || a->N % a->Nk != 0) return -1;
+  if (!paged && (a->S <= 0 || a->kv_len <= 0)) return -1;
+  if (paged && (!a->cu_seqlens || !a->past_seqlens || a->T <= 0 || a->block_size <= 0 || a->block_size % kKT != 0 || a->max_blocks <= 0 ||
+                a->num_blocks <= 0))
+    return -1;
   if (a->H != 64 && a->H != 128) return -2;
   if (a->dtype != ORTB200_BF16 && a->dtype != ORTB200_F16) return -4;
-  for (int i = 0; i < 3; ++i)
-    if (a->q_strides[i] % 8 || a->o_strides[i] % 8 || a->kv_strides[i] % 8) return -3;
+  for (int i = paged ? 1 : 0; i < 3; ++i)
+    if (a->q_strides[i] % 8 || a->o_strides[i] % 8 || (!paged && a->kv_strides[i] % 8)) return -3;
   if ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) | reinterpret_cast<uintptr_t>(a->v) |
        reinterpret_cast<uintptr_t>(a->out)) & 15)
     return -3;
-  return a->H == 128 ? launch_attn<128>(a, stream) : launch_attn<64>(a, stream);
+  if (a->split_weights) return a->H == 128 ? launch_attn<128, true>(a, stream) : launch_attn<64, true>(a, stream);
+  return a->H == 128 ? launch_attn<128, false>(a, stream) : launch_attn<64, false>(a, stream);
 }

@@ -391,7 +391,7 @@ gemm_2cta_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
 
 int launch_gemm_2cta(const ortb200_gemm_args* a, cudaStream_t stream) {
   const bool fp8 = a->in_dtype == ORTB200_F8E4M3;
-  if (a->act == ORTB200_ACT_SWIGLU || (a->in_dtype != 0 && !fp8) || a->rms_eps > 0.f) return -16;
+  if (is_gated_act(a->act) || (a->in_dtype != 0 && !fp8) || a->rms_eps > 0.f) return -16;
   if (fp8 && (a->world > 1 || a->K % 16 != 0)) return -16;
   if (a->alpha_dev != nullptr && !fp8) return -16;
   if (a->world > 1 && (a->act != ORTB200_ACT_NONE || a->ldo != a->N || a->N % 8 != 0 || a->world > 8)) return -12;
@@ -466,7 +466,7 @@ int launch_gemm_2cta(const ortb200_gemm_args* a, cudaStream_t stream) {
 
 // Grouped GEMM (mixture of experts) on CTA pairs: 256-token tiles from the device-side tile list.
 int launch_gemm_grouped_2cta(const ortb200_gemm_grouped_args* a, cudaStream_t stream) {
-  if (a->act == ORTB200_ACT_SWIGLU || a->tile_rows != 256) return -16;
+  if (is_gated_act(a->act) || a->tile_rows != 256) return -16;
   CUtensorMap tw, tx;
   const CUtensorMapDataType dt = a->dtype == ORTB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   const int64_t w_rows = static_cast<int64_t>(a->num_experts) * a->w_rows_per_expert;

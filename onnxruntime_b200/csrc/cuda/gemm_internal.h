@@ -5,6 +5,9 @@
 
 namespace ortb200 {
 
+// activations that combine two weight tiles (gate rows, up rows)
+inline bool is_gated_act(int act) { return act == ORTB200_ACT_SWIGLU || act == ORTB200_ACT_GEGLU; }
+
 struct SmallGemmParams {
   int M, N, K;
   int num_kb;

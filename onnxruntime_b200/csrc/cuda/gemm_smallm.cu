@@ -562,7 +562,7 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         const float row_scale = p.rms_eps > 0.f ? s_rstd[j] * p.alpha : p.alpha;
         float y = v * row_scale + bias_v;
         if (DUAL) {
-          const float g = y / (1.0f + __expf(-y));
+          const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
           y = g * (u * row_scale);
         } else {
           y = act_apply(p.act, y);
@@ -715,7 +715,7 @@ int pick_cluster(int tiles, int num_kb, int bn, int force) {
 }
 
 int launch_gemm_smallm(const ortb200_gemm_args* a, int bn, cudaStream_t stream, int* cluster_out, int* stages_out) {
-  const bool dual = a->act == ORTB200_ACT_SWIGLU;
+  const bool dual = is_gated_act(a->act);
   const int num_kb = (a->K + kBK - 1) / kBK;
   const int tiles_n = (a->N + kBM - 1) / kBM, tiles_m = (a->M + bn - 1) / bn;
   const int cluster = pick_cluster(tiles_n * tiles_m, num_kb, bn, a->force_splits);
@@ -788,7 +788,7 @@ int launch_gemm_smallm(const ortb200_gemm_args* a, int bn, cudaStream_t stream, 
 }
 
 int launch_gemm_grouped(const ortb200_gemm_grouped_args* a, cudaStream_t stream) {
-  const bool dual = a->act == ORTB200_ACT_SWIGLU;
+  const bool dual = is_gated_act(a->act);
   const int bn = a->tile_rows;
   if (bn != 16 && bn != 32 && bn != 64) return -8;
   const int num_kb = (a->K + kBK - 1) / kBK;
@@ -824,9 +824,9 @@ extern "C" int ortb200_gemm_grouped(const ortb200_gemm_grouped_args* a, ortb200_
   if (!a || !a->x || !a->w || !a->out || !a->tile_info || !a->num_tiles) return -1;
   if (a->rows <= 0 || a->N <= 0 || a->K <= 0 || a->K % 8 != 0 || a->num_experts <= 0 || a->max_tiles <= 0 || a->max_tiles > 65535) return -1;
   if (a->dtype != ORTB200_BF16 && a->dtype != ORTB200_F16) return -4;
-  if (a->act == ORTB200_ACT_SWIGLU && a->dual_offset <= 0) return -2;
+  if (ortb200::is_gated_act(a->act) && a->dual_offset <= 0) return -2;
   if ((reinterpret_cast<uintptr_t>(a->x) | reinterpret_cast<uintptr_t>(a->w) | reinterpret_cast<uintptr_t>(a->tile_info)) & 15) return -3;
-  if (a->tile_rows == 256 && a->act != ORTB200_ACT_SWIGLU) return ortb200::launch_gemm_grouped_2cta(a, static_cast<cudaStream_t>(stream));
+  if (a->tile_rows == 256 && !ortb200::is_gated_act(a->act)) return ortb200::launch_gemm_grouped_2cta(a, static_cast<cudaStream_t>(stream));
   if (a->tile_rows >= 128) return ortb200::launch_gemm_grouped_large(a, static_cast<cudaStream_t>(stream));
   return ortb200::launch_gemm_grouped(a, static_cast<cudaStream_t>(stream));
 }

@@ -491,7 +491,7 @@ __device__ __forceinline__ void gemm_tcgen05_body(const CUtensorMap* tmap_w, con
                 // than the gated one are applied on the way out, on the 16-bit value, as a separate op would
                 float y = v[j] * alpha_v + bias_v;
                 if (DUAL) {
-                  const float g = y / (1.0f + __expf(-y));
+                  const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
                   y = g * (uu[j] * alpha_v);
                 }
                 uint16_t bits;
@@ -586,7 +586,7 @@ __device__ __forceinline__ void gemm_tcgen05_body(const CUtensorMap* tmap_w, con
                 if (m < p.M) {
                   float y = v[j] * alpha_v + bias_v;
                   if (DUAL) {
-                    const float g = y / (1.0f + __expf(-y));
+                    const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
                     y = g * (uu[j] * alpha_v);
                   } else {
                     y = apply_act(p.act, y);
@@ -844,7 +844,7 @@ extern "C" int ortb200_allgather_gemm(const ortb200_allgather_gemm_args* a, ortb
   if (a->dtype != ORTB200_BF16 && a->dtype != ORTB200_F16) return -2;
   if (a->world < 1 || a->world > 8 || a->rank < 0 || a->rank >= a->world) return -12;
   if (a->rows_local <= 0 || a->N <= 0 || a->K <= 0 || a->K % 8 != 0) return -3;
-  if (a->act == ORTB200_ACT_SWIGLU) return -8;
+  if (is_gated_act(a->act)) return -8;
   if ((reinterpret_cast<uintptr_t>(a->x_local) | reinterpret_cast<uintptr_t>(a->w)) & 15) return -3;
   if (a->rows_local > ortb200_allgather_gemm_max_rows(a->world, a->K, a->symm_bytes)) return -13;
   for (int i = 0; i < a->world; ++i)
@@ -882,9 +882,9 @@ extern "C" int ortb200_allgather_gemm(const ortb200_allgather_gemm_args* a, ortb
 
 extern "C" int64_t ortb200_gemm_workspace_bytes(int M, int N, int K, int act) {
   GemmPlan pl, pl128;
-  if (M <= 0 || N <= 0 || K <= 0 || plan_gemm(M, N, K, act == ORTB200_ACT_SWIGLU, 0, 0, -1, &pl) != 0) return 65536;
+  if (M <= 0 || N <= 0 || K <= 0 || plan_gemm(M, N, K, is_gated_act(act), 0, 0, -1, &pl) != 0) return 65536;
   int64_t need = pl.ws_need;
-  if (plan_gemm(M, N, K, act == ORTB200_ACT_SWIGLU, 0, 0, -1, &pl128, 128) == 0 && pl128.ws_need > need) need = pl128.ws_need;
+  if (plan_gemm(M, N, K, is_gated_act(act), 0, 0, -1, &pl128, 128) == 0 && pl128.ws_need > need) need = pl128.ws_need;
   return need > 65536 ? need : 65536;
 }
 
@@ -905,7 +905,7 @@ extern "C" int ortb200_gemm(const ortb200_gemm_args* a, ortb200_stream_t stream_
   if (a->K % (fp8 ? 16 : 8) != 0) return -2;                     // TMA row pitch must be a multiple of 16 bytes
   if ((reinterpret_cast<uintptr_t>(a->x) & 15) || (reinterpret_cast<uintptr_t>(a->w) & 15)) return -3;
   if (a->dtype != ORTB200_F16 && a->dtype != ORTB200_BF16) return -4;
-  const bool dual = a->act == ORTB200_ACT_SWIGLU;
+  const bool dual = is_gated_act(a->act);
   if (dual && (a->dual_offset <= 0 || a->w_rows < a->dual_offset + a->N)) return -5;
   if (!dual && a->w_rows < a->N) return -5;
   if (q4 && (a->force_bn ? a->force_bn : pick_bn(a->M)) > 64) return -15;  // packed weights: decode-shaped problems only
@@ -1002,7 +1002,7 @@ extern "C" int ortb200_gemm(const ortb200_gemm_args* a, ortb200_stream_t stream_
 // Grouped GEMM on the persistent kernel: token tiles of 128 or 256 rows taken from the device-side tile list.
 namespace ortb200 {
 int launch_gemm_grouped_large(const ortb200_gemm_grouped_args* a, cudaStream_t stream) {
-  const bool dual = a->act == ORTB200_ACT_SWIGLU;
+  const bool dual = is_gated_act(a->act);
   const int bn = a->tile_rows;
   if ((bn != 128 && bn != 256) || (dual && bn != 128)) return -8;
   const int num_kb = (a->K + kBK - 1) / kBK;

@@ -77,7 +77,7 @@ __global__ void __launch_bounds__(256) argmax_kernel(const T* __restrict__ x, in
 __device__ __forceinline__ float act_fn(int act, float v, float alpha) {
   switch (act) {
     case ORTB200_ACT_GELU: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
-    case ORTB200_ACT_FASTGELU: return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * v * (1.0f + 0.044715f * v * v)));
+    case ORTB200_ACT_FASTGELU: return gelu_tanh(v);
     case ORTB200_ACT_RELU: return fmaxf(v, 0.0f);
     case ORTB200_ACT_SILU: return v / (1.0f + __expf(-v));
     case ORTB200_ACT_QUICKGELU: return v / (1.0f + __expf(-alpha * v));
@@ -98,7 +98,7 @@ __global__ void bias_act_kernel(const T* __restrict__ x, const T* __restrict__ b
   pdl_launch_dependents();
 }
 
-template <typename T>
+template <typename T, bool GELU>
 __global__ void swiglu_kernel(const T* __restrict__ x, T* __restrict__ y, int64_t rows, int cols) {
   pdl_wait_prior_grids();
   const int64_t total = rows * cols;
@@ -106,13 +106,13 @@ __global__ void swiglu_kernel(const T* __restrict__ x, T* __restrict__ y, int64_
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
     const int64_t r = i / cols, c = i % cols;
     const float g = to_float<T>(x[r * 2 * cols + c]), u = to_float<T>(x[r * 2 * cols + cols + c]);
-    y[i] = from_float<T>(g / (1.0f + __expf(-g)) * u);
+    y[i] = from_float<T>(gated_act(GELU, g) * u);
   }
   pdl_launch_dependents();
 }
 
 // 16-bit types, cols a multiple of 8: one thread combines 8 gate values with 8 up values (16-byte accesses)
-template <typename T>
+template <typename T, bool GELU>
 __global__ void __launch_bounds__(256) swiglu_vec8_kernel(const uint4* __restrict__ x, uint4* __restrict__ y, int64_t rows, int cols8) {
   pdl_wait_prior_grids();
   const int64_t total = rows * cols8;
@@ -126,7 +126,7 @@ __global__ void __launch_bounds__(256) swiglu_vec8_kernel(const uint4* __restric
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float gv = to_float<T>(g[e]);
-      o[e] = from_float<T>(gv / (1.0f + __expf(-gv)) * to_float<T>(u[e]));
+      o[e] = from_float<T>(gated_act(GELU, gv) * to_float<T>(u[e]));
     }
     y[i] = *reinterpret_cast<const uint4*>(o);
   }
@@ -226,27 +226,36 @@ extern "C" int ortb200_bias_act(const void* x, const void* bias, void* y, int64_
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
-extern "C" int ortb200_swiglu(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream) {
+template <bool GELU>
+static int launch_gated_unit(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream) {
   if (!x || !y || rows < 0 || cols <= 0) return -1;
   if (rows == 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dtype != ORTB200_F32 && cols % 8 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y)) & 15) == 0) {
     const int gv = grid_for(rows * (cols / 8), 256);
     if (dtype == ORTB200_BF16)
-      swiglu_vec8_kernel<__nv_bfloat16><<<gv, 256, 0, st>>>(static_cast<const uint4*>(x), static_cast<uint4*>(y), rows, cols / 8);
+      swiglu_vec8_kernel<__nv_bfloat16, GELU><<<gv, 256, 0, st>>>(static_cast<const uint4*>(x), static_cast<uint4*>(y), rows, cols / 8);
     else
-      swiglu_vec8_kernel<__half><<<gv, 256, 0, st>>>(static_cast<const uint4*>(x), static_cast<uint4*>(y), rows, cols / 8);
+      swiglu_vec8_kernel<__half, GELU><<<gv, 256, 0, st>>>(static_cast<const uint4*>(x), static_cast<uint4*>(y), rows, cols / 8);
     return cudaGetLastError() == cudaSuccess ? 0 : -11;
   }
   const int g = grid_for(rows * cols, 256);
   if (dtype == ORTB200_BF16)
-    swiglu_kernel<__nv_bfloat16><<<g, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(y), rows, cols);
+    swiglu_kernel<__nv_bfloat16, GELU><<<g, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(y), rows, cols);
   else if (dtype == ORTB200_F16)
-    swiglu_kernel<__half><<<g, 256, 0, st>>>(static_cast<const __half*>(x), static_cast<__half*>(y), rows, cols);
+    swiglu_kernel<__half, GELU><<<g, 256, 0, st>>>(static_cast<const __half*>(x), static_cast<__half*>(y), rows, cols);
   else if (dtype == ORTB200_F32)
-    swiglu_kernel<float><<<g, 256, 0, st>>>(static_cast<const float*>(x), static_cast<float*>(y), rows, cols);
+    swiglu_kernel<float, GELU><<<g, 256, 0, st>>>(static_cast<const float*>(x), static_cast<float*>(y), rows, cols);
   else return -4;
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int ortb200_swiglu(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream) {
+  return launch_gated_unit<false>(x, y, rows, cols, dtype, stream);
+}
+
+extern "C" int ortb200_geglu(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream) {
+  return launch_gated_unit<true>(x, y, rows, cols, dtype, stream);
 }
 
 extern "C" int ortb200_rotary(const void* x, void* y, const int64_t* position_ids, int64_t position_offset,

@@ -27,6 +27,7 @@ enum ortb200_act {
   ORTB200_ACT_SILU = 4,
   ORTB200_ACT_SWIGLU = 5,    // silu(W1 x) * (W2 x); W2 rows start `dual_offset` rows after W1 rows
   ORTB200_ACT_QUICKGELU = 6,
+  ORTB200_ACT_GEGLU = 7,     // gelu_tanh(W1 x) * (W2 x), rows laid out as for SWIGLU
 };
 
 // out[M, N] = act(alpha * X[M, K] * W[N, K]^T + bias[N]) + residual[M, N]
@@ -372,6 +373,17 @@ typedef struct {
   int dtype;
   int* status;
   const int* key_mask;     // optional [B, kv_len] int32, 0 = this key is padding for every query of the batch entry
+  // Packed queries over a paged cache: when block_table is given, q / out hold T tokens of B sequences (token, head
+  // strides; the batch stride is ignored), sequence b owns rows [cu_seqlens[b], cu_seqlens[b + 1]) and has
+  // past_seqlens[b] cached keys in front of them; k / v are [num_blocks, block_size, Nk, H] with block_size a multiple of
+  // 128.  S, kv_len, seqlens_k, kv_strides, first_prompt and key_mask are ignored.
+  const int* block_table;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  int T, block_size, max_blocks, num_blocks;
+  // Softmax weights enter the second product as the sum of two 16-bit terms instead of one (fp32-like weights for 1.5x
+  // the tensor-core work).
+  int split_weights;
 } ortb200_attn_prefill_args;
 int ortb200_attn_prefill(const ortb200_attn_prefill_args* args, ortb200_stream_t stream);
 
@@ -388,8 +400,9 @@ int64_t ortb200_argmax_workspace_bytes(int64_t rows);
 // y = act(x + bias[col]) elementwise; bias optional, cols = last dimension
 int ortb200_bias_act(const void* x, const void* bias, void* y, int64_t rows, int cols, int act, float alpha, int dtype,
                      ortb200_stream_t stream);
-// y = silu(gate) * up for x = [rows, 2 * cols] split in halves (gate | up)
+// y = act(gate) * up for x = [rows, 2 * cols] split in halves (gate | up): silu, or the tanh form of gelu (GEGLU)
 int ortb200_swiglu(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream);
+int ortb200_geglu(const void* x, void* y, int64_t rows, int cols, int dtype, ortb200_stream_t stream);
 // standalone rotary embedding on [B, S, N, H] (in -> out, may alias)
 int ortb200_rotary(const void* x, void* y, const int64_t* position_ids, int64_t position_offset, const void* cos_cache,
                    const void* sin_cache, int B, int S, int N, int H, int rot_dim, int interleaved, int bnsh, int dtype,
@@ -486,6 +499,147 @@ int ortb200_nbits_prepack(const void* B, void* out, int64_t bytes, ortb200_strea
 // block_size a power of two >= 16, ldo a multiple of 8.
 int ortb200_nbits_dequant(const void* B, const void* scales, const void* zero_points, int zp_is_packed, void* out,
                           int64_t N, int K, int bits, int block_size, int64_t ldo, int dtype, ortb200_stream_t stream);
+
+// ---------------------------------------------------------------------------
+// Packed-sequence mechanisms of hybrid decoders (recurrent layers, hyper-connections, gated attention).
+// Tokens of all sequences are packed along one axis: sequence b owns rows [cu_seqlens[b], cu_seqlens[b + 1]) and its
+// first row sits at position past_seqlens[b].  Recurrent state lives in pools of slots; sequence b uses slot slots[b].
+// A sequence whose past length is 0 starts from the zero state whatever its slot holds, so a slot needs no clearing when
+// it changes hands.  When T == B every sequence brings exactly one token and the one-launch decode kernels run.
+
+// Gated delta rule with one decay per key channel.  With x_t the inputs of the short convolution (columns of `qkvb`):
+//   (q, k, v) = silu(sum_j conv[:, taps - 1 - j] x_{t - j});  q, k unit vectors per head (q also times key_dim^-1/2)
+//   g = exp(-exp(A_log[h]) softplus(a + dt_bias)), beta = sigmoid(b)
+//   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   out = o / rms(o) * norm * sigmoid(gate)
+typedef struct {
+  const void* qkvb;        // [T, ld]: q (kv_heads * dk) | k (kv_heads * dk) | v (heads * dv) | b (heads) | padding
+  const void* low;         // [T, heads * (dk + dv)]: decay pre-activation a (heads * dk) | output gate (heads * dv)
+  const float* conv;       // [channels, taps], channels = 2 kv_heads dk + heads dv, newest token last
+  const float* a_log;      // [heads]
+  const float* dt_bias;    // [heads * dk]
+  const float* norm;       // [dv]
+  void* conv_state;        // [num_slots, taps, channels], dtype: ring of inputs, position p in entry p % taps
+  float* state;            // [num_slots, heads, dk, dv]
+  const int* cu_seqlens;   // [B + 1]
+  const int* past_seqlens; // [B]
+  const int* slots;        // [B]
+  void* out;               // [T, heads * dv]
+  float* workspace;        // T > B: ortb200_recurrent_workspace_bytes()
+  int64_t workspace_bytes;
+  int T, B, ld;
+  int heads, kv_heads, dk, dv, taps, num_slots;
+  float norm_eps, unit_eps;
+  int dtype;               // F16, BF16 or F32: qkvb, low, conv_state, out
+  int use_pdl;
+  int* status;
+} ortb200_gated_delta_args;
+int ortb200_gated_delta(const ortb200_gated_delta_args* args, ortb200_stream_t stream);
+
+// Matrix memory with exponential gating (mLSTM).  Log gates i = cap tanh((z_i + i_bias) / cap),
+// f = logsigmoid(cap tanh((z_f + f_bias) / cap)); q is scaled by key_dim^-1/2.  With m_0 = 0:
+//   m_t = max(f + m_{t-1}, i);  (S, n) <- exp(f + m_{t-1} - m_t) (S, n) + exp(i - m_t) (k v^T, k)
+//   o = S^T q / (max(|n . q|, exp(-m_t)) + den_eps);  out = o / rms(o) * norm * sigmoid(g)
+typedef struct {
+  const void* packed;      // [T, ld]: q (heads * dk) | k (heads * dk) | v (heads * dv) | g (heads * dv) | i (heads) | f (heads) | padding
+  const float* i_bias;     // [heads]
+  const float* f_bias;     // [heads]
+  const float* norm;       // [heads * dv]
+  float* state;            // [num_slots, heads, dk, dv]
+  float* aux;              // [num_slots, heads, dk + 1]: n, then m
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* slots;
+  void* out;               // [T, heads * dv]
+  float* workspace;
+  int64_t workspace_bytes;
+  int T, B, ld;
+  int heads, dk, dv, num_slots;
+  float gate_cap, norm_eps, den_eps;
+  int dtype;
+  int use_pdl;
+  int* status;
+} ortb200_mlstm_args;
+int ortb200_mlstm(const ortb200_mlstm_args* args, ortb200_stream_t stream);
+// Scratch of a multi-token call (0 when T == B).  Head sizes up to 256.
+int64_t ortb200_recurrent_workspace_bytes(int T, int B, int heads, int kv_heads, int dk, int dv);
+
+// Hyper-connections around a sublayer: write the previous sublayer's output back into `streams` residual copies, read the
+// next sublayer's input from them and normalise it, in one pass:
+//   x'_t = sum_s mix[s, t] x_s + w_out[t] y      (y == null: x' = x)
+//   u = sum_t w_in[t] x'_t;   out = u / sqrt(mean(u^2) + eps) * gamma
+typedef struct {
+  const void* x;           // [T, streams, width] fp32; with x_shared: [T, width] of `dtype`, every stream equals that row
+  const void* y;           // [T, width] dtype, or null
+  const float* mix;        // [streams, streams], [from, to]
+  const float* w_out;      // [streams]
+  const float* w_in;       // [streams]
+  const float* gamma;      // [width]
+  float* x_out;            // [T, streams, width] or null
+  void* out;               // [num_rows, width] dtype
+  const int64_t* rows;     // optional: tokens whose `out` row is wanted (x_out must then be null)
+  int T, num_rows, streams, width;
+  int x_shared;
+  float eps;
+  int dtype;
+  int use_pdl;
+  int* status;
+} ortb200_hyper_norm_args;
+int ortb200_hyper_norm(const ortb200_hyper_norm_args* args, ortb200_stream_t stream);
+
+// y = cap * tanh(x / cap), x of `dtype`, y fp32
+int ortb200_softcap(const void* x, float* y, int64_t n, float cap, int dtype, ortb200_stream_t stream);
+
+// Step 1 of the gated paged attention: per-head RMS norm of q and k (optional), rotary embedding on the first rot_dim
+// entries (rotate-half layout, fp32 tables), K / V appended to the paged cache, heads zero-padded to the cache's widths.
+typedef struct {
+  const void* packed;      // [T, ld]: q (N * dk) | k (Nk * dk) | v (Nk * dv) | ...; q only when kv_shared
+  void* q_out;             // [T, N, dk_pad] dtype
+  void* k_cache;           // [num_blocks, block_size, Nk, dk_pad]
+  void* v_cache;           // [num_blocks, block_size, Nk, dv_pad]
+  const float* q_norm;     // optional [dk]
+  const float* k_norm;     // optional [dk]
+  const float* cos_table;  // [rows, rot_dim / 2]
+  const float* sin_table;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* block_table;  // [B, max_blocks]
+  int T, B, ld, N, Nk, dk, dv, dk_pad, dv_pad;
+  int rot_dim, table_rows;
+  int block_size, max_blocks, num_blocks;
+  int kv_shared;
+  float eps;
+  int dtype;
+  int use_pdl;
+  int* status;
+} ortb200_qk_norm_rope_args;
+int ortb200_qk_norm_rope(const ortb200_qk_norm_rope_args* args, ortb200_stream_t stream);
+
+// Step 2 for any head sizes up to 256 and any of the three types: causal attention of packed queries over the paged cache
+// on CUDA cores, fp32 throughout, optional sink per head and sigmoid output gate.
+typedef struct {
+  const void* q;           // [T, N, dk_pad]
+  const void* k_cache;
+  const void* v_cache;
+  const float* sink;       // optional [N]
+  const void* gate;        // optional: row t at gate + t * gate_ld elements, N * dv entries
+  void* out;               // [T, N * dv]
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* block_table;
+  int64_t gate_ld;
+  int T, B, N, Nk, dk, dv, dk_pad, dv_pad;
+  int block_size, max_blocks, num_blocks;
+  int window;              // <= 0: none
+  float scale;
+  int dtype;
+  int use_pdl;
+} ortb200_paged_attn_args;
+int ortb200_paged_attn(const ortb200_paged_attn_args* args, ortb200_stream_t stream);
+
+// out[t, h * dv + j] = x[t, h, j] * sigmoid(gate[t, h * dv + j]) for x [T, heads, x_pad] (gate null: plain compaction)
+int ortb200_head_gate(const void* x, const void* gate, void* out, int T, int heads, int dv, int x_pad, int64_t gate_ld, int dtype,
+                      int use_pdl, ortb200_stream_t stream);
 
 #ifdef __cplusplus
 }

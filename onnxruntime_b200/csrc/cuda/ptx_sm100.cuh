@@ -340,6 +340,11 @@ __device__ __forceinline__ void tmem_st_x16_u32(uint32_t taddr, const uint32_t* 
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
+// tanh form of gelu, written as v * sigmoid(2 z): 0.5 (1 + tanh z) = 1 / (1 + exp(-2 z))
+__device__ __forceinline__ float gelu_tanh(float v) { return v / (1.0f + __expf(-1.5957691216057308f * v * (1.0f + 0.044715f * v * v))); }
+// gate activation of the gated (two-weight) epilogues: silu, or the tanh form of gelu
+__device__ __forceinline__ float gated_act(bool gelu, float v) { return gelu ? gelu_tanh(v) : v / (1.0f + __expf(-v)); }
+
 // Exact-form GELU, 0.5 x (1 + erf(x / sqrt 2)), with erf from the rational approximation 7.1.26 of Abramowitz &
 // Stegun (absolute error below 1.5e-7, far under the resolution of the 16-bit outputs it feeds): one reciprocal, one
 // exponential and a degree-5 polynomial, no branches - about a third of the instructions of the library erff.

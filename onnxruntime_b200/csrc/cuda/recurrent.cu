@@ -1,0 +1,845 @@
+// Recurrent token mixers over packed sequences: the gated delta rule with a decay per key channel, and the
+// exponentially gated matrix memory (mLSTM).  The state is fp32 everywhere, and the recurrence runs token by token in
+// fp32, so a result does not depend on how a prompt is cut.
+//
+// Several tokens per sequence (prompts): three launches.
+//   prep   one block per token: short convolution + silu, unit norms, decays, gates -> fp32 rows, heads padded
+//   scan   one block per (16 * warps state columns, head, sequence).  State columns are independent of each other, so
+//          the grid splits them; a warp holds a [dk, 16] slice of S in registers (8 row groups x 4 column groups of
+//          lanes), streams the token rows through double-buffered shared memory with cp.async, and does the decay, the
+//          two matrix-vector products and the rank-one update with packed fp32x2 instructions
+//   post   one block per token: norm over the value dimension, output gate, ring of convolution inputs
+// One token per sequence (decode): one launch, one block per (head, sequence) that does all of it; the state is read
+// once and written once, which is what bounds the step.
+//
+// Both products of a delta-rule step come from one pass over the old state: with S' = diag(g) S,
+// o = (S' + k u^T)^T q = S'^T q + (k . q) u.
+#include <cuda_runtime.h>
+#include <math.h>
+#include <type_traits>
+#include "launch_util.cuh"
+#include "ortb200_kernels.h"
+#include "ptx_sm100.cuh"
+
+namespace ortb200 {
+
+namespace {
+
+constexpr int kMaxHead = 256;     // key / value head sizes
+constexpr int kChunk = 16;        // tokens per shared-memory stage of the scan
+constexpr int kMaxTaps = 16;
+
+int pad_dk(int dk) { return dk <= 64 ? 64 : (dk <= 128 ? 128 : 256); }
+int pad4(int n) { return (n + 3) / 4 * 4; }
+
+// fp32 scratch of a multi-token call
+struct Scratch {
+  float* qk;      // [T, G, 2, dkp]: q row, then k row
+  float* decay;   // [T, H, dkp] (delta rule only)
+  float* v;       // [T, H, dvp]
+  float* scal;    // [T, H, 4]: delta: beta, q.k, -, -;  mLSTM: i, f, q.k, -
+  float* o;       // [T, H, dvp]
+  float* aux_out; // [B, H, dk + 1] (mLSTM only): n and m after the last token
+};
+
+int64_t scratch_floats(int T, int H, int G, int dkp, int dvp) {
+  return static_cast<int64_t>(T) * (static_cast<int64_t>(G) * 2 * dkp + static_cast<int64_t>(H) * (dkp + 2 * dvp + 4));
+}
+Scratch split_scratch(float* w, int T, int H, int G, int dkp, int dvp) {
+  Scratch s;
+  s.qk = w;
+  s.decay = s.qk + static_cast<int64_t>(T) * G * 2 * dkp;
+  s.v = s.decay + static_cast<int64_t>(T) * H * dkp;
+  s.scal = s.v + static_cast<int64_t>(T) * H * dvp;
+  s.o = s.scal + static_cast<int64_t>(T) * H * 4;
+  s.aux_out = s.o + static_cast<int64_t>(T) * H * dvp;
+  return s;
+}
+
+// ------------------------------------------------------------------------------------------------ delta rule pieces
+// Convolution + silu of one channel for the token in packed row t (position pos, `before` rows of its sequence in this
+// call); earlier inputs come from the packed rows, then from the ring, and are zero in front of the sequence.
+template <typename T>
+__device__ __forceinline__ float conv_silu(const ortb200_gated_delta_args& a, const T* ring, int channels, int ch, long long t, int pos,
+                                           int before) {
+  const T* x = static_cast<const T*>(a.qkvb) + t * a.ld + ch;
+  const float* w = a.conv + static_cast<long long>(ch) * a.taps;
+  float acc = 0.f;
+  for (int j = a.taps - 1; j >= 1; --j) {
+    float xv = 0.f;
+    if (j <= before) xv = to_float<T>(x[-static_cast<long long>(j) * a.ld]);
+    else if (pos - j >= 0) xv = to_float<T>(ring[static_cast<long long>((pos - j) % a.taps) * channels + ch]);
+    acc = fmaf(w[a.taps - 1 - j], xv, acc);
+  }
+  acc = fmaf(w[a.taps - 1], to_float<T>(x[0]), acc);
+  return acc * sigmoid_f(acc);
+}
+
+__device__ __forceinline__ bool slot_ok(int slot, int num_slots, int* status) {
+  if (slot >= 0 && slot < num_slots) return true;
+  if (status && threadIdx.x == 0) atomicExch(status, kStatusBadArgument);
+  return false;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const ortb200_gated_delta_args a, const Scratch s, int dkp, int dvp) {
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = a.heads, G = a.kv_heads, dk = a.dk, dv = a.dv;
+  const int channels = 2 * G * dk + H * dv;
+  pdl_wait_prior_grids();
+  const int b = sequence_of(a.cu_seqlens, a.B, t);
+  const int before = t - a.cu_seqlens[b];
+  const int pos = a.past_seqlens[b] + before;
+  const int slot = a.slots[b];
+  const bool ok = slot_ok(slot, a.num_slots, a.status);
+  const T* ring = static_cast<const T*>(a.conv_state) + static_cast<long long>(ok ? slot : 0) * a.taps * channels;
+  // units of work: G (q and k of a key head), H value heads, H decay heads
+  for (int u = warp; u < G + 2 * H; u += 8) {
+    if (u < G) {
+      float q[kMaxHead / 32], k[kMaxHead / 32];
+      float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int i = 0; i < kMaxHead / 32; ++i) {
+        const int d = i * 32 + lane;
+        q[i] = d < dk ? conv_silu<T>(a, ring, channels, u * dk + d, t, pos, before) : 0.f;
+        k[i] = d < dk ? conv_silu<T>(a, ring, channels, (G + u) * dk + d, t, pos, before) : 0.f;
+        qq = fmaf(q[i], q[i], qq);
+        kk = fmaf(k[i], k[i], kk);
+        qk = fmaf(q[i], k[i], qk);
+      }
+      qq = warp_sum(qq);
+      kk = warp_sum(kk);
+      qk = warp_sum(qk);
+      const float qs = 1.f / (sqrtf(qq + a.unit_eps) * sqrtf(static_cast<float>(dk)));
+      const float ks = 1.f / sqrtf(kk + a.unit_eps);
+      float* row = s.qk + (static_cast<long long>(t) * G + u) * 2 * dkp;
+#pragma unroll
+      for (int i = 0; i < kMaxHead / 32; ++i) {
+        const int d = i * 32 + lane;
+        if (d < dkp) {
+          row[d] = q[i] * qs;
+          row[dkp + d] = k[i] * ks;
+        }
+      }
+      const int group = H / G;
+      for (int j = lane; j < group; j += 32) s.scal[(static_cast<long long>(t) * H + u * group + j) * 4 + 1] = qk * qs * ks;
+    } else if (u < G + H) {
+      const int h = u - G;
+      float* row = s.v + (static_cast<long long>(t) * H + h) * dvp;
+      for (int d = lane; d < dvp; d += 32) row[d] = d < dv ? conv_silu<T>(a, ring, channels, 2 * G * dk + h * dv + d, t, pos, before) : 0.f;
+    } else {
+      const int h = u - G - H;
+      const T* low = static_cast<const T*>(a.low) + static_cast<long long>(t) * H * (dk + dv) + h * dk;
+      const float rate = expf(a.a_log[h]);
+      float* row = s.decay + (static_cast<long long>(t) * H + h) * dkp;
+      for (int d = lane; d < dkp; d += 32) row[d] = d < dk ? expf(-rate * softplus_f(to_float<T>(low[d]) + a.dt_bias[h * dk + d])) : 0.f;
+    }
+  }
+  const T* bp = static_cast<const T*>(a.qkvb) + static_cast<long long>(t) * a.ld + channels;
+  for (int h = threadIdx.x; h < H; h += blockDim.x) s.scal[(static_cast<long long>(t) * H + h) * 4] = sigmoid_f(to_float<T>(bp[h]));
+  pdl_launch_dependents();
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) mlstm_prep_kernel(const ortb200_mlstm_args a, const Scratch s, int dkp, int dvp) {
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = a.heads, dk = a.dk, dv = a.dv;
+  pdl_wait_prior_grids();
+  const T* row = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld;
+  const float qs = 1.f / sqrtf(static_cast<float>(dk));
+  for (int h = warp; h < H; h += 8) {
+    float* qk = s.qk + (static_cast<long long>(t) * H + h) * 2 * dkp;
+    float dot = 0.f;
+    for (int d = lane; d < dkp; d += 32) {
+      const float q = d < dk ? to_float<T>(row[h * dk + d]) * qs : 0.f;
+      const float k = d < dk ? to_float<T>(row[(H + h) * dk + d]) : 0.f;
+      qk[d] = q;
+      qk[dkp + d] = k;
+      dot = fmaf(q, k, dot);
+    }
+    dot = warp_sum(dot);
+    const T* v = row + 2 * H * dk + h * dv;
+    float* vr = s.v + (static_cast<long long>(t) * H + h) * dvp;
+    for (int d = lane; d < dvp; d += 32) vr[d] = d < dv ? to_float<T>(v[d]) : 0.f;
+    if (lane == 0) {
+      const T* gates = row + 2 * H * (dk + dv);
+      float* sc = s.scal + (static_cast<long long>(t) * H + h) * 4;
+      sc[0] = a.gate_cap * tanhf((to_float<T>(gates[h]) + a.i_bias[h]) / a.gate_cap);
+      sc[1] = logsigmoid_f(a.gate_cap * tanhf((to_float<T>(gates[H + h]) + a.f_bias[h]) / a.gate_cap));
+      sc[2] = dot;
+    }
+  }
+  pdl_launch_dependents();
+}
+
+// ---------------------------------------------------------------------------------------------------------- the scan
+struct ScanParams {
+  Scratch s;
+  float* state;            // [num_slots, H, dk, dv]
+  float* aux;              // mLSTM: [num_slots, H, dk + 1]
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* slots;
+  int H, G, dk, dv, dvp, num_slots;
+  float den_eps;
+  int* status;
+};
+
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// R = state rows per lane; dkp = 8 R.  Lane (rg = lane & 7, cg = lane >> 3) holds rows j * 32 + rg * 4 + {0..3},
+// j < R / 4, of columns col0 .. col0 + 3.
+template <bool DELTA, int R>
+__global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
+  constexpr int DKP = 8 * R, NJ = R / 4;
+  constexpr int kRows = DELTA ? 3 : 2;             // q, k (, decay)
+  const int warps = blockDim.x >> 5;
+  const int cs = warps * 16;                       // columns per block
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7, cg = lane >> 3;
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int g = h / (p.H / p.G);
+  const int base_col = blockIdx.x * cs;
+  const int wcol = warp * 16 + cg * 4;             // column within the block's slice
+  const int col0 = base_col + wcol;
+  extern __shared__ __align__(16) float sm[];
+  const int stage_floats = kChunk * (kRows * DKP + cs + 4);
+
+  pdl_wait_prior_grids();
+  const int t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len <= 0) return;
+  const int slot = p.slots[b];
+  if (!slot_ok(slot, p.num_slots, p.status)) return;
+  const bool fresh = p.past_seqlens[b] == 0;
+
+  auto fetch = [&](int chunk) {
+    float* st = sm + (chunk & 1) * stage_floats;
+    const int first = chunk * kChunk, n = min(kChunk, len - first);
+    for (int i = threadIdx.x; i < n * (2 * DKP / 4); i += blockDim.x) {
+      const int tt = i / (2 * DKP / 4), c = i % (2 * DKP / 4);
+      cp_async16(st + tt * kRows * DKP + c * 4, p.s.qk + ((static_cast<long long>(t0 + first + tt) * p.G + g) * 2 * DKP) + c * 4);
+    }
+    if (DELTA) {
+      for (int i = threadIdx.x; i < n * (DKP / 4); i += blockDim.x) {
+        const int tt = i / (DKP / 4), c = i % (DKP / 4);
+        cp_async16(st + tt * kRows * DKP + 2 * DKP + c * 4, p.s.decay + (static_cast<long long>(t0 + first + tt) * p.H + h) * DKP + c * 4);
+      }
+    }
+    float* sv = st + kChunk * kRows * DKP;
+    const int vq = cs / 4;
+    for (int i = threadIdx.x; i < n * vq; i += blockDim.x) {
+      const int tt = i / vq, c = i % vq;
+      if (base_col + c * 4 < p.dvp) cp_async16(sv + tt * cs + c * 4, p.s.v + (static_cast<long long>(t0 + first + tt) * p.H + h) * p.dvp + base_col + c * 4);
+    }
+    float* sc = sv + kChunk * cs;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) cp_async16(sc + i * 4, p.s.scal + (static_cast<long long>(t0 + first + i) * p.H + h) * 4);
+    cp_async_commit();
+  };
+
+  float* gst = p.state + (static_cast<long long>(slot) * p.H + h) * p.dk * p.dv;
+  f32x2 S[NJ][4][2];
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int r = j * 32 + rg * 4 + hh * 2;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float lo = 0.f, hi = 0.f;
+        if (!fresh && col0 + c < p.dv) {
+          if (r < p.dk) lo = gst[static_cast<long long>(r) * p.dv + col0 + c];
+          if (r + 1 < p.dk) hi = gst[static_cast<long long>(r + 1) * p.dv + col0 + c];
+        }
+        S[j][c][hh] = pack2(lo, hi);
+      }
+    }
+  }
+  float* gaux = DELTA ? nullptr : p.aux + (static_cast<long long>(slot) * p.H + h) * (p.dk + 1);
+  f32x2 nrm[DELTA ? 1 : NJ][2];
+  float m = 0.f;
+  if (!DELTA) {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const int r = j * 32 + rg * 4 + hh * 2;
+        nrm[DELTA ? 0 : j][hh] = pack2(!fresh && r < p.dk ? gaux[r] : 0.f, !fresh && r + 1 < p.dk ? gaux[r + 1] : 0.f);
+      }
+    }
+    m = fresh ? 0.f : gaux[p.dk];
+  }
+
+  const int chunks = (len + kChunk - 1) / kChunk;
+  fetch(0);
+  for (int ch = 0; ch < chunks; ++ch) {
+    if (ch + 1 < chunks) {
+      fetch(ch + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const float* st = sm + (ch & 1) * stage_floats;
+    const float* sv = st + kChunk * kRows * DKP;
+    const float* sc = sv + kChunk * cs;
+    const int n = min(kChunk, len - ch * kChunk);
+    for (int tt = 0; tt < n; ++tt) {
+      const float* qr = st + tt * kRows * DKP;
+      const float* kr = qr + DKP;
+      const float4 vv = *reinterpret_cast<const float4*>(sv + tt * cs + wcol);
+      const float4 scal = *reinterpret_cast<const float4*>(sc + tt * 4);
+      float* orow = p.s.o + (static_cast<long long>(t0 + ch * kChunk + tt) * p.H + h) * p.dvp;
+      if (DELTA) {
+        const float* gr = kr + DKP;
+        f32x2 accA[4], accO[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) { accA[c] = 0ull; accO[c] = 0ull; }
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
+          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
+          const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(gr + j * 32 + rg * 4);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            S[j][c][0] = mul2(S[j][c][0], g2.x);
+            S[j][c][1] = mul2(S[j][c][1], g2.y);
+            accA[c] = fma2(S[j][c][0], k2.x, accA[c]);
+            accO[c] = fma2(S[j][c][0], q2.x, accO[c]);
+            accA[c] = fma2(S[j][c][1], k2.y, accA[c]);
+            accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
+          }
+        }
+        // eight sums (S^T k and S^T q of four columns) over the eight row-group lanes: reduce-scatter, lane rg ends with
+        // sum number rg (0..3: S^T k of column rg, 4..7: S^T q of column rg - 4)
+        float x[8];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          float lo, hi;
+          unpack2(accA[c], lo, hi);
+          x[c] = lo + hi;
+          unpack2(accO[c], lo, hi);
+          x[4 + c] = lo + hi;
+        }
+        float y[4], z[2], w;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float send = (rg & 4) ? x[i] : x[4 + i], keep = (rg & 4) ? x[4 + i] : x[i];
+          y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float send = (rg & 2) ? y[i] : y[2 + i], keep = (rg & 2) ? y[2 + i] : y[i];
+          z[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+        }
+        {
+          const float send = (rg & 1) ? z[0] : z[1], keep = (rg & 1) ? z[1] : z[0];
+          w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+        }
+        const float a0 = __shfl_sync(0xffffffffu, w, (lane & 24) | 0), a1 = __shfl_sync(0xffffffffu, w, (lane & 24) | 1);
+        const float a2 = __shfl_sync(0xffffffffu, w, (lane & 24) | 2), a3 = __shfl_sync(0xffffffffu, w, (lane & 24) | 3);
+        const float u0 = scal.x * (vv.x - a0), u1 = scal.x * (vv.y - a1), u2 = scal.x * (vv.z - a2), u3 = scal.x * (vv.w - a3);
+        const f32x2 uu[4] = {pack2(u0, u0), pack2(u1, u1), pack2(u2, u2), pack2(u3, u3)};
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            S[j][c][0] = fma2(k2.x, uu[c], S[j][c][0]);
+            S[j][c][1] = fma2(k2.y, uu[c], S[j][c][1]);
+          }
+        }
+        if (rg >= 4) {
+          const int c = rg - 4;
+          const float u = c == 0 ? u0 : (c == 1 ? u1 : (c == 2 ? u2 : u3));
+          if (col0 + c < p.dv) orow[col0 + c] = fmaf(scal.y, u, w);
+        }
+      } else {
+        const float m_new = fmaxf(scal.y + m, scal.x);
+        const float fw = expf(scal.y + m - m_new), iw = expf(scal.x - m_new);
+        m = m_new;
+        const f32x2 f2 = pack2(fw, fw), i2 = pack2(iw, iw);
+        const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
+        f32x2 accO[4], accN = 0ull;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) accO[c] = 0ull;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
+          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
+          const f32x2 ik0 = mul2(k2.x, i2), ik1 = mul2(k2.y, i2);
+          nrm[DELTA ? 0 : j][0] = fma2(nrm[DELTA ? 0 : j][0], f2, ik0);
+          nrm[DELTA ? 0 : j][1] = fma2(nrm[DELTA ? 0 : j][1], f2, ik1);
+          accN = fma2(nrm[DELTA ? 0 : j][0], q2.x, accN);
+          accN = fma2(nrm[DELTA ? 0 : j][1], q2.y, accN);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            S[j][c][0] = fma2(ik0, v2[c], mul2(S[j][c][0], f2));
+            S[j][c][1] = fma2(ik1, v2[c], mul2(S[j][c][1], f2));
+            accO[c] = fma2(S[j][c][0], q2.x, accO[c]);
+            accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
+          }
+        }
+        float x[4], lo, hi;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          unpack2(accO[c], lo, hi);
+          x[c] = lo + hi;
+        }
+        unpack2(accN, lo, hi);
+        float nq = lo + hi;
+#pragma unroll
+        for (int off = 1; off <= 4; off <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, off);
+        float y[2], w;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float send = (rg & 2) ? x[i] : x[2 + i], keep = (rg & 2) ? x[2 + i] : x[i];
+          y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+        }
+        {
+          const float send = (rg & 1) ? y[0] : y[1], keep = (rg & 1) ? y[1] : y[0];
+          w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+        }
+        w += __shfl_xor_sync(0xffffffffu, w, 4);
+        if (rg < 4 && col0 + rg < p.dv) orow[col0 + rg] = w / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
+      }
+    }
+    __syncthreads();   // the stage may be refilled
+  }
+  pdl_launch_dependents();
+
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int r = j * 32 + rg * 4 + hh * 2;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        if (col0 + c >= p.dv) continue;
+        float lo, hi;
+        unpack2(S[j][c][hh], lo, hi);
+        if (r < p.dk) gst[static_cast<long long>(r) * p.dv + col0 + c] = lo;
+        if (r + 1 < p.dk) gst[static_cast<long long>(r + 1) * p.dv + col0 + c] = hi;
+      }
+    }
+  }
+  // n and m: every block of a (head, sequence) computes the same values, and another block may still have to read the
+  // old ones, so they leave through scratch and the post kernel moves them into the state
+  if (!DELTA && blockIdx.x == 0 && warp == 0 && cg == 0) {
+    float* ao = p.s.aux_out + (static_cast<long long>(b) * p.H + h) * (p.dk + 1);
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const int r = j * 32 + rg * 4 + hh * 2;
+        float lo, hi;
+        unpack2(nrm[DELTA ? 0 : j][hh], lo, hi);
+        if (r < p.dk) ao[r] = lo;
+        if (r + 1 < p.dk) ao[r + 1] = hi;
+      }
+    }
+    if (rg == 0) ao[p.dk] = m;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------- post
+struct PostParams {
+  const float* o;          // [T, H, dvp]
+  const float* norm;       // [dv] (norm_stride 0) or [H * dv] (norm_stride dv)
+  const void* gate;        // row t at gate + t * gate_ld elements, H * dv entries
+  void* out;               // [T, H * dv]
+  long long gate_ld;
+  int H, dv, dvp, norm_stride;
+  float eps;
+  // convolution inputs of the last `taps` tokens -> ring
+  const void* conv_in;
+  void* conv_state;
+  int conv_ld, channels, taps;
+  // n and m of the sequence -> state
+  const float* aux_out;
+  float* aux;
+  int dk;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* slots;
+  int B, num_slots;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) recurrent_post_kernel(const PostParams p) {
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_wait_prior_grids();
+  for (int h = warp; h < p.H; h += 8) {
+    const float* o = p.o + (static_cast<long long>(t) * p.H + h) * p.dvp;
+    float x[kMaxHead / 32], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxHead / 32; ++i) {
+      const int d = i * 32 + lane;
+      x[i] = d < p.dv ? o[d] : 0.f;
+      ss = fmaf(x[i], x[i], ss);
+    }
+    ss = warp_sum(ss);
+    const float r = 1.f / sqrtf(ss / p.dv + p.eps);
+    const T* gate = static_cast<const T*>(p.gate) + t * p.gate_ld + h * p.dv;
+    T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.H + h) * p.dv;
+#pragma unroll
+    for (int i = 0; i < kMaxHead / 32; ++i) {
+      const int d = i * 32 + lane;
+      if (d < p.dv) out[d] = from_float<T>(x[i] * r * p.norm[h * p.norm_stride + d] * sigmoid_f(to_float<T>(gate[d])));
+    }
+  }
+  const int b = sequence_of(p.cu_seqlens, p.B, t);
+  const int end = p.cu_seqlens[b + 1];
+  const int slot = p.slots[b];
+  if (slot >= 0 && slot < p.num_slots) {
+    if (p.conv_state && t >= end - p.taps) {
+      const int pos = p.past_seqlens[b] + t - p.cu_seqlens[b];
+      const T* src = static_cast<const T*>(p.conv_in) + static_cast<long long>(t) * p.conv_ld;
+      T* dst = static_cast<T*>(p.conv_state) + (static_cast<long long>(slot) * p.taps + pos % p.taps) * p.channels;
+      for (int c = threadIdx.x; c < p.channels; c += blockDim.x) dst[c] = src[c];
+    }
+    if (p.aux && t == end - 1) {
+      const long long n = static_cast<long long>(p.H) * (p.dk + 1);
+      for (int i = threadIdx.x; i < n; i += blockDim.x) p.aux[slot * n + i] = p.aux_out[b * n + i];
+    }
+  }
+  pdl_launch_dependents();
+}
+
+// ----------------------------------------------------------------------------------------------------------- decode
+// One block per (head, sequence), one token.  Lane l of warp w holds rows w, w + 8, ... of four columns; RPW rows.
+template <typename T, typename A, int RPW>
+__global__ void __launch_bounds__(256) recurrent_decode_kernel(const A a) {
+  constexpr bool DELTA = std::is_same<A, ortb200_gated_delta_args>::value;
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = a.heads, dk = a.dk, dv = a.dv;
+  __shared__ float sq[kMaxHead], sk[kMaxHead], sg[kMaxHead], sv[kMaxHead], so[kMaxHead];
+  __shared__ float redA[8][128], redO[8][128], su[128];
+  __shared__ float red[8], scal[4];
+  pdl_wait_prior_grids();
+  const int slot = a.slots[b];
+  if (!slot_ok(slot, a.num_slots, a.status)) return;
+  const int pos = a.past_seqlens[b];
+  const bool fresh = pos == 0;
+  float* gst = a.state + (static_cast<long long>(slot) * H + h) * dk * dv;
+  const bool vec = (dv & 3) == 0;
+
+  float4 S[RPW];
+  auto load_state = [&](int c0) {
+    const int col = c0 + lane * 4;
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      const int r = warp + 8 * i;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!fresh && r < dk && col < dv) {
+        const float* src = gst + static_cast<long long>(r) * dv + col;
+        if (vec) {
+          v = __ldcs(reinterpret_cast<const float4*>(src));
+        } else {
+          v.x = src[0];
+          if (col + 1 < dv) v.y = src[1];
+          if (col + 2 < dv) v.z = src[2];
+          if (col + 3 < dv) v.w = src[3];
+        }
+      }
+      S[i] = v;
+    }
+  };
+  load_state(0);   // in flight while the inputs are prepared
+
+  if constexpr (DELTA) {
+    const int G = a.kv_heads, g = h / (H / G);
+    const int channels = 2 * G * dk + H * dv;
+    T* ring = static_cast<T*>(a.conv_state) + static_cast<long long>(slot) * a.taps * channels;
+    T* ring_new = ring + static_cast<long long>(pos % a.taps) * channels;
+    const T* x = static_cast<const T*>(a.qkvb) + static_cast<long long>(b) * a.ld;
+    const T* low = static_cast<const T*>(a.low) + static_cast<long long>(b) * H * (dk + dv) + h * dk;
+    const bool first_of_group = h % (H / G) == 0;
+    float qq = 0.f, kk = 0.f, qk = 0.f;
+    if (tid < dk) {
+      const int cq = g * dk + tid, ck = (G + g) * dk + tid;
+      const float q = conv_silu<T>(a, ring, channels, cq, b, pos, 0), k = conv_silu<T>(a, ring, channels, ck, b, pos, 0);
+      sq[tid] = q;
+      sk[tid] = k;
+      qq = q * q;
+      kk = k * k;
+      qk = q * k;
+      sg[tid] = expf(-expf(a.a_log[h]) * softplus_f(to_float<T>(low[tid]) + a.dt_bias[h * dk + tid]));
+      if (first_of_group) {   // the ring entry of this position is read by nobody in this step
+        ring_new[cq] = x[cq];
+        ring_new[ck] = x[ck];
+      }
+    }
+    if (tid < dv) {
+      const int cv = 2 * G * dk + h * dv + tid;
+      sv[tid] = conv_silu<T>(a, ring, channels, cv, b, pos, 0);
+      ring_new[cv] = x[cv];
+    }
+    qq = block_sum_all(qq, red);
+    kk = block_sum_all(kk, red);
+    qk = block_sum_all(qk, red);
+    const float qs = 1.f / (sqrtf(qq + a.unit_eps) * sqrtf(static_cast<float>(dk))), ks = 1.f / sqrtf(kk + a.unit_eps);
+    if (tid < dk) {
+      sq[tid] *= qs;
+      sk[tid] *= ks;
+    }
+    if (tid == 0) {
+      scal[0] = sigmoid_f(to_float<T>(x[channels + h]));
+      scal[1] = qk * qs * ks;
+    }
+  } else {
+    const T* x = static_cast<const T*>(a.packed) + static_cast<long long>(b) * a.ld;
+    float* aux = a.aux + (static_cast<long long>(slot) * H + h) * (dk + 1);
+    const T* gates = x + 2 * H * (dk + dv);
+    const float iv = a.gate_cap * tanhf((to_float<T>(gates[h]) + a.i_bias[h]) / a.gate_cap);
+    const float fv = logsigmoid_f(a.gate_cap * tanhf((to_float<T>(gates[H + h]) + a.f_bias[h]) / a.gate_cap));
+    const float m_old = fresh ? 0.f : aux[dk];
+    const float m = fmaxf(fv + m_old, iv);
+    const float fw = expf(fv + m_old - m), iw = expf(iv - m);
+    float nq = 0.f;
+    __syncthreads();   // every thread has read m before thread 0 replaces it
+    if (tid < dk) {
+      const float q = to_float<T>(x[h * dk + tid]) / sqrtf(static_cast<float>(dk));
+      const float k = to_float<T>(x[(H + h) * dk + tid]) * iw;
+      const float n = fmaf(fresh ? 0.f : aux[tid], fw, k);
+      aux[tid] = n;
+      sq[tid] = q;
+      sk[tid] = k;
+      nq = n * q;
+    }
+    if (tid < dv) sv[tid] = to_float<T>(x[2 * H * dk + h * dv + tid]);
+    nq = block_sum_all(nq, red);
+    if (tid == 0) {
+      aux[dk] = m;
+      scal[0] = fw;
+      scal[1] = 1.f / (fmaxf(fabsf(nq), expf(-m)) + a.den_eps);
+    }
+  }
+  __syncthreads();
+
+  for (int c0 = 0; c0 < dv; c0 += 128) {
+    if (c0 > 0) load_state(c0);
+    const int col = c0 + lane * 4;
+    float4 pa = make_float4(0.f, 0.f, 0.f, 0.f), po = pa;
+    float4 v4 = pa;
+    if (!DELTA) {
+      if (col < dv) v4.x = sv[col];
+      if (col + 1 < dv) v4.y = sv[col + 1];
+      if (col + 2 < dv) v4.z = sv[col + 2];
+      if (col + 3 < dv) v4.w = sv[col + 3];
+    }
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      const int r = warp + 8 * i;
+      if (r >= dk) break;
+      const float q = sq[r], k = sk[r];
+      if (DELTA) {
+        const float gr = sg[r];
+        S[i].x *= gr; S[i].y *= gr; S[i].z *= gr; S[i].w *= gr;
+        pa.x = fmaf(S[i].x, k, pa.x); pa.y = fmaf(S[i].y, k, pa.y); pa.z = fmaf(S[i].z, k, pa.z); pa.w = fmaf(S[i].w, k, pa.w);
+      } else {
+        const float f = scal[0];
+        S[i].x = fmaf(k, v4.x, S[i].x * f); S[i].y = fmaf(k, v4.y, S[i].y * f);
+        S[i].z = fmaf(k, v4.z, S[i].z * f); S[i].w = fmaf(k, v4.w, S[i].w * f);
+      }
+      po.x = fmaf(S[i].x, q, po.x); po.y = fmaf(S[i].y, q, po.y); po.z = fmaf(S[i].z, q, po.z); po.w = fmaf(S[i].w, q, po.w);
+    }
+    if (DELTA) *reinterpret_cast<float4*>(&redA[warp][lane * 4]) = pa;
+    *reinterpret_cast<float4*>(&redO[warp][lane * 4]) = po;
+    __syncthreads();
+    if (tid < 128) {
+      float o = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) o += redO[w][tid];
+      const bool in = c0 + tid < dv;
+      if (DELTA) {
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) s += redA[w][tid];
+        const float u = in ? scal[0] * (sv[c0 + tid] - s) : 0.f;
+        su[tid] = u;
+        if (in) so[c0 + tid] = fmaf(scal[1], u, o);
+      } else if (in) {
+        so[c0 + tid] = o * scal[1];
+      }
+    }
+    __syncthreads();
+    float4 u4 = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (DELTA) u4 = *reinterpret_cast<const float4*>(&su[lane * 4]);
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      const int r = warp + 8 * i;
+      if (r >= dk || col >= dv) break;
+      float4 v = S[i];
+      if (DELTA) {
+        const float k = sk[r];
+        v.x = fmaf(k, u4.x, v.x); v.y = fmaf(k, u4.y, v.y); v.z = fmaf(k, u4.z, v.z); v.w = fmaf(k, u4.w, v.w);
+      }
+      float* dst = gst + static_cast<long long>(r) * dv + col;
+      if (vec) {
+        __stcs(reinterpret_cast<float4*>(dst), v);
+      } else {
+        dst[0] = v.x;
+        if (col + 1 < dv) dst[1] = v.y;
+        if (col + 2 < dv) dst[2] = v.z;
+        if (col + 3 < dv) dst[3] = v.w;
+      }
+    }
+    // redA / redO / su are rewritten by the next column pass only after its first barrier
+    if (c0 + 128 < dv) __syncthreads();
+  }
+  pdl_launch_dependents();
+
+  const float o = tid < dv ? so[tid] : 0.f;
+  const float r = 1.f / sqrtf(block_sum_all(o * o, red) / dv + a.norm_eps);
+  if (tid < dv) {
+    float gate, w;
+    if constexpr (DELTA) {
+      gate = to_float<T>(static_cast<const T*>(a.low)[static_cast<long long>(b) * H * (dk + dv) + H * dk + h * dv + tid]);
+      w = a.norm[tid];
+    } else {
+      gate = to_float<T>(static_cast<const T*>(a.packed)[static_cast<long long>(b) * a.ld + H * (2 * dk + dv) + h * dv + tid]);
+      w = a.norm[h * dv + tid];
+    }
+    static_cast<T*>(a.out)[(static_cast<long long>(b) * H + h) * dv + tid] = from_float<T>(o * r * w * sigmoid_f(gate));
+  }
+}
+
+template <typename T, typename A>
+int launch_decode(const A& a, cudaStream_t stream) {
+  const dim3 grid(a.heads, a.B);
+  const bool pdl = a.use_pdl != 0;
+  if (a.dk <= 64) return launch_kernel(recurrent_decode_kernel<T, A, 8>, grid, 256, 0, stream, pdl, a);
+  if (a.dk <= 128) return launch_kernel(recurrent_decode_kernel<T, A, 16>, grid, 256, 0, stream, pdl, a);
+  return launch_kernel(recurrent_decode_kernel<T, A, 32>, grid, 256, 0, stream, pdl, a);
+}
+
+template <bool DELTA, int R>
+int launch_scan_r(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl) {
+  constexpr int DKP = 8 * R;
+  // columns per block: a quarter of the value head per warp, fewer when the grid would not fill the machine
+  int warps = (p.dv + 15) / 16;
+  if (warps > 4) warps = 4;
+  while (warps > 1 && static_cast<long long>(B) * p.H * ((p.dv + warps * 16 - 1) / (warps * 16)) < 148) warps /= 2;
+  const int cs = warps * 16;
+  const int smem = 2 * kChunk * ((DELTA ? 3 : 2) * DKP + cs + 4) * 4;
+  auto kern = scan_kernel<DELTA, R>;
+  static int attr_smem = 0;
+  if (smem > 48 * 1024 && smem > attr_smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
+    attr_smem = smem;
+  }
+  const dim3 grid((p.dv + cs - 1) / cs, p.H, B);
+  return launch_kernel(kern, grid, warps * 32, smem, stream, pdl, p);
+}
+
+template <bool DELTA>
+int launch_scan(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl) {
+  switch (pad_dk(p.dk)) {
+    case 64: return launch_scan_r<DELTA, 8>(p, B, T, stream, pdl);
+    case 128: return launch_scan_r<DELTA, 16>(p, B, T, stream, pdl);
+    default: return launch_scan_r<DELTA, 32>(p, B, T, stream, pdl);
+  }
+}
+
+template <typename T>
+int run_delta(const ortb200_gated_delta_args& a, cudaStream_t stream) {
+  if (a.T == a.B) return launch_decode<T, ortb200_gated_delta_args>(a, stream);
+  const bool pdl = a.use_pdl != 0;
+  const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
+  const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.kv_heads, dkp, dvp);
+  int rc = launch_kernel(delta_prep_kernel<T>, dim3(a.T), 256, 0, stream, pdl, a, s, dkp, dvp);
+  if (rc) return rc;
+  ScanParams p{s, a.state, nullptr, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.kv_heads, a.dk, a.dv, dvp, a.num_slots, 0.f, a.status};
+  rc = launch_scan<true>(p, a.B, a.T, stream, pdl);
+  if (rc) return rc;
+  PostParams q{};
+  q.o = s.o; q.norm = a.norm; q.norm_stride = 0;
+  q.gate = static_cast<const T*>(a.low) + static_cast<int64_t>(a.heads) * a.dk;
+  q.gate_ld = static_cast<long long>(a.heads) * (a.dk + a.dv);
+  q.out = a.out; q.H = a.heads; q.dv = a.dv; q.dvp = dvp; q.eps = a.norm_eps;
+  q.conv_in = a.qkvb; q.conv_state = a.conv_state; q.conv_ld = a.ld;
+  q.channels = 2 * a.kv_heads * a.dk + a.heads * a.dv; q.taps = a.taps;
+  q.cu_seqlens = a.cu_seqlens; q.past_seqlens = a.past_seqlens; q.slots = a.slots; q.B = a.B; q.num_slots = a.num_slots;
+  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T), 256, 0, stream, pdl, q);
+}
+
+template <typename T>
+int run_mlstm(const ortb200_mlstm_args& a, cudaStream_t stream) {
+  if (a.T == a.B) return launch_decode<T, ortb200_mlstm_args>(a, stream);
+  const bool pdl = a.use_pdl != 0;
+  const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
+  const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.heads, dkp, dvp);
+  int rc = launch_kernel(mlstm_prep_kernel<T>, dim3(a.T), 256, 0, stream, pdl, a, s, dkp, dvp);
+  if (rc) return rc;
+  ScanParams p{s, a.state, a.aux, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.heads, a.dk, a.dv, dvp, a.num_slots, a.den_eps, a.status};
+  rc = launch_scan<false>(p, a.B, a.T, stream, pdl);
+  if (rc) return rc;
+  PostParams q{};
+  q.o = s.o; q.norm = a.norm; q.norm_stride = a.dv;
+  q.gate = static_cast<const T*>(a.packed) + static_cast<int64_t>(a.heads) * (2 * a.dk + a.dv);
+  q.gate_ld = a.ld;
+  q.out = a.out; q.H = a.heads; q.dv = a.dv; q.dvp = dvp; q.eps = a.norm_eps;
+  q.aux_out = s.aux_out; q.aux = a.aux; q.dk = a.dk;
+  q.cu_seqlens = a.cu_seqlens; q.past_seqlens = a.past_seqlens; q.slots = a.slots; q.B = a.B; q.num_slots = a.num_slots;
+  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T), 256, 0, stream, pdl, q);
+}
+
+bool sizes_ok(int T, int B, int heads, int dk, int dv, int num_slots) {
+  return T > 0 && B > 0 && B <= T && heads > 0 && dk > 0 && dk <= kMaxHead && dv > 0 && dv <= kMaxHead && num_slots > 0 && B <= 65535 &&
+         heads <= 65535;
+}
+
+}  // namespace
+
+}  // namespace ortb200
+
+using namespace ortb200;
+
+extern "C" int64_t ortb200_recurrent_workspace_bytes(int T, int B, int heads, int kv_heads, int dk, int dv) {
+  if (T == B) return 0;
+  return 4 * (scratch_floats(T, heads, kv_heads, pad_dk(dk), pad4(dv)) + static_cast<int64_t>(B) * heads * (dk + 1));
+}
+
+extern "C" int ortb200_gated_delta(const ortb200_gated_delta_args* a, ortb200_stream_t stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (!a || !a->qkvb || !a->low || !a->conv || !a->a_log || !a->dt_bias || !a->norm || !a->conv_state || !a->state || !a->cu_seqlens ||
+      !a->past_seqlens || !a->slots || !a->out)
+    return -1;
+  if (!sizes_ok(a->T, a->B, a->heads, a->dk, a->dv, a->num_slots) || a->kv_heads <= 0 || a->heads % a->kv_heads != 0) return -2;
+  if (a->taps < 1 || a->taps > kMaxTaps || a->ld < 2 * a->kv_heads * a->dk + a->heads * (a->dv + 1)) return -2;
+  if (a->T != a->B && (!a->workspace || a->workspace_bytes < ortb200_recurrent_workspace_bytes(a->T, a->B, a->heads, a->kv_heads, a->dk, a->dv)))
+    return -5;
+  if ((reinterpret_cast<uintptr_t>(a->workspace) | reinterpret_cast<uintptr_t>(a->state)) & 15) return -3;
+  switch (a->dtype) {
+    case ORTB200_F16: return run_delta<__half>(*a, stream);
+    case ORTB200_BF16: return run_delta<__nv_bfloat16>(*a, stream);
+    case ORTB200_F32: return run_delta<float>(*a, stream);
+    default: return -4;
+  }
+}
+
+extern "C" int ortb200_mlstm(const ortb200_mlstm_args* a, ortb200_stream_t stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (!a || !a->packed || !a->i_bias || !a->f_bias || !a->norm || !a->state || !a->aux || !a->cu_seqlens || !a->past_seqlens || !a->slots ||
+      !a->out)
+    return -1;
+  if (!sizes_ok(a->T, a->B, a->heads, a->dk, a->dv, a->num_slots) || a->gate_cap <= 0.f) return -2;
+  if (a->ld < a->heads * (2 * a->dk + 2 * a->dv + 2)) return -2;
+  if (a->T != a->B && (!a->workspace || a->workspace_bytes < ortb200_recurrent_workspace_bytes(a->T, a->B, a->heads, a->heads, a->dk, a->dv)))
+    return -5;
+  if ((reinterpret_cast<uintptr_t>(a->workspace) | reinterpret_cast<uintptr_t>(a->state)) & 15) return -3;
+  switch (a->dtype) {
+    case ORTB200_F16: return run_mlstm<__half>(*a, stream);
+    case ORTB200_BF16: return run_mlstm<__nv_bfloat16>(*a, stream);
+    case ORTB200_F32: return run_mlstm<float>(*a, stream);
+    default: return -4;
+  }
+}

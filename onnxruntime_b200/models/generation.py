@@ -10,12 +10,13 @@ session captures it on the first step and replays it afterwards.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, Hashable, List, Optional, Sequence, Tuple, Union
 
 import torch
 
 from ..capi import InferenceSession, RunOptions
-from .llama import LlamaConfig, empty_kv_cache, empty_paged_cache
+from .decoder_cache import CacheFull, CachePool
+from .llama import LlamaConfig, empty_kv_cache
 
 
 class DecoderRunner:
@@ -145,94 +146,231 @@ class DecoderRunner:
 
 
 class PagedDecoderRunner:
-    """Greedy decoding over a block (paged) KV cache: the serving form of the decoder, where all sequences share
-    one pool of cache blocks and ``block_table[b, j]`` names the block that holds tokens [j * block_size,
-    (j + 1) * block_size) of sequence b (the inputs of com.microsoft.PagedAttention,
-    onnxruntime/contrib_ops/cuda/bert/paged_attention.cc).  Blocks are handed out round-robin over the sequences,
-    so no sequence owns a contiguous range and every access goes through the table.  The decode step has fixed
-    shapes and addresses and is captured as one CUDA graph."""
+    """Decoding over pooled caches: the serving form of a decoder.  Tokens of all sequences of a step are packed along
+    one axis; all sequences share one pool of cache blocks (``block_table[b, j]`` names the block that holds tokens
+    [j * block_size, (j + 1) * block_size) of sequence b, as in com.microsoft.PagedAttention,
+    onnxruntime/contrib_ops/cuda/bert/paged_attention.cc) and one pool of state slots for models with recurrent layers
+    (``state_slots[b]``).  What a model keeps is declared by ``cfg.cache_tensors()``.
 
-    def __init__(self, session: InferenceSession, cfg: LlamaConfig, batch: int, max_len: int, block_size: int = 256,
-                 tp_size: int = 1, device: Optional[torch.device] = None, graph_id: int = 1):
+    ``step`` runs one batch of any composition - whole prompts, portions of prompts, single tokens - for sequences named
+    by the caller and returns the wanted logits; ``release`` gives a sequence's blocks and slot back.  ``prefill`` /
+    ``decode_step`` drive a fixed batch of ``batch`` rows on top of the same pool.  A step that brings one token per
+    sequence has fixed shapes and addresses and is captured as one CUDA graph per batch size."""
+
+    def __init__(self, session: InferenceSession, cfg, batch: int, max_len: int, block_size: int = 256,
+                 tp_size: int = 1, device: Optional[torch.device] = None, graph_id: int = 1, num_blocks: Optional[int] = None,
+                 num_slots: Optional[int] = None):
+        """``num_blocks``: size of the block pool (default: ``batch`` sequences of ``max_len`` tokens); ``max_len`` bounds
+        one sequence; ``num_slots`` (default ``batch``) bounds the sequences that are open at a time."""
         self.sess, self.cfg, self.batch, self.max_len, self.block_size = session, cfg, batch, max_len, block_size
         self.device = device if device is not None else (
             torch.device("cuda", torch.cuda.current_device()) if "CUDAExecutionProvider" in session.get_providers() else torch.device("cpu"))
-        per_seq = (max_len + block_size - 1) // block_size
-        self.cache = empty_paged_cache(cfg, batch * per_seq, block_size, self.device, tp_size)
-        self.block_table = torch.arange(batch * per_seq, dtype=torch.int32).view(per_seq, batch).t().contiguous().to(self.device)
-        dt = self.cache[0][0].dtype
-        self.step_ids = torch.zeros(batch, dtype=torch.int64, device=self.device)
-        self.step_cum = torch.arange(batch + 1, dtype=torch.int32, device=self.device)
-        self.step_past = torch.zeros(batch, dtype=torch.int32, device=self.device)
-        self.step_rows = torch.arange(batch, dtype=torch.int64, device=self.device)
-        self.step_logits = torch.zeros(batch, cfg.vocab_size, dtype=dt, device=self.device)
-        self.step_next = torch.zeros(batch, dtype=torch.int64, device=self.device)
-        self.has_argmax = "next_tokens" in [o.name for o in session.get_outputs()]
-        self._decode_binding = None
-        self._ro_decode = RunOptions()
-        self._ro_decode.add_run_config_entry("gpu_graph_id", str(graph_id))  # one captured graph per (session, shape)
+        self.blocks_per_seq = (max_len + block_size - 1) // block_size
+        self.pool = CachePool(cfg.cache_tensors(tp_size), num_blocks or batch * self.blocks_per_seq, block_size, num_slots or batch, self.device)
+        out_info = {o.name: o for o in session.get_outputs()}
+        in_names = {i.name for i in session.get_inputs()}
+        self.has_argmax = "next_tokens" in out_info
+        self.has_slots = "state_slots" in in_names
+        self.logits_dtype = {"tensor(float)": torch.float32, "tensor(float16)": torch.float16,
+                             "tensor(bfloat16)": torch.bfloat16}[out_info["logits"].type]
+        self._steps: Dict[int, "_DecodeBuffers"] = {}
+        self._graph_id = graph_id             # graph ids graph_id, graph_id + 1, ...: one captured graph per batch size
         self._ro_prefill = RunOptions()
         self._ro_prefill.add_run_config_entry("gpu_graph_id", "-1")
-        self.cur_len = 0
+        self._rows: List[Tuple[str, int]] = [("row", b) for b in range(batch)]   # sequences of prefill / decode_step
+        self.prefill_logits = self.step_logits = None
 
-    def _bind(self, binding, ids, cum, past, rows, logits, nxt) -> None:
+    @property
+    def cur_len(self) -> int:
+        """Tokens held by the longest row of the fixed batch."""
+        return max((self.pool.sequences[r].length for r in self._rows if r in self.pool.sequences), default=0)
+
+    @cur_len.setter
+    def cur_len(self, length: int) -> None:
+        self.assume_context(length)
+
+    @property
+    def block_table(self) -> torch.Tensor:
+        """Block table of the fixed batch."""
+        return self._table(self._rows).to(self.device)
+
+    def _table(self, seqs) -> torch.Tensor:
+        t = torch.zeros(len(seqs), self.blocks_per_seq, dtype=torch.int32)
+        for b, s in enumerate(seqs):
+            blocks = self.pool.sequences[s].blocks
+            t[b, :len(blocks)] = torch.tensor(blocks, dtype=torch.int32)
+        return t
+
+    def _slots(self, seqs) -> torch.Tensor:
+        return torch.tensor([self.pool.sequences[s].slot for s in seqs], dtype=torch.int32)
+
+    def _bind(self, binding, ids, cum, past, table, slots, rows, logits, nxt) -> None:
         binding.bind_torch_input("input_ids", ids)
         binding.bind_torch_input("cumulative_sequence_length", cum)
         binding.bind_torch_input("past_seqlens", past)
-        binding.bind_torch_input("block_table", self.block_table)
+        binding.bind_torch_input("block_table", table)
         binding.bind_torch_input("logits_indices", rows)
-        for i, (k, v) in enumerate(self.cache):
-            binding.bind_torch_input(f"key_cache.{i}", k)
-            binding.bind_torch_input(f"value_cache.{i}", v)
-            binding.bind_torch_output(f"key_cache_out.{i}", k)
-            binding.bind_torch_output(f"value_cache_out.{i}", v)
+        if self.has_slots:
+            binding.bind_torch_input("state_slots", slots)
+        for c in self.pool.spec:
+            binding.bind_torch_input(c.input, self.pool.tensors[c.input])
+            binding.bind_torch_output(c.output, self.pool.tensors[c.input])
         binding.bind_torch_output("logits", logits)
         if self.has_argmax:
             binding.bind_torch_output("next_tokens", nxt)
 
-    def prefill(self, input_ids: torch.Tensor) -> torch.Tensor:
-        """Prompts [B, S] of equal length, packed to [B * S] tokens; returns the first generated token [B]."""
-        B, S = input_ids.shape
-        assert B == self.batch and S <= self.max_len
-        ids = input_ids.reshape(-1).to(self.device)
-        cum = (torch.arange(B + 1, dtype=torch.int32) * S).to(self.device)
-        past = torch.zeros(B, dtype=torch.int32, device=self.device)
-        rows = (torch.arange(1, B + 1, dtype=torch.int64) * S - 1).to(self.device)
-        logits = torch.empty(B, self.cfg.vocab_size, dtype=self.step_logits.dtype, device=self.device)
-        nxt = torch.empty(B, dtype=torch.int64, device=self.device)
+    # ------------------------------------------------------------------------------------------------- general steps
+    def step(self, entries: Sequence[Tuple[Hashable, Sequence[int], Sequence[int]]]) -> torch.Tensor:
+        """One batch: ``entries`` = (sequence, its next tokens, places among them whose logits are wanted).  A sequence
+        seen for the first time is opened.  Returns the logits [wanted, vocab] in the order of the entries."""
+        entries = [e for e in entries if len(e[1]) > 0]
+        opened = []
+        try:
+            for seq, tokens, want in entries:
+                if any(not 0 <= w < len(tokens) for w in want):
+                    raise ValueError(f"sequence {seq!r}: a wanted place lies outside its {len(tokens)} tokens")
+                if seq not in self.pool.sequences:
+                    self.pool.open(seq)
+                    opened.append(seq)
+                if self.pool.sequences[seq].length + len(tokens) > self.max_len:
+                    raise CacheFull(f"sequence {seq!r} would exceed {self.max_len} tokens")
+                self.pool.reserve(seq, len(tokens))
+        except Exception:
+            for seq in opened:
+                self.pool.close(seq)
+            raise
+        if not entries:
+            return torch.empty(0, self.cfg.vocab_size, dtype=self.logits_dtype, device=self.device)
+        seqs = [e[0] for e in entries]
+        if all(len(e[1]) == 1 for e in entries):
+            buf = self._decode_buffers(len(entries))
+            buf.ids.copy_(torch.tensor([int(e[1][0]) for e in entries], dtype=torch.int64))
+            self._run_decode(buf, seqs)
+            wanted = [b for b, e in enumerate(entries) for _ in e[2]]
+            return buf.logits[torch.tensor(wanted, dtype=torch.int64, device=self.device)]
+        ids = torch.cat([torch.as_tensor(e[1], dtype=torch.int64).reshape(-1).cpu() for e in entries])
+        starts, rows = [0], []
+        for _, tokens, want in entries:
+            rows += [starts[-1] + int(w) for w in want]
+            starts.append(starts[-1] + len(tokens))
+        logits, _ = self._run_packed(ids, starts, seqs, rows or [0])
+        return logits if rows else logits[:0]
+
+    def release(self, seq: Hashable) -> None:
+        """The sequence is finished: its blocks and slot go back to the pool."""
+        self.pool.close(seq)
+
+    def _run_packed(self, ids: torch.Tensor, starts, seqs, rows) -> Tuple[torch.Tensor, torch.Tensor]:
+        dev = self.device
+        past = torch.tensor([self.pool.sequences[s].length for s in seqs], dtype=torch.int32)
+        logits = torch.empty(len(rows), self.cfg.vocab_size, dtype=self.logits_dtype, device=dev)
+        nxt = torch.empty(len(rows), dtype=torch.int64, device=dev)
         binding = self.sess.io_binding()
-        self._bind(binding, ids, cum, past, rows, logits, nxt)
+        self._bind(binding, ids.to(dev), torch.tensor(starts, dtype=torch.int32).to(dev), past.to(dev), self._table(seqs).to(dev),
+                   self._slots(seqs).to(dev), torch.tensor(rows, dtype=torch.int64).to(dev), logits, nxt)
         self.sess.run_with_iobinding(binding, self._ro_prefill)
-        self.cur_len = S
+        for b, s in enumerate(seqs):
+            self.pool.advance(s, starts[b + 1] - starts[b])
         if not self.has_argmax:
             nxt = logits.float().argmax(-1)
+        return logits, nxt
+
+    def _decode_buffers(self, rows: int) -> "_DecodeBuffers":
+        if rows not in self._steps:
+            buf = _DecodeBuffers(rows, self.blocks_per_seq, self.cfg.vocab_size, self.logits_dtype, self.device)
+            buf.binding = self.sess.io_binding()
+            self._bind(buf.binding, buf.ids, buf.cum, buf.past, buf.table, buf.slots, buf.rows, buf.logits, buf.next)
+            buf.options.add_run_config_entry("gpu_graph_id", str(self._graph_id + len(self._steps)))
+            self._steps[rows] = buf
+        return self._steps[rows]
+
+    def _run_decode(self, buf: "_DecodeBuffers", seqs) -> None:
+        """One token per sequence, ids already in ``buf.ids``; room has been reserved."""
+        layout = [(s, self.pool.sequences[s].slot, tuple(self.pool.sequences[s].blocks)) for s in seqs]
+        if layout != buf.layout:
+            buf.table.copy_(self._table(seqs))
+            buf.slots.copy_(self._slots(seqs))
+            buf.layout = layout
+        lengths = [self.pool.sequences[s].length for s in seqs]
+        if lengths.count(lengths[0]) == len(lengths):
+            buf.past.fill_(lengths[0])
+        else:
+            buf.past.copy_(torch.tensor(lengths, dtype=torch.int32))
+        self.sess.run_with_iobinding(buf.binding, buf.options)
+        for s in seqs:
+            self.pool.advance(s, 1)
+        if not self.has_argmax:
+            buf.next.copy_(buf.logits.float().argmax(-1))
+
+    # ------------------------------------------------------------------------------------------- the fixed batch of rows
+    def _reopen_rows(self) -> None:
+        for r in self._rows:
+            if r in self.pool.sequences:
+                self.pool.close(r)
+        for r in self._rows:
+            self.pool.open(r)
+        # full capacity at once, one block per row in turn: the block table of a row is fixed from here on, and no row owns
+        # a contiguous range
+        for j in range(self.blocks_per_seq):
+            for r in self._rows:
+                self.pool.reserve(r, min((j + 1) * self.block_size, self.max_len))
+
+    def prefill(self, input_ids) -> torch.Tensor:
+        """Prompts of the fixed batch: a tensor [B, S] or a list of B prompts of any lengths, packed without padding.
+        Returns the first generated token of every row [B]."""
+        prompts = [torch.as_tensor(p, dtype=torch.int64).reshape(-1) for p in input_ids]
+        assert len(prompts) == self.batch and all(1 <= len(p) <= self.max_len for p in prompts)
+        self._reopen_rows()
+        starts = [0]
+        for p in prompts:
+            starts.append(starts[-1] + len(p))
+        self.prefill_logits, nxt = self._run_packed(torch.cat(prompts), starts, self._rows, [s - 1 for s in starts[1:]])
+        self._decode_buffers(self.batch).next.copy_(nxt)
         return nxt
 
     def assume_context(self, length: int) -> None:
         """Treat the caches as holding ``length`` tokens per sequence (benchmarks that time decode over a cache
         filled with arbitrary values instead of running a prompt first)."""
         assert 0 <= length < self.max_len
-        self.cur_len = length
+        if any(r not in self.pool.sequences for r in self._rows):
+            self._reopen_rows()
+        for r in self._rows:
+            self.pool.sequences[r].length = length
 
     def decode_step(self, tokens: Optional[torch.Tensor] = None) -> torch.Tensor:
         """One token per sequence; ``tokens`` [B] or None to feed back the previous step's output."""
-        if self._decode_binding is None:
-            self._decode_binding = self.sess.io_binding()
-            self._bind(self._decode_binding, self.step_ids, self.step_cum, self.step_past, self.step_rows, self.step_logits,
-                       self.step_next)
-        self.step_ids.copy_(tokens.reshape(-1) if tokens is not None else self.step_next, non_blocking=True)
-        self.step_past.fill_(self.cur_len)
-        self.sess.run_with_iobinding(self._decode_binding, self._ro_decode)
-        self.cur_len += 1
-        if not self.has_argmax:
-            self.step_next.copy_(self.step_logits.float().argmax(-1))
-        return self.step_next
+        buf = self._decode_buffers(self.batch)
+        buf.ids.copy_(tokens.reshape(-1) if tokens is not None else buf.next, non_blocking=True)
+        self._run_decode(buf, self._rows)
+        self.step_logits = buf.logits
+        return buf.next
 
-    def generate(self, input_ids: torch.Tensor, max_new_tokens: int) -> torch.Tensor:
+    def reorder_cache(self, rows: torch.Tensor) -> None:
+        """Row i takes the content of row rows[i] (beam search: beams follow their parents)."""
+        self.pool.copy_sequence_state([self._rows[int(r)] for r in rows.tolist()], self._rows)
+
+    def generate(self, input_ids, max_new_tokens: int) -> torch.Tensor:
         out = [self.prefill(input_ids).clone()]
         for _ in range(max_new_tokens - 1):
             out.append(self.decode_step(out[-1]).clone())
         return torch.stack(out, dim=1)
+
+
+class _DecodeBuffers:
+    """Device buffers of the one-token step of one batch size; their addresses are frozen into its CUDA graph."""
+
+    def __init__(self, rows: int, max_blocks: int, vocab: int, logits_dtype: torch.dtype, device: torch.device):
+        self.ids = torch.zeros(rows, dtype=torch.int64, device=device)
+        self.cum = torch.arange(rows + 1, dtype=torch.int32, device=device)
+        self.past = torch.zeros(rows, dtype=torch.int32, device=device)
+        self.table = torch.zeros(rows, max_blocks, dtype=torch.int32, device=device)
+        self.slots = torch.zeros(rows, dtype=torch.int32, device=device)
+        self.rows = torch.arange(rows, dtype=torch.int64, device=device)
+        self.logits = torch.zeros(rows, vocab, dtype=logits_dtype, device=device)
+        self.next = torch.zeros(rows, dtype=torch.int64, device=device)
+        self.layout = None
+        self.binding = None
+        self.options = RunOptions()
 
 
 # ----------------------------------------------------------------------------------------------------------------
@@ -293,7 +431,7 @@ def top_k_top_p_filter(logits: torch.Tensor, top_k: int, top_p: float) -> torch.
     return logits
 
 
-def generate(runner: DecoderRunner, input_ids: torch.Tensor, cfg: GenerationConfig) -> torch.Tensor:
+def generate(runner: Union[DecoderRunner, PagedDecoderRunner], input_ids: torch.Tensor, cfg: GenerationConfig) -> torch.Tensor:
     """Greedy (``num_beams == 1``, ``top_k == 0``, ``top_p == 1``, temperature 1), sampling or beam search.
     Returns [batch * num_return_sequences, prompt + generated] token ids, padded with ``pad_token_id`` after EOS.
     For beam search the runner must have been created with ``batch = prompts * num_beams``."""
@@ -325,6 +463,60 @@ def generate(runner: DecoderRunner, input_ids: torch.Tensor, cfg: GenerationConf
             runner.decode_step(nxt.view(-1, 1))
             logits = _last_logits(runner, prefill=False)
     return seqs
+
+
+def generate_requests(runner: PagedDecoderRunner, prompts: Sequence[Sequence[int]], cfg: GenerationConfig) -> List[List[int]]:
+    """Greedy or sampled continuations of prompts of any lengths, with the processors and knobs of ``generate``.  At most
+    ``runner.batch`` requests run at a time; a finished one frees its blocks and slot, and the next waiting prompt joins
+    the running batch in a step of its own.  Returns the generated tokens of every request (end token included)."""
+    if cfg.num_beams > 1:
+        raise ValueError("beam search needs a fixed batch: use generate()")
+    sampling = cfg.top_k > 0 or cfg.top_p < 1.0 or cfg.seed is not None
+    gen = torch.Generator(device=runner.device)
+    if cfg.seed is not None:
+        gen.manual_seed(cfg.seed)
+    texts = [[int(t) for t in p] for p in prompts]
+    done: List[Optional[List[int]]] = [None] * len(texts)
+    new: Dict[int, List[int]] = {}
+    waiting, running = list(range(len(texts))), []
+
+    def pick(i: int, logits: torch.Tensor) -> None:
+        seq = torch.tensor([texts[i] + new[i]], dtype=torch.int64, device=runner.device)
+        scores = process_logits(logits.reshape(1, -1), seq, len(new[i]), cfg)
+        if sampling:
+            tok = int(torch.multinomial(torch.softmax(top_k_top_p_filter(scores, cfg.top_k, cfg.top_p), -1), 1, generator=gen))
+        else:
+            tok = int(scores.argmax(-1))
+        new[i].append(tok)
+        if len(new[i]) >= cfg.max_new_tokens or tok == cfg.eos_token_id:
+            done[i] = new.pop(i)
+            running.remove(i)
+            runner.release(("request", i))
+
+    while waiting or running:
+        joining = waiting[:runner.batch - len(running)]
+        while joining:   # prompts that fit into the free blocks together with the tokens they will generate
+            room = len(runner.pool.free_blocks)
+            need = [(len(texts[i]) + cfg.max_new_tokens + runner.block_size - 1) // runner.block_size for i in joining]
+            held = sum(max(0, (len(texts[i]) + cfg.max_new_tokens + runner.block_size - 1) // runner.block_size
+                           - len(runner.pool.sequences[("request", i)].blocks)) for i in running)
+            if sum(need) + held <= room:
+                break
+            joining.pop()
+        if joining:
+            logits = runner.step([(("request", i), texts[i], [len(texts[i]) - 1]) for i in joining])
+            waiting = waiting[len(joining):]
+            running += joining
+            for i in joining:
+                new[i] = []
+        elif running:
+            joining = list(running)
+            logits = runner.step([(("request", i), [new[i][-1]], [0]) for i in joining])
+        else:
+            raise CacheFull(f"request {waiting[0]} does not fit into the cache")
+        for row, i in enumerate(joining):
+            pick(i, logits[row])
+    return done
 
 
 def _last_logits(runner: DecoderRunner, prefill: bool) -> torch.Tensor:

@@ -18,12 +18,13 @@ from __future__ import annotations
 import math
 import zlib
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Tuple
+from typing import Any, Dict, List, Mapping, Optional, Tuple
 
 import numpy as np
 import torch
 
 from .. import onnx_lite as ol
+from .decoder_cache import CacheTensor
 
 T = ol.TensorProto
 
@@ -59,6 +60,23 @@ class LlamaConfig:
         base.update(kw)
         return LlamaConfig(**base)
 
+    @staticmethod
+    def from_json(d: Mapping[str, Any], dtype: str = "bf16", max_seq_len: int = 2048) -> "LlamaConfig":
+        """From the keys of a Llama checkpoint's config.json."""
+        if d.get("rope_scaling"):
+            raise ValueError("rope_scaling is not supported by this graph")
+        heads, hidden = int(d["num_attention_heads"]), int(d["hidden_size"])
+        return LlamaConfig(vocab_size=int(d["vocab_size"]), hidden_size=hidden, num_layers=int(d["num_hidden_layers"]), num_heads=heads,
+                           num_kv_heads=int(d.get("num_key_value_heads", heads)), head_dim=int(d.get("head_dim") or hidden // heads),
+                           ffn_size=int(d["intermediate_size"]), rope_theta=float(d.get("rope_theta", 10000.0)), max_seq_len=max_seq_len,
+                           rms_eps=float(d.get("rms_norm_eps", 1e-5)), dtype=dtype)
+
+    def cache_tensors(self, tp_size: int = 1) -> List[CacheTensor]:
+        """Cache of the paged graph: one key and one value pool per layer."""
+        shape = (self.num_kv_heads // tp_size, self.head_dim)
+        return [CacheTensor(f"{kv}_cache.{i}", f"{kv}_cache_out.{i}", "paged", shape, _TORCH_DT[self.dtype])
+                for i in range(self.num_layers) for kv in ("key", "value")]
+
 
 _TORCH_DT = {"bf16": torch.bfloat16, "fp16": torch.float16, "fp32": torch.float32}
 _ONNX_DT = {"bf16": T.BFLOAT16, "fp16": T.FLOAT16, "fp32": T.FLOAT}
@@ -77,8 +95,9 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
                 device: str = "cpu", with_argmax: bool = True, last_token_logits: bool = True,
                 weight_std: float = 0.02, shard_lm_head: bool = True, quant_bits: int = 0,
                 quant_block: int = 32, paged: bool = False, moe_experts: int = 0, moe_top_k: int = 2, ep_rank: int = 0,
-                ep_size: int = 1) -> Tuple[bytes, Dict[str, torch.Tensor]]:
-    """Returns (ModelProto bytes, weights).  With ``external_weights`` the dict holds every weight (on
+                ep_size: int = 1, state: Optional[Mapping[str, torch.Tensor]] = None) -> Tuple[bytes, Dict[str, torch.Tensor]]:
+    """Returns (ModelProto bytes, weights).  ``state`` holds a checkpoint's tensors under their usual names
+    (``model.layers.0.self_attn.q_proj.weight`` [out, in], ...); without it the weights are random.  With ``external_weights`` the dict holds every weight (on
     ``device``) to pass to ``SessionOptions.add_external_initializers``; otherwise it is empty and the
     weights are embedded in the model.
 
@@ -100,6 +119,7 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
     holding experts ``[ep_rank * E / ep_size, (ep_rank + 1) * E / ep_size)`` when ``ep_size > 1`` (expert parallelism:
     attention and router weights are replicated, every rank sees all tokens, as the operator's contract has it,
     onnxruntime/contrib_ops/cuda/collective/sharded_moe.cc:54-189)."""
+    assert state is None or not (moe_experts or quant_bits), "checkpoints are loaded into the dense form"
     assert not (moe_experts and (tp_size > 1 or quant_bits)), "the mixture-of-experts form is dense and expert-parallel only"
     assert moe_experts % max(ep_size, 1) == 0
     if paged:
@@ -117,17 +137,30 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
     def randn(name: str, shape, std: float = weight_std, shard: Optional[Tuple[int, int]] = None) -> str:
         """Full-size tensor from a per-name seed, then the rank's shard (so ranks agree on the full model)."""
         gen.manual_seed(seed * 1000003 + zlib.crc32(name.encode()))
-        full = tuple(shape)
+        full = list(shape)
         if shard is not None:
             axis, parts = shard
-            full = list(shape)
             full[axis] *= parts
-        w = (torch.randn(full, generator=gen, device=device, dtype=torch.float32) * std).to(dt)
+        if state is not None:
+            w = checkpoint(name.replace(".attn.", ".self_attn."), full)
+        else:
+            w = (torch.randn(full, generator=gen, device=device, dtype=torch.float32) * std).to(dt)
         if shard is not None:
             axis, parts = shard
             w = w.chunk(parts, dim=axis)[tp_rank].contiguous()
         add_weight(name, w)
         return name
+
+    def checkpoint(name: str, shape) -> torch.Tensor:
+        """A matrix of the checkpoint as this graph stores it: [in, out], the embedding as it is."""
+        if name == "lm_head.weight" and name not in state:
+            name = "model.embed_tokens.weight"   # tied head
+            w = state[name].t()
+        else:
+            w = state[name] if name == "model.embed_tokens.weight" else state[name].t()
+        if list(w.shape) != list(shape):
+            raise ValueError(f"tensor {name!r} has shape {tuple(state[name].shape)}, which does not fit the configuration")
+        return w.to(device=device, dtype=dt).contiguous()
 
     def add_weight(name: str, w: torch.Tensor) -> None:
         if external_weights:
@@ -173,7 +206,7 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
                                   domain="com.microsoft", K=k, N=n, bits=quant_bits, block_size=quant_block))
 
     def ones(name: str, n: int) -> str:
-        add_weight(name, torch.ones(n, dtype=dt, device=device))
+        add_weight(name, torch.ones(n, dtype=dt, device=device) if state is None else state[name].to(device=device, dtype=dt).contiguous())
         return name
 
     cos, sin = rope_caches(cfg, device)
@@ -213,8 +246,12 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
             residual = f"{p}.res1"
         # packed QKV projection: column-parallel, columns ordered [q heads | k heads | v heads] of this rank
         gen.manual_seed(seed * 1000003 + zlib.crc32(f"{p}.qkv".encode()))
-        full = (torch.randn((hidden, (cfg.num_heads + 2 * cfg.num_kv_heads) * H), generator=gen, device=device,
-                            dtype=torch.float32) * weight_std).to(dt)
+        if state is not None:
+            full = torch.cat([checkpoint(f"{p}.self_attn.{n}_proj.weight", (hidden, h * H))
+                              for n, h in (("q", cfg.num_heads), ("k", cfg.num_kv_heads), ("v", cfg.num_kv_heads))], dim=1)
+        else:
+            full = (torch.randn((hidden, (cfg.num_heads + 2 * cfg.num_kv_heads) * H), generator=gen, device=device,
+                                dtype=torch.float32) * weight_std).to(dt)
         q_full, k_full, v_full = full.split([cfg.num_heads * H, cfg.num_kv_heads * H, cfg.num_kv_heads * H], dim=1)
         wqkv = torch.cat([q_full.chunk(tp_size, 1)[tp_rank], k_full.chunk(tp_size, 1)[tp_rank],
                           v_full.chunk(tp_size, 1)[tp_rank]], dim=1).contiguous()

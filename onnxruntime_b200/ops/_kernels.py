@@ -16,7 +16,7 @@ import torch
 _LIB: Optional[ctypes.CDLL] = None
 
 F16, BF16, F32 = 0, 1, 2
-ACT = {"none": 0, "gelu": 1, "fastgelu": 2, "relu": 3, "silu": 4, "swiglu": 5, "quickgelu": 6}
+ACT = {"none": 0, "gelu": 1, "fastgelu": 2, "relu": 3, "silu": 4, "swiglu": 5, "quickgelu": 6, "geglu": 7}
 
 
 def lib_path() -> str:
@@ -294,7 +294,10 @@ class AttnPrefillArgs(ctypes.Structure):
                 ("N", ctypes.c_int), ("Nk", ctypes.c_int), ("H", ctypes.c_int), ("kv_len", ctypes.c_int),
                 ("q_strides", ctypes.c_int64 * 3), ("o_strides", ctypes.c_int64 * 3), ("kv_strides", ctypes.c_int64 * 3),
                 ("first_prompt", ctypes.c_int), ("causal", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
-                ("softcap", ctypes.c_float), ("dtype", ctypes.c_int), ("status", ctypes.c_void_p), ("key_mask", ctypes.c_void_p)]
+                ("softcap", ctypes.c_float), ("dtype", ctypes.c_int), ("status", ctypes.c_void_p), ("key_mask", ctypes.c_void_p),
+                ("block_table", ctypes.c_void_p), ("cu_seqlens", ctypes.c_void_p), ("past_seqlens", ctypes.c_void_p),
+                ("T", ctypes.c_int), ("block_size", ctypes.c_int), ("max_blocks", ctypes.c_int), ("num_blocks", ctypes.c_int),
+                ("split_weights", ctypes.c_int)]
 
 
 def attn_prefill(q, k, v, seqlens_k=None, first_prompt=True, causal=True, window=-1, scale=0.0, softcap=0.0,
