@@ -140,8 +140,9 @@ class MatMulNBitsKernel final : public WithFallback {
 };
 
 // ---------------------------------------------------------------------------------------------------------------
-// PagedAttention, decode form (one new token per sequence): rotary + cache write, then the split-KV kernel reading
-// the cache through the block table.  Other forms (prompt chunks) take the generic path.
+// PagedAttention.  One new token per sequence: rotary + cache write, then the split-KV kernel reading the cache through
+// the block table.  Prompts and portions of prompts: rotary + cache write, then the tcgen05 flash kernel over packed
+// queries (cache blocks of a multiple of 128 tokens; other block sizes take the generic path).
 class PagedAttentionKernel final : public WithFallback {
  public:
   explicit PagedAttentionKernel(const OpKernelInfo& info) : WithFallback(info) {
@@ -166,7 +167,7 @@ class PagedAttentionKernel final : public WithFallback {
     const bool packed = !ctx.HasInput(1);
     const int dt = DtypeCode(query.scalar_type());
     const bool decode = T == B;
-    if (dt < 0 || !decode || (H != 64 && H != 128) || kc.scalar_type() != query.scalar_type() || !kc.is_contiguous() ||
+    if (dt < 0 || T == 0 || (!decode && block_size % 128 != 0) || (H != 64 && H != 128) || kc.scalar_type() != query.scalar_type() || !kc.is_contiguous() ||
         !vc.is_contiguous() || !cum.is_cuda() || !past.is_cuda() || !table.is_cuda() || cum.scalar_type() != at::kInt ||
         past.scalar_type() != at::kInt || table.scalar_type() != at::kInt ||
         (do_rotary_ && (!ctx.HasInput(8) || ctx.Input(8).scalar_type() != query.scalar_type()))) {
@@ -177,7 +178,7 @@ class PagedAttentionKernel final : public WithFallback {
     at::Tensor q_rot = at::empty({T, N_, H}, query.options());
     at::Tensor tb = table.contiguous();
     // head size 128: the tcgen05 decode kernel rotates, appends and attends in one launch
-    const bool fuse = packed && H == 128 && window_ <= 0 && (block_size & (block_size - 1)) == 0 && block_size >= 8 &&
+    const bool fuse = decode && packed && H == 128 && window_ <= 0 && (block_size & (block_size - 1)) == 0 && block_size >= 8 &&
                       (!do_rotary_ || ctx.Input(8).size(1) * 2 == H) && ctx.session()->config().Get("ortb200.fused_gqa_prep", "auto") != "0" &&
                       ctx.session()->config().Get("ortb200.decode_attention_algo", "0") != "1";
     ortb200_paged_prep_args pa{};
@@ -209,6 +210,32 @@ class PagedAttentionKernel final : public WithFallback {
     if (!fuse) CheckLaunch(ortb200_paged_prep(&pa, ctx.cuda_stream()), "ortb200_paged_prep");
 
     at::Tensor out = at::empty({T, N_ * H}, query.options());
+    if (!decode) {
+      ortb200_attn_prefill_args fa{};
+      fa.q = q_rot.data_ptr();
+      fa.k = kc.data_ptr();
+      fa.v = vc.data_ptr();
+      fa.out = out.data_ptr();
+      fa.B = pa.B; fa.N = pa.N; fa.Nk = pa.Nk; fa.H = pa.H;
+      fa.q_strides[1] = fa.o_strides[1] = N_ * H;
+      fa.q_strides[2] = fa.o_strides[2] = H;
+      fa.causal = 1;
+      fa.window = static_cast<int>(window_);
+      fa.scale = scale_;
+      fa.softcap = softcap_;
+      fa.dtype = dt;
+      fa.status = pa.status;
+      fa.block_table = pa.block_table;
+      fa.cu_seqlens = pa.cu_seqlens;
+      fa.past_seqlens = pa.past_seqlens;
+      fa.T = pa.T; fa.block_size = pa.block_size; fa.max_blocks = pa.max_blocks; fa.num_blocks = pa.num_blocks;
+      CheckLaunch(ortb200_attn_prefill(&fa, ctx.cuda_stream()), "ortb200_attn_prefill(paged)");
+      ctx.session()->AddLaunches(2);
+      ctx.SetOutput(0, out);
+      if (ctx.OutputCount() > 1) ctx.SetOutput(1, kc);
+      if (ctx.OutputCount() > 2) ctx.SetOutput(2, vc);
+      return;
+    }
     at::Tensor& ws = ctx.session()->AttnWorkspace(ortb200_gqa_decode_workspace_bytes(static_cast<int>(B), static_cast<int>(N_), static_cast<int>(H)));
     ortb200_gqa_decode_args da{};
     da.q = q_rot.data_ptr();

@@ -165,6 +165,11 @@ def rotary_tables(rot: Mapping[str, Any], rows: int, device="cpu") -> Tuple[torc
     return angles.cos().float().to(device), angles.sin().float().to(device)
 
 
+def default_rank(cfg: FegilixConfig) -> int:
+    """Rank of the low-rank maps for random weights: the key head size of the first delta-rule layer."""
+    return next((layer["mixer"]["dim"] for layer in cfg.layers if layer["type"] == "channel_delta"), 16)
+
+
 def random_weights(cfg: FegilixConfig, seed: int = 0, device="cpu", low_rank: int = 16, dtype: torch.dtype = torch.bfloat16,
                    gain: float = 1.0) -> Dict[str, torch.Tensor]:
     """Random tensors of the checkpoint's shapes, scaled so that activations and gates stay in a useful range."""

@@ -190,6 +190,12 @@ class PagedDecoderRunner:
         self.assume_context(length)
 
     @property
+    def cache(self) -> List[Tuple[torch.Tensor, torch.Tensor]]:
+        """(key, value) block pools of the attention layers that own them."""
+        paged = [self.pool.tensors[c.input] for c in self.pool.spec if c.kind == "paged"]
+        return list(zip(paged[::2], paged[1::2]))
+
+    @property
     def block_table(self) -> torch.Tensor:
         """Block table of the fixed batch."""
         return self._table(self._rows).to(self.device)

@@ -18,9 +18,9 @@ from .generation import PagedDecoderRunner
 @dataclass(frozen=True)
 class DecoderFamily:
     """``config(json, dtype, max_seq_len)`` parses config.json; ``build(config, tensors, device)`` returns the packed serving
-    graph and its initializers.  The config object declares what the model keeps per sequence (``cache_tensors()``)."""
+    graph and its initializers; ``tensors`` None means random weights.  The config object declares what the model keeps per sequence (``cache_tensors()``)."""
     config: Callable[[Mapping[str, Any], str, int], Any]
-    build: Callable[[Any, Mapping[str, torch.Tensor], str], Tuple[bytes, Dict[str, torch.Tensor]]]
+    build: Callable[[Any, Optional[Mapping[str, torch.Tensor]], str], Tuple[bytes, Dict[str, torch.Tensor]]]
 
 
 FAMILIES: Dict[str, DecoderFamily] = {}
@@ -30,7 +30,8 @@ def register_family(name: str, family: DecoderFamily) -> None:
     FAMILIES[name] = family
 
 
-register_family("Fegilix", DecoderFamily(fegilix.FegilixConfig.from_json, lambda cfg, w, dev: fegilix.build_fegilix(cfg, w, device=dev)))
+register_family("Fegilix", DecoderFamily(fegilix.FegilixConfig.from_json, lambda cfg, w, dev: fegilix.build_fegilix(
+    cfg, w if w is not None else fegilix.random_weights(cfg, device=dev, low_rank=fegilix.default_rank(cfg)), device=dev)))
 register_family("LlamaForCausalLM", DecoderFamily(
     llama.LlamaConfig.from_json, lambda cfg, w, dev: llama.build_llama(cfg, external_weights=True, device=dev, paged=True, state=w)))
 
@@ -44,7 +45,7 @@ def family_of(config: Mapping[str, Any]) -> DecoderFamily:
     return FAMILIES[name]
 
 
-def create_decoder(config: Mapping[str, Any], tensors: Mapping[str, torch.Tensor], dtype: str = "bfloat16", *, batch: int = 1,
+def create_decoder(config: Mapping[str, Any], tensors: Optional[Mapping[str, torch.Tensor]], dtype: str = "bfloat16", *, batch: int = 1,
                    max_len: int = 2048, max_tokens: Optional[int] = None, block_size: int = 256, provider: str = "CUDAExecutionProvider",
                    cuda_graph: bool = True, session_entries: Optional[Mapping[str, str]] = None) -> PagedDecoderRunner:
     """A decoder with room for ``batch`` sequences of at most ``max_len`` tokens; ``max_tokens`` bounds the tokens that all

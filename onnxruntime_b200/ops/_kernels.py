@@ -320,6 +320,20 @@ def attn_prefill(q, k, v, seqlens_k=None, first_prompt=True, causal=True, window
     return out
 
 
+def attn_prefill_paged(q, k_cache, v_cache, cu_seqlens, past_seqlens, block_table, scale=0.0, head_sink=None, split_weights=False, status=None,
+                       window=-1):
+    """Packed queries q [T,N,H] of several sequences over a paged cache [num_blocks,block_size,Nk,H].  Returns [T,N,H]."""
+    T, N, H = q.shape
+    nb, bs, Nk, _ = k_cache.shape
+    out = torch.empty_like(q)
+    st = (ctypes.c_int64 * 3)(0, N * H, H)
+    a = AttnPrefillArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), None, _ptr(head_sink), _ptr(out), past_seqlens.numel(), 0, N, Nk, H, 0, st, st,
+                        (ctypes.c_int64 * 3)(0, 0, 0), 0, 1, window, scale, 0.0, dtype_code(q.dtype), _ptr(status), None, _ptr(block_table),
+                        _ptr(cu_seqlens), _ptr(past_seqlens), T, bs, block_table.shape[1], nb, 1 if split_weights else 0)
+    _check(lib().ortb200_attn_prefill(ctypes.byref(a), ctypes.c_void_p(stream_ptr())), "ortb200_attn_prefill(paged)")
+    return out
+
+
 class PagedPrepArgs(ctypes.Structure):
     _fields_ = [("qkv", ctypes.c_void_p), ("k", ctypes.c_void_p), ("v", ctypes.c_void_p), ("q_out", ctypes.c_void_p),
                 ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p), ("cu_seqlens", ctypes.c_void_p),
@@ -450,4 +464,101 @@ def gather_rows(table, ids):
     _check(lib().ortb200_gather_rows(ctypes.c_void_p(_ptr(table)), ctypes.c_void_p(_ptr(ids)), ctypes.c_void_p(_ptr(out)),
                                      ctypes.c_int64(ids.numel()), ctypes.c_int64(table.shape[0]), table.shape[1],
                                      table.element_size(), ctypes.c_void_p(stream_ptr())), "ortb200_gather_rows")
+    return out
+
+
+# ---------------------------------------------------------------------------------------- packed hybrid-decoder kernels
+_P, _I, _L, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float
+
+
+class GatedDeltaArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("qkvb", "low", "conv", "a_log", "dt_bias", "norm", "conv_state", "state", "cu_seqlens", "past_seqlens",
+                                  "slots", "out", "workspace")] + [("workspace_bytes", _L)] + \
+               [(n, _I) for n in ("T", "B", "ld", "heads", "kv_heads", "dk", "dv", "taps", "num_slots")] + \
+               [("norm_eps", _F), ("unit_eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P)]
+
+
+class MLstmArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("packed", "i_bias", "f_bias", "norm", "state", "aux", "cu_seqlens", "past_seqlens", "slots", "out",
+                                  "workspace")] + [("workspace_bytes", _L)] + \
+               [(n, _I) for n in ("T", "B", "ld", "heads", "dk", "dv", "num_slots")] + \
+               [("gate_cap", _F), ("norm_eps", _F), ("den_eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P)]
+
+
+class HyperNormArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("x", "y", "mix", "w_out", "w_in", "gamma", "x_out", "out", "rows")] + \
+               [(n, _I) for n in ("T", "num_rows", "streams", "width", "x_shared")] + \
+               [("eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P)]
+
+
+class QkNormRopeArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("packed", "q_out", "k_cache", "v_cache", "q_norm", "k_norm", "cos_table", "sin_table", "cu_seqlens",
+                                  "past_seqlens", "block_table")] + \
+               [(n, _I) for n in ("T", "B", "ld", "N", "Nk", "dk", "dv", "dk_pad", "dv_pad", "rot_dim", "table_rows", "block_size", "max_blocks",
+                                  "num_blocks", "kv_shared")] + [("eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P)]
+
+
+def _call(name, args):
+    _check(getattr(lib(), name)(ctypes.byref(args), ctypes.c_void_p(stream_ptr())), name)
+
+
+def _recurrent_workspace(T, B, heads, kv_heads, dk, dv, device):
+    f = lib().ortb200_recurrent_workspace_bytes
+    f.restype = ctypes.c_int64
+    n = f(T, B, heads, kv_heads, dk, dv)
+    return torch.empty(max(n, 16), dtype=torch.uint8, device=device), n
+
+
+def gated_delta(qkvb, low, conv, a_log, dt_bias, norm, conv_state, state, cu, past, slots, kv_heads, norm_eps=1e-6, unit_eps=1e-6):
+    """Packed gated delta rule (ortb200_gated_delta_args); conv_state and state are updated in place.  Returns [T, heads * dv]."""
+    T, B = qkvb.shape[0], past.numel()
+    ns, heads, dk, dv = state.shape
+    out = torch.empty(T, heads * dv, dtype=qkvb.dtype, device=qkvb.device)
+    ws, n = _recurrent_workspace(T, B, heads, kv_heads, dk, dv, qkvb.device)
+    _call("ortb200_gated_delta", GatedDeltaArgs(_ptr(qkvb), _ptr(low), _ptr(conv), _ptr(a_log), _ptr(dt_bias), _ptr(norm), _ptr(conv_state),
+                                                _ptr(state), _ptr(cu), _ptr(past), _ptr(slots), _ptr(out), _ptr(ws), n, T, B, qkvb.shape[1], heads,
+                                                kv_heads, dk, dv, conv.shape[1], ns, norm_eps, unit_eps, dtype_code(qkvb.dtype), 0, None))
+    return out
+
+
+def mlstm(packed, i_bias, f_bias, norm, state, aux, cu, past, slots, gate_cap, norm_eps=1e-6, den_eps=1e-6):
+    """Packed mLSTM (ortb200_mlstm_args); state and aux are updated in place.  Returns [T, heads * dv]."""
+    T, B = packed.shape[0], past.numel()
+    ns, heads, dk, dv = state.shape
+    out = torch.empty(T, heads * dv, dtype=packed.dtype, device=packed.device)
+    ws, n = _recurrent_workspace(T, B, heads, heads, dk, dv, packed.device)
+    _call("ortb200_mlstm", MLstmArgs(_ptr(packed), _ptr(i_bias), _ptr(f_bias), _ptr(norm), _ptr(state), _ptr(aux), _ptr(cu), _ptr(past),
+                                     _ptr(slots), _ptr(out), _ptr(ws), n, T, B, packed.shape[1], heads, dk, dv, ns, gate_cap, norm_eps, den_eps,
+                                     dtype_code(packed.dtype), 0, None))
+    return out
+
+
+def hyper_norm(x, y, mix, w_out, w_in, gamma, eps, keep=True):
+    """x [T, streams, width] fp32, y [T, width].  Returns (normed [T, width], new streams or None)."""
+    T, n, W = x.shape
+    out = torch.empty(T, W, dtype=y.dtype, device=x.device)
+    xo = torch.empty_like(x) if keep else None
+    _call("ortb200_hyper_norm", HyperNormArgs(_ptr(x), _ptr(y), _ptr(mix), _ptr(w_out), _ptr(w_in), _ptr(gamma), _ptr(xo), _ptr(out), None, T, T, n,
+                                              W, 0, eps, dtype_code(y.dtype), 0, None))
+    return out, xo
+
+
+def qk_norm_rope(packed, k_cache, v_cache, q_norm, k_norm, cos, sin, cu, past, table, N, dk, dv, eps=1e-6):
+    """Packed q | k | v rows; caches [num_blocks, block_size, Nk, padded head] updated in place.  Returns q [T, N, padded head]."""
+    T = packed.shape[0]
+    nb, bs, Nk, dkp = k_cache.shape
+    q = torch.empty(T, N, dkp, dtype=packed.dtype, device=packed.device)
+    _call("ortb200_qk_norm_rope", QkNormRopeArgs(_ptr(packed), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin),
+                                                 _ptr(cu), _ptr(past), _ptr(table), T, past.numel(), packed.shape[1], N, Nk, dk, dv, dkp,
+                                                 v_cache.shape[3], cos.shape[1] * 2, cos.shape[0], bs, table.shape[1], nb, 0, eps,
+                                                 dtype_code(packed.dtype), 0, None))
+    return q
+
+
+def head_gate(x, gate, gate_ld, dv):
+    """out[t, h * dv + j] = x[t, h, j] * sigmoid(gate row t); ``gate`` points at the first gate column of packed rows."""
+    T, heads, x_pad = x.shape
+    out = torch.empty(T, heads * dv, dtype=x.dtype, device=x.device)
+    _check(lib().ortb200_head_gate(ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(gate.data_ptr()), ctypes.c_void_p(out.data_ptr()), T, heads, dv, x_pad,
+                                   ctypes.c_int64(gate_ld), dtype_code(x.dtype), 0, ctypes.c_void_p(stream_ptr())), "ortb200_head_gate")
     return out

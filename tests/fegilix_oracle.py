@@ -79,8 +79,8 @@ def gated_delta_scan(q, k, v, beta, decay):
     return torch.stack(out)
 
 
-def mlstm_scan(q, k, v, i_gate, f_gate):
-    """q, k [T, H, dk], v [T, H, dv], log gates [T, H]; returns [T, H, dv]."""
+def mlstm_scan(q, k, v, i_gate, f_gate, floor=True):
+    """``floor=False`` plants a mistake: the denominator is |n . q| alone.  q, k [T, H, dk], v [T, H, dv], log gates [T, H]; returns [T, H, dv]."""
     T, H, dk = q.shape
     S = torch.zeros(H, dk, v.shape[-1], dtype=q.dtype)
     n = torch.zeros(H, dk, dtype=q.dtype)
@@ -93,7 +93,7 @@ def mlstm_scan(q, k, v, i_gate, f_gate):
         n = keep[:, None] * n + add[:, None] * k[t]
         m = m_new
         num = (S * q[t][:, :, None]).sum(1)
-        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m) * float(floor)) + 1e-6
         out.append(num / den[:, None])
     return torch.stack(out)
 
@@ -103,6 +103,16 @@ def softmax_with_sink(scores, sink):
     top = torch.maximum(scores.max(-1, keepdim=True).values, sink[:, None, None])
     e = torch.exp(scores - top)
     return e / (e.sum(-1, keepdim=True) + torch.exp(sink[:, None, None] - top))
+
+
+def causal_attention(q, k, v, scale, sink):
+    """q [T, H, d], k [T, G, d], v [T, G, dv]: query head h reads key / value head h // (H / G)."""
+    rep = q.shape[1] // k.shape[1]
+    k, v = k.repeat_interleave(rep, 1), v.repeat_interleave(rep, 1)
+    s = torch.einsum("thd,lhd->htl", q, k) * scale
+    pos = torch.arange(q.shape[0])
+    s = s.masked_fill(pos[None, None, :] > pos[None, :, None], float("-inf"))
+    return torch.einsum("htl,lhv->thv", softmax_with_sink(s, sink), v)
 
 
 def channel_delta(h, w, p, m, eps):
@@ -138,15 +148,13 @@ def attention(h, w, p, m, eps, kv=None):
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     pos = torch.arange(T)
-    q = rotate(rms_norm((h @ w[p + "q"].T).view(T, H, d), w[p + "q.norm"], eps), pos, m["rot"])
+    turn = (lambda x: rotate(x, pos, m["rot"])) if m.get("rot") else (lambda x: x)
+    q = turn(rms_norm((h @ w[p + "q"].T).view(T, H, d), w[p + "q.norm"], eps))
     if kv is None:
-        k = rotate(rms_norm((h @ w[p + "k"].T).view(T, G, d), w[p + "k.norm"], eps), pos, m["rot"])
+        k = turn(rms_norm((h @ w[p + "k"].T).view(T, G, d), w[p + "k.norm"], eps))
         v = (h @ w[p + "v"].T).view(T, G, dv)
         kv = (k, v)
-    k, v = kv[0].repeat_interleave(H // G, 1), kv[1].repeat_interleave(H // G, 1)
-    s = torch.einsum("thd,lhd->htl", q, k) * m["scale"]
-    s = s.masked_fill(pos[None, None, :] > pos[None, :, None], float("-inf"))
-    o = torch.einsum("htl,lhv->thv", softmax_with_sink(s, w[p + "sink"]), v).reshape(T, H * dv)
+    o = causal_attention(q, kv[0], kv[1], m["scale"], w[p + "sink"]).reshape(T, H * dv)
     return (o * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T, kv
 
 
@@ -162,12 +170,24 @@ def hyper_write(streams, mix, w_out, y):
     return torch.einsum("st,nsw->ntw", mix, streams) + w_out[None, :, None] * y[:, None, :]
 
 
+class PlainStream(dict):
+    """Weights of a model without hyper-connections: every read, write and mix factor is 1."""
+
+    def __missing__(self, name):
+        assert ".hc" in name, name
+        return torch.ones((1, 1) if name.endswith("mix") else 1, dtype=F64)
+
+
 def forward(config, weights, tokens, layers_out=None):
     """Logits [T, vocab] of one sequence; ``layers_out`` (a list) receives the stream sum after every layer."""
     w = {k: v.to(F64) for k, v in weights.items()}
     eps = config["norm"]["eps"]
     x = w["embed"][torch.as_tensor(tokens)]
-    streams = x[:, None, :].repeat(1, config["streams"], 1)
+    plain = config.get("streams") is None       # one residual stream, x <- x + y
+    n = 1 if plain else config["streams"]
+    if plain:
+        w = PlainStream(w)
+    streams = x[:, None, :].repeat(1, n, 1)
     caches = {}
     for i, layer in enumerate(config["layers"]):
         L, m = f"l{i}.", layer["mixer"]
@@ -185,5 +205,5 @@ def forward(config, weights, tokens, layers_out=None):
         if layers_out is not None:
             layers_out.append(streams.sum(1))
     logits = rms_norm(streams.sum(1), w["final.norm"], eps) @ w["head"].T
-    cap = config["logit_softcap"]
-    return cap * torch.tanh(logits / cap)
+    cap = config.get("logit_softcap")
+    return cap * torch.tanh(logits / cap) if cap else logits
