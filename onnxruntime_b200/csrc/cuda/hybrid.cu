@@ -47,9 +47,9 @@ __device__ __forceinline__ void store4(T* p, const float (&v)[4]) {
 // One block per token.  E = elements per access (4 when the width allows it).  u stays in shared memory between the sum of
 // squares and the scaled store.
 template <typename T, int N, int E>
-__global__ void __launch_bounds__(256) hyper_norm_kernel(const ortb200_hyper_norm_args a) {
+__global__ void __launch_bounds__(N <= 4 ? 1024 : 256) hyper_norm_kernel(const ortb200_hyper_norm_args a) {
   extern __shared__ __align__(16) float u[];
-  __shared__ float red[8];
+  __shared__ float red[32];
   float mix[N][N], w_out[N], w_in[N];
 #pragma unroll
   for (int s = 0; s < N; ++s) {
@@ -133,7 +133,11 @@ int launch_hyper(const ortb200_hyper_norm_args& a, cudaStream_t stream) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
     attr_smem[vec] = smem;
   }
-  return launch_kernel(kern, dim3(a.rows ? a.num_rows : a.T), 256, smem, stream, a.use_pdl != 0, a);
+  // few tokens: enough threads that a row is one round of loads per thread
+  const int blocks = a.rows ? a.num_rows : a.T;
+  int threads = 256;
+  while (N <= 4 && blocks <= 296 && threads < 1024 && threads * (vec ? 4 : 1) < a.width) threads *= 2;
+  return launch_kernel(kern, dim3(blocks), threads, smem, stream, a.use_pdl != 0, a);
 }
 
 template <typename T>

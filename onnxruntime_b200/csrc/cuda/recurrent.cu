@@ -3,12 +3,13 @@
 // fp32, so a result does not depend on how a prompt is cut.
 //
 // Several tokens per sequence (prompts): three launches.
-//   prep   one block per token: short convolution + silu, unit norms, decays, gates -> fp32 rows, heads padded
+//   prep   short convolution + silu, unit norms, decays, gates -> fp32 rows, heads padded; a warp owns the channels of one
+//          head and walks a run of tokens with the convolution window in registers
 //   scan   one block per (16 * warps state columns, head, sequence).  State columns are independent of each other, so
 //          the grid splits them; a warp holds a [dk, 16] slice of S in registers (8 row groups x 4 column groups of
 //          lanes), streams the token rows through double-buffered shared memory with cp.async, and does the decay, the
 //          two matrix-vector products and the rank-one update with packed fp32x2 instructions
-//   post   one block per token: norm over the value dimension, output gate, ring of convolution inputs
+//   post   norm over the value dimension, output gate, ring of convolution inputs
 // One token per sequence (decode): one launch, one block per (head, sequence) that does all of it; the state is read
 // once and written once, which is what bounds the step.
 //
@@ -26,7 +27,8 @@ namespace ortb200 {
 namespace {
 
 constexpr int kMaxHead = 256;     // key / value head sizes
-constexpr int kChunk = 16;        // tokens per shared-memory stage of the scan
+constexpr int kChunk = 8;         // tokens per shared-memory stage of the scan
+constexpr int kPrepRun = 16;      // tokens a prep warp walks
 constexpr int kMaxTaps = 16;
 
 int pad_dk(int dk) { return dk <= 64 ? 64 : (dk <= 128 ? 128 : 256); }
@@ -57,6 +59,14 @@ Scratch split_scratch(float* w, int T, int H, int G, int dkp, int dvp) {
 }
 
 // ------------------------------------------------------------------------------------------------ delta rule pieces
+// silu behind the short convolution and sigmoid of the output gate: results that 16-bit models round to 16 bits take the
+// fast exponential and division
+template <typename T>
+__device__ __forceinline__ float act_sigmoid(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  else return sigmoid_f(x);
+}
+
 // Convolution + silu of one channel for the token in packed row t (position pos, `before` rows of its sequence in this
 // call); earlier inputs come from the packed rows, then from the ring, and are zero in front of the sequence.
 template <typename T>
@@ -72,7 +82,7 @@ __device__ __forceinline__ float conv_silu(const ortb200_gated_delta_args& a, co
     acc = fmaf(w[a.taps - 1 - j], xv, acc);
   }
   acc = fmaf(w[a.taps - 1], to_float<T>(x[0]), acc);
-  return acc * sigmoid_f(acc);
+  return acc * act_sigmoid<T>(acc);
 }
 
 __device__ __forceinline__ bool slot_ok(int slot, int num_slots, int* status) {
@@ -81,64 +91,185 @@ __device__ __forceinline__ bool slot_ok(int slot, int num_slots, int* status) {
   return false;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const ortb200_gated_delta_args a, const Scratch s, int dkp, int dvp) {
-  const int t = blockIdx.x;
+// Inputs of one channel per lane and 32-column group, TAPS - 1 tokens back (newest last), for a warp that walks packed rows.
+template <typename T, int TAPS, int NI>
+struct ConvWindow {
+  float w[NI][TAPS], x[NI][TAPS - 1 > 0 ? TAPS - 1 : 1];
+  __device__ __forceinline__ void load_taps(const float* conv, int ch0, int n, int lane) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = i * 32 + lane;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[i][j] = d < n ? conv[static_cast<long long>(ch0 + d) * TAPS + j] : 0.f;
+    }
+  }
+  // `row` points at channel ch0 of the token's packed row
+  __device__ __forceinline__ void refill(const T* row, long long ld, const T* ring, int channels, int ch0, int n, int lane, int pos, int before) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = i * 32 + lane;
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j) {
+        float v = 0.f;
+        if (d < n) {
+          if (j <= before) v = to_float<T>(row[d - j * ld]);
+          else if (pos - j >= 0) v = to_float<T>(ring[static_cast<long long>((pos - j) % TAPS) * channels + ch0 + d]);
+        }
+        x[i][TAPS - 1 - j] = v;
+      }
+    }
+  }
+  __device__ __forceinline__ void step(const T* row, int n, int lane, float (&y)[NI]) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = i * 32 + lane;
+      const float now = d < n ? to_float<T>(row[d]) : 0.f;
+      float acc = now * w[i][TAPS - 1];
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) acc = fmaf(x[i][j], w[i][j], acc);
+#pragma unroll
+      for (int j = 0; j + 2 < TAPS; ++j) x[i][j] = x[i][j + 1];
+      if (TAPS > 1) x[i][TAPS - 2 > 0 ? TAPS - 2 : 0] = now;
+      y[i] = acc * act_sigmoid<T>(acc);
+    }
+  }
+};
+// any number of taps: every input is fetched again
+template <typename T, int NI>
+struct ConvWindow<T, 0, NI> {
+  const ortb200_gated_delta_args* a;
+  const T* ring;
+  int channels, ch0, pos, before;
+  long long t;
+  __device__ __forceinline__ void step(int n, int lane, float (&y)[NI]) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = i * 32 + lane;
+      y[i] = d < n ? conv_silu<T>(*a, ring, channels, ch0 + d, t, pos, before) : 0.f;
+    }
+  }
+};
+
+template <typename T, int TAPS, int NI>
+__global__ void __launch_bounds__(256, NI <= 4 ? 3 : 1) delta_prep_kernel(const ortb200_gated_delta_args a, const Scratch s, int dkp, int dvp) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.heads, G = a.kv_heads, dk = a.dk, dv = a.dv;
   const int channels = 2 * G * dk + H * dv;
+  const int u = blockIdx.y * 8 + warp;              // G (q and k of a key head), then H value heads, then H decay heads
   pdl_wait_prior_grids();
-  const int b = sequence_of(a.cu_seqlens, a.B, t);
-  const int before = t - a.cu_seqlens[b];
-  const int pos = a.past_seqlens[b] + before;
-  const int slot = a.slots[b];
-  const bool ok = slot_ok(slot, a.num_slots, a.status);
-  const T* ring = static_cast<const T*>(a.conv_state) + static_cast<long long>(ok ? slot : 0) * a.taps * channels;
-  // units of work: G (q and k of a key head), H value heads, H decay heads
-  for (int u = warp; u < G + 2 * H; u += 8) {
-    if (u < G) {
-      float q[kMaxHead / 32], k[kMaxHead / 32];
+  pdl_launch_dependents();
+  if (u >= G + 2 * H) return;
+  const int t0 = blockIdx.x * kPrepRun, t1 = min(a.T, t0 + kPrepRun);
+  if (u >= G + H) {
+    const int h = u - G - H;
+    const float rate = expf(a.a_log[h]);
+    for (int t = t0; t < t1; ++t) {
+      const T* low = static_cast<const T*>(a.low) + static_cast<long long>(t) * H * (dk + dv) + h * dk;
+      float* row = s.decay + (static_cast<long long>(t) * H + h) * dkp;
+      for (int d = lane; d < dkp; d += 32) row[d] = d < dk ? expf(-rate * softplus_f(to_float<T>(low[d]) + a.dt_bias[h * dk + d])) : 0.f;
+      if (lane == 0) s.scal[(static_cast<long long>(t) * H + h) * 4] = sigmoid_f(to_float<T>(static_cast<const T*>(a.qkvb)[static_cast<long long>(t) * a.ld + channels + h]));
+    }
+    return;
+  }
+  int b = sequence_of(a.cu_seqlens, a.B, t0), next = a.cu_seqlens[b + 1];
+  bool fill = true;
+  const T* ring = nullptr;
+  int pos = 0, before = 0;
+  // position of token t; true when the window has to be (re)loaded
+  auto locate = [&](int t) {
+    if (fill || t >= next) {
+      while (t >= next) next = a.cu_seqlens[++b + 1];
+      const int slot = a.slots[b];
+      const bool ok = slot >= 0 && slot < a.num_slots;
+      if (!ok && a.status && lane == 0) atomicExch(a.status, kStatusBadArgument);
+      ring = static_cast<const T*>(a.conv_state) + static_cast<long long>(ok ? slot : 0) * a.taps * channels;
+      before = t - a.cu_seqlens[b];
+      pos = a.past_seqlens[b] + before;
+      fill = false;
+      return true;
+    }
+    ++before;
+    ++pos;
+    return false;
+  };
+  const T* base = static_cast<const T*>(a.qkvb);
+  if (u < G) {
+    ConvWindow<T, TAPS, NI> wq, wk;
+    const int cq = u * dk, ck = (G + u) * dk;
+    if constexpr (TAPS > 0) {
+      wq.load_taps(a.conv, cq, dk, lane);
+      wk.load_taps(a.conv, ck, dk, lane);
+    }
+    const float root = 1.f / sqrtf(static_cast<float>(dk));
+    const int group = H / G;
+    for (int t = t0; t < t1; ++t) {
+      const bool refill = locate(t);
+      const T* row = base + static_cast<long long>(t) * a.ld;
+      float q[NI], k[NI];
+      if constexpr (TAPS > 0) {
+        if (refill) {
+          wq.refill(row + cq, a.ld, ring, channels, cq, dk, lane, pos, before);
+          wk.refill(row + ck, a.ld, ring, channels, ck, dk, lane, pos, before);
+        }
+        wq.step(row + cq, dk, lane, q);
+        wk.step(row + ck, dk, lane, k);
+      } else {
+        wq = {&a, ring, channels, cq, pos, before, t};
+        wk = {&a, ring, channels, ck, pos, before, t};
+        wq.step(dk, lane, q);
+        wk.step(dk, lane, k);
+      }
       float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
-      for (int i = 0; i < kMaxHead / 32; ++i) {
-        const int d = i * 32 + lane;
-        q[i] = d < dk ? conv_silu<T>(a, ring, channels, u * dk + d, t, pos, before) : 0.f;
-        k[i] = d < dk ? conv_silu<T>(a, ring, channels, (G + u) * dk + d, t, pos, before) : 0.f;
+      for (int i = 0; i < NI; ++i) {
         qq = fmaf(q[i], q[i], qq);
         kk = fmaf(k[i], k[i], kk);
         qk = fmaf(q[i], k[i], qk);
       }
-      qq = warp_sum(qq);
-      kk = warp_sum(kk);
-      qk = warp_sum(qk);
-      const float qs = 1.f / (sqrtf(qq + a.unit_eps) * sqrtf(static_cast<float>(dk)));
-      const float ks = 1.f / sqrtf(kk + a.unit_eps);
-      float* row = s.qk + (static_cast<long long>(t) * G + u) * 2 * dkp;
 #pragma unroll
-      for (int i = 0; i < kMaxHead / 32; ++i) {
-        const int d = i * 32 + lane;
-        if (d < dkp) {
-          row[d] = q[i] * qs;
-          row[dkp + d] = k[i] * ks;
-        }
+      for (int off = 16; off > 0; off >>= 1) {
+        qq += __shfl_xor_sync(0xffffffffu, qq, off);
+        kk += __shfl_xor_sync(0xffffffffu, kk, off);
+        qk += __shfl_xor_sync(0xffffffffu, qk, off);
       }
-      const int group = H / G;
+      const float qs = root / sqrtf(qq + a.unit_eps), ks = 1.f / sqrtf(kk + a.unit_eps);
+      float* out = s.qk + (static_cast<long long>(t) * G + u) * 2 * dkp;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {   // dkp == 32 * NI
+        out[i * 32 + lane] = q[i] * qs;
+        out[dkp + i * 32 + lane] = k[i] * ks;
+      }
       for (int j = lane; j < group; j += 32) s.scal[(static_cast<long long>(t) * H + u * group + j) * 4 + 1] = qk * qs * ks;
-    } else if (u < G + H) {
-      const int h = u - G;
-      float* row = s.v + (static_cast<long long>(t) * H + h) * dvp;
-      for (int d = lane; d < dvp; d += 32) row[d] = d < dv ? conv_silu<T>(a, ring, channels, 2 * G * dk + h * dv + d, t, pos, before) : 0.f;
-    } else {
-      const int h = u - G - H;
-      const T* low = static_cast<const T*>(a.low) + static_cast<long long>(t) * H * (dk + dv) + h * dk;
-      const float rate = expf(a.a_log[h]);
-      float* row = s.decay + (static_cast<long long>(t) * H + h) * dkp;
-      for (int d = lane; d < dkp; d += 32) row[d] = d < dk ? expf(-rate * softplus_f(to_float<T>(low[d]) + a.dt_bias[h * dk + d])) : 0.f;
+    }
+  } else {
+    const int h = u - G, cv = 2 * G * dk + h * dv;
+    for (int c0 = 0; c0 < dv; c0 += NI * 32) {
+      const int n = dv - c0;
+      ConvWindow<T, TAPS, NI> wv;
+      if constexpr (TAPS > 0) wv.load_taps(a.conv, cv + c0, n, lane);
+      if (c0 > 0) {
+        b = sequence_of(a.cu_seqlens, a.B, t0);
+        next = a.cu_seqlens[b + 1];
+        fill = true;
+      }
+      for (int t = t0; t < t1; ++t) {
+        const bool refill = locate(t);
+        const T* row = base + static_cast<long long>(t) * a.ld + cv + c0;
+        float v[NI];
+        if constexpr (TAPS > 0) {
+          if (refill) wv.refill(row, a.ld, ring, channels, cv + c0, n, lane, pos, before);
+          wv.step(row, n, lane, v);
+        } else {
+          wv = {&a, ring, channels, cv + c0, pos, before, t};
+          wv.step(n, lane, v);
+        }
+        float* out = s.v + (static_cast<long long>(t) * H + h) * dvp + c0;
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (c0 + i * 32 + lane < dvp) out[i * 32 + lane] = v[i];
+      }
     }
   }
-  const T* bp = static_cast<const T*>(a.qkvb) + static_cast<long long>(t) * a.ld + channels;
-  for (int h = threadIdx.x; h < H; h += blockDim.x) s.scal[(static_cast<long long>(t) * H + h) * 4] = sigmoid_f(to_float<T>(bp[h]));
-  pdl_launch_dependents();
 }
 
 template <typename T>
@@ -146,10 +277,12 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const ortb200_mlstm_arg
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.heads, dk = a.dk, dv = a.dv;
+  const int h = blockIdx.y * 8 + warp;
   pdl_wait_prior_grids();
+  pdl_launch_dependents();
   const T* row = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld;
   const float qs = 1.f / sqrtf(static_cast<float>(dk));
-  for (int h = warp; h < H; h += 8) {
+  if (h < H) {
     float* qk = s.qk + (static_cast<long long>(t) * H + h) * 2 * dkp;
     float dot = 0.f;
     for (int d = lane; d < dkp; d += 32) {
@@ -171,7 +304,6 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const ortb200_mlstm_arg
       sc[2] = dot;
     }
   }
-  pdl_launch_dependents();
 }
 
 // ---------------------------------------------------------------------------------------------------------- the scan
@@ -197,7 +329,7 @@ __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_gr
 // R = state rows per lane; dkp = 8 R.  Lane (rg = lane & 7, cg = lane >> 3) holds rows j * 32 + rg * 4 + {0..3},
 // j < R / 4, of columns col0 .. col0 + 3.
 template <bool DELTA, int R>
-__global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) scan_kernel(const ScanParams p) {
   constexpr int DKP = 8 * R, NJ = R / 4;
   constexpr int kRows = DELTA ? 3 : 2;             // q, k (, decay)
   const int warps = blockDim.x >> 5;
@@ -261,19 +393,16 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
     }
   }
   float* gaux = DELTA ? nullptr : p.aux + (static_cast<long long>(slot) * p.H + h) * (p.dk + 1);
-  f32x2 nrm[DELTA ? 1 : NJ][2];
+  constexpr int NR = DKP / 32;                     // mLSTM: every warp keeps n, lane l its rows l, l + 32, ...
+  float nrm[NR];
   float m = 0.f;
   if (!DELTA) {
 #pragma unroll
-    for (int j = 0; j < NJ; ++j) {
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const int r = j * 32 + rg * 4 + hh * 2;
-        nrm[DELTA ? 0 : j][hh] = pack2(!fresh && r < p.dk ? gaux[r] : 0.f, !fresh && r + 1 < p.dk ? gaux[r + 1] : 0.f);
-      }
-    }
+    for (int i = 0; i < NR; ++i) nrm[i] = !fresh && i * 32 + lane < p.dk ? gaux[i * 32 + lane] : 0.f;
     m = fresh ? 0.f : gaux[p.dk];
   }
+  float* orow = p.s.o + (static_cast<long long>(t0) * p.H + h) * p.dvp + col0;
+  const long long ostep = static_cast<long long>(p.H) * p.dvp;
 
   const int chunks = (len + kChunk - 1) / kChunk;
   fetch(0);
@@ -294,12 +423,9 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
       const float* kr = qr + DKP;
       const float4 vv = *reinterpret_cast<const float4*>(sv + tt * cs + wcol);
       const float4 scal = *reinterpret_cast<const float4*>(sc + tt * 4);
-      float* orow = p.s.o + (static_cast<long long>(t0 + ch * kChunk + tt) * p.H + h) * p.dvp;
       if (DELTA) {
         const float* gr = kr + DKP;
         f32x2 accA[4], accO[4];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) { accA[c] = 0ull; accO[c] = 0ull; }
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
@@ -309,8 +435,8 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
           for (int c = 0; c < 4; ++c) {
             S[j][c][0] = mul2(S[j][c][0], g2.x);
             S[j][c][1] = mul2(S[j][c][1], g2.y);
-            accA[c] = fma2(S[j][c][0], k2.x, accA[c]);
-            accO[c] = fma2(S[j][c][0], q2.x, accO[c]);
+            accA[c] = j == 0 ? mul2(S[j][c][0], k2.x) : fma2(S[j][c][0], k2.x, accA[c]);
+            accO[c] = j == 0 ? mul2(S[j][c][0], q2.x) : fma2(S[j][c][0], q2.x, accO[c]);
             accA[c] = fma2(S[j][c][1], k2.y, accA[c]);
             accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
           }
@@ -357,7 +483,7 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
         if (rg >= 4) {
           const int c = rg - 4;
           const float u = c == 0 ? u0 : (c == 1 ? u1 : (c == 2 ? u2 : u3));
-          if (col0 + c < p.dv) orow[col0 + c] = fmaf(scal.y, u, w);
+          if (col0 + c < p.dv) orow[c] = fmaf(scal.y, u, w);
         }
       } else {
         const float m_new = fmaxf(scal.y + m, scal.x);
@@ -365,23 +491,23 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
         m = m_new;
         const f32x2 f2 = pack2(fw, fw), i2 = pack2(iw, iw);
         const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
-        f32x2 accO[4], accN = 0ull;
+        f32x2 accO[4];
+        float nq = 0.f;
 #pragma unroll
-        for (int c = 0; c < 4; ++c) accO[c] = 0ull;
+        for (int i = 0; i < NR; ++i) {
+          nrm[i] = fmaf(nrm[i], fw, iw * kr[i * 32 + lane]);
+          nq = fmaf(nrm[i], qr[i * 32 + lane], nq);
+        }
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
           const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
           const f32x2 ik0 = mul2(k2.x, i2), ik1 = mul2(k2.y, i2);
-          nrm[DELTA ? 0 : j][0] = fma2(nrm[DELTA ? 0 : j][0], f2, ik0);
-          nrm[DELTA ? 0 : j][1] = fma2(nrm[DELTA ? 0 : j][1], f2, ik1);
-          accN = fma2(nrm[DELTA ? 0 : j][0], q2.x, accN);
-          accN = fma2(nrm[DELTA ? 0 : j][1], q2.y, accN);
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
             S[j][c][0] = fma2(ik0, v2[c], mul2(S[j][c][0], f2));
             S[j][c][1] = fma2(ik1, v2[c], mul2(S[j][c][1], f2));
-            accO[c] = fma2(S[j][c][0], q2.x, accO[c]);
+            accO[c] = j == 0 ? mul2(S[j][c][0], q2.x) : fma2(S[j][c][0], q2.x, accO[c]);
             accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
           }
         }
@@ -391,10 +517,8 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
           unpack2(accO[c], lo, hi);
           x[c] = lo + hi;
         }
-        unpack2(accN, lo, hi);
-        float nq = lo + hi;
 #pragma unroll
-        for (int off = 1; off <= 4; off <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, off);
+        for (int off = 1; off <= 16; off <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, off);
         float y[2], w;
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -406,8 +530,9 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
           w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
         }
         w += __shfl_xor_sync(0xffffffffu, w, 4);
-        if (rg < 4 && col0 + rg < p.dv) orow[col0 + rg] = w / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
+        if (rg < 4 && col0 + rg < p.dv) orow[rg] = w / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
       }
+      orow += ostep;
     }
     __syncthreads();   // the stage may be refilled
   }
@@ -430,20 +555,12 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
   }
   // n and m: every block of a (head, sequence) computes the same values, and another block may still have to read the
   // old ones, so they leave through scratch and the post kernel moves them into the state
-  if (!DELTA && blockIdx.x == 0 && warp == 0 && cg == 0) {
+  if (!DELTA && blockIdx.x == 0 && warp == 0) {
     float* ao = p.s.aux_out + (static_cast<long long>(b) * p.H + h) * (p.dk + 1);
 #pragma unroll
-    for (int j = 0; j < NJ; ++j) {
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const int r = j * 32 + rg * 4 + hh * 2;
-        float lo, hi;
-        unpack2(nrm[DELTA ? 0 : j][hh], lo, hi);
-        if (r < p.dk) ao[r] = lo;
-        if (r + 1 < p.dk) ao[r + 1] = hi;
-      }
-    }
-    if (rg == 0) ao[p.dk] = m;
+    for (int i = 0; i < NR; ++i)
+      if (i * 32 + lane < p.dk) ao[i * 32 + lane] = nrm[i];
+    if (lane == 0) ao[p.dk] = m;
   }
 }
 
@@ -468,32 +585,65 @@ struct PostParams {
   const int* past_seqlens;
   const int* slots;
   int B, num_slots;
+  int vec;                 // gate, out and dv allow four-element accesses
 };
 
+template <typename T>
+__device__ __forceinline__ void copy4(T* dst, const T* src) {
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(src);
+  else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(src);
+}
+template <typename T>
+int post_vec(const PostParams& p) {
+  return p.dv % 4 == 0 && p.gate_ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & (4 * sizeof(T) - 1)) == 0;
+}
+
+// One warp per (token, head); lane l holds the columns 4 l ... 4 l + 3 of every 128.
 template <typename T>
 __global__ void __launch_bounds__(256) recurrent_post_kernel(const PostParams p) {
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y * 8 + warp;
   pdl_wait_prior_grids();
-  for (int h = warp; h < p.H; h += 8) {
+  pdl_launch_dependents();
+  if (h < p.H) {
     const float* o = p.o + (static_cast<long long>(t) * p.H + h) * p.dvp;
     float x[kMaxHead / 32], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < kMaxHead / 32; ++i) {
-      const int d = i * 32 + lane;
-      x[i] = d < p.dv ? o[d] : 0.f;
-      ss = fmaf(x[i], x[i], ss);
+    for (int i = 0; i < kMaxHead / 128; ++i) {
+      const int d = i * 128 + lane * 4;
+      const float4 v = d < p.dvp ? *reinterpret_cast<const float4*>(o + d) : make_float4(0.f, 0.f, 0.f, 0.f);   // rows padded to fours
+      x[i * 4] = v.x;
+      x[i * 4 + 1] = d + 1 < p.dv ? v.y : 0.f;
+      x[i * 4 + 2] = d + 2 < p.dv ? v.z : 0.f;
+      x[i * 4 + 3] = d + 3 < p.dv ? v.w : 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss = fmaf(x[i * 4 + e], x[i * 4 + e], ss);
     }
     ss = warp_sum(ss);
     const float r = 1.f / sqrtf(ss / p.dv + p.eps);
     const T* gate = static_cast<const T*>(p.gate) + t * p.gate_ld + h * p.dv;
     T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.H + h) * p.dv;
+    const float* norm = p.norm + h * p.norm_stride;
 #pragma unroll
-    for (int i = 0; i < kMaxHead / 32; ++i) {
-      const int d = i * 32 + lane;
-      if (d < p.dv) out[d] = from_float<T>(x[i] * r * p.norm[h * p.norm_stride + d] * sigmoid_f(to_float<T>(gate[d])));
+    for (int i = 0; i < kMaxHead / 128; ++i) {
+      const int d = i * 128 + lane * 4;
+      if (p.vec) {
+        if (d < p.dv) {
+          __align__(16) T g[4], y[4];
+          copy4(g, gate + d);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[e] = from_float<T>(x[i * 4 + e] * r * norm[d + e] * act_sigmoid<T>(to_float<T>(g[e])));
+          copy4(out + d, y);
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (d + e < p.dv) out[d + e] = from_float<T>(x[i * 4 + e] * r * norm[d + e] * act_sigmoid<T>(to_float<T>(gate[d + e])));
+      }
     }
   }
+  if (blockIdx.y != 0) return;
   const int b = sequence_of(p.cu_seqlens, p.B, t);
   const int end = p.cu_seqlens[b + 1];
   const int slot = p.slots[b];
@@ -509,7 +659,6 @@ __global__ void __launch_bounds__(256) recurrent_post_kernel(const PostParams p)
       for (int i = threadIdx.x; i < n; i += blockDim.x) p.aux[slot * n + i] = p.aux_out[b * n + i];
     }
   }
-  pdl_launch_dependents();
 }
 
 // ----------------------------------------------------------------------------------------------------------- decode
@@ -523,6 +672,7 @@ __global__ void __launch_bounds__(256) recurrent_decode_kernel(const A a) {
   __shared__ float sq[kMaxHead], sk[kMaxHead], sg[kMaxHead], sv[kMaxHead], so[kMaxHead];
   __shared__ float redA[8][128], redO[8][128], su[128];
   __shared__ float red[8], scal[4];
+  __shared__ float4 red3[8];
   pdl_wait_prior_grids();
   const int slot = a.slots[b];
   if (!slot_ok(slot, a.num_slots, a.status)) return;
@@ -582,9 +732,18 @@ __global__ void __launch_bounds__(256) recurrent_decode_kernel(const A a) {
       sv[tid] = conv_silu<T>(a, ring, channels, cv, b, pos, 0);
       ring_new[cv] = x[cv];
     }
-    qq = block_sum_all(qq, red);
-    kk = block_sum_all(kk, red);
-    qk = block_sum_all(qk, red);
+    qq = warp_sum(qq);
+    kk = warp_sum(kk);
+    qk = warp_sum(qk);
+    if (lane == 0) red3[warp] = make_float4(qq, kk, qk, 0.f);
+    __syncthreads();
+    qq = kk = qk = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      qq += red3[w].x;
+      kk += red3[w].y;
+      qk += red3[w].z;
+    }
     const float qs = 1.f / (sqrtf(qq + a.unit_eps) * sqrtf(static_cast<float>(dk))), ks = 1.f / sqrtf(kk + a.unit_eps);
     if (tid < dk) {
       sq[tid] *= qs;
@@ -708,7 +867,7 @@ __global__ void __launch_bounds__(256) recurrent_decode_kernel(const A a) {
       gate = to_float<T>(static_cast<const T*>(a.packed)[static_cast<long long>(b) * a.ld + H * (2 * dk + dv) + h * dv + tid]);
       w = a.norm[h * dv + tid];
     }
-    static_cast<T*>(a.out)[(static_cast<long long>(b) * H + h) * dv + tid] = from_float<T>(o * r * w * sigmoid_f(gate));
+    static_cast<T*>(a.out)[(static_cast<long long>(b) * H + h) * dv + tid] = from_float<T>(o * r * w * act_sigmoid<T>(gate));
   }
 }
 
@@ -724,10 +883,19 @@ int launch_decode(const A& a, cudaStream_t stream) {
 template <bool DELTA, int R>
 int launch_scan_r(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl) {
   constexpr int DKP = 8 * R;
-  // columns per block: a quarter of the value head per warp, fewer when the grid would not fill the machine
-  int warps = (p.dv + 15) / 16;
-  if (warps > 4) warps = 4;
-  while (warps > 1 && static_cast<long long>(B) * p.H * ((p.dv + warps * 16 - 1) / (warps * 16)) < 148) warps /= 2;
+  // Warps (16 columns each) per block: as many as share the staged q / k / decay rows without loading one SM more than
+  // another - all warps run from the first token to the last, so the fullest SM decides.
+  const int most = p.dv <= 16 ? 1 : (p.dv <= 32 ? 2 : 4);
+  int warps = most;
+  long long best = -1;
+  for (int w = most; w >= 1; w /= 2) {
+    const long long blocks = static_cast<long long>(B) * p.H * ((p.dv + w * 16 - 1) / (w * 16));
+    const long long load = (blocks + 147) / 148 * w;
+    if (best < 0 || load < best) {
+      best = load;
+      warps = w;
+    }
+  }
   const int cs = warps * 16;
   const int smem = 2 * kChunk * ((DELTA ? 3 : 2) * DKP + cs + 4) * 4;
   auto kern = scan_kernel<DELTA, R>;
@@ -749,13 +917,21 @@ int launch_scan(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl
   }
 }
 
+template <typename T, int TAPS>
+int launch_delta_prep(const ortb200_gated_delta_args& a, const Scratch& s, int dkp, int dvp, cudaStream_t stream, bool pdl) {
+  const dim3 grid((a.T + kPrepRun - 1) / kPrepRun, (a.kv_heads + 2 * a.heads + 7) / 8);
+  if (dkp == 64) return launch_kernel(delta_prep_kernel<T, TAPS, 2>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
+  if (dkp == 128) return launch_kernel(delta_prep_kernel<T, TAPS, 4>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
+  return launch_kernel(delta_prep_kernel<T, TAPS, 8>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
+}
+
 template <typename T>
 int run_delta(const ortb200_gated_delta_args& a, cudaStream_t stream) {
   if (a.T == a.B) return launch_decode<T, ortb200_gated_delta_args>(a, stream);
   const bool pdl = a.use_pdl != 0;
   const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
   const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.kv_heads, dkp, dvp);
-  int rc = launch_kernel(delta_prep_kernel<T>, dim3(a.T), 256, 0, stream, pdl, a, s, dkp, dvp);
+  int rc = a.taps == 4 ? launch_delta_prep<T, 4>(a, s, dkp, dvp, stream, pdl) : launch_delta_prep<T, 0>(a, s, dkp, dvp, stream, pdl);
   if (rc) return rc;
   ScanParams p{s, a.state, nullptr, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.kv_heads, a.dk, a.dv, dvp, a.num_slots, 0.f, a.status};
   rc = launch_scan<true>(p, a.B, a.T, stream, pdl);
@@ -768,7 +944,8 @@ int run_delta(const ortb200_gated_delta_args& a, cudaStream_t stream) {
   q.conv_in = a.qkvb; q.conv_state = a.conv_state; q.conv_ld = a.ld;
   q.channels = 2 * a.kv_heads * a.dk + a.heads * a.dv; q.taps = a.taps;
   q.cu_seqlens = a.cu_seqlens; q.past_seqlens = a.past_seqlens; q.slots = a.slots; q.B = a.B; q.num_slots = a.num_slots;
-  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T), 256, 0, stream, pdl, q);
+  q.vec = post_vec<T>(q);
+  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T, (a.heads + 7) / 8), 256, 0, stream, pdl, q);
 }
 
 template <typename T>
@@ -777,7 +954,7 @@ int run_mlstm(const ortb200_mlstm_args& a, cudaStream_t stream) {
   const bool pdl = a.use_pdl != 0;
   const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
   const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.heads, dkp, dvp);
-  int rc = launch_kernel(mlstm_prep_kernel<T>, dim3(a.T), 256, 0, stream, pdl, a, s, dkp, dvp);
+  int rc = launch_kernel(mlstm_prep_kernel<T>, dim3(a.T, (a.heads + 7) / 8), 256, 0, stream, pdl, a, s, dkp, dvp);
   if (rc) return rc;
   ScanParams p{s, a.state, a.aux, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.heads, a.dk, a.dv, dvp, a.num_slots, a.den_eps, a.status};
   rc = launch_scan<false>(p, a.B, a.T, stream, pdl);
@@ -789,7 +966,8 @@ int run_mlstm(const ortb200_mlstm_args& a, cudaStream_t stream) {
   q.out = a.out; q.H = a.heads; q.dv = a.dv; q.dvp = dvp; q.eps = a.norm_eps;
   q.aux_out = s.aux_out; q.aux = a.aux; q.dk = a.dk;
   q.cu_seqlens = a.cu_seqlens; q.past_seqlens = a.past_seqlens; q.slots = a.slots; q.B = a.B; q.num_slots = a.num_slots;
-  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T), 256, 0, stream, pdl, q);
+  q.vec = post_vec<T>(q);
+  return launch_kernel(recurrent_post_kernel<T>, dim3(a.T, (a.heads + 7) / 8), 256, 0, stream, pdl, q);
 }
 
 bool sizes_ok(int T, int B, int heads, int dk, int dv, int num_slots) {

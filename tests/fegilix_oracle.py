@@ -10,6 +10,17 @@ import torch
 F64 = torch.float64
 
 
+ROUND_16 = False     # round what enters and leaves every projection to bfloat16: shows how much a model amplifies rounding
+
+
+def round_16(x):
+    return x.to(torch.bfloat16).to(x.dtype) if ROUND_16 else x
+
+
+def lin(x, w):
+    return round_16(round_16(x) @ w.T)
+
+
 def rms(x, eps):
     return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
 
@@ -118,29 +129,29 @@ def causal_attention(q, k, v, scale, sink):
 def channel_delta(h, w, p, m, eps):
     T = h.shape[0]
     H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = causal_conv_silu(h @ w[p + "q"].T, w[p + "q.conv"]).view(T, G, dk)
-    k = causal_conv_silu(h @ w[p + "k"].T, w[p + "k.conv"]).view(T, G, dk)
-    v = causal_conv_silu(h @ w[p + "v"].T, w[p + "v.conv"]).view(T, H, dv)
+    q = causal_conv_silu(lin(h, w[p + "q"]), w[p + "q.conv"]).view(T, G, dk)
+    k = causal_conv_silu(lin(h, w[p + "k"]), w[p + "k.conv"]).view(T, G, dk)
+    v = causal_conv_silu(lin(h, w[p + "v"]), w[p + "v.conv"]).view(T, H, dv)
     q, k = unit(q) * dk ** -0.5, unit(k)
     q, k = q.repeat_interleave(H // G, 1), k.repeat_interleave(H // G, 1)
-    beta = torch.sigmoid(h @ w[p + "b"].T)
-    rate = torch.nn.functional.softplus((h @ w[p + "a1"].T) @ w[p + "a2"].T + w[p + "dt_bias"], threshold=1e9).view(T, H, dk)
+    beta = torch.sigmoid(lin(h, w[p + "b"]))
+    rate = torch.nn.functional.softplus(lin(lin(h, w[p + "a1"]), w[p + "a2"]) + w[p + "dt_bias"], threshold=1e9).view(T, H, dk)
     decay = torch.exp(-torch.exp(w[p + "A_log"])[None, :, None] * rate)
     o = rms_norm(gated_delta_scan(q, k, v, beta, decay), w[p + "norm"], eps)
-    gate = torch.sigmoid((h @ w[p + "g1"].T) @ w[p + "g2"].T).view(T, H, dv)
-    return (o * gate).reshape(T, H * dv) @ w[p + "o"].T
+    gate = torch.sigmoid(lin(lin(h, w[p + "g1"]), w[p + "g2"])).view(T, H, dv)
+    return lin((o * gate).reshape(T, H * dv), w[p + "o"])
 
 
 def mlstm(h, w, p, m, eps):
     T = h.shape[0]
     H, dk, dv, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
-    q = (h @ w[p + "q"].T * dk ** -0.5).view(T, H, dk)
-    k = (h @ w[p + "k"].T).view(T, H, dk)
-    v = (h @ w[p + "v"].T).view(T, H, dv)
-    i_gate = cap * torch.tanh((h @ w[p + "i"].T + w[p + "i.b"]) / cap)
-    f_gate = torch.nn.functional.logsigmoid(cap * torch.tanh((h @ w[p + "f"].T + w[p + "f.b"]) / cap))
+    q = (lin(h, w[p + "q"]) * dk ** -0.5).view(T, H, dk)
+    k = (lin(h, w[p + "k"])).view(T, H, dk)
+    v = (lin(h, w[p + "v"])).view(T, H, dv)
+    i_gate = cap * torch.tanh((lin(h, w[p + "i"]) + w[p + "i.b"]) / cap)
+    f_gate = torch.nn.functional.logsigmoid(cap * torch.tanh((lin(h, w[p + "f"]) + w[p + "f.b"]) / cap))
     o = rms(mlstm_scan(q, k, v, i_gate, f_gate), eps).reshape(T, H * dv)
-    return (o * w[p + "norm"] * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+    return lin(o * w[p + "norm"] * torch.sigmoid(lin(h, w[p + "g"])), w[p + "o"])
 
 
 def attention(h, w, p, m, eps, kv=None):
@@ -149,17 +160,17 @@ def attention(h, w, p, m, eps, kv=None):
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     pos = torch.arange(T)
     turn = (lambda x: rotate(x, pos, m["rot"])) if m.get("rot") else (lambda x: x)
-    q = turn(rms_norm((h @ w[p + "q"].T).view(T, H, d), w[p + "q.norm"], eps))
+    q = turn(rms_norm((lin(h, w[p + "q"])).view(T, H, d), w[p + "q.norm"], eps))
     if kv is None:
-        k = turn(rms_norm((h @ w[p + "k"].T).view(T, G, d), w[p + "k.norm"], eps))
-        v = (h @ w[p + "v"].T).view(T, G, dv)
+        k = turn(rms_norm((lin(h, w[p + "k"])).view(T, G, d), w[p + "k.norm"], eps))
+        v = (lin(h, w[p + "v"])).view(T, G, dv)
         kv = (k, v)
     o = causal_attention(q, kv[0], kv[1], m["scale"], w[p + "sink"]).reshape(T, H * dv)
-    return (o * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T, kv
+    return lin(o * torch.sigmoid(lin(h, w[p + "g"])), w[p + "o"]), kv
 
 
 def dense_ff(h, w, p):
-    return (gelu_tanh(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
+    return lin(gelu_tanh(lin(h, w[p + "gate"])) * lin(h, w[p + "up"]), w[p + "down"])
 
 
 def hyper_read(streams, w_in):
@@ -207,3 +218,14 @@ def forward(config, weights, tokens, layers_out=None):
     logits = rms_norm(streams.sum(1), w["final.norm"], eps) @ w["head"].T
     cap = config.get("logit_softcap")
     return cap * torch.tanh(logits / cap) if cap else logits
+
+
+def rounding_noise(config, weights, tokens):
+    """Difference of the logits that 16-bit projections alone make, [T, vocab]."""
+    global ROUND_16
+    exact = forward(config, weights, tokens)
+    ROUND_16 = True
+    try:
+        return forward(config, weights, tokens) - exact
+    finally:
+        ROUND_16 = False
