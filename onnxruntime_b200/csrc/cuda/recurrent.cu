@@ -13,8 +13,12 @@
 // One token per sequence (decode): one launch, one block per (head, sequence) that does all of it; the state is read
 // once and written once, which is what bounds the step.
 //
-// Both products of a delta-rule step come from one pass over the old state: with S' = diag(g) S,
-// o = (S' + k u^T)^T q = S'^T q + (k . q) u.
+// The delta-rule scan takes four tokens at a time.  With P_t = g_1 ... g_t the decays since the block began,
+//   S_t^T k_{t+1} etc. need only products with the state at the block's start:
+//   a_t = S^T (P_t k_t) + sum_{j<t} (k_t . g_{j+1..t} k_j) u_j,   u_t = beta_t (v_t - a_t)
+//   o_t = S^T (P_t q_t) + sum_{j<=t} (q_t . g_{j+1..t} k_j) u_j,  S' = P_4 S + sum_j (g_{j+1..4} k_j) u_j^T
+// All factors are products of decays (no quotients), so nothing can overflow; the prep kernel forms them, and the scan
+// does 13 multiply-adds per state element and block instead of 16, with one chain of reductions instead of four.
 #include <cuda_runtime.h>
 #include <math.h>
 #include <type_traits>
@@ -34,27 +38,37 @@ constexpr int kMaxTaps = 16;
 int pad_dk(int dk) { return dk <= 64 ? 64 : (dk <= 128 ? 128 : 256); }
 int pad4(int n) { return (n + 3) / 4 * 4; }
 
-// fp32 scratch of a multi-token call
+// fp32 scratch of a multi-token call.  mLSTM rows are indexed by packed token; the delta rule keeps blocks of kBlock tokens
+// of one sequence: block i of sequence b is number cu_seqlens[b] / kBlock + b + i, which never collides.
+constexpr int kBlock = 4;
+constexpr int kVecs = 3 * kBlock + 1;     // P_t k_t, P_t q_t, g_{j+1..4} k_j, P_4
+constexpr int kScal = 20;                 // beta_t (4), k_t . g k_j for j < t (6), q_t . g k_j for j <= t (10)
 struct Scratch {
-  float* qk;      // [T, G, 2, dkp]: q row, then k row
-  float* decay;   // [T, H, dkp] (delta rule only)
-  float* v;       // [T, H, dvp]
-  float* scal;    // [T, H, 4]: delta: beta, q.k, -, -;  mLSTM: i, f, q.k, -
+  float* vec;     // delta: [blocks, H, kVecs, dkp];  mLSTM: [T, H, 2, dkp] q row, then k row
+  float* v;       // delta: [blocks, kBlock, H, dvp];  mLSTM: [T, H, dvp]
+  float* scal;    // delta: [blocks, H, kScal];        mLSTM: [T, H, 4] log gates i, f
   float* o;       // [T, H, dvp]
-  float* aux_out; // [B, H, dk + 1] (mLSTM only): n and m after the last token
+  float* aux_out; // mLSTM: [B, H, dk + 1] n and m after the last token
 };
 
-int64_t scratch_floats(int T, int H, int G, int dkp, int dvp) {
-  return static_cast<int64_t>(T) * (static_cast<int64_t>(G) * 2 * dkp + static_cast<int64_t>(H) * (dkp + 2 * dvp + 4));
+struct ScratchSizes {
+  int64_t vec, v, scal, o, aux;
+  int64_t total() const { return vec + v + scal + o + aux; }
+};
+ScratchSizes delta_scratch(int64_t T, int64_t B, int64_t H, int64_t dkp, int64_t dvp) {
+  const int64_t blocks = T / kBlock + B;
+  return {blocks * H * kVecs * dkp, blocks * kBlock * H * dvp, blocks * H * kScal, T * H * dvp, 0};
 }
-Scratch split_scratch(float* w, int T, int H, int G, int dkp, int dvp) {
+ScratchSizes mlstm_scratch(int64_t T, int64_t B, int64_t H, int64_t dk, int64_t dkp, int64_t dvp) {
+  return {T * H * 2 * dkp, T * H * dvp, T * H * 4, T * H * dvp, B * H * (dk + 1)};
+}
+Scratch split_scratch(float* w, const ScratchSizes& n) {
   Scratch s;
-  s.qk = w;
-  s.decay = s.qk + static_cast<int64_t>(T) * G * 2 * dkp;
-  s.v = s.decay + static_cast<int64_t>(T) * H * dkp;
-  s.scal = s.v + static_cast<int64_t>(T) * H * dvp;
-  s.o = s.scal + static_cast<int64_t>(T) * H * 4;
-  s.aux_out = s.o + static_cast<int64_t>(T) * H * dvp;
+  s.vec = w;
+  s.v = s.vec + n.vec;
+  s.scal = s.v + n.v;
+  s.o = s.scal + n.scal;
+  s.aux_out = s.o + n.o;
   return s;
 }
 
@@ -150,123 +164,174 @@ struct ConvWindow<T, 0, NI> {
   }
 };
 
+// Sums of 16 values over the warp: lane l ends with the sum of x[l & 15].
+__device__ __forceinline__ float reduce16(const float (&x)[16], int lane) {
+  float y[8], z[4], w[2];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const float send = (lane & 8) ? x[i] : x[8 + i], keep = (lane & 8) ? x[8 + i] : x[i];
+    y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float send = (lane & 4) ? y[i] : y[4 + i], keep = (lane & 4) ? y[4 + i] : y[i];
+    z[i] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const float send = (lane & 2) ? z[i] : z[2 + i], keep = (lane & 2) ? z[2 + i] : z[i];
+    w[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+  }
+  const float send = (lane & 1) ? w[0] : w[1], keep = (lane & 1) ? w[1] : w[0];
+  const float r = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+  return r + __shfl_xor_sync(0xffffffffu, r, 16);
+}
+
+// A warp owns one head (q, k and decays, or values) and a run of kPrepRun tokens of one sequence.
 template <typename T, int TAPS, int NI>
-__global__ void __launch_bounds__(256, NI <= 4 ? 3 : 1) delta_prep_kernel(const ortb200_gated_delta_args a, const Scratch s, int dkp, int dvp) {
+__global__ void __launch_bounds__(256, NI <= 4 ? 2 : 1) delta_prep_kernel(const ortb200_gated_delta_args a, const Scratch s, int dkp, int dvp) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.heads, G = a.kv_heads, dk = a.dk, dv = a.dv;
   const int channels = 2 * G * dk + H * dv;
-  const int u = blockIdx.y * 8 + warp;              // G (q and k of a key head), then H value heads, then H decay heads
+  const int unit = blockIdx.y * 8 + warp;           // H key heads (one per value head: each has its own decays), H value heads
   pdl_wait_prior_grids();
   pdl_launch_dependents();
-  if (u >= G + 2 * H) return;
-  const int t0 = blockIdx.x * kPrepRun, t1 = min(a.T, t0 + kPrepRun);
-  if (u >= G + H) {
-    const int h = u - G - H;
-    const float rate = expf(a.a_log[h]);
-    for (int t = t0; t < t1; ++t) {
-      const T* low = static_cast<const T*>(a.low) + static_cast<long long>(t) * H * (dk + dv) + h * dk;
-      float* row = s.decay + (static_cast<long long>(t) * H + h) * dkp;
-      for (int d = lane; d < dkp; d += 32) row[d] = d < dk ? expf(-rate * softplus_f(to_float<T>(low[d]) + a.dt_bias[h * dk + d])) : 0.f;
-      if (lane == 0) s.scal[(static_cast<long long>(t) * H + h) * 4] = sigmoid_f(to_float<T>(static_cast<const T*>(a.qkvb)[static_cast<long long>(t) * a.ld + channels + h]));
-    }
-    return;
+  if (unit >= 2 * H) return;
+  int run = blockIdx.x, b = 0, first = 0, len = 0;  // runs of all sequences are numbered consecutively
+  for (; b < a.B; ++b) {
+    first = a.cu_seqlens[b];
+    len = a.cu_seqlens[b + 1] - first;
+    const int runs = (len + kPrepRun - 1) / kPrepRun;
+    if (run < runs) break;
+    run -= runs;
   }
-  int b = sequence_of(a.cu_seqlens, a.B, t0), next = a.cu_seqlens[b + 1];
-  bool fill = true;
-  const T* ring = nullptr;
-  int pos = 0, before = 0;
-  // position of token t; true when the window has to be (re)loaded
-  auto locate = [&](int t) {
-    if (fill || t >= next) {
-      while (t >= next) next = a.cu_seqlens[++b + 1];
-      const int slot = a.slots[b];
-      const bool ok = slot >= 0 && slot < a.num_slots;
-      if (!ok && a.status && lane == 0) atomicExch(a.status, kStatusBadArgument);
-      ring = static_cast<const T*>(a.conv_state) + static_cast<long long>(ok ? slot : 0) * a.taps * channels;
-      before = t - a.cu_seqlens[b];
-      pos = a.past_seqlens[b] + before;
-      fill = false;
-      return true;
-    }
-    ++before;
-    ++pos;
-    return false;
-  };
+  if (b == a.B) return;
+  const int slot = a.slots[b], past = a.past_seqlens[b];
+  const bool ok = slot >= 0 && slot < a.num_slots;
+  if (!ok && a.status && lane == 0) atomicExch(a.status, kStatusBadArgument);
+  const T* ring = static_cast<const T*>(a.conv_state) + static_cast<long long>(ok ? slot : 0) * a.taps * channels;
+  const int i0 = run * kPrepRun, i1 = min(len, i0 + kPrepRun);
+  const long long block0 = first / kBlock + b;
   const T* base = static_cast<const T*>(a.qkvb);
-  if (u < G) {
+  if (unit < H) {
+    const int h = unit, u = h / (H / G), cq = u * dk, ck = (G + u) * dk;
     ConvWindow<T, TAPS, NI> wq, wk;
-    const int cq = u * dk, ck = (G + u) * dk;
     if constexpr (TAPS > 0) {
       wq.load_taps(a.conv, cq, dk, lane);
       wk.load_taps(a.conv, ck, dk, lane);
+      const T* row = base + static_cast<long long>(first + i0) * a.ld;
+      wq.refill(row + cq, a.ld, ring, channels, cq, dk, lane, past + i0, i0);
+      wk.refill(row + ck, a.ld, ring, channels, ck, dk, lane, past + i0, i0);
     }
-    const float root = 1.f / sqrtf(static_cast<float>(dk));
-    const int group = H / G;
-    for (int t = t0; t < t1; ++t) {
-      const bool refill = locate(t);
-      const T* row = base + static_cast<long long>(t) * a.ld;
-      float q[NI], k[NI];
-      if constexpr (TAPS > 0) {
-        if (refill) {
-          wq.refill(row + cq, a.ld, ring, channels, cq, dk, lane, pos, before);
-          wk.refill(row + ck, a.ld, ring, channels, ck, dk, lane, pos, before);
+    const float root = 1.f / sqrtf(static_cast<float>(dk)), rate = expf(a.a_log[h]);
+    for (int ib = i0; ib < i1; ib += kBlock) {
+      float q[kBlock][NI], k[kBlock][NI], g[kBlock][NI], beta = 0.f;
+#pragma unroll
+      for (int j = 0; j < kBlock; ++j) {
+        const int i = ib + j;
+        if (i < i1) {
+          const long long t = first + i;
+          if constexpr (TAPS > 0) {
+            const T* row = base + t * a.ld;
+            wq.step(row + cq, dk, lane, q[j]);
+            wk.step(row + ck, dk, lane, k[j]);
+          } else {
+            wq = {&a, ring, channels, cq, past + i, i, t};
+            wk = {&a, ring, channels, ck, past + i, i, t};
+            wq.step(dk, lane, q[j]);
+            wk.step(dk, lane, k[j]);
+          }
+          float qq = 0.f, kk = 0.f;
+#pragma unroll
+          for (int n = 0; n < NI; ++n) {
+            qq = fmaf(q[j][n], q[j][n], qq);
+            kk = fmaf(k[j][n], k[j][n], kk);
+          }
+#pragma unroll
+          for (int off = 16; off > 0; off >>= 1) {
+            qq += __shfl_xor_sync(0xffffffffu, qq, off);
+            kk += __shfl_xor_sync(0xffffffffu, kk, off);
+          }
+          const float qs = root / sqrtf(qq + a.unit_eps), ks = 1.f / sqrtf(kk + a.unit_eps);
+          const T* low = static_cast<const T*>(a.low) + t * H * (dk + dv) + h * dk;
+#pragma unroll
+          for (int n = 0; n < NI; ++n) {
+            const int d = n * 32 + lane;
+            q[j][n] *= qs;
+            k[j][n] *= ks;
+            g[j][n] = d < dk ? expf(-rate * softplus_f(to_float<T>(low[d]) + a.dt_bias[h * dk + d])) : 1.f;
+          }
+          if (lane == j) beta = sigmoid_f(to_float<T>(base[t * a.ld + channels + h]));
+        } else {   // behind the end: tokens that leave the state alone
+#pragma unroll
+          for (int n = 0; n < NI; ++n) {
+            q[j][n] = k[j][n] = 0.f;
+            g[j][n] = 1.f;
+          }
         }
-        wq.step(row + cq, dk, lane, q);
-        wk.step(row + ck, dk, lane, k);
-      } else {
-        wq = {&a, ring, channels, cq, pos, before, t};
-        wk = {&a, ring, channels, ck, pos, before, t};
-        wq.step(dk, lane, q);
-        wk.step(dk, lane, k);
       }
-      float qq = 0.f, kk = 0.f, qk = 0.f;
+      const long long blk = block0 + ib / kBlock;
+      float* out = s.vec + (blk * H + h) * kVecs * dkp + lane;
+      float dots[16];
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        qq = fmaf(q[i], q[i], qq);
-        kk = fmaf(k[i], k[i], kk);
-        qk = fmaf(q[i], k[i], qk);
-      }
+      for (int n = 0; n < 16; ++n) dots[n] = 0.f;
 #pragma unroll
-      for (int off = 16; off > 0; off >>= 1) {
-        qq += __shfl_xor_sync(0xffffffffu, qq, off);
-        kk += __shfl_xor_sync(0xffffffffu, kk, off);
-        qk += __shfl_xor_sync(0xffffffffu, qk, off);
-      }
-      const float qs = root / sqrtf(qq + a.unit_eps), ks = 1.f / sqrtf(kk + a.unit_eps);
-      float* out = s.qk + (static_cast<long long>(t) * G + u) * 2 * dkp;
+      for (int n = 0; n < NI; ++n) {
+        float P = 1.f;
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {   // dkp == 32 * NI
-        out[i * 32 + lane] = q[i] * qs;
-        out[dkp + i * 32 + lane] = k[i] * ks;
+        for (int j = 0; j < kBlock; ++j) {
+          P *= g[j][n];
+          out[j * dkp + n * 32] = P * k[j][n];
+          out[(kBlock + j) * dkp + n * 32] = P * q[j][n];
+        }
+        out[3 * kBlock * dkp + n * 32] = P;
+        // k_t . g k_j ordered by t, then j < t; behind them q_t . g k_j ordered by t, then j <= t
+#pragma unroll
+        for (int j = 0; j < kBlock; ++j) {
+          float x = k[j][n];
+          dots[6 + j * (j + 1) / 2 + j] = fmaf(q[j][n], x, dots[6 + j * (j + 1) / 2 + j]);
+#pragma unroll
+          for (int t = j + 1; t < kBlock; ++t) {
+            x *= g[t][n];
+            dots[t * (t - 1) / 2 + j] = fmaf(k[t][n], x, dots[t * (t - 1) / 2 + j]);
+            dots[6 + t * (t + 1) / 2 + j] = fmaf(q[t][n], x, dots[6 + t * (t + 1) / 2 + j]);
+          }
+          out[(2 * kBlock + j) * dkp + n * 32] = x;
+        }
       }
-      for (int j = lane; j < group; j += 32) s.scal[(static_cast<long long>(t) * H + u * group + j) * 4 + 1] = qk * qs * ks;
+      const float sum = reduce16(dots, lane);
+      float* sc = s.scal + (blk * H + h) * kScal;
+      if (lane < kBlock) sc[lane] = beta;
+      if (lane < 16) sc[kBlock + lane] = sum;
     }
   } else {
-    const int h = u - G, cv = 2 * G * dk + h * dv;
-    for (int c0 = 0; c0 < dv; c0 += NI * 32) {
+    const int h = unit - H, cv = 2 * G * dk + h * dv;
+    for (int c0 = 0; c0 < dvp; c0 += NI * 32) {
       const int n = dv - c0;
       ConvWindow<T, TAPS, NI> wv;
-      if constexpr (TAPS > 0) wv.load_taps(a.conv, cv + c0, n, lane);
-      if (c0 > 0) {
-        b = sequence_of(a.cu_seqlens, a.B, t0);
-        next = a.cu_seqlens[b + 1];
-        fill = true;
+      if constexpr (TAPS > 0) {
+        wv.load_taps(a.conv, cv + c0, n, lane);
+        wv.refill(base + static_cast<long long>(first + i0) * a.ld + cv + c0, a.ld, ring, channels, cv + c0, n, lane, past + i0, i0);
       }
-      for (int t = t0; t < t1; ++t) {
-        const bool refill = locate(t);
-        const T* row = base + static_cast<long long>(t) * a.ld + cv + c0;
+      const int padded = (i1 + kBlock - 1) / kBlock * kBlock;
+      for (int i = i0; i < padded; ++i) {
+        const long long t = first + i;
         float v[NI];
-        if constexpr (TAPS > 0) {
-          if (refill) wv.refill(row, a.ld, ring, channels, cv + c0, n, lane, pos, before);
-          wv.step(row, n, lane, v);
+        if (i < i1) {
+          if constexpr (TAPS > 0) {
+            wv.step(base + t * a.ld + cv + c0, n, lane, v);
+          } else {
+            wv = {&a, ring, channels, cv + c0, past + i, i, t};
+            wv.step(n, lane, v);
+          }
         } else {
-          wv = {&a, ring, channels, cv + c0, pos, before, t};
-          wv.step(n, lane, v);
-        }
-        float* out = s.v + (static_cast<long long>(t) * H + h) * dvp + c0;
 #pragma unroll
-        for (int i = 0; i < NI; ++i)
-          if (c0 + i * 32 + lane < dvp) out[i * 32 + lane] = v[i];
+          for (int e = 0; e < NI; ++e) v[e] = 0.f;
+        }
+        float* out = s.v + ((block0 * kBlock + i) * H + h) * dvp + c0;
+#pragma unroll
+        for (int e = 0; e < NI; ++e)
+          if (c0 + e * 32 + lane < dvp) out[e * 32 + lane] = v[e];
       }
     }
   }
@@ -283,16 +348,13 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const ortb200_mlstm_arg
   const T* row = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld;
   const float qs = 1.f / sqrtf(static_cast<float>(dk));
   if (h < H) {
-    float* qk = s.qk + (static_cast<long long>(t) * H + h) * 2 * dkp;
-    float dot = 0.f;
+    float* qk = s.vec + (static_cast<long long>(t) * H + h) * 2 * dkp;
     for (int d = lane; d < dkp; d += 32) {
       const float q = d < dk ? to_float<T>(row[h * dk + d]) * qs : 0.f;
       const float k = d < dk ? to_float<T>(row[(H + h) * dk + d]) : 0.f;
       qk[d] = q;
       qk[dkp + d] = k;
-      dot = fmaf(q, k, dot);
     }
-    dot = warp_sum(dot);
     const T* v = row + 2 * H * dk + h * dv;
     float* vr = s.v + (static_cast<long long>(t) * H + h) * dvp;
     for (int d = lane; d < dvp; d += 32) vr[d] = d < dv ? to_float<T>(v[d]) : 0.f;
@@ -301,12 +363,11 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const ortb200_mlstm_arg
       float* sc = s.scal + (static_cast<long long>(t) * H + h) * 4;
       sc[0] = a.gate_cap * tanhf((to_float<T>(gates[h]) + a.i_bias[h]) / a.gate_cap);
       sc[1] = logsigmoid_f(a.gate_cap * tanhf((to_float<T>(gates[H + h]) + a.f_bias[h]) / a.gate_cap));
-      sc[2] = dot;
     }
   }
 }
 
-// ---------------------------------------------------------------------------------------------------------- the scan
+// --------------------------------------------------------------------------------------------------------- the scans
 struct ScanParams {
   Scratch s;
   float* state;            // [num_slots, H, dk, dv]
@@ -314,7 +375,7 @@ struct ScanParams {
   const int* cu_seqlens;
   const int* past_seqlens;
   const int* slots;
-  int H, G, dk, dv, dvp, num_slots;
+  int H, dk, dv, dvp, num_slots;
   float den_eps;
   int* status;
 };
@@ -326,22 +387,218 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// R = state rows per lane; dkp = 8 R.  Lane (rg = lane & 7, cg = lane >> 3) holds rows j * 32 + rg * 4 + {0..3},
-// j < R / 4, of columns col0 .. col0 + 3.
-template <bool DELTA, int R>
-__global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) scan_kernel(const ScanParams p) {
+// The warp's slice of the state in registers: lane (rg = lane & 7, cg = lane >> 3) holds rows j * 32 + rg * 4 + {0..3},
+// j < NJ, of the columns col0 ... col0 + 3, as pairs of rows.
+template <int NJ>
+struct StateSlice {
+  f32x2 S[NJ][4][2];
+  __device__ __forceinline__ void load(const float* g, int rg, int col0, int dk, int dv, bool fresh) {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const int r = j * 32 + rg * 4 + hh * 2;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          float lo = 0.f, hi = 0.f;
+          if (!fresh && col0 + c < dv) {
+            if (r < dk) lo = g[static_cast<long long>(r) * dv + col0 + c];
+            if (r + 1 < dk) hi = g[static_cast<long long>(r + 1) * dv + col0 + c];
+          }
+          S[j][c][hh] = pack2(lo, hi);
+        }
+      }
+    }
+  }
+  __device__ __forceinline__ void store(float* g, int rg, int col0, int dk, int dv) const {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const int r = j * 32 + rg * 4 + hh * 2;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          if (col0 + c >= dv) continue;
+          float lo, hi;
+          unpack2(S[j][c][hh], lo, hi);
+          if (r < dk) g[static_cast<long long>(r) * dv + col0 + c] = lo;
+          if (r + 1 < dk) g[static_cast<long long>(r + 1) * dv + col0 + c] = hi;
+        }
+      }
+    }
+  }
+};
+__device__ __forceinline__ float hsum(f32x2 v) {
+  float lo, hi;
+  unpack2(v, lo, hi);
+  return lo + hi;
+}
+
+constexpr int kStageBlocks = 2;   // delta blocks per shared-memory stage
+
+// R = state rows per lane; dkp = 8 R.
+template <int R>
+__global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) delta_scan_kernel(const ScanParams p) {
   constexpr int DKP = 8 * R, NJ = R / 4;
-  constexpr int kRows = DELTA ? 3 : 2;             // q, k (, decay)
-  const int warps = blockDim.x >> 5;
-  const int cs = warps * 16;                       // columns per block
+  const int cs = (blockDim.x >> 5) * 16;           // columns per block
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7, cg = lane >> 3;
   const int h = blockIdx.y, b = blockIdx.z;
-  const int g = h / (p.H / p.G);
   const int base_col = blockIdx.x * cs;
   const int wcol = warp * 16 + cg * 4;             // column within the block's slice
   const int col0 = base_col + wcol;
   extern __shared__ __align__(16) float sm[];
-  const int stage_floats = kChunk * (kRows * DKP + cs + 4);
+  const int block_floats = kVecs * DKP + kBlock * cs + kScal;
+  const int stage_floats = kStageBlocks * block_floats;
+
+  pdl_wait_prior_grids();
+  const int t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len <= 0) return;
+  const int slot = p.slots[b];
+  if (!slot_ok(slot, p.num_slots, p.status)) return;
+  const bool fresh = p.past_seqlens[b] == 0;
+  const long long block0 = t0 / kBlock + b;
+  const int blocks = (len + kBlock - 1) / kBlock;
+
+  auto fetch = [&](int stage) {
+    float* st = sm + (stage & 1) * stage_floats;
+    const int n = min(kStageBlocks, blocks - stage * kStageBlocks);
+    for (int i = 0; i < n; ++i) {
+      const long long blk = block0 + stage * kStageBlocks + i;
+      float* dst = st + i * block_floats;
+      const float* vec = p.s.vec + (blk * p.H + h) * kVecs * DKP;
+      for (int c = threadIdx.x; c < kVecs * DKP / 4; c += blockDim.x) cp_async16(dst + c * 4, vec + c * 4);
+      dst += kVecs * DKP;
+      const int vq = cs / 4;
+      for (int c = threadIdx.x; c < kBlock * vq; c += blockDim.x) {
+        const int tt = c / vq, x = c % vq;
+        if (base_col + x * 4 < p.dvp) cp_async16(dst + tt * cs + x * 4, p.s.v + ((blk * kBlock + tt) * p.H + h) * p.dvp + base_col + x * 4);
+      }
+      dst += kBlock * cs;
+      if (threadIdx.x < kScal / 4) cp_async16(dst + threadIdx.x * 4, p.s.scal + (blk * p.H + h) * kScal + threadIdx.x * 4);
+    }
+    cp_async_commit();
+  };
+
+  float* gst = p.state + (static_cast<long long>(slot) * p.H + h) * p.dk * p.dv;
+  StateSlice<NJ> st;
+  st.load(gst, rg, col0, p.dk, p.dv, fresh);
+  const long long ostep = static_cast<long long>(p.H) * p.dvp;
+  float* orow = p.s.o + (static_cast<long long>(t0) * p.H + h) * p.dvp + col0 + (rg & 3);
+  const bool writes = rg >= 4 && col0 + (rg & 3) < p.dv;
+
+  const int stages = (blocks + kStageBlocks - 1) / kStageBlocks;
+  fetch(0);
+  for (int stage = 0; stage < stages; ++stage) {
+    if (stage + 1 < stages) {
+      fetch(stage + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const int n = min(kStageBlocks, blocks - stage * kStageBlocks);
+    for (int i = 0; i < n; ++i) {
+      const float* vec = sm + (stage & 1) * stage_floats + i * block_floats + rg * 4;
+      const float* vrow = sm + (stage & 1) * stage_floats + i * block_floats + kVecs * DKP + wcol + (rg & 3);
+      const float* sc = sm + (stage & 1) * stage_floats + i * block_floats + kVecs * DKP + kBlock * cs;
+      // lane rg ends with S^T (P_t k_t) of column rg (rg < 4), or S^T (P_t q_t) of column rg - 4
+      float w[kBlock];
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) {
+        f32x2 accA[4], accO[4];
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(vec + t * DKP + j * 32);
+          const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(vec + (kBlock + t) * DKP + j * 32);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            accA[c] = j == 0 ? mul2(st.S[j][c][0], k2.x) : fma2(st.S[j][c][0], k2.x, accA[c]);
+            accO[c] = j == 0 ? mul2(st.S[j][c][0], q2.x) : fma2(st.S[j][c][0], q2.x, accO[c]);
+            accA[c] = fma2(st.S[j][c][1], k2.y, accA[c]);
+            accO[c] = fma2(st.S[j][c][1], q2.y, accO[c]);
+          }
+        }
+        float y[4], z[2];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float xa = hsum(accA[c]), xo = hsum(accO[c]);
+          const float send = (rg & 4) ? xa : xo, keep = (rg & 4) ? xo : xa;
+          y[c] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+        }
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const float send = (rg & 2) ? y[c] : y[2 + c], keep = (rg & 2) ? y[2 + c] : y[c];
+          z[c] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+        }
+        const float send = (rg & 1) ? z[0] : z[1], keep = (rg & 1) ? z[1] : z[0];
+        w[t] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+      }
+      // forward substitution (meaningful on the lanes rg < 4)
+      const float4 beta = *reinterpret_cast<const float4*>(sc), kk0 = *reinterpret_cast<const float4*>(sc + 4);
+      const float2 kk1 = *reinterpret_cast<const float2*>(sc + 8);
+      float u[kBlock];
+      u[0] = beta.x * (vrow[0] - w[0]);
+      u[1] = beta.y * (vrow[cs] - w[1] - kk0.x * u[0]);
+      u[2] = beta.z * (vrow[2 * cs] - w[2] - kk0.y * u[0] - kk0.z * u[1]);
+      u[3] = beta.w * (vrow[3 * cs] - w[3] - kk0.w * u[0] - kk1.x * u[1] - kk1.y * u[2]);
+      // S' = P_4 S + sum_j K_j u_j^T
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const ulonglong2 P = *reinterpret_cast<const ulonglong2*>(vec + 3 * kBlock * DKP + j * 32);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          st.S[j][c][0] = mul2(st.S[j][c][0], P.x);
+          st.S[j][c][1] = mul2(st.S[j][c][1], P.y);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) {
+        f32x2 uu[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float x = __shfl_sync(0xffffffffu, u[t], (lane & 24) | c);
+          uu[c] = pack2(x, x);
+        }
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(vec + (2 * kBlock + t) * DKP + j * 32);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            st.S[j][c][0] = fma2(k2.x, uu[c], st.S[j][c][0]);
+            st.S[j][c][1] = fma2(k2.y, uu[c], st.S[j][c][1]);
+          }
+        }
+      }
+      // outputs (lanes rg >= 4)
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) u[t] = __shfl_sync(0xffffffffu, u[t], (lane & 24) | (rg & 3));
+      const int left = len - (stage * kStageBlocks + i) * kBlock;
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) {
+        float o = w[t];
+#pragma unroll
+        for (int j = 0; j <= t; ++j) o = fmaf(sc[10 + t * (t + 1) / 2 + j], u[j], o);
+        if (writes && t < left) orow[t * ostep] = o;
+      }
+      orow += kBlock * ostep;
+    }
+    __syncthreads();   // the stage may be refilled
+  }
+  pdl_launch_dependents();
+  st.store(gst, rg, col0, p.dk, p.dv);
+}
+
+template <int R>
+__global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) mlstm_scan_kernel(const ScanParams p) {
+  constexpr int DKP = 8 * R, NJ = R / 4;
+  const int cs = (blockDim.x >> 5) * 16;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7, cg = lane >> 3;
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int base_col = blockIdx.x * cs;
+  const int wcol = warp * 16 + cg * 4;
+  const int col0 = base_col + wcol;
+  extern __shared__ __align__(16) float sm[];
+  const int stage_floats = kChunk * (2 * DKP + cs + 4);
 
   pdl_wait_prior_grids();
   const int t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
@@ -355,15 +612,9 @@ __global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) scan_kernel(const ScanPa
     const int first = chunk * kChunk, n = min(kChunk, len - first);
     for (int i = threadIdx.x; i < n * (2 * DKP / 4); i += blockDim.x) {
       const int tt = i / (2 * DKP / 4), c = i % (2 * DKP / 4);
-      cp_async16(st + tt * kRows * DKP + c * 4, p.s.qk + ((static_cast<long long>(t0 + first + tt) * p.G + g) * 2 * DKP) + c * 4);
+      cp_async16(st + tt * 2 * DKP + c * 4, p.s.vec + ((static_cast<long long>(t0 + first + tt) * p.H + h) * 2 * DKP) + c * 4);
     }
-    if (DELTA) {
-      for (int i = threadIdx.x; i < n * (DKP / 4); i += blockDim.x) {
-        const int tt = i / (DKP / 4), c = i % (DKP / 4);
-        cp_async16(st + tt * kRows * DKP + 2 * DKP + c * 4, p.s.decay + (static_cast<long long>(t0 + first + tt) * p.H + h) * DKP + c * 4);
-      }
-    }
-    float* sv = st + kChunk * kRows * DKP;
+    float* sv = st + kChunk * 2 * DKP;
     const int vq = cs / 4;
     for (int i = threadIdx.x; i < n * vq; i += blockDim.x) {
       const int tt = i / vq, c = i % vq;
@@ -375,32 +626,14 @@ __global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) scan_kernel(const ScanPa
   };
 
   float* gst = p.state + (static_cast<long long>(slot) * p.H + h) * p.dk * p.dv;
-  f32x2 S[NJ][4][2];
-#pragma unroll
-  for (int j = 0; j < NJ; ++j) {
-#pragma unroll
-    for (int hh = 0; hh < 2; ++hh) {
-      const int r = j * 32 + rg * 4 + hh * 2;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        float lo = 0.f, hi = 0.f;
-        if (!fresh && col0 + c < p.dv) {
-          if (r < p.dk) lo = gst[static_cast<long long>(r) * p.dv + col0 + c];
-          if (r + 1 < p.dk) hi = gst[static_cast<long long>(r + 1) * p.dv + col0 + c];
-        }
-        S[j][c][hh] = pack2(lo, hi);
-      }
-    }
-  }
-  float* gaux = DELTA ? nullptr : p.aux + (static_cast<long long>(slot) * p.H + h) * (p.dk + 1);
-  constexpr int NR = DKP / 32;                     // mLSTM: every warp keeps n, lane l its rows l, l + 32, ...
+  const float* gaux = p.aux + (static_cast<long long>(slot) * p.H + h) * (p.dk + 1);
+  StateSlice<NJ> s;
+  s.load(gst, rg, col0, p.dk, p.dv, fresh);
+  constexpr int NR = DKP / 32;                     // every warp keeps n, lane l its rows l, l + 32, ...
   float nrm[NR];
-  float m = 0.f;
-  if (!DELTA) {
 #pragma unroll
-    for (int i = 0; i < NR; ++i) nrm[i] = !fresh && i * 32 + lane < p.dk ? gaux[i * 32 + lane] : 0.f;
-    m = fresh ? 0.f : gaux[p.dk];
-  }
+  for (int i = 0; i < NR; ++i) nrm[i] = !fresh && i * 32 + lane < p.dk ? gaux[i * 32 + lane] : 0.f;
+  float m = fresh ? 0.f : gaux[p.dk];
   float* orow = p.s.o + (static_cast<long long>(t0) * p.H + h) * p.dvp + col0;
   const long long ostep = static_cast<long long>(p.H) * p.dvp;
 
@@ -415,147 +648,64 @@ __global__ void __launch_bounds__(128, R <= 16 ? 4 : 2) scan_kernel(const ScanPa
     }
     __syncthreads();
     const float* st = sm + (ch & 1) * stage_floats;
-    const float* sv = st + kChunk * kRows * DKP;
+    const float* sv = st + kChunk * 2 * DKP;
     const float* sc = sv + kChunk * cs;
     const int n = min(kChunk, len - ch * kChunk);
     for (int tt = 0; tt < n; ++tt) {
-      const float* qr = st + tt * kRows * DKP;
+      const float* qr = st + tt * 2 * DKP;
       const float* kr = qr + DKP;
       const float4 vv = *reinterpret_cast<const float4*>(sv + tt * cs + wcol);
-      const float4 scal = *reinterpret_cast<const float4*>(sc + tt * 4);
-      if (DELTA) {
-        const float* gr = kr + DKP;
-        f32x2 accA[4], accO[4];
+      const float2 gate = *reinterpret_cast<const float2*>(sc + tt * 4);
+      const float m_new = fmaxf(gate.y + m, gate.x);
+      const float fw = expf(gate.y + m - m_new), iw = expf(gate.x - m_new);
+      m = m_new;
+      const f32x2 f2 = pack2(fw, fw), i2 = pack2(iw, iw);
+      const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
+      f32x2 accO[4];
+      float nq = 0.f;
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
-          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
-          const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(gr + j * 32 + rg * 4);
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            S[j][c][0] = mul2(S[j][c][0], g2.x);
-            S[j][c][1] = mul2(S[j][c][1], g2.y);
-            accA[c] = j == 0 ? mul2(S[j][c][0], k2.x) : fma2(S[j][c][0], k2.x, accA[c]);
-            accO[c] = j == 0 ? mul2(S[j][c][0], q2.x) : fma2(S[j][c][0], q2.x, accO[c]);
-            accA[c] = fma2(S[j][c][1], k2.y, accA[c]);
-            accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
-          }
-        }
-        // eight sums (S^T k and S^T q of four columns) over the eight row-group lanes: reduce-scatter, lane rg ends with
-        // sum number rg (0..3: S^T k of column rg, 4..7: S^T q of column rg - 4)
-        float x[8];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          float lo, hi;
-          unpack2(accA[c], lo, hi);
-          x[c] = lo + hi;
-          unpack2(accO[c], lo, hi);
-          x[4 + c] = lo + hi;
-        }
-        float y[4], z[2], w;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float send = (rg & 4) ? x[i] : x[4 + i], keep = (rg & 4) ? x[4 + i] : x[i];
-          y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
-        }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const float send = (rg & 2) ? y[i] : y[2 + i], keep = (rg & 2) ? y[2 + i] : y[i];
-          z[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
-        }
-        {
-          const float send = (rg & 1) ? z[0] : z[1], keep = (rg & 1) ? z[1] : z[0];
-          w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
-        }
-        const float a0 = __shfl_sync(0xffffffffu, w, (lane & 24) | 0), a1 = __shfl_sync(0xffffffffu, w, (lane & 24) | 1);
-        const float a2 = __shfl_sync(0xffffffffu, w, (lane & 24) | 2), a3 = __shfl_sync(0xffffffffu, w, (lane & 24) | 3);
-        const float u0 = scal.x * (vv.x - a0), u1 = scal.x * (vv.y - a1), u2 = scal.x * (vv.z - a2), u3 = scal.x * (vv.w - a3);
-        const f32x2 uu[4] = {pack2(u0, u0), pack2(u1, u1), pack2(u2, u2), pack2(u3, u3)};
-#pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            S[j][c][0] = fma2(k2.x, uu[c], S[j][c][0]);
-            S[j][c][1] = fma2(k2.y, uu[c], S[j][c][1]);
-          }
-        }
-        if (rg >= 4) {
-          const int c = rg - 4;
-          const float u = c == 0 ? u0 : (c == 1 ? u1 : (c == 2 ? u2 : u3));
-          if (col0 + c < p.dv) orow[c] = fmaf(scal.y, u, w);
-        }
-      } else {
-        const float m_new = fmaxf(scal.y + m, scal.x);
-        const float fw = expf(scal.y + m - m_new), iw = expf(scal.x - m_new);
-        m = m_new;
-        const f32x2 f2 = pack2(fw, fw), i2 = pack2(iw, iw);
-        const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
-        f32x2 accO[4];
-        float nq = 0.f;
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-          nrm[i] = fmaf(nrm[i], fw, iw * kr[i * 32 + lane]);
-          nq = fmaf(nrm[i], qr[i * 32 + lane], nq);
-        }
-#pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
-          const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
-          const f32x2 ik0 = mul2(k2.x, i2), ik1 = mul2(k2.y, i2);
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            S[j][c][0] = fma2(ik0, v2[c], mul2(S[j][c][0], f2));
-            S[j][c][1] = fma2(ik1, v2[c], mul2(S[j][c][1], f2));
-            accO[c] = j == 0 ? mul2(S[j][c][0], q2.x) : fma2(S[j][c][0], q2.x, accO[c]);
-            accO[c] = fma2(S[j][c][1], q2.y, accO[c]);
-          }
-        }
-        float x[4], lo, hi;
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          unpack2(accO[c], lo, hi);
-          x[c] = lo + hi;
-        }
-#pragma unroll
-        for (int off = 1; off <= 16; off <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, off);
-        float y[2], w;
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const float send = (rg & 2) ? x[i] : x[2 + i], keep = (rg & 2) ? x[2 + i] : x[i];
-          y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
-        }
-        {
-          const float send = (rg & 1) ? y[0] : y[1], keep = (rg & 1) ? y[1] : y[0];
-          w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
-        }
-        w += __shfl_xor_sync(0xffffffffu, w, 4);
-        if (rg < 4 && col0 + rg < p.dv) orow[rg] = w / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
+      for (int i = 0; i < NR; ++i) {
+        nrm[i] = fmaf(nrm[i], fw, iw * kr[i * 32 + lane]);
+        nq = fmaf(nrm[i], qr[i * 32 + lane], nq);
       }
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qr + j * 32 + rg * 4);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(kr + j * 32 + rg * 4);
+        const f32x2 ik0 = mul2(k2.x, i2), ik1 = mul2(k2.y, i2);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          s.S[j][c][0] = fma2(ik0, v2[c], mul2(s.S[j][c][0], f2));
+          s.S[j][c][1] = fma2(ik1, v2[c], mul2(s.S[j][c][1], f2));
+          accO[c] = j == 0 ? mul2(s.S[j][c][0], q2.x) : fma2(s.S[j][c][0], q2.x, accO[c]);
+          accO[c] = fma2(s.S[j][c][1], q2.y, accO[c]);
+        }
+      }
+#pragma unroll
+      for (int off = 1; off <= 16; off <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, off);
+      float x[4], y[2], w;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) x[c] = hsum(accO[c]);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float send = (rg & 2) ? x[i] : x[2 + i], keep = (rg & 2) ? x[2 + i] : x[i];
+        y[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+      }
+      {
+        const float send = (rg & 1) ? y[0] : y[1], keep = (rg & 1) ? y[1] : y[0];
+        w = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+      }
+      w += __shfl_xor_sync(0xffffffffu, w, 4);
+      if (rg < 4 && col0 + rg < p.dv) orow[rg] = w / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
       orow += ostep;
     }
     __syncthreads();   // the stage may be refilled
   }
   pdl_launch_dependents();
-
-#pragma unroll
-  for (int j = 0; j < NJ; ++j) {
-#pragma unroll
-    for (int hh = 0; hh < 2; ++hh) {
-      const int r = j * 32 + rg * 4 + hh * 2;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        if (col0 + c >= p.dv) continue;
-        float lo, hi;
-        unpack2(S[j][c][hh], lo, hi);
-        if (r < p.dk) gst[static_cast<long long>(r) * p.dv + col0 + c] = lo;
-        if (r + 1 < p.dk) gst[static_cast<long long>(r + 1) * p.dv + col0 + c] = hi;
-      }
-    }
-  }
+  s.store(gst, rg, col0, p.dk, p.dv);
   // n and m: every block of a (head, sequence) computes the same values, and another block may still have to read the
   // old ones, so they leave through scratch and the post kernel moves them into the state
-  if (!DELTA && blockIdx.x == 0 && warp == 0) {
+  if (blockIdx.x == 0 && warp == 0) {
     float* ao = p.s.aux_out + (static_cast<long long>(b) * p.H + h) * (p.dk + 1);
 #pragma unroll
     for (int i = 0; i < NR; ++i)
@@ -880,46 +1030,48 @@ int launch_decode(const A& a, cudaStream_t stream) {
   return launch_kernel(recurrent_decode_kernel<T, A, 32>, grid, 256, 0, stream, pdl, a);
 }
 
-template <bool DELTA, int R>
-int launch_scan_r(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl) {
-  constexpr int DKP = 8 * R;
-  // Warps (16 columns each) per block: as many as share the staged q / k / decay rows without loading one SM more than
-  // another - all warps run from the first token to the last, so the fullest SM decides.
-  const int most = p.dv <= 16 ? 1 : (p.dv <= 32 ? 2 : 4);
+// Warps (16 columns each) per scan block: as many as share the staged rows without loading one SM more than another - all
+// warps run from the first token to the last, so the fullest SM decides.
+int scan_warps(int B, int H, int dv) {
+  const int most = dv <= 16 ? 1 : (dv <= 32 ? 2 : 4);
   int warps = most;
-  long long best = -1;
+  int64_t best = -1;
   for (int w = most; w >= 1; w /= 2) {
-    const long long blocks = static_cast<long long>(B) * p.H * ((p.dv + w * 16 - 1) / (w * 16));
-    const long long load = (blocks + 147) / 148 * w;
+    const int64_t blocks = static_cast<int64_t>(B) * H * ((dv + w * 16 - 1) / (w * 16));
+    const int64_t load = (blocks + 147) / 148 * w;
     if (best < 0 || load < best) {
       best = load;
       warps = w;
     }
   }
-  const int cs = warps * 16;
-  const int smem = 2 * kChunk * ((DELTA ? 3 : 2) * DKP + cs + 4) * 4;
-  auto kern = scan_kernel<DELTA, R>;
-  static int attr_smem = 0;
-  if (smem > 48 * 1024 && smem > attr_smem) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
-    attr_smem = smem;
-  }
-  const dim3 grid((p.dv + cs - 1) / cs, p.H, B);
-  return launch_kernel(kern, grid, warps * 32, smem, stream, pdl, p);
+  return warps;
 }
 
-template <bool DELTA>
-int launch_scan(const ScanParams& p, int B, int T, cudaStream_t stream, bool pdl) {
-  switch (pad_dk(p.dk)) {
-    case 64: return launch_scan_r<DELTA, 8>(p, B, T, stream, pdl);
-    case 128: return launch_scan_r<DELTA, 16>(p, B, T, stream, pdl);
-    default: return launch_scan_r<DELTA, 32>(p, B, T, stream, pdl);
+template <typename K>
+int launch_scan(K kern, const ScanParams& p, int B, int warps, int smem, int* attr_smem, cudaStream_t stream, bool pdl) {
+  if (smem > 48 * 1024 && smem > *attr_smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
+    *attr_smem = smem;
   }
+  const int cs = warps * 16;
+  return launch_kernel(kern, dim3((p.dv + cs - 1) / cs, p.H, B), warps * 32, smem, stream, pdl, p);
+}
+template <int R>
+int launch_delta_scan(const ScanParams& p, int B, cudaStream_t stream, bool pdl) {
+  static int attr = 0;
+  const int warps = scan_warps(B, p.H, p.dv);
+  return launch_scan(delta_scan_kernel<R>, p, B, warps, 2 * kStageBlocks * (kVecs * 8 * R + kBlock * warps * 16 + kScal) * 4, &attr, stream, pdl);
+}
+template <int R>
+int launch_mlstm_scan(const ScanParams& p, int B, cudaStream_t stream, bool pdl) {
+  static int attr = 0;
+  const int warps = scan_warps(B, p.H, p.dv);
+  return launch_scan(mlstm_scan_kernel<R>, p, B, warps, 2 * kChunk * (2 * 8 * R + warps * 16 + 4) * 4, &attr, stream, pdl);
 }
 
 template <typename T, int TAPS>
 int launch_delta_prep(const ortb200_gated_delta_args& a, const Scratch& s, int dkp, int dvp, cudaStream_t stream, bool pdl) {
-  const dim3 grid((a.T + kPrepRun - 1) / kPrepRun, (a.kv_heads + 2 * a.heads + 7) / 8);
+  const dim3 grid(a.T / kPrepRun + a.B, (2 * a.heads + 7) / 8);   // every sequence has at most one partly filled run
   if (dkp == 64) return launch_kernel(delta_prep_kernel<T, TAPS, 2>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
   if (dkp == 128) return launch_kernel(delta_prep_kernel<T, TAPS, 4>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
   return launch_kernel(delta_prep_kernel<T, TAPS, 8>, grid, 256, 0, stream, pdl, a, s, dkp, dvp);
@@ -930,11 +1082,11 @@ int run_delta(const ortb200_gated_delta_args& a, cudaStream_t stream) {
   if (a.T == a.B) return launch_decode<T, ortb200_gated_delta_args>(a, stream);
   const bool pdl = a.use_pdl != 0;
   const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
-  const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.kv_heads, dkp, dvp);
+  const Scratch s = split_scratch(a.workspace, delta_scratch(a.T, a.B, a.heads, dkp, dvp));
   int rc = a.taps == 4 ? launch_delta_prep<T, 4>(a, s, dkp, dvp, stream, pdl) : launch_delta_prep<T, 0>(a, s, dkp, dvp, stream, pdl);
   if (rc) return rc;
-  ScanParams p{s, a.state, nullptr, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.kv_heads, a.dk, a.dv, dvp, a.num_slots, 0.f, a.status};
-  rc = launch_scan<true>(p, a.B, a.T, stream, pdl);
+  ScanParams p{s, a.state, nullptr, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.dk, a.dv, dvp, a.num_slots, 0.f, a.status};
+  rc = dkp == 64 ? launch_delta_scan<8>(p, a.B, stream, pdl) : dkp == 128 ? launch_delta_scan<16>(p, a.B, stream, pdl) : launch_delta_scan<32>(p, a.B, stream, pdl);
   if (rc) return rc;
   PostParams q{};
   q.o = s.o; q.norm = a.norm; q.norm_stride = 0;
@@ -953,11 +1105,11 @@ int run_mlstm(const ortb200_mlstm_args& a, cudaStream_t stream) {
   if (a.T == a.B) return launch_decode<T, ortb200_mlstm_args>(a, stream);
   const bool pdl = a.use_pdl != 0;
   const int dkp = pad_dk(a.dk), dvp = pad4(a.dv);
-  const Scratch s = split_scratch(a.workspace, a.T, a.heads, a.heads, dkp, dvp);
+  const Scratch s = split_scratch(a.workspace, mlstm_scratch(a.T, a.B, a.heads, a.dk, dkp, dvp));
   int rc = launch_kernel(mlstm_prep_kernel<T>, dim3(a.T, (a.heads + 7) / 8), 256, 0, stream, pdl, a, s, dkp, dvp);
   if (rc) return rc;
-  ScanParams p{s, a.state, a.aux, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.heads, a.dk, a.dv, dvp, a.num_slots, a.den_eps, a.status};
-  rc = launch_scan<false>(p, a.B, a.T, stream, pdl);
+  ScanParams p{s, a.state, a.aux, a.cu_seqlens, a.past_seqlens, a.slots, a.heads, a.dk, a.dv, dvp, a.num_slots, a.den_eps, a.status};
+  rc = dkp == 64 ? launch_mlstm_scan<8>(p, a.B, stream, pdl) : dkp == 128 ? launch_mlstm_scan<16>(p, a.B, stream, pdl) : launch_mlstm_scan<32>(p, a.B, stream, pdl);
   if (rc) return rc;
   PostParams q{};
   q.o = s.o; q.norm = a.norm; q.norm_stride = a.dv;
@@ -983,7 +1135,9 @@ using namespace ortb200;
 
 extern "C" int64_t ortb200_recurrent_workspace_bytes(int T, int B, int heads, int kv_heads, int dk, int dv) {
   if (T == B) return 0;
-  return 4 * (scratch_floats(T, heads, kv_heads, pad_dk(dk), pad4(dv)) + static_cast<int64_t>(B) * heads * (dk + 1));
+  (void)kv_heads;
+  const int64_t delta = delta_scratch(T, B, heads, pad_dk(dk), pad4(dv)).total(), mem = mlstm_scratch(T, B, heads, dk, pad_dk(dk), pad4(dv)).total();
+  return 4 * (delta > mem ? delta : mem);
 }
 
 extern "C" int ortb200_gated_delta(const ortb200_gated_delta_args* a, ortb200_stream_t stream_) {
