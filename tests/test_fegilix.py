@@ -413,12 +413,15 @@ def small_config(name):
                       ("attention", dict(att, heads=6, kv_heads=1, dim=16, vdim=48, scale=1.0, rot={"base": 50.0, "dims": 4}), ff(24)),
                       ("attention", dict(att, heads=4, kv_heads=1, dim=16, vdim=48, scale=0.3, rot={"base": 50.0, "dims": 4}, kv_from=1), ff(24))],
         "recurrent": [("mlstm", mem, None), ("mlstm", dict(mem, heads=1, dim=8, vdim=8, gate_cap=2.0), ff(16)), ("channel_delta", delta, None)],
+        # sizes that no tensor-core or vector path takes
+        "odd": [("attention", dict(att, heads=3, kv_heads=1, dim=10, vdim=14, rot={"base": 30.0, "dims": 6}), ff(20)),
+                ("channel_delta", dict(delta, heads=3, kv_heads=1, dim=9, vdim=7, conv=4), None), ("mlstm", dict(mem, heads=5, dim=11, vdim=6), ff(12))],
         "plain": [("attention", att, ff(24)), ("mlstm", mem, None), ("channel_delta", delta, ff(32))],
     }[name]
-    cfg = {"architecture": "Fegilix", "vocab": 97 if name != "attention" else 120, "width": 48 if name != "recurrent" else 40, "norm": {"eps": 1e-5},
+    cfg = {"architecture": "Fegilix", "vocab": 97 if name != "attention" else 120, "width": {"recurrent": 40, "odd": 36}.get(name, 48), "norm": {"eps": 1e-5},
            "layers": [{"type": t, "mixer": dict(m), "mlp": f} for t, m, f in layers]}
     if name != "plain":
-        cfg.update(streams={"mixed": 3, "attention": 2, "recurrent": 1}[name], logit_softcap=8.0)
+        cfg.update(streams={"mixed": 3, "attention": 2, "recurrent": 1, "odd": 5}[name], logit_softcap=8.0)
     return cfg
 
 
@@ -485,7 +488,7 @@ def feed(runner, seq, tokens, cuts):
 
 
 @pytest.mark.parametrize("kind", KINDS)
-@pytest.mark.parametrize("name", ["mixed", "attention", "recurrent", "plain"])
+@pytest.mark.parametrize("name", ["mixed", "attention", "recurrent", "plain", "odd"])
 def test_model_matches_the_restatement(kind, name):
     """Whole prompt, portions down to two tokens, token by token, and a prompt followed by decoding."""
     cfg, w = model_pair(name)
