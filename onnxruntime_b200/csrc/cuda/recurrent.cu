@@ -1,6 +1,6 @@
 // Recurrent token mixers over packed sequences: the gated delta rule with a decay per key channel, and the
-// exponentially gated matrix memory (mLSTM).  The state is fp32 everywhere, and the recurrence runs token by token in
-// fp32, so a result does not depend on how a prompt is cut.
+// exponentially gated matrix memory (mLSTM).  State and arithmetic are fp32 everywhere, and every token
+// sees the exact state of the tokens before it, so a result does not depend on how a prompt is cut.
 //
 // Several tokens per sequence (prompts): three launches.
 //   prep   short convolution + silu, unit norms, decays, gates -> fp32 rows, heads padded; a warp owns the channels of one

@@ -358,15 +358,6 @@ def build_llama(cfg: LlamaConfig, tp_rank: int = 0, tp_size: int = 1, external_w
     return model.serialize(), weights
 
 
-def empty_paged_cache(cfg: LlamaConfig, num_blocks: int, block_size: int, device,
-                      tp_size: int = 1) -> List[Tuple[torch.Tensor, torch.Tensor]]:
-    """Per layer (key_cache, value_cache) of shape [num_blocks, block_size, kv_heads / tp, head_dim]."""
-    dt = _TORCH_DT[cfg.dtype]
-    nk = cfg.num_kv_heads // tp_size
-    return [(torch.zeros(num_blocks, block_size, nk, cfg.head_dim, dtype=dt, device=device),
-             torch.zeros(num_blocks, block_size, nk, cfg.head_dim, dtype=dt, device=device)) for _ in range(cfg.num_layers)]
-
-
 def empty_kv_cache(cfg: LlamaConfig, batch: int, max_len: int, device, tp_size: int = 1) -> List[Tuple[torch.Tensor, torch.Tensor]]:
     dt = _TORCH_DT[cfg.dtype]
     nk = cfg.num_kv_heads // tp_size
