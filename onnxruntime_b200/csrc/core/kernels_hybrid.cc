@@ -1,6 +1,6 @@
 // com.ortb200 operators of hybrid decoders in packed serving form: hyper-connections, the gated delta rule with short
-// convolutions, the exponentially gated matrix memory, gated paged attention and the soft cap.  These are the
-// device-agnostic versions (tensor library, one token at a time where the mathematics is a recurrence); the GPU provider
+// convolutions, the exponentially gated matrix memory, gated paged attention, latent paged attention, the clamped gated
+// linear unit and the soft cap.  These are the device-agnostic versions (tensor library, one token at a time where the mathematics is a recurrence); the GPU provider
 // has its own kernels (kernels_cuda4.cc).
 //
 // Packed form: the tokens of all sequences lie behind one another, sequence b owns rows [cu[b], cu[b + 1]) and its first
@@ -158,13 +158,34 @@ void PackedMLstmImpl(Ctx& ctx) {
   if (ctx.OutputCount() > 2) ctx.SetOutput(2, aux);
 }
 
-// inputs: packed, key_cache, value_cache, cu, past, block_table, cos?, sin?, q_norm?, k_norm?, sink?
+// A parallel block writes its two sublayers into the columns of one tensor: `base` (when given) receives y in its first
+// columns and is the result.
+void SetColumns(Ctx& ctx, int base, const at::Tensor& y) {
+  if (!ctx.HasInput(base)) {
+    ctx.SetOutput(0, y);
+    return;
+  }
+  at::Tensor b = ctx.Input(base);
+  ORTB_ENFORCE_ARG(b.dim() == 2 && b.size(0) == y.size(0) && b.size(1) >= y.size(1) && b.scalar_type() == y.scalar_type(), ctx.node().op_type,
+                   ": base does not fit the result");
+  b.narrow(1, 0, y.size(1)).copy_(y);
+  ctx.SetOutput(0, b);
+}
+
+// softmax over the last axis of s [heads, L, total], optionally with one more term per head in the denominator
+at::Tensor SoftmaxWithSink(at::Tensor s, Ctx& ctx, int sink) {
+  const int64_t N = s.size(0), L = s.size(1), total = s.size(2);
+  if (ctx.HasInput(sink)) s = at::cat({s, F32(ctx.Input(sink)).reshape({N, 1, 1}).expand({N, L, 1})}, 2);
+  return at::softmax(s, -1).narrow(2, 0, total);
+}
+
+// inputs: packed, key_cache, value_cache, cu, past, block_table, cos?, sin?, q_norm?, k_norm?, sink?, first_values?, v_mix?, base?
 void GatedPagedAttentionImpl(Ctx& ctx) {
   const Node& n = ctx.node();
   const int64_t N = n.attr_i("num_heads", 0), Nk = n.attr_i("kv_num_heads", 0), dk = n.attr_i("head_size", 0), dv = n.attr_i("v_head_size", 0);
   const bool shared = n.attr_i("kv_shared", 0) != 0, gated = n.attr_i("gated", 0) != 0;
   const double eps = n.attr_f("epsilon", 1e-6f), scale = n.attr_f("scale", 1.f);
-  const int64_t window = n.attr_i("local_window_size", -1);
+  const int64_t window = n.attr_i("local_window_size", -1), chunk = n.attr_i("chunk_size", 0);
   const at::Tensor& packed = ctx.RequiredInput(0);
   at::Tensor kc = ctx.RequiredInput(1), vc = ctx.RequiredInput(2);
   const int64_t T = packed.size(0), block_size = kc.size(1), kv_cols = shared ? 0 : Nk * (dk + dv);
@@ -179,6 +200,11 @@ void GatedPagedAttentionImpl(Ctx& ctx) {
     k = xf.narrow(1, N * dk, Nk * dk).reshape({T, Nk, dk});
     v = packed.narrow(1, (N + Nk) * dk, Nk * dv).reshape({T, Nk, dv});
     if (ctx.HasInput(9)) k = Rms(k, eps) * F32(ctx.Input(9));
+    if (ctx.HasInput(11)) {   // values of another layer for the same tokens, mixed in before they are stored
+      at::Tensor first = F32(ctx.Input(11).narrow(1, n.attr_i("first_values_offset", 0), Nk * dv)).reshape({T, Nk, dv});
+      at::Tensor m = F32(ctx.RequiredInput(12)).reshape({1, 1, 1});
+      v = ((1 - m) * F32(v) + m * first).to(vc.scalar_type());
+    }
   }
   auto rotate = [&](const at::Tensor& x, int64_t first) {   // x [L, heads, dk]
     if (!ctx.HasInput(6)) return x;
@@ -212,16 +238,96 @@ void GatedPagedAttentionImpl(Ctx& ctx) {
     at::Tensor kpos = at::arange(total, s.options().dtype(at::kLong)).unsqueeze(0);
     at::Tensor hidden = kpos.gt(qpos);
     if (window > 0) hidden = hidden.logical_or(kpos.le(qpos - window));
+    if (chunk > 0) hidden = hidden.logical_or(kpos.lt(qpos - qpos.remainder(chunk)));
     s = s.masked_fill(hidden.unsqueeze(0), -std::numeric_limits<float>::infinity());
-    if (ctx.HasInput(10)) s = at::cat({s, F32(ctx.Input(10)).reshape({N, 1, 1}).expand({N, L, 1})}, 2);
-    at::Tensor w = at::softmax(s, -1).narrow(2, 0, total);
+    at::Tensor w = SoftmaxWithSink(s, ctx, 10);
     out.narrow(0, t0, L).copy_(at::matmul(w, gather(vc, dv)).permute({1, 0, 2}));
   }
   out = out.reshape({T, N * dv});
   if (gated) out = out * at::sigmoid(xf.narrow(1, N * dk + kv_cols, N * dv));
-  ctx.SetOutput(0, out.to(packed.scalar_type()));
+  SetColumns(ctx, 13, out.to(packed.scalar_type()));
   if (ctx.OutputCount() > 1) ctx.SetOutput(1, kc);
   if (ctx.OutputCount() > 2) ctx.SetOutput(2, vc);
+}
+
+// inputs: packed, cache, cu, past, block_table, cos?, sin?, norm, up, sink?, base?, key_starts?
+// packed: q (heads * (head_size + rot)) | latent (rank) | rotated key part (rot) | gate (heads).  A cache entry is the
+// normed latent, zero-padded to `latent_width`, and the rotated key part behind it.  up: rows of the key map (heads *
+// head_size), then of the value map (heads * v_head_size), each of `rank` columns.
+void LatentPagedAttentionImpl(Ctx& ctx) {
+  const Node& n = ctx.node();
+  const int64_t N = n.attr_i("num_heads", 0), dk = n.attr_i("head_size", 0), dr = n.attr_i("rotary_size", 0), dv = n.attr_i("v_head_size", 0),
+                rank = n.attr_i("latent_size", 0), wide = n.attr_i("latent_width", rank);
+  const bool gated = n.attr_i("gated", 0) != 0;
+  const double eps = n.attr_f("epsilon", 1e-6f), scale = n.attr_f("scale", 1.f);
+  const at::Tensor& packed = ctx.RequiredInput(0);
+  at::Tensor cache = ctx.RequiredInput(1);
+  const at::Tensor& up = ctx.RequiredInput(8);
+  const int64_t T = packed.size(0), block_size = cache.size(1), q_cols = N * (dk + dr);
+  ORTB_ENFORCE_ARG(N > 0 && rank > 0 && wide >= rank && cache.dim() == 3 && cache.size(2) >= wide + dr && up.dim() == 2 && up.size(0) == N * (dk + dv) &&
+                       up.size(1) == rank && packed.size(1) >= q_cols + rank + dr + (gated ? N : 0),
+                   "LatentPagedAttention: sizes disagree");
+  const Packing p = ReadPacking(ctx, 2, 3, -1);
+  at::Tensor table = ctx.RequiredInput(4).to(at::kCPU, at::kLong);
+  at::Tensor xf = F32(packed);
+  at::Tensor q = xf.narrow(1, 0, q_cols).reshape({T, N, dk + dr});
+  at::Tensor c = (Rms(xf.narrow(1, q_cols, rank), eps) * F32(ctx.RequiredInput(7))).to(cache.scalar_type());
+  at::Tensor kr = xf.narrow(1, q_cols + rank, dr).unsqueeze(1);
+  // x [L, heads, dr]: neighbours (2 i, 2 i + 1) turn together
+  auto rotate = [&](const at::Tensor& x, int64_t first) {
+    if (!ctx.HasInput(5)) return x;
+    const int64_t half = ctx.Input(5).size(1), L = x.size(0);
+    ORTB_ENFORCE_ARG(first + L <= ctx.Input(5).size(0) && 2 * half <= dr, "LatentPagedAttention: position or size beyond the rotary tables");
+    at::Tensor cs = F32(ctx.Input(5)).narrow(0, first, L).unsqueeze(1), sn = F32(ctx.RequiredInput(6)).narrow(0, first, L).unsqueeze(1);
+    at::Tensor pairs = x.narrow(2, 0, 2 * half).reshape({L, x.size(1), half, 2});
+    at::Tensor u = pairs.select(3, 0), v = pairs.select(3, 1);
+    at::Tensor turned = at::stack({u * cs - v * sn, v * cs + u * sn}, 3).reshape({L, x.size(1), 2 * half});
+    return at::cat({turned, x.narrow(2, 2 * half, dr - 2 * half)}, 2);
+  };
+  at::Tensor upf = F32(up);
+  at::Tensor uk = upf.narrow(0, 0, N * dk).reshape({N, dk, rank}), uv = upf.narrow(0, N * dk, N * dv).reshape({N, dv, rank});
+  at::Tensor out = at::zeros({T, N, dv}, xf.options());
+  for (int64_t b = 0; b < p.B(); ++b) {
+    const int64_t t0 = p.cu[b], L = p.cu[b + 1] - t0, past = p.past[b], total = past + L;
+    if (L == 0) continue;
+    at::Tensor krb = rotate(kr.narrow(0, t0, L), past).to(cache.scalar_type());
+    for (int64_t s = 0; s < L; ++s) {
+      at::Tensor entry = cache[table[b][(past + s) / block_size].item<int64_t>()][(past + s) % block_size];
+      entry.narrow(0, 0, rank).copy_(c[t0 + s]);
+      entry.narrow(0, wide, dr).copy_(krb[s][0]);
+    }
+    const int64_t nblk = (total + block_size - 1) / block_size;
+    at::Tensor all = F32(cache.index_select(0, table[b].narrow(0, 0, nblk).to(cache.device())).reshape({nblk * block_size, cache.size(2)}).narrow(0, 0, total));
+    at::Tensor cl = all.narrow(1, 0, rank), qb = q.narrow(0, t0, L);
+    at::Tensor qa = at::matmul(qb.narrow(2, 0, dk).permute({1, 0, 2}), uk);                                            // [N, L, rank]
+    at::Tensor qr = rotate(qb.narrow(2, dk, dr), past).permute({1, 0, 2});
+    at::Tensor s = (at::matmul(qa, cl.t()) + at::matmul(qr, all.narrow(1, wide, dr).t())) * scale;                     // [N, L, total]
+    at::Tensor qpos = (at::arange(L, s.options().dtype(at::kLong)) + past).unsqueeze(1);
+    at::Tensor kpos = at::arange(total, s.options().dtype(at::kLong)).unsqueeze(0);
+    s = s.masked_fill(kpos.gt(qpos).unsqueeze(0), -std::numeric_limits<float>::infinity());
+    at::Tensor o = at::matmul(at::matmul(SoftmaxWithSink(s, ctx, 9), cl), uv.transpose(1, 2));                         // [N, L, dv]
+    out.narrow(0, t0, L).copy_(o.permute({1, 0, 2}));
+  }
+  if (gated) out = out * at::sigmoid(xf.narrow(1, q_cols + rank + dr, N)).unsqueeze(2);
+  SetColumns(ctx, 10, out.reshape({T, N * dv}).to(packed.scalar_type()));
+  if (ctx.OutputCount() > 1) ctx.SetOutput(1, cache);
+}
+
+// y = g sigmoid(alpha g) (u + offset), g = min(gate, limit), u = clamp(up, -limit, limit), behind `lead_columns` columns
+// that another operator fills
+void ClampedSwiGLUImpl(Ctx& ctx) {
+  const Node& n = ctx.node();
+  const double limit = n.attr_f("limit", std::numeric_limits<float>::infinity()), alpha = n.attr_f("alpha", 1.f), offset = n.attr_f("offset", 0.f);
+  const at::Tensor& gate = ctx.RequiredInput(0);
+  at::Tensor g = F32(gate).clamp_max(limit), u = F32(ctx.RequiredInput(1)).clamp(-limit, limit);
+  at::Tensor y = (g * at::sigmoid(alpha * g) * (u + offset)).to(gate.scalar_type());
+  const int64_t lead = n.attr_i("lead_columns", 0);
+  if (lead > 0) {
+    std::vector<int64_t> shape = y.sizes().vec();
+    shape.back() = lead;
+    y = at::cat({at::zeros(shape, y.options()), y}, -1);
+  }
+  ctx.SetOutput(0, y);
 }
 
 }  // namespace
@@ -231,6 +337,8 @@ void RegisterHybridKernels(KernelRegistry& r) {
   r.RegisterFn(FUSED, "PackedGatedDelta", 1, kMax, PackedGatedDeltaImpl);
   r.RegisterFn(FUSED, "PackedMLstm", 1, kMax, PackedMLstmImpl);
   r.RegisterFn(FUSED, "GatedPagedAttention", 1, kMax, GatedPagedAttentionImpl);
+  r.RegisterFn(FUSED, "LatentPagedAttention", 1, kMax, LatentPagedAttentionImpl, {11});
+  r.RegisterFn(FUSED, "ClampedSwiGLU", 1, kMax, ClampedSwiGLUImpl);
   r.RegisterFn(FUSED, "SoftCap", 1, kMax, [](Ctx& ctx) {
     const double cap = ctx.node().attr_f("cap", 1.f);
     ctx.SetOutput(0, at::tanh(F32(ctx.RequiredInput(0)) / cap) * cap);

@@ -678,7 +678,9 @@ void RegisterBuiltinSchemas(std::map<std::string, OpSchema>& t) {
   Reg(t, FUSED, "HyperConnectionNorm", 5, 7);
   Reg(t, FUSED, "PackedGatedDelta", 11, 11);
   Reg(t, FUSED, "PackedMLstm", 9, 9);
-  Reg(t, FUSED, "GatedPagedAttention", 6, 11);
+  Reg(t, FUSED, "GatedPagedAttention", 6, 14);
+  Reg(t, FUSED, "LatentPagedAttention", 9, 12);
+  Reg(t, FUSED, "ClampedSwiGLU", 2, 2);
   Reg(t, FUSED, "SoftCap", 1, 1);
   Reg(t, FUSED, "SwiGLU", 1, 1, [](Ctx& c) {
     if (!c.HasShape(0) || c.Rank(0) < 1) return;

@@ -23,12 +23,10 @@ import torch
 
 from .. import onnx_lite as ol
 from .decoder_cache import CacheTensor
+from .packed_graph import TORCH_DT, PackedGraph, padded_head_widths
+from .rotary import rotary_tables  # noqa: F401
 
 T = ol.TensorProto
-FUSED = "com.ortb200"
-
-_TORCH_DT = {"bf16": torch.bfloat16, "fp16": torch.float16, "fp32": torch.float32}
-_ONNX_DT = {"bf16": T.BFLOAT16, "fp16": T.FLOAT16, "fp32": T.FLOAT}
 
 UNIT_EPS = 1e-6          # inside the root of the unit norms of the delta rule's q and k
 DENOMINATOR_EPS = 1e-6   # added to the mLSTM denominator
@@ -88,17 +86,12 @@ class FegilixConfig:
         return any(layer["type"] != "attention" for layer in self.layers)
 
     def cache_widths(self, m: Mapping[str, Any]) -> Tuple[int, int]:
-        """Stored widths of a key and a value head: 16-bit heads are padded to the sizes of the tensor-core kernels (zeros
-        change neither a score nor an output), others to a multiple of four."""
-        wide = max(m["dim"], m["vdim"])
-        if self.dtype != "fp32" and wide <= 128:
-            return (64, 64) if wide <= 64 else (128, 128)
-        return -(-m["dim"] // 4) * 4, -(-m["vdim"] // 4) * 4
+        return padded_head_widths(self.dtype, m["dim"], m["vdim"])
 
     def cache_tensors(self, tp_size: int = 1) -> List[CacheTensor]:
         if tp_size != 1:
             raise ValueError("this graph is built for one device")
-        dt = _TORCH_DT[self.dtype]
+        dt = TORCH_DT[self.dtype]
         out: List[CacheTensor] = []
         for i, layer in enumerate(self.layers):
             m = layer["mixer"]
@@ -150,21 +143,6 @@ class FegilixConfig:
         return shapes
 
 
-def rotary_tables(rot: Mapping[str, Any], rows: int, device="cpu") -> Tuple[torch.Tensor, torch.Tensor]:
-    """fp32 cos / sin [rows, dims / 2] of positions 0 .. rows - 1 (angles in float64), with the three-band frequency
-    rescaling of long-context Llama models when ``rot`` has "scaling"."""
-    half = rot["dims"] // 2
-    f = float(rot["base"]) ** (-2.0 * torch.arange(half, dtype=torch.float64) / rot["dims"])
-    sc = rot.get("scaling")
-    if sc:
-        wavelength = 2.0 * math.pi / f
-        s = (sc["original"] / wavelength - sc["low"]) / (sc["high"] - sc["low"])
-        blend = (1.0 - s) * f / sc["factor"] + s * f
-        f = torch.where(wavelength < sc["original"] / sc["high"], f, torch.where(wavelength > sc["original"] / sc["low"], f / sc["factor"], blend))
-    angles = torch.outer(torch.arange(rows, dtype=torch.float64), f)
-    return angles.cos().float().to(device), angles.sin().float().to(device)
-
-
 def default_rank(cfg: FegilixConfig) -> int:
     """Rank of the low-rank maps for random weights: the key head size of the first delta-rule layer."""
     return next((layer["mixer"]["dim"] for layer in cfg.layers if layer["type"] == "channel_delta"), 16)
@@ -204,78 +182,13 @@ def build_fegilix(cfg: FegilixConfig, weights: Mapping[str, torch.Tensor], devic
     """Returns (ModelProto bytes, initializers); the initializers lie on ``device`` and are handed to
     ``SessionOptions.add_external_initializers``."""
     cfg.validate()
-    dt, odt = _TORCH_DT[cfg.dtype], _ONNX_DT[cfg.dtype]
-    W, eps = cfg.width, cfg.norm_eps
-    nodes: List[ol.Node] = []
-    inits: List[ol.Tensor] = []
-    store: Dict[str, torch.Tensor] = {}
-    expected = cfg.tensor_shapes()
-
-    def tensor(name: str) -> torch.Tensor:
-        if name not in weights:
-            raise KeyError(f"the checkpoint has no tensor {name!r}")
-        w, want = weights[name], expected[name]
-        if len(w.shape) != len(want) or any(e >= 0 and e != s for e, s in zip(want, w.shape)):
-            raise ValueError(f"tensor {name!r} has shape {tuple(w.shape)}, the configuration wants {want}")
-        return w.to(device)
-
-    def add(name: str, w: torch.Tensor, dtype: Optional[torch.dtype] = None) -> str:
-        if name not in store:
-            w = w.to(dtype or dt).contiguous()
-            store[name] = w
-            inits.append(ol.make_external_tensor(name, odt if w.dtype == dt else T.FLOAT, w.shape))
-        return name
-
-    def const32(name: str, w: Optional[torch.Tensor] = None) -> str:
-        return add(name, tensor(name) if w is None else w.to(device), torch.float32)
-
-    def node(op: str, inputs: List[str], outputs: List[str], domain: str = FUSED, **attrs) -> str:
-        nodes.append(ol.make_node(op, inputs, outputs, name=outputs[0] + "/" + op, domain=domain, **attrs))
-        return outputs[0]
-
-    def linear(x: str, name: str, rows: torch.Tensor, out: str) -> str:
-        """out = x @ rows^T (rows [out, in] as in the checkpoint)."""
-        add(name, rows.to(dt).t())
-        return node("MatMul", [x, name], [out], domain="")
-
-    def stacked(x: str, name: str, parts: List[torch.Tensor], out: str) -> str:
-        rows = torch.cat([p.to(dt) for p in parts])
-        pad = -rows.shape[0] % 8
-        if pad:
-            rows = torch.cat([rows, rows.new_zeros(pad, rows.shape[1])])
-        return linear(x, name, rows, out)
-
-    inputs = [ol.make_tensor_value_info("input_ids", T.INT64, ["tokens"]),
-              ol.make_tensor_value_info("cumulative_sequence_length", T.INT32, ["batch_plus_1"]),
-              ol.make_tensor_value_info("past_seqlens", T.INT32, ["batch"]),
-              ol.make_tensor_value_info("block_table", T.INT32, ["batch", "max_blocks"]),
-              ol.make_tensor_value_info("logits_indices", T.INT64, ["rows"])]
-    if cfg.is_recurrent:
-        inputs.append(ol.make_tensor_value_info("state_slots", T.INT32, ["batch"]))
-    outputs = []
-    for c in cfg.cache_tensors():
-        lead = ["num_blocks", "block_size"] if c.kind == "paged" else ["num_slots"]
-        elem = odt if c.dtype == dt else T.FLOAT
-        inputs.append(ol.make_tensor_value_info(c.input, elem, lead + list(c.shape)))
-        outputs.append(ol.make_tensor_value_info(c.output, elem, lead + list(c.shape)))
-
-    tables: Dict[str, Tuple[str, str]] = {}
-
-    def rotary(rot: Optional[Mapping[str, Any]]) -> List[str]:
-        if not rot:
-            return ["", ""]
-        key = repr(sorted(rot.items(), key=lambda kv: kv[0]))
-        if key not in tables:
-            cos, sin = rotary_tables(rot, cfg.max_seq_len, device)
-            k = len(tables)
-            tables[key] = (const32(f"rotary.{k}.cos", cos), const32(f"rotary.{k}.sin", sin))
-        return list(tables[key])
+    g = PackedGraph(cfg, weights, device, state_slots=cfg.is_recurrent)
+    tensor, const32, node, linear, stacked, rotary = g.tensor, g.const32, g.node, g.linear, g.stacked, g.rotary
+    dt, eps = g.dt, cfg.norm_eps
 
     # ---- residual streams
     streams = cfg.streams if cfg.streams is not None else 1
-    add("embed", tensor("embed"))
-    node("Gather", ["embed", "input_ids"], ["x0"], domain="", axis=0)
-    residual, pending = "x0", None        # pending: (sublayer output, mix, w_out) still to be written back
+    residual, pending = g.embed("x0"), None        # pending: (sublayer output, mix, w_out) still to be written back
 
     def hyper_weights(prefix: str) -> Tuple[str, str, str]:
         if cfg.streams is None:
@@ -351,16 +264,10 @@ def build_fegilix(cfg: FegilixConfig, weights: Mapping[str, torch.Tensor], devic
             pending = (linear(prod, f + ".down", tensor(f + ".down"), f + ".out"), mix, w_out)
 
     rows = read(const32("streams.sum", torch.ones(streams)), const32("final.norm"), "final_rows", rows="logits_indices")
-    logit_type = odt
+    logit_type = g.odt
     if cfg.logit_softcap is None:
         linear(rows, "head", tensor("head"), "logits")
     else:
         node("SoftCap", [linear(rows, "head", tensor("head"), "raw_logits")], ["logits"], cap=cfg.logit_softcap)
         logit_type = T.FLOAT
-    outputs.insert(0, ol.make_tensor_value_info("logits", logit_type, ["rows", cfg.vocab_size]))
-    if with_argmax:
-        node("ArgMax", ["logits"], ["next_tokens"], domain="", axis=-1, keepdims=0)
-        outputs.insert(1, ol.make_tensor_value_info("next_tokens", T.INT64, ["rows"]))
-    graph = ol.make_graph(nodes, "fegilix", inputs, outputs, inits)
-    model = ol.make_model(graph, opset=17, metadata={"architecture": cfg.architecture}, extra_opsets={FUSED: 1})
-    return model.serialize(), store
+    return g.finish("fegilix", cfg.vocab_size, logit_type, with_argmax)

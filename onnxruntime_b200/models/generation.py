@@ -171,6 +171,7 @@ class PagedDecoderRunner:
         in_names = {i.name for i in session.get_inputs()}
         self.has_argmax = "next_tokens" in out_info
         self.has_slots = "state_slots" in in_names
+        self.has_key_starts = "key_starts" in in_names
         self.logits_dtype = {"tensor(float)": torch.float32, "tensor(float16)": torch.float16,
                              "tensor(bfloat16)": torch.bfloat16}[out_info["logits"].type]
         self._steps: Dict[int, "_DecodeBuffers"] = {}
@@ -191,7 +192,7 @@ class PagedDecoderRunner:
 
     @property
     def cache(self) -> List[Tuple[torch.Tensor, torch.Tensor]]:
-        """(key, value) block pools of the attention layers that own them."""
+        """(key, value) block pools of the attention layers that own them (models that cache keys and values in every layer)."""
         paged = [self.pool.tensors[c.input] for c in self.pool.spec if c.kind == "paged"]
         return list(zip(paged[::2], paged[1::2]))
 
@@ -210,7 +211,7 @@ class PagedDecoderRunner:
     def _slots(self, seqs) -> torch.Tensor:
         return torch.tensor([self.pool.sequences[s].slot for s in seqs], dtype=torch.int32)
 
-    def _bind(self, binding, ids, cum, past, table, slots, rows, logits, nxt) -> None:
+    def _bind(self, binding, ids, cum, past, table, slots, key_starts, rows, logits, nxt) -> None:
         binding.bind_torch_input("input_ids", ids)
         binding.bind_torch_input("cumulative_sequence_length", cum)
         binding.bind_torch_input("past_seqlens", past)
@@ -218,6 +219,8 @@ class PagedDecoderRunner:
         binding.bind_torch_input("logits_indices", rows)
         if self.has_slots:
             binding.bind_torch_input("state_slots", slots)
+        if self.has_key_starts:
+            binding.bind_torch_input("key_starts", key_starts)
         for c in self.pool.spec:
             binding.bind_torch_input(c.input, self.pool.tensors[c.input])
             binding.bind_torch_output(c.output, self.pool.tensors[c.input])
@@ -268,12 +271,15 @@ class PagedDecoderRunner:
 
     def _run_packed(self, ids: torch.Tensor, starts, seqs, rows) -> Tuple[torch.Tensor, torch.Tensor]:
         dev = self.device
-        past = torch.tensor([self.pool.sequences[s].length for s in seqs], dtype=torch.int32)
+        lengths = [self.pool.sequences[s].length for s in seqs]
+        past = torch.tensor(lengths, dtype=torch.int32)
+        # host tensor: the keys of sequence b, cached and new, are rows [key_starts[b], key_starts[b + 1]) of an expansion
+        key_starts = torch.tensor([starts[b] + sum(lengths[:b]) for b in range(len(seqs) + 1)], dtype=torch.int32)
         logits = torch.empty(len(rows), self.cfg.vocab_size, dtype=self.logits_dtype, device=dev)
         nxt = torch.empty(len(rows), dtype=torch.int64, device=dev)
         binding = self.sess.io_binding()
         self._bind(binding, ids.to(dev), torch.tensor(starts, dtype=torch.int32).to(dev), past.to(dev), self._table(seqs).to(dev),
-                   self._slots(seqs).to(dev), torch.tensor(rows, dtype=torch.int64).to(dev), logits, nxt)
+                   self._slots(seqs).to(dev), key_starts, torch.tensor(rows, dtype=torch.int64).to(dev), logits, nxt)
         self.sess.run_with_iobinding(binding, self._ro_prefill)
         for b, s in enumerate(seqs):
             self.pool.advance(s, starts[b + 1] - starts[b])
@@ -285,7 +291,7 @@ class PagedDecoderRunner:
         if rows not in self._steps:
             buf = _DecodeBuffers(rows, self.blocks_per_seq, self.cfg.vocab_size, self.logits_dtype, self.device)
             buf.binding = self.sess.io_binding()
-            self._bind(buf.binding, buf.ids, buf.cum, buf.past, buf.table, buf.slots, buf.rows, buf.logits, buf.next)
+            self._bind(buf.binding, buf.ids, buf.cum, buf.past, buf.table, buf.slots, buf.key_starts, buf.rows, buf.logits, buf.next)
             buf.options.add_run_config_entry("gpu_graph_id", str(self._graph_id + len(self._steps)))
             self._steps[rows] = buf
         return self._steps[rows]
@@ -371,6 +377,7 @@ class _DecodeBuffers:
         self.past = torch.zeros(rows, dtype=torch.int32, device=device)
         self.table = torch.zeros(rows, max_blocks, dtype=torch.int32, device=device)
         self.slots = torch.zeros(rows, dtype=torch.int32, device=device)
+        self.key_starts = torch.zeros(rows + 1, dtype=torch.int32)     # one-token steps read the cache as it lies
         self.rows = torch.arange(rows, dtype=torch.int64, device=device)
         self.logits = torch.zeros(rows, vocab, dtype=logits_dtype, device=device)
         self.next = torch.zeros(rows, dtype=torch.int64, device=device)

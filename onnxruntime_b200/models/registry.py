@@ -11,7 +11,7 @@ import torch
 
 from ..capi import InferenceSession, SessionOptions
 from ..safetensors_lite import load_file
-from . import fegilix, llama
+from . import fegilix, llama, rovurax
 from .generation import PagedDecoderRunner
 
 
@@ -32,6 +32,8 @@ def register_family(name: str, family: DecoderFamily) -> None:
 
 register_family("Fegilix", DecoderFamily(fegilix.FegilixConfig.from_json, lambda cfg, w, dev: fegilix.build_fegilix(
     cfg, w if w is not None else fegilix.random_weights(cfg, device=dev, low_rank=fegilix.default_rank(cfg)), device=dev)))
+register_family("Rovurax", DecoderFamily(rovurax.RovuraxConfig.from_json, lambda cfg, w, dev: rovurax.build_rovurax(
+    cfg, w if w is not None else rovurax.random_weights(cfg, device=dev), device=dev)))
 register_family("LlamaForCausalLM", DecoderFamily(
     llama.LlamaConfig.from_json, lambda cfg, w, dev: llama.build_llama(cfg, external_weights=True, device=dev, paged=True, state=w)))
 
