@@ -36,7 +36,7 @@ NVCC_FLAGS = [
 
 # Kernels whose arithmetic is specified in 32-bit (recurrences, norms, softmax of fp32 models) keep the accurate divisions,
 # square roots and transcendentals.
-ACCURATE_MATH = {"recurrent.cu", "hybrid.cu"}
+ACCURATE_MATH = {"recurrent.cu", "hybrid.cu", "latent.cu"}
 
 
 def _cuda_home() -> str:

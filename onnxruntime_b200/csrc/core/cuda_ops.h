@@ -8,6 +8,13 @@ namespace ortb {
 
 void CheckLaunch(int rc, const char* what);
 
+// Constants of a clamped gated epilogue, and where a gated product goes: columns [lead, lead + n_out) of a tensor of
+// lead + n_out columns whose first columns another operator fills.
+struct GatedOutput {
+  float limit = 0.f, alpha = 1.f, offset = 0.f;
+  int64_t lead = 0;
+};
+
 // out[M,N] = act(alpha * x[M,K] @ w_nk[N,K]^T + bias) + residual on the tcgen05 GEMM kernel.
 // act == SWIGLU: w_nk holds gate rows then up rows, `dual_offset` rows apart.
 // fused_allreduce: the kernel also sums the result over all ranks through the session's symmetric workspace.
@@ -15,7 +22,7 @@ void CheckLaunch(int rc, const char* what);
 at::Tensor LaunchGemm(OpKernelContext& ctx, const at::Tensor& x2d, const at::Tensor& w_nk, int64_t n_out,
                       int64_t dual_offset, const at::Tensor& bias, const at::Tensor& residual2d, int act, float alpha,
                       bool fused_allreduce = false, at::ScalarType out_type = at::ScalarType::Undefined, float rms_eps = 0.f,
-                      const at::Tensor& alpha_dev = at::Tensor());
+                      const at::Tensor& alpha_dev = at::Tensor(), const GatedOutput* gated = nullptr);
 // MatMulNBits (4-bit) weights as the tile-blob array the decode GEMM expands in shared memory, and that GEMM (M <= 64).
 at::Tensor NbitsBuildBlobs(const at::Tensor& B, const at::Tensor& scales, const at::Tensor& zp_bytes, int64_t N, int64_t K,
                            int64_t block);

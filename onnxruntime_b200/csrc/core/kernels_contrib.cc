@@ -839,6 +839,7 @@ void RegisterContribKernels(KernelRegistry& r) {
   r.RegisterFn("com.ortb200", "GemmSwiGLU", 1, kMax, [normed_input](Ctx& ctx) {
     at::Tensor x = normed_input(ctx, 3);
     at::Tensor gate = at::matmul(x, ctx.RequiredInput(1));
+    if (ctx.node().attr_s("activation", "swiglu") == "clamped_swiglu") ORTB_THROW(NOT_IMPLEMENTED, "GemmSwiGLU: the clamped form is a GPU lowering");
     gate = ctx.node().attr_s("activation", "swiglu") == "geglu" ? at::gelu(gate, "tanh") : at::silu(gate);
     ctx.SetOutput(0, gate * at::matmul(x, ctx.RequiredInput(2)));
   });

@@ -8,6 +8,7 @@
 // onnxruntime/contrib_ops/cuda/bert/{skip_layer_norm.cc,rotary_embedding.cc,
 // group_query_attention.cc,fast_gelu.cc}, quantization/matmul_nbits.cc, moe/moe.cc.
 #include <ATen/ATen.h>
+#include <limits>
 #include <sstream>
 #include <chrono>
 #include <ATen/cuda/CUDAContext.h>
@@ -42,6 +43,7 @@ int ActCode(const std::string& a) {
   if (a == "quickgelu") return ORTB200_ACT_QUICKGELU;
   if (a == "swiglu") return ORTB200_ACT_SWIGLU;
   if (a == "geglu") return ORTB200_ACT_GEGLU;
+  if (a == "clamped_swiglu") return ORTB200_ACT_CLAMPED_SWIGLU;
   ORTB_THROW(INVALID_ARGUMENT, "unknown activation ", a);
 }
 
@@ -75,7 +77,7 @@ void ApplyTunedConfig(Ctx& ctx, ortb200_gemm_args* a, at::ScalarType out_type) {
         if (bn < a->M && bn != 64) continue;  // one token tile per weight tile: the weights stream once
         for (int splits : {1, 2, 4, 8}) cands.push_back({splits, bn, 0});
       }
-    } else if (a->M > 128 && a->in_dtype == 0 && a->act != ORTB200_ACT_SWIGLU) {
+    } else if (a->M > 128 && a->in_dtype == 0 && a->act != ORTB200_ACT_SWIGLU && a->act != ORTB200_ACT_GEGLU && a->act != ORTB200_ACT_CLAMPED_SWIGLU) {
       cands.push_back({0, 0, 128});
       cands.push_back({0, 0, 512});
     }
@@ -130,22 +132,28 @@ void ApplyTunedConfig(Ctx& ctx, ortb200_gemm_args* a, at::ScalarType out_type) {
 // out[M,N] = act(x[M,K] @ w_nk[N,K]^T + bias) + residual on the tcgen05 GEMM.
 at::Tensor LaunchGemm(Ctx& ctx, const at::Tensor& x2d, const at::Tensor& w_nk, int64_t n_out, int64_t dual_offset,
                       const at::Tensor& bias, const at::Tensor& residual2d, int act, float alpha, bool fused_allreduce,
-                      at::ScalarType out_type, float rms_eps, const at::Tensor& alpha_dev) {
+                      at::ScalarType out_type, float rms_eps, const at::Tensor& alpha_dev, const GatedOutput* gated) {
   InferenceSession* s = ctx.session();
   const int64_t M = x2d.size(0), K = x2d.size(1);
   const bool fp8 = x2d.scalar_type() == at::kFloat8_e4m3fn;
   if (out_type == at::ScalarType::Undefined) out_type = x2d.scalar_type();
-  at::Tensor out = at::empty({M, n_out}, x2d.options().dtype(out_type));
+  const int64_t lead = gated ? gated->lead : 0;
+  at::Tensor out = at::empty({M, lead + n_out}, x2d.options().dtype(out_type));
   if (M == 0) return out;
   const int64_t ws_bytes = ortb200_gemm_workspace_bytes(static_cast<int>(M), static_cast<int>(n_out), static_cast<int>(K), act);
   at::Tensor& ws = s->GemmWorkspace(ws_bytes);
   ortb200_gemm_args a{};
   a.x = x2d.data_ptr();
   a.w = w_nk.data_ptr();
-  a.out = out.data_ptr();
+  a.out = static_cast<char*>(out.data_ptr()) + lead * out.element_size();
   a.bias = bias.defined() ? bias.data_ptr() : nullptr;
   a.residual = residual2d.defined() ? residual2d.data_ptr() : nullptr;
-  a.ldo = n_out;
+  a.ldo = lead + n_out;
+  if (gated) {
+    a.gate_limit = gated->limit;
+    a.gate_alpha = gated->alpha;
+    a.gate_offset = gated->offset;
+  }
   a.ldr = residual2d.defined() ? residual2d.stride(0) : 0;
   a.M = static_cast<int>(M);
   a.N = static_cast<int>(n_out);
@@ -201,12 +209,12 @@ at::Tensor RmsNormalizeRows(Ctx& ctx, const at::Tensor& x2d, const at::Tensor& u
 // Runs a GEMM whose weights carry the gamma of a preceding RMS normalisation (rms_eps > 0).
 at::Tensor LaunchNormedGemm(Ctx& ctx, const at::Tensor& x2d, const at::Tensor& w_nk, int64_t n_out, int64_t dual_offset,
                             const at::Tensor& bias, const at::Tensor& residual2d, int act, float alpha, float rms_eps,
-                            const at::Tensor& unit_gamma) {
+                            const at::Tensor& unit_gamma, const GatedOutput* gated = nullptr) {
   if (rms_eps > 0.f && x2d.size(0) > 64) {
     at::Tensor xn = RmsNormalizeRows(ctx, x2d, unit_gamma, rms_eps);
-    return LaunchGemm(ctx, xn, w_nk, n_out, dual_offset, bias, residual2d, act, alpha);
+    return LaunchGemm(ctx, xn, w_nk, n_out, dual_offset, bias, residual2d, act, alpha, false, at::ScalarType::Undefined, 0.f, at::Tensor(), gated);
   }
-  return LaunchGemm(ctx, x2d, w_nk, n_out, dual_offset, bias, residual2d, act, alpha, false, at::ScalarType::Undefined, rms_eps);
+  return LaunchGemm(ctx, x2d, w_nk, n_out, dual_offset, bias, residual2d, act, alpha, false, at::ScalarType::Undefined, rms_eps, at::Tensor(), gated);
 }
 
 // MatMulNBits weights -> the tile-blob array of the in-kernel expansion (layout: ortb200_gemm_args, in_dtype Q4).
@@ -425,7 +433,11 @@ class GemmSwiGLUKernel final : public OpKernel {
     const at::Tensor* wu = info.constant_input(2);
     ORTB_ENFORCE(wg && wu, "GemmSwiGLU needs constant weights");
     I_ = wg->size(1);
-    gelu_ = info.node.attr_s("activation", "swiglu") == "geglu";
+    act_ = ActCode(info.node.attr_s("activation", "swiglu"));
+    gated_.limit = info.node.attr_f("limit", std::numeric_limits<float>::infinity());
+    gated_.alpha = info.node.attr_f("alpha", 1.f);
+    gated_.offset = info.node.attr_f("offset", 0.f);
+    gated_.lead = info.node.attr_i("lead_columns", 0);
     w_ = at::cat({wg->t(), wu->t()}, 0).contiguous();  // [2I, K]: gate rows then up rows
     rms_eps_ = info.node.attr_f("rms_eps", 0.f);
     if (rms_eps_ > 0.f) {
@@ -443,24 +455,32 @@ class GemmSwiGLUKernel final : public OpKernel {
       // Large M: the two-accumulator kernel is limited to 128-token tiles (tensor memory), which costs more than it
       // saves; one plain GEMM over the stacked gate | up rows at 256-token tiles plus a streaming SwiGLU is faster.
       at::Tensor gu = LaunchNormedGemm(ctx, x2, w_, 2 * I_, 0, at::Tensor(), at::Tensor(), ORTB200_ACT_NONE, 1.f, rms_eps_, unit_gamma_);
-      at::Tensor y = at::empty({x2.size(0), I_}, x2.options());
-      CheckLaunch((gelu_ ? ortb200_geglu : ortb200_swiglu)(gu.data_ptr(), y.data_ptr(), x2.size(0), static_cast<int>(I_), DtypeCode(x2.scalar_type()),
-                                                           ctx.cuda_stream()),
-                  "ortb200_swiglu");
+      const int64_t cols = gated_.lead + I_, esize = x2.element_size();
+      at::Tensor y = at::empty({x2.size(0), cols}, x2.options());
+      if (act_ == ORTB200_ACT_CLAMPED_SWIGLU || gated_.lead > 0) {
+        CheckLaunch(ortb200_gated_unit(gu.data_ptr(), static_cast<char*>(gu.data_ptr()) + I_ * esize, static_cast<char*>(y.data_ptr()) + gated_.lead * esize,
+                                       x2.size(0), static_cast<int>(I_), 2 * I_, cols, act_, gated_.limit, gated_.alpha, gated_.offset,
+                                       DtypeCode(x2.scalar_type()), 0, ctx.cuda_stream()),
+                    "ortb200_gated_unit");
+      } else {
+        CheckLaunch((act_ == ORTB200_ACT_GEGLU ? ortb200_geglu : ortb200_swiglu)(gu.data_ptr(), y.data_ptr(), x2.size(0), static_cast<int>(I_),
+                                                                                 DtypeCode(x2.scalar_type()), ctx.cuda_stream()),
+                    "ortb200_swiglu");
+      }
       ctx.session()->AddLaunches(1);
-      ctx.SetOutput(0, y.reshape(OutShape(x, I_)));
+      ctx.SetOutput(0, y.reshape(OutShape(x, cols)));
       return;
     }
-    at::Tensor y = LaunchNormedGemm(ctx, x2, w_, I_, I_, at::Tensor(), at::Tensor(), gelu_ ? ORTB200_ACT_GEGLU : ORTB200_ACT_SWIGLU, 1.f,
-                                    rms_eps_, unit_gamma_);
-    ctx.SetOutput(0, y.reshape(OutShape(x, I_)));
+    at::Tensor y = LaunchNormedGemm(ctx, x2, w_, I_, I_, at::Tensor(), at::Tensor(), act_, 1.f, rms_eps_, unit_gamma_, &gated_);
+    ctx.SetOutput(0, y.reshape(OutShape(x, gated_.lead + I_)));
   }
 
  private:
   at::Tensor w_, unit_gamma_;
   float rms_eps_ = 0.f;
   int64_t I_ = 0;
-  bool gelu_ = false;
+  int act_ = ORTB200_ACT_SWIGLU;
+  GatedOutput gated_;
 };
 
 // com.ortb200.SwiGLU: [..., 2 I] -> silu(x[..., :I]) * x[..., I:], one streaming kernel (behind the stacked gate | up

@@ -6,7 +6,7 @@
 //    add (the reference runs cuBLAS followed by separate BiasGelu / Add kernels).
 //  * SwiGLUFusion:  Mul(silu(MatMul(x, Wg)), MatMul(x, Wu)) -> com.ortb200.GemmSwiGLU(x, Wg, Wu)
 //    one kernel with two TMEM accumulators sharing the activation tile; FastGelu in place of silu sets
-//    activation = "geglu".
+//    activation = "geglu"; com.ortb200.ClampedSwiGLU over the two MatMuls becomes activation = "clamped_swiglu".
 //  * MatMulAllReduceFusion:  AllReduce(GEMM) -> the GEMM carries all_reduce=1 and
 //    its kernel finishes the row-parallel sum over NVLink itself.
 #include "optimizer.h"
@@ -77,6 +77,30 @@ int SwiGLUFusion(PassContext& c) {
       ++count;
       break;
     }
+  }
+  return count;
+}
+
+int ClampedSwiGLUFusion(PassContext& c) {
+  Graph& g = c.g;
+  int count = 0;
+  for (Node* top : g.Nodes()) {
+    if (top->op_type != "ClampedSwiGLU" || top->domain != kFusedDomain) continue;
+    Node *gate = g.Producer(top->inputs[0]), *up = g.Producer(top->inputs[1]);
+    if (!gate || !up || gate == up) continue;
+    if (gate->op_type != "MatMul" || !gate->domain.empty() || up->op_type != "MatMul" || !up->domain.empty() || gate->inputs[0] != up->inputs[0]) continue;
+    if (!IsHalfWeight2D(g, gate->inputs[1]) || !IsHalfWeight2D(g, up->inputs[1])) continue;
+    if (g.GetConstant(gate->inputs[1])->sizes() != g.GetConstant(up->inputs[1])->sizes()) continue;
+    if (SoleConsumer(g, gate->outputs[0]) != top || SoleConsumer(g, up->outputs[0]) != top) continue;
+    Node* f = g.AddNode("GemmSwiGLU", {gate->inputs[0], gate->inputs[1], up->inputs[1]}, {top->outputs[0]}, kFusedDomain, g.UniqueName("GemmSwiGLU"));
+    f->set_attr_s("activation", "clamped_swiglu");
+    for (const char* k : {"limit", "alpha", "offset"})
+      if (top->has_attr(k)) f->set_attr_f(k, top->attr_f(k, 0.f));
+    f->set_attr_i("lead_columns", top->attr_i("lead_columns", 0));
+    g.RemoveNode(top);
+    g.RemoveNode(gate);
+    g.RemoveNode(up);
+    ++count;
   }
   return count;
 }
@@ -403,6 +427,7 @@ void AddGpuPasses(std::vector<Pass>& v) {
   v.push_back({"NBitsSwiGLUFusion", 2, true, NBitsSwiGLUFusion});
   v.push_back({"NBitsAllReduceFusion", 2, true, NBitsAllReduceFusion});
   v.push_back({"SwiGLUFusion", 2, true, SwiGLUFusion});
+  v.push_back({"ClampedSwiGLUFusion", 2, true, ClampedSwiGLUFusion});
   v.push_back({"AllGatherMatMulFusion", 2, true, AllGatherMatMulFusion});
   v.push_back({"MatMulAllReduceFusion", 2, true, MatMulAllReduceFusion});
   v.push_back({"AllReduceResidualFusion", 2, true, AllReduceResidualFusion});

@@ -1,12 +1,21 @@
 // Internal interface between the GEMM dispatcher (gemm_tcgen05.cu) and the decode-shaped kernel (gemm_smallm.cu).
 #pragma once
 #include <cuda_runtime.h>
+#include <math.h>
 #include "ortb200_kernels.h"
+#include "ptx_sm100.cuh"
 
 namespace ortb200 {
 
 // activations that combine two weight tiles (gate rows, up rows)
-inline bool is_gated_act(int act) { return act == ORTB200_ACT_SWIGLU || act == ORTB200_ACT_GEGLU; }
+inline bool is_gated_act(int act) { return act == ORTB200_ACT_SWIGLU || act == ORTB200_ACT_GEGLU || act == ORTB200_ACT_CLAMPED_SWIGLU; }
+
+// The clamped form takes limit (+inf: none), slope and offset from the caller.
+inline GateFn make_gate_fn(int act, float limit, float alpha, float offset) {
+  if (act == ORTB200_ACT_GEGLU) return {INFINITY, 0.f, -1.5957691216057308f, -1.5957691216057308f * 0.044715f};
+  if (act == ORTB200_ACT_CLAMPED_SWIGLU) return {limit, offset, -alpha, 0.f};
+  return {INFINITY, 0.f, -1.f, 0.f};
+}
 
 struct SmallGemmParams {
   int M, N, K;
@@ -16,6 +25,7 @@ struct SmallGemmParams {
   int dtype;
   int act;
   float alpha;
+  GateFn gate;       // gated activations
   void* out;
   long long ldo;
   const void* bias;
@@ -57,9 +67,6 @@ int launch_gemm_grouped_2cta(const ortb200_gemm_grouped_args* a, cudaStream_t st
 int launch_gemm_smallm(const ortb200_gemm_args* a, int bn, cudaStream_t stream, int* cluster_out, int* stages_out);
 
 #ifdef __CUDACC__
-}  // namespace ortb200
-#include "ptx_sm100.cuh"
-namespace ortb200 {
 // ---- epilogue store pass shared by the large-M GEMM kernels (device code)
 template <int ACT>
 __device__ __forceinline__ float act_const(float v) {

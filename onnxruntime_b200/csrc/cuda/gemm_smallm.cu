@@ -562,8 +562,7 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         const float row_scale = p.rms_eps > 0.f ? s_rstd[j] * p.alpha : p.alpha;
         float y = v * row_scale + bias_v;
         if (DUAL) {
-          const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
-          y = g * (u * row_scale);
+          y = gated_unit(p.gate, y, u * row_scale);
         } else {
           y = act_apply(p.act, y);
         }
@@ -734,7 +733,9 @@ int launch_gemm_smallm(const ortb200_gemm_args* a, int bn, cudaStream_t stream, 
   SmallGemmParams p;
   p.nbits_blob = nbits ? a->w : nullptr;
   p.M = a->M; p.N = a->N; p.K = a->K; p.num_kb = num_kb; p.cluster = cluster; p.dual_offset = a->dual_offset;
-  p.dtype = a->dtype; p.act = a->act; p.alpha = a->alpha; p.out = a->out; p.ldo = a->ldo; p.bias = a->bias;
+  p.dtype = a->dtype; p.act = a->act; p.alpha = a->alpha;
+  p.gate = make_gate_fn(a->act, a->gate_limit, a->gate_alpha, a->gate_offset);
+  p.out = a->out; p.ldo = a->ldo; p.bias = a->bias;
   p.residual = a->residual; p.ldr = a->ldr; p.status = a->status;
   p.world = 1; p.rank = 0; p.staging_offset = 0; p.slot_elems = 0; p.epoch = nullptr; p.done = nullptr;
   p.tile_info = nullptr; p.num_tiles = nullptr; p.w_rows_per_expert = 0;
@@ -800,7 +801,9 @@ int launch_gemm_grouped(const ortb200_gemm_grouped_args* a, cudaStream_t stream)
   if (make_tensor_map_2d(&tx, a->x, dt, 2, a->K, a->rows, static_cast<int64_t>(a->K) * 2, kBK, bn) != 0) return -6;
   SmallGemmParams p;
   p.M = a->rows; p.N = a->N; p.K = a->K; p.num_kb = num_kb; p.cluster = 1; p.dual_offset = a->dual_offset;
-  p.dtype = a->dtype; p.act = a->act; p.alpha = 1.0f; p.out = a->out; p.ldo = a->N; p.bias = a->bias;
+  p.dtype = a->dtype; p.act = a->act; p.alpha = 1.0f;
+  p.gate = make_gate_fn(a->act, INFINITY, 1.f, 0.f);
+  p.out = a->out; p.ldo = a->N; p.bias = a->bias;
   p.residual = nullptr; p.ldr = 0; p.status = a->status;
   p.world = 1; p.rank = 0; p.staging_offset = 0; p.slot_elems = 0; p.epoch = nullptr; p.done = nullptr;
   for (int i = 0; i < 8; ++i) p.peers[i] = nullptr;

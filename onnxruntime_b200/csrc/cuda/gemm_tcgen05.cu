@@ -50,6 +50,7 @@ struct GemmKernelParams {
   int k_per_block;    // K elements per pipeline stage: 64 (16-bit operands) or 128 (fp8)
   int act;
   float alpha;
+  GateFn gate;             // gated activations
   const float* alpha_dev;  // optional device scalar multiplied into alpha (runtime scales: no host read)
   void* out;
   long long ldo;
@@ -491,8 +492,7 @@ __device__ __forceinline__ void gemm_tcgen05_body(const CUtensorMap* tmap_w, con
                 // than the gated one are applied on the way out, on the 16-bit value, as a separate op would
                 float y = v[j] * alpha_v + bias_v;
                 if (DUAL) {
-                  const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
-                  y = g * (uu[j] * alpha_v);
+                  y = gated_unit(p.gate, y, uu[j] * alpha_v);
                 }
                 uint16_t bits;
                 if (bf16) {
@@ -586,8 +586,7 @@ __device__ __forceinline__ void gemm_tcgen05_body(const CUtensorMap* tmap_w, con
                 if (m < p.M) {
                   float y = v[j] * alpha_v + bias_v;
                   if (DUAL) {
-                    const float g = gated_act(p.act == ORTB200_ACT_GEGLU, y);
-                    y = g * (uu[j] * alpha_v);
+                    y = gated_unit(p.gate, y, uu[j] * alpha_v);
                   } else {
                     y = apply_act(p.act, y);
                   }
@@ -868,6 +867,7 @@ extern "C" int ortb200_allgather_gemm(const ortb200_allgather_gemm_args* a, ortb
   p.tiles = p.tiles_n * p.tiles_m;
   p.tile_aligned = 1; p.max_contrib = 1;
   p.dtype = a->dtype; p.in_fp8 = 0; p.k_per_block = kBK; p.act = a->act; p.alpha = 1.0f; p.alpha_dev = nullptr;
+  p.gate = make_gate_fn(a->act, INFINITY, 1.f, 0.f);
   p.out = a->out; p.ldo = a->N; p.bias = a->bias; p.residual = nullptr; p.ldr = 0;
   p.status = a->status;
   p.gather_world = a->world; p.gather_rank = a->rank; p.gather_rows = a->rows_local;
@@ -964,6 +964,7 @@ extern "C" int ortb200_gemm(const ortb200_gemm_args* a, ortb200_stream_t stream_
   p.tile_info = nullptr; p.num_tiles = nullptr; p.tiles_n = 0; p.w_rows_per_expert = 0;
   p.tile_aligned = tile_aligned ? 1 : 0; p.max_contrib = max_contrib;
   p.dual_offset = a->dual_offset; p.dtype = a->dtype; p.act = a->act; p.alpha = a->alpha; p.alpha_dev = a->alpha_dev;
+  p.gate = make_gate_fn(a->act, a->gate_limit, a->gate_alpha, a->gate_offset);
   p.out = a->out; p.ldo = a->ldo; p.bias = a->bias; p.residual = a->residual; p.ldr = a->ldr;
   p.counters = reinterpret_cast<unsigned int*>(a->workspace);
   p.ws = a->workspace ? reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(a->workspace) + 65536) : nullptr;
@@ -1017,6 +1018,7 @@ int launch_gemm_grouped_large(const ortb200_gemm_grouped_args* a, cudaStream_t s
   p.num_kb = num_kb; p.tiles = 0; p.tiles_m = 0;
   p.tile_aligned = 1; p.max_contrib = 1;
   p.dual_offset = a->dual_offset; p.dtype = a->dtype; p.in_fp8 = 0; p.k_per_block = kBK; p.act = a->act; p.alpha = 1.0f; p.alpha_dev = nullptr;
+  p.gate = make_gate_fn(a->act, INFINITY, 1.f, 0.f);
   p.out = a->out; p.ldo = a->N; p.bias = a->bias; p.residual = nullptr; p.ldr = 0;
   p.counters = nullptr; p.ws = nullptr; p.status = a->status;
   p.tile_info = static_cast<const int4*>(a->tile_info);

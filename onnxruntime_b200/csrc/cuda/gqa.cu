@@ -205,7 +205,8 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const DecodeParams p) {
     if (tid == 0 && p.status) atomicExch(p.status, kStatusBadLength);
     total = total < 0 ? 0 : p.Smax;
   }
-  const int start0 = p.window > 0 ? max(0, total - p.window) : 0;
+  int start0 = p.window > 0 ? max(0, total - p.window) : 0;
+  if (p.chunk > 0) start0 = max(start0, (total - 1) / p.chunk * p.chunk);
   const int len = max(total - start0, 0);
   const int chunk = (len + p.splits - 1) / p.splits;
   const int k_begin = start0 + split * chunk;
@@ -294,7 +295,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const DecodeParams p) {
   for (int g = 0; g < G; ++g) {
     const int hd = head0 + (g < n_heads ? g : 0);
     const T* qp = fused ? static_cast<const T*>(p.qkv) + qkv_row + static_cast<long long>(hd) * H + d0
-                        : static_cast<const T*>(p.q) + (static_cast<long long>(b) * p.N + hd) * H + d0;
+                        : static_cast<const T*>(p.q) + b * p.q_ld + static_cast<long long>(hd) * H + d0;
     float x[DPL];
 #pragma unroll
     for (int i = 0; i < DPL; ++i) x[i] = to_float<T>(qp[i]);
@@ -530,7 +531,8 @@ static int launch_decode(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
     // about three resident CTAs per SM, but at least two key tiles per CTA at full cache occupancy
     const int ctas = a->B * a->Nk * gparts;
     splits = (2 * 148) / ctas;  // one wave of (register-limited) two CTAs per SM
-    const int max_by_len = (a->Smax + 2 * kDecTile - 1) / (2 * kDecTile);
+    const int longest = a->chunk > 0 && a->chunk < a->Smax ? a->chunk : a->Smax;
+    const int max_by_len = (longest + 2 * kDecTile - 1) / (2 * kDecTile);
     if (splits > max_by_len) splits = max_by_len;
     if (splits > 32) splits = 32;
     if (splits < 1) splits = 1;
@@ -550,6 +552,9 @@ static int launch_decode(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   p.block_table = a->block_table; p.block_size = a->block_size; p.max_blocks = a->max_blocks;
   p.qkv = a->qkv; p.cos_cache = a->cos_cache; p.sin_cache = a->sin_cache; p.cos_rows = a->cos_rows;
   p.prefetch = nullptr; p.prefetch_bytes = 0; p.prefetch_per_cta = 0;
+  p.chunk = a->chunk;
+  p.q_ld = a->q_ld > 0 ? a->q_ld : static_cast<long long>(a->N) * H;
+  p.out_ld = a->out_ld > 0 ? a->out_ld : static_cast<long long>(a->N) * H;
   p.do_rotary = a->do_rotary; p.interleaved = a->rotary_interleaved;
   dim3 grid(splits, a->Nk * gparts, a->B);
   if (a->block_table) {

@@ -506,6 +506,7 @@ int launch_tc_g(int group, const CUtensorMap& tq, const CUtensorMap& tk, const C
 bool gqa_decode_tc_supported(const ortb200_gqa_decode_args* a) {
   if (a->H != 128 || (a->dtype != ORTB200_BF16 && a->dtype != ORTB200_F16)) return false;
   if (a->qkv == nullptr && a->q == nullptr) return false;
+  if (a->chunk > 0 || a->q_ld > 0 || a->out_ld > 0) return false;
   if (a->qkv != nullptr && (reinterpret_cast<uintptr_t>(a->qkv) & 15)) return false;
   const int group = a->N / a->Nk;
   if (group > 16 || !a->workspace) return false;
@@ -573,6 +574,7 @@ int launch_gqa_decode_tc(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   p.qkv = a->qkv; p.cos_cache = a->cos_cache; p.sin_cache = a->sin_cache; p.cos_rows = a->cos_rows;
   p.do_rotary = a->do_rotary; p.interleaved = a->rotary_interleaved;
   dim3 grid(splits, a->Nk, a->B);
+  p.q_ld = p.out_ld = static_cast<long long>(a->N) * H;
   p.prefetch = nullptr; p.prefetch_bytes = 0; p.prefetch_per_cta = 0;
   if (a->prefetch != nullptr && a->prefetch_bytes >= 16 && (reinterpret_cast<uintptr_t>(a->prefetch) & 15) == 0) {
     const long long bytes = (a->prefetch_bytes < (48LL << 20) ? a->prefetch_bytes : (48LL << 20)) & ~15LL;

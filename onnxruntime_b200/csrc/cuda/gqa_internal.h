@@ -34,6 +34,8 @@ struct DecodeParams {
   const unsigned char* prefetch;
   long long prefetch_bytes;
   int prefetch_per_cta;
+  int chunk;               // CUDA-core kernel: > 0 = keys of the new token's own chunk only
+  long long q_ld, out_ld;  // elements between the rows of q and of out
 };
 
 // Running maxima start at a large negative finite value so that exp(m_old - m_new) never sees inf - inf.
@@ -113,7 +115,7 @@ __device__ __forceinline__ void decode_finish(const DecodeParams& p, int tile, i
         fa[g] *= c;
       }
       const float o = ll > 0.f ? fa[g] / ll : 0.f;
-      static_cast<T*>(p.out)[(static_cast<long long>(b) * p.N + head0 + g) * H + tid] = from_float<T>(o);
+      static_cast<T*>(p.out)[b * p.out_ld + static_cast<long long>(head0 + g) * H + tid] = from_float<T>(o);
     }
   }
 }

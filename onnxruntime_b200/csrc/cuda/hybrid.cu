@@ -6,8 +6,10 @@
 //   paged_attn     causal attention over the paged cache for any head sizes and types, fp32 on CUDA cores: the path for
 //                  fp32 models and for head sizes outside the tensor-core kernels
 //   head_gate      sigmoid output gate + removal of the head padding behind the tensor-core kernels
+//   gated_unit     act(gate) * up of two inputs, written into columns of a wider tensor
 #include <cuda_runtime.h>
 #include <math.h>
+#include "gemm_internal.h"
 #include "launch_util.cuh"
 #include "ortb200_kernels.h"
 #include "ptx_sm100.cuh"
@@ -182,13 +184,21 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kernel(const ortb200_qk_norm
   const float* sn = a.sin_table + static_cast<long long>(ok ? pos : 0) * half;
   const T* row = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld;
   const int units = a.N + (a.kv_shared ? 0 : 2 * a.Nk);
-  for (int u = blockIdx.y * 8 + warp; u < units; u += 8 * gridDim.y) {
+  const int first_unit = a.q_out ? 0 : a.N;
+  for (int u = first_unit + blockIdx.y * 8 + warp; u < units; u += 8 * gridDim.y) {
     const bool is_q = u < a.N, is_v = u >= a.N + a.Nk;
     if (!is_q && !ok) continue;
     if (is_v) {
       const int h = u - a.N - a.Nk;
       const T* src = row + (a.N + a.Nk) * a.dk + h * a.dv;
       T* dst = static_cast<T*>(a.v_cache) + (entry * a.Nk + h) * a.dv_pad;
+      if (a.first_values) {
+        const T* first = static_cast<const T*>(a.first_values) + t * a.first_ld + h * a.dv;
+        const float m = *a.v_mix;
+        for (int d = lane; d < a.dv_pad; d += 32)
+          dst[d] = from_float<T>(d < a.dv ? fmaf(m, to_float<T>(first[d]), (1.f - m) * to_float<T>(src[d])) : 0.f);
+        continue;
+      }
       for (int d = lane; d < a.dv_pad; d += 32) dst[d] = d < a.dv ? src[d] : from_float<T>(0.f);
       continue;
     }
@@ -238,7 +248,8 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const ortb200_paged_att
   const T* qp = static_cast<const T*>(a.q) + (static_cast<long long>(t) * a.N + h) * a.dk_pad;
   for (int d = tid; d < a.dk_pad; d += 128) q[d] = to_float<T>(qp[d]);
   __syncthreads();
-  const int begin = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  int begin = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  if (a.chunk > 0) begin = max(begin, pos / a.chunk * a.chunk);
   const int end = min(pos + 1, a.max_blocks * a.block_size);
   float m = kNeg, l = 0.f, acc[kMaxHead / 32];
 #pragma unroll
@@ -302,7 +313,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const ortb200_paged_att
   }
   const float inv = den > 0.f ? 1.f / den : 0.f;
   const T* gate = a.gate ? static_cast<const T*>(a.gate) + t * a.gate_ld + h * a.dv : nullptr;
-  T* out = static_cast<T*>(a.out) + (static_cast<long long>(t) * a.N + h) * a.dv;
+  T* out = static_cast<T*>(a.out) + t * (a.out_ld > 0 ? a.out_ld : static_cast<long long>(a.N) * a.dv) + h * a.dv;
   for (int d = tid; d < a.dv; d += 128) {
     float o = 0.f;
 #pragma unroll
@@ -315,7 +326,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const ortb200_paged_att
 
 template <typename T>
 __global__ void __launch_bounds__(256) head_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, T* __restrict__ out, int64_t n,
-                                                        int heads, int dv, int x_pad, int64_t gate_ld) {
+                                                        int heads, int dv, int x_pad, int64_t gate_ld, int64_t out_ld) {
   pdl_wait_prior_grids();
   const int64_t stride = static_cast<int64_t>(gridDim.x) * blockDim.x;
   const int row = heads * dv;
@@ -324,7 +335,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const T* __restrict__ x,
     const int c = static_cast<int>(i % row), h = c / dv, j = c % dv;
     float v = to_float<T>(x[(t * heads + h) * x_pad + j]);
     if (gate) v *= sigmoid_f(to_float<T>(gate[t * gate_ld + c]));
-    out[i] = from_float<T>(v);
+    out[t * out_ld + c] = from_float<T>(v);
   }
   pdl_launch_dependents();
 }
@@ -332,7 +343,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const T* __restrict__ x,
 // the same for 16-bit types with dv, x_pad and gate_ld multiples of 8: one 16-byte access each
 template <typename T>
 __global__ void __launch_bounds__(256) head_gate_vec8_kernel(const T* __restrict__ x, const T* __restrict__ gate, T* __restrict__ out,
-                                                             int64_t n8, int heads, int dv, int x_pad, int64_t gate_ld) {
+                                                             int64_t n8, int heads, int dv, int x_pad, int64_t gate_ld, int64_t out_ld) {
   pdl_wait_prior_grids();
   const int64_t stride = static_cast<int64_t>(gridDim.x) * blockDim.x;
   const int row8 = heads * dv / 8, dv8 = dv / 8;
@@ -347,7 +358,46 @@ __global__ void __launch_bounds__(256) head_gate_vec8_kernel(const T* __restrict
     __align__(16) T o[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) o[e] = from_float<T>(gate ? to_float<T>(xe[e]) * sigmoid_f(to_float<T>(ge[e])) : to_float<T>(xe[e]));
-    reinterpret_cast<uint4*>(out)[i] = *reinterpret_cast<const uint4*>(o);
+    *reinterpret_cast<uint4*>(out + t * out_ld + static_cast<int64_t>(c) * 8) = *reinterpret_cast<const uint4*>(o);
+  }
+  pdl_launch_dependents();
+}
+
+// 16-bit results: fast exponential and division; 32-bit: the accurate ones this file is compiled with
+template <typename T>
+__device__ __forceinline__ float gated_value(const GateFn& f, float gate, float up) {
+  if constexpr (sizeof(T) == 2) {
+    const float g = fminf(gate, f.limit);
+    const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
+    return __fdividef(g, 1.f + __expf(g * (f.c1 + f.c3 * g * g))) * u;
+  } else {
+    const float g = fminf(gate, f.limit);
+    const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
+    return g / (1.f + expf(g * (f.c1 + f.c3 * g * g))) * u;
+  }
+}
+
+// E elements per access: 8 for 16-bit types on aligned rows, else 1
+template <typename T, int E>
+__global__ void __launch_bounds__(256) gated_unit_kernel(const T* __restrict__ gate, const T* __restrict__ up, T* __restrict__ out, int64_t rows,
+                                                         int cols, int64_t ld_in, int64_t ld_out, const GateFn f) {
+  pdl_wait_prior_grids();
+  const int per_row = cols / E;
+  const int64_t n = rows * per_row, stride = static_cast<int64_t>(gridDim.x) * blockDim.x;
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const int64_t r = i / per_row;
+    const int c = static_cast<int>(i % per_row) * E;
+    if constexpr (E == 8) {
+      const uint4 gv = *reinterpret_cast<const uint4*>(gate + r * ld_in + c), uv = *reinterpret_cast<const uint4*>(up + r * ld_in + c);
+      const T* ge = reinterpret_cast<const T*>(&gv);
+      const T* ue = reinterpret_cast<const T*>(&uv);
+      __align__(16) T o[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = from_float<T>(gated_value<T>(f, to_float<T>(ge[e]), to_float<T>(ue[e])));
+      *reinterpret_cast<uint4*>(out + r * ld_out + c) = *reinterpret_cast<const uint4*>(o);
+    } else {
+      out[r * ld_out + c] = from_float<T>(gated_value<T>(f, to_float<T>(gate[r * ld_in + c]), to_float<T>(up[r * ld_in + c])));
+    }
   }
   pdl_launch_dependents();
 }
@@ -358,14 +408,28 @@ unsigned grid_1d(int64_t n) {
 }
 
 template <typename T>
-int run_head_gate(const void* x, const void* gate, void* out, int T_, int heads, int dv, int x_pad, int64_t gate_ld, bool pdl, cudaStream_t st) {
+int run_head_gate(const void* x, const void* gate, void* out, int T_, int heads, int dv, int x_pad, int64_t gate_ld, int64_t out_ld, bool pdl,
+                  cudaStream_t st) {
   const int64_t n = static_cast<int64_t>(T_) * heads * dv;
   const uintptr_t align = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out);
   const T *xp = static_cast<const T*>(x), *gp = static_cast<const T*>(gate);
   T* op = static_cast<T*>(out);
-  if (sizeof(T) == 2 && dv % 8 == 0 && x_pad % 8 == 0 && gate_ld % 8 == 0 && (align & 15) == 0)
-    return launch_kernel(head_gate_vec8_kernel<T>, dim3(grid_1d(n / 8)), 256, 0, st, pdl, xp, gp, op, n / 8, heads, dv, x_pad, gate_ld);
-  return launch_kernel(head_gate_kernel<T>, dim3(grid_1d(n)), 256, 0, st, pdl, xp, gp, op, n, heads, dv, x_pad, gate_ld);
+  if (sizeof(T) == 2 && dv % 8 == 0 && x_pad % 8 == 0 && gate_ld % 8 == 0 && out_ld % 8 == 0 && (align & 15) == 0)
+    return launch_kernel(head_gate_vec8_kernel<T>, dim3(grid_1d(n / 8)), 256, 0, st, pdl, xp, gp, op, n / 8, heads, dv, x_pad, gate_ld, out_ld);
+  return launch_kernel(head_gate_kernel<T>, dim3(grid_1d(n)), 256, 0, st, pdl, xp, gp, op, n, heads, dv, x_pad, gate_ld, out_ld);
+}
+
+template <typename T>
+int run_gated_unit(const void* gate, const void* up, void* out, int64_t rows, int cols, int64_t ld_in, int64_t ld_out, const GateFn& f, bool pdl,
+                   cudaStream_t st) {
+  const uintptr_t align = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out);
+  const T *g = static_cast<const T*>(gate), *u = static_cast<const T*>(up);
+  T* o = static_cast<T*>(out);
+  if constexpr (sizeof(T) == 2) {
+    if (cols % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && (align & 15) == 0)
+      return launch_kernel(gated_unit_kernel<T, 8>, dim3(grid_1d(rows * cols / 8)), 256, 0, st, pdl, g, u, o, rows, cols, ld_in, ld_out, f);
+  }
+  return launch_kernel(gated_unit_kernel<T, 1>, dim3(grid_1d(rows * cols)), 256, 0, st, pdl, g, u, o, rows, cols, ld_in, ld_out, f);
 }
 
 }  // namespace
@@ -373,6 +437,20 @@ int run_head_gate(const void* x, const void* gate, void* out, int T_, int heads,
 }  // namespace ortb200
 
 using namespace ortb200;
+
+extern "C" int ortb200_gated_unit(const void* gate, const void* up, void* out, int64_t rows, int cols, int64_t ld_in, int64_t ld_out, int act,
+                                  float limit, float alpha, float offset, int dtype, int use_pdl, ortb200_stream_t stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (!gate || !up || !out || rows < 0 || cols <= 0 || ld_in < cols || ld_out < cols || !is_gated_act(act)) return -1;
+  if (rows == 0) return 0;
+  const GateFn f = make_gate_fn(act, limit, alpha, offset);
+  switch (dtype) {
+    case ORTB200_F16: return run_gated_unit<__half>(gate, up, out, rows, cols, ld_in, ld_out, f, use_pdl != 0, stream);
+    case ORTB200_BF16: return run_gated_unit<__nv_bfloat16>(gate, up, out, rows, cols, ld_in, ld_out, f, use_pdl != 0, stream);
+    case ORTB200_F32: return run_gated_unit<float>(gate, up, out, rows, cols, ld_in, ld_out, f, use_pdl != 0, stream);
+    default: return -4;
+  }
+}
 
 extern "C" int ortb200_hyper_norm(const ortb200_hyper_norm_args* a, ortb200_stream_t stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
@@ -408,14 +486,16 @@ extern "C" int ortb200_softcap(const void* x, float* y, int64_t n, float cap, in
 
 extern "C" int ortb200_qk_norm_rope(const ortb200_qk_norm_rope_args* a, ortb200_stream_t stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (!a || !a->packed || !a->q_out || !a->cu_seqlens || !a->past_seqlens || !a->block_table) return -1;
+  if (!a || !a->packed || !a->cu_seqlens || !a->past_seqlens || !a->block_table) return -1;
+  if (!a->q_out && (a->kv_shared || a->q_norm || a->rot_dim > 0)) return -1;
   if (!a->kv_shared && (!a->k_cache || !a->v_cache)) return -1;
+  if (a->first_values && (!a->v_mix || a->first_ld < static_cast<int64_t>(a->Nk) * a->dv)) return -1;
   if (a->T <= 0 || a->B <= 0 || a->N <= 0 || a->Nk <= 0 || a->N % a->Nk != 0) return -2;
   if (a->dk <= 0 || a->dk > kMaxHead || a->dv <= 0 || a->dk_pad < a->dk || a->dv_pad < a->dv || a->dk_pad > kMaxHead) return -2;
   if (a->rot_dim < 0 || a->rot_dim > a->dk || a->rot_dim % 2 != 0 || (a->rot_dim > 0 && (!a->cos_table || !a->sin_table))) return -2;
   if (a->table_rows <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->num_blocks <= 0) return -2;
   if (a->ld < a->N * a->dk + (a->kv_shared ? 0 : a->Nk * (a->dk + a->dv))) return -2;
-  const int units = a->N + (a->kv_shared ? 0 : 2 * a->Nk);
+  const int units = (a->q_out ? a->N : 0) + (a->kv_shared ? 0 : 2 * a->Nk);
   int gy = 1;   // few tokens: several blocks share the heads of one token
   while (gy * a->T < 148 && gy * 8 < units) gy *= 2;
   const dim3 grid(a->T, gy);
@@ -443,14 +523,16 @@ extern "C" int ortb200_paged_attn(const ortb200_paged_attn_args* a, ortb200_stre
   }
 }
 
-extern "C" int ortb200_head_gate(const void* x, const void* gate, void* out, int T, int heads, int dv, int x_pad, int64_t gate_ld, int dtype,
-                                 int use_pdl, ortb200_stream_t stream_) {
+extern "C" int ortb200_head_gate(const void* x, const void* gate, void* out, int T, int heads, int dv, int x_pad, int64_t gate_ld, int64_t out_ld,
+                                 int dtype, int use_pdl, ortb200_stream_t stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (!x || !out || T <= 0 || heads <= 0 || dv <= 0 || x_pad < dv || (gate && gate_ld < static_cast<int64_t>(heads) * dv)) return -1;
+  if (!x || !out || T <= 0 || heads <= 0 || dv <= 0 || x_pad < dv || out_ld < static_cast<int64_t>(heads) * dv ||
+      (gate && gate_ld < static_cast<int64_t>(heads) * dv))
+    return -1;
   switch (dtype) {
-    case ORTB200_F16: return run_head_gate<__half>(x, gate, out, T, heads, dv, x_pad, gate_ld, use_pdl != 0, stream);
-    case ORTB200_BF16: return run_head_gate<__nv_bfloat16>(x, gate, out, T, heads, dv, x_pad, gate_ld, use_pdl != 0, stream);
-    case ORTB200_F32: return run_head_gate<float>(x, gate, out, T, heads, dv, x_pad, gate_ld, use_pdl != 0, stream);
+    case ORTB200_F16: return run_head_gate<__half>(x, gate, out, T, heads, dv, x_pad, gate_ld, out_ld, use_pdl != 0, stream);
+    case ORTB200_BF16: return run_head_gate<__nv_bfloat16>(x, gate, out, T, heads, dv, x_pad, gate_ld, out_ld, use_pdl != 0, stream);
+    case ORTB200_F32: return run_head_gate<float>(x, gate, out, T, heads, dv, x_pad, gate_ld, out_ld, use_pdl != 0, stream);
     default: return -4;
   }
 }

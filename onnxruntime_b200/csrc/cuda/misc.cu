@@ -106,7 +106,7 @@ __global__ void swiglu_kernel(const T* __restrict__ x, T* __restrict__ y, int64_
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
     const int64_t r = i / cols, c = i % cols;
     const float g = to_float<T>(x[r * 2 * cols + c]), u = to_float<T>(x[r * 2 * cols + cols + c]);
-    y[i] = from_float<T>(gated_act(GELU, g) * u);
+    y[i] = from_float<T>((GELU ? gelu_tanh(g) : g / (1.0f + __expf(-g))) * u);
   }
   pdl_launch_dependents();
 }
@@ -126,7 +126,7 @@ __global__ void __launch_bounds__(256) swiglu_vec8_kernel(const uint4* __restric
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float gv = to_float<T>(g[e]);
-      o[e] = from_float<T>(gated_act(GELU, gv) * to_float<T>(u[e]));
+      o[e] = from_float<T>((GELU ? gelu_tanh(gv) : gv / (1.0f + __expf(-gv))) * to_float<T>(u[e]));
     }
     y[i] = *reinterpret_cast<const uint4*>(o);
   }

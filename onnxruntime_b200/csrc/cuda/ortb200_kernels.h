@@ -28,6 +28,7 @@ enum ortb200_act {
   ORTB200_ACT_SWIGLU = 5,    // silu(W1 x) * (W2 x); W2 rows start `dual_offset` rows after W1 rows
   ORTB200_ACT_QUICKGELU = 6,
   ORTB200_ACT_GEGLU = 7,     // gelu_tanh(W1 x) * (W2 x), rows laid out as for SWIGLU
+  ORTB200_ACT_CLAMPED_SWIGLU = 8,  // g sigmoid(alpha g) (u + offset), g = min(W1 x, limit), u = clamp(W2 x, -limit, limit); rows as for SWIGLU
 };
 
 // out[M, N] = act(alpha * X[M, K] * W[N, K]^T + bias[N]) + residual[M, N]
@@ -105,6 +106,7 @@ typedef struct {
   // Optional device scalar (fp32) multiplied into alpha by the kernel: scales that only exist on the device (GemmFloat8 with
   // runtime scale inputs) need no host read.  fp8 operand mode only; null otherwise.
   const float* alpha_dev;
+  float gate_limit, gate_alpha, gate_offset;  // CLAMPED_SWIGLU only (limit +inf: none)
 } ortb200_gemm_args;
 
 int ortb200_gemm(const ortb200_gemm_args* args, ortb200_stream_t stream);
@@ -342,6 +344,10 @@ typedef struct {
   const void* prefetch;
   int64_t prefetch_bytes;
   int cos_rows;           // rows of cos_cache / sin_cache; the rotary position is clamped to it (0 = not checked)
+  // CUDA-core kernel only: attend within chunks of this many positions (the new token sees its own chunk; <= 0: none), and
+  // elements between the rows of q and of out (0 = N H)
+  int chunk;
+  int64_t q_ld, out_ld;
 } ortb200_gqa_decode_args;
 int ortb200_gqa_decode(const ortb200_gqa_decode_args* args, ortb200_stream_t stream);
 int64_t ortb200_gqa_decode_workspace_bytes(int B, int N, int H);
@@ -384,6 +390,7 @@ typedef struct {
   // Softmax weights enter the second product as the sum of two 16-bit terms instead of one (fp32-like weights for 1.5x
   // the tensor-core work).
   int split_weights;
+  int chunk;               // > 0: a query sees only keys of its own chunk of this many positions (positions count from 0)
 } ortb200_attn_prefill_args;
 int ortb200_attn_prefill(const ortb200_attn_prefill_args* args, ortb200_stream_t stream);
 
@@ -594,7 +601,7 @@ int ortb200_softcap(const void* x, float* y, int64_t n, float cap, int dtype, or
 // entries (rotate-half layout, fp32 tables), K / V appended to the paged cache, heads zero-padded to the cache's widths.
 typedef struct {
   const void* packed;      // [T, ld]: q (N * dk) | k (Nk * dk) | v (Nk * dv) | ...; q only when kv_shared
-  void* q_out;             // [T, N, dk_pad] dtype
+  void* q_out;             // [T, N, dk_pad] dtype; null: the queries are used as they lie in `packed`
   void* k_cache;           // [num_blocks, block_size, Nk, dk_pad]
   void* v_cache;           // [num_blocks, block_size, Nk, dv_pad]
   const float* q_norm;     // optional [dk]
@@ -612,6 +619,11 @@ typedef struct {
   int dtype;
   int use_pdl;
   int* status;
+  // Optional: values of another layer for the same tokens (row t at first_values + t * first_ld elements, Nk * dv of them);
+  // the stored value is (1 - m) v + m first with m = *v_mix.
+  const void* first_values;
+  int64_t first_ld;
+  const float* v_mix;
 } ortb200_qk_norm_rope_args;
 int ortb200_qk_norm_rope(const ortb200_qk_norm_rope_args* args, ortb200_stream_t stream);
 
@@ -634,12 +646,123 @@ typedef struct {
   float scale;
   int dtype;
   int use_pdl;
+  int chunk;               // > 0: keys of the query's own chunk only
+  int64_t out_ld;          // elements between rows of out (0 = N * dv)
 } ortb200_paged_attn_args;
 int ortb200_paged_attn(const ortb200_paged_attn_args* args, ortb200_stream_t stream);
 
-// out[t, h * dv + j] = x[t, h, j] * sigmoid(gate[t, h * dv + j]) for x [T, heads, x_pad] (gate null: plain compaction)
-int ortb200_head_gate(const void* x, const void* gate, void* out, int T, int heads, int dv, int x_pad, int64_t gate_ld, int dtype,
-                      int use_pdl, ortb200_stream_t stream);
+// out[t * out_ld + h * dv + j] = x[t, h, j] * sigmoid(gate[t, h * dv + j]) for x [T, heads, x_pad] (gate null: plain
+// compaction)
+int ortb200_head_gate(const void* x, const void* gate, void* out, int T, int heads, int dv, int x_pad, int64_t gate_ld, int64_t out_ld,
+                      int dtype, int use_pdl, ortb200_stream_t stream);
+
+// A gated unit (ortb200_act: SWIGLU, GEGLU or CLAMPED_SWIGLU) of two inputs [rows, cols] with ld_in elements between rows;
+// out has ld_out.  32-bit inputs are computed with accurate exponentials and divisions.
+int ortb200_gated_unit(const void* gate, const void* up, void* out, int64_t rows, int cols, int64_t ld_in, int64_t ld_out, int act,
+                       float limit, float alpha, float offset, int dtype, int use_pdl, ortb200_stream_t stream);
+
+// ---------------------------------------------------------------------------
+// Latent attention: per token one latent c of `rank` entries (RMS-normed) and one rotated key part of dr entries that all
+// heads share.  Per head the unrotated key is Uk c and the value Uv c, the score (q . Uk c + q_r . k_r) scale.  A cache
+// entry is [c, zero-padded to `wide` | k_r, zero-padded to `width` - wide]; caches are [num_blocks, block_size, width].
+//
+// Two forms.  Absorbed (few tokens): ortb200_latent_absorb turns the query into Uk^T q and appends the new entries,
+// ortb200_latent_decode attends over the cache as it lies, ortb200_latent_out merges, applies Uv and the output gate.
+// Expanded (prompts): ortb200_latent_prep rotates and appends, ortb200_latent_gather collects cached latents behind one
+// another when there are any, a GEMM expands keys and values of all heads, ortb200_latent_prefill is the flash kernel.
+typedef struct {
+  const void* packed;      // [T, ld]: q (N * (dk + dr)) | latent (rank) | key part (dr) | gate (N) | padding
+  void* cache;
+  const float* norm;       // [rank]
+  const float* cos_table;  // [rows, rot_dim / 2], pairs (2 i, 2 i + 1) of the first rot_dim of the dr entries turn; null: none
+  const float* sin_table;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* block_table;
+  int T, B, ld, N, dk, dr, rank, wide, width;
+  int rot_dim, table_rows;
+  int block_size, max_blocks, num_blocks;
+  float eps;
+  int dtype;               // F16, BF16 or F32: packed, cache
+  int use_pdl;
+  int* status;
+  // absorbed form
+  const void* up;          // [N * (dk + dv), rank]: rows of Uk, then of Uv
+  void* q_abs;             // [T, N, width], `dtype` or (q_abs_f32) fp32: Uk^T q | rotated q_r, laid out as a cache entry
+  int q_abs_f32;
+  // expanded form
+  void* q_rot;             // [T, N, dr]
+  void* c_out;             // optional copies of the new entries: [T, rank]
+  void* k_rot_out;         // [T, width - wide]
+} ortb200_latent_prep_args;
+int ortb200_latent_absorb(const ortb200_latent_prep_args* args, ortb200_stream_t stream);
+int ortb200_latent_prep(const ortb200_latent_prep_args* args, ortb200_stream_t stream);
+
+// All cached entries of the B sequences (past_seqlens[b] + new tokens each), sequence behind sequence: c_out [rows, rank],
+// k_rot_out [rows, width - wide].  `rows` is their number.
+int ortb200_latent_gather(const void* cache, const int* cu_seqlens, const int* past_seqlens, const int* block_table, void* c_out, void* k_rot_out,
+                          int rows, int B, int rank, int wide, int width, int block_size, int max_blocks, int num_blocks, int dtype, int use_pdl,
+                          int* status, ortb200_stream_t stream);
+
+// Attention of absorbed queries over the cache.  Key ranges are split into `parts` (from ortb200_latent_decode_plan); per
+// (token, head, part) the result is sum_j p_j c_j (unnormalised, `wide` floats), the maximum of the base-2 scores and the
+// sum of p_j = 2^(score - maximum).
+typedef struct {
+  const void* q_abs;       // [T, N, width]
+  const void* cache;
+  const int* cu_seqlens;
+  const int* past_seqlens;
+  const int* block_table;
+  float* o;                // [T, N, parts, wide]
+  float* ml;               // [T, N, parts, 2]
+  int T, B, N, rank, wide, width, parts;
+  int block_size, max_blocks, num_blocks;
+  float scale;
+  int dtype;               // of the cache; q_abs has it in the tensor-core form and is fp32 in the other
+  int tensor_cores;        // from ortb200_latent_decode_plan
+  int use_pdl;
+  int* status;
+} ortb200_latent_decode_args;
+// Whether the tensor-core kernel takes these sizes (else the CUDA-core kernel runs, with one part), and the parts to use.
+int ortb200_latent_decode_plan(int T, int N, int wide, int width, int block_size, int max_blocks, int dtype, int* parts);
+int ortb200_latent_decode(const ortb200_latent_decode_args* args, ortb200_stream_t stream);
+
+// out[t * out_ld + h * dv + j] = sigmoid(gate[t, h]) sum_c Uv[h * dv + j, c] o[t, h, c], o merged over the parts and divided
+// by the sum of exponentials (plus that of the head's sink).
+typedef struct {
+  const float* o;          // [T, N, parts, wide]
+  const float* ml;
+  const float* sink;       // optional [N]
+  const void* up_v;        // [N * dv, rank]
+  const void* gate;        // optional: row t at gate + t * gate_ld elements, N entries
+  void* out;
+  int64_t gate_ld, out_ld;
+  int T, N, dv, rank, wide, parts;
+  int dtype;
+  int use_pdl;
+} ortb200_latent_out_args;
+int ortb200_latent_out(const ortb200_latent_out_args* args, ortb200_stream_t stream);
+
+// Causal flash attention of packed queries over expanded keys and values (16-bit types, softmax weights as the sum of two
+// 16-bit terms).  Sizes: dk, dr, dv multiples of 8, dv <= 128, ceil(dk / 64) + ceil(dr / 64) <= 3.
+typedef struct {
+  const void* q;           // row t at q + t * q_ld elements: per head dk unrotated entries, then dr that are not read
+  const void* q_rot;       // [T, N, dr]
+  const void* kv;          // [key_rows, kv_ld]: unrotated keys (N * dk) | values (N * dv)
+  const void* k_rot;       // [key_rows, k_rot_ld]
+  const void* head_sink;   // optional [N], dtype
+  const void* gate;        // optional: row t at gate + t * gate_ld elements, N entries; sigmoid factor of a head's output
+  void* out;               // row t at out + t * out_ld elements: N * dv
+  const int* cu_seqlens;
+  const int* past_seqlens; // keys of sequence b: past_seqlens[b] + its new tokens, behind those of the sequences before it
+  int64_t q_ld, kv_ld, k_rot_ld, gate_ld, out_ld;
+  int T, B, N, dk, dr, dv, key_rows;
+  float scale;
+  int dtype;
+  int* status;
+} ortb200_latent_prefill_args;
+int ortb200_latent_prefill_supported(int dk, int dr, int dv, int dtype);
+int ortb200_latent_prefill(const ortb200_latent_prefill_args* args, ortb200_stream_t stream);
 
 #ifdef __cplusplus
 }

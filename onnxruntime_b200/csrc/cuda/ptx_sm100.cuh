@@ -342,8 +342,17 @@ __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.
 
 // tanh form of gelu, written as v * sigmoid(2 z): 0.5 (1 + tanh z) = 1 / (1 + exp(-2 z))
 __device__ __forceinline__ float gelu_tanh(float v) { return v / (1.0f + __expf(-1.5957691216057308f * v * (1.0f + 0.044715f * v * v))); }
-// gate activation of the gated (two-weight) epilogues: silu, or the tanh form of gelu
-__device__ __forceinline__ float gated_act(bool gelu, float v) { return gelu ? gelu_tanh(v) : v / (1.0f + __expf(-v)); }
+// Gated (two-weight) units as one formula, so that an unrolled epilogue holds no switch:
+//   g = min(gate, limit), u = clamp(up, -limit, limit) + offset, result = g / (1 + exp(g (c1 + c3 g^2))) u
+// silu: c1 = -1; a sigmoid of slope alpha: c1 = -alpha; the tanh form of gelu: c1 = -2 sqrt(2 / pi), c3 = 0.044715 c1.
+struct GateFn {
+  float limit, offset, c1, c3;
+};
+__device__ __forceinline__ float gated_unit(const GateFn& f, float gate, float up) {
+  const float g = fminf(gate, f.limit);
+  const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
+  return g / (1.0f + __expf(g * (f.c1 + f.c3 * g * g))) * u;
+}
 
 // Exact-form GELU, 0.5 x (1 + erf(x / sqrt 2)), with erf from the rational approximation 7.1.26 of Abramowitz &
 // Stegun (absolute error below 1.5e-7, far under the resolution of the 16-bit outputs it feeds): one reciprocal, one

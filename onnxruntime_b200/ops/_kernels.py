@@ -16,7 +16,8 @@ import torch
 _LIB: Optional[ctypes.CDLL] = None
 
 F16, BF16, F32 = 0, 1, 2
-ACT = {"none": 0, "gelu": 1, "fastgelu": 2, "relu": 3, "silu": 4, "swiglu": 5, "quickgelu": 6, "geglu": 7}
+ACT = {"none": 0, "gelu": 1, "fastgelu": 2, "relu": 3, "silu": 4, "swiglu": 5, "quickgelu": 6, "geglu": 7, "clamped_swiglu": 8}
+GATED = ("swiglu", "geglu", "clamped_swiglu")
 
 
 def lib_path() -> str:
@@ -55,7 +56,7 @@ class GemmArgs(ctypes.Structure):
         ("force_splits", ctypes.c_int), ("force_bn", ctypes.c_int), ("use_pdl", ctypes.c_int),
         ("world", ctypes.c_int), ("rank", ctypes.c_int), ("peers", ctypes.c_void_p * 8), ("symm_bytes", ctypes.c_int64),
         ("in_dtype", ctypes.c_int), ("rms_eps", ctypes.c_float), ("force_tile_rows", ctypes.c_int), ("mc_ptr", ctypes.c_void_p),
-        ("alpha_dev", ctypes.c_void_p),
+        ("alpha_dev", ctypes.c_void_p), ("gate_limit", ctypes.c_float), ("gate_alpha", ctypes.c_float), ("gate_offset", ctypes.c_float),
     ]
 
 
@@ -86,7 +87,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          force_splits: int = 0, force_bn: int = 0, status: Optional[torch.Tensor] = None,
          use_pdl: bool = False, peers=None, rank: int = 0, symm_bytes: int = 0,
          out_dtype: Optional[torch.dtype] = None, rms_eps: float = 0.0, force_tile_rows: int = 0,
-         q4: bool = False, mc_ptr: int = 0) -> torch.Tensor:
+         q4: bool = False, mc_ptr: int = 0, gate=(float("inf"), 1.0, 0.0)) -> torch.Tensor:
     """out[M, N] = act(alpha * x[M, K] @ w[N, K].T + bias) + residual  (tcgen05 kernel).
     x / w of dtype float8_e4m3fn use the 8-bit tensor-core mode; out_dtype (fp16 / bf16) is then required."""
     assert x.is_cuda and w.is_cuda and (x.dtype == w.dtype or q4) and x.dim() == 2
@@ -97,8 +98,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
     M, K = x.shape
     w_rows = w.shape[0]
     if n is None:
-        n = w_rows // 2 if act == "swiglu" else w_rows
-        if act == "swiglu" and dual_offset == 0:
+        n = w_rows // 2 if act in GATED else w_rows
+        if act in GATED and dual_offset == 0:
             dual_offset = n
     fp8 = x.dtype == torch.float8_e4m3fn
     odt = out_dtype if out_dtype is not None else (out.dtype if out is not None else x.dtype)
@@ -111,7 +112,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
                  dtype_code(odt), ACT[act], alpha, _ptr(ws), ws.numel(), _ptr(status), force_splits, force_bn,
                  1 if use_pdl else 0, len(peers) if peers else 1, rank,
                  (ctypes.c_void_p * 8)(*(list(peers) + [None] * (8 - len(peers)))) if peers else (ctypes.c_void_p * 8)(),
-                 symm_bytes, 4 if q4 else (3 if fp8 else 0), rms_eps, force_tile_rows, mc_ptr or None, None)
+                 symm_bytes, 4 if q4 else (3 if fp8 else 0), rms_eps, force_tile_rows, mc_ptr or None, None, *gate)
     rc = lib().ortb200_gemm(ctypes.byref(a), ctypes.c_void_p(stream_ptr()))
     if rc != 0:
         raise RuntimeError(f"ortb200_gemm rejected its arguments (code {rc})")
@@ -246,7 +247,7 @@ class GqaDecodeArgs(ctypes.Structure):
                 ("block_size", ctypes.c_int), ("max_blocks", ctypes.c_int), ("qkv", ctypes.c_void_p), ("cos_cache", ctypes.c_void_p),
                 ("sin_cache", ctypes.c_void_p), ("do_rotary", ctypes.c_int), ("rotary_interleaved", ctypes.c_int),
                 ("num_blocks", ctypes.c_int), ("algo", ctypes.c_int), ("prefetch", ctypes.c_void_p), ("prefetch_bytes", ctypes.c_int64),
-                ("cos_rows", ctypes.c_int)]
+                ("cos_rows", ctypes.c_int), ("chunk", ctypes.c_int), ("q_ld", ctypes.c_int64), ("out_ld", ctypes.c_int64)]
 
 
 _ATTN_WS = {}
@@ -297,7 +298,7 @@ class AttnPrefillArgs(ctypes.Structure):
                 ("softcap", ctypes.c_float), ("dtype", ctypes.c_int), ("status", ctypes.c_void_p), ("key_mask", ctypes.c_void_p),
                 ("block_table", ctypes.c_void_p), ("cu_seqlens", ctypes.c_void_p), ("past_seqlens", ctypes.c_void_p),
                 ("T", ctypes.c_int), ("block_size", ctypes.c_int), ("max_blocks", ctypes.c_int), ("num_blocks", ctypes.c_int),
-                ("split_weights", ctypes.c_int)]
+                ("split_weights", ctypes.c_int), ("chunk", ctypes.c_int)]
 
 
 def attn_prefill(q, k, v, seqlens_k=None, first_prompt=True, causal=True, window=-1, scale=0.0, softcap=0.0,
@@ -495,7 +496,7 @@ class QkNormRopeArgs(ctypes.Structure):
     _fields_ = [(n, _P) for n in ("packed", "q_out", "k_cache", "v_cache", "q_norm", "k_norm", "cos_table", "sin_table", "cu_seqlens",
                                   "past_seqlens", "block_table")] + \
                [(n, _I) for n in ("T", "B", "ld", "N", "Nk", "dk", "dv", "dk_pad", "dv_pad", "rot_dim", "table_rows", "block_size", "max_blocks",
-                                  "num_blocks", "kv_shared")] + [("eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P)]
+                                  "num_blocks", "kv_shared")] + [("eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P), ("first_values", _P), ("first_ld", _L), ("v_mix", _P)]
 
 
 def _call(name, args):
@@ -560,5 +561,5 @@ def head_gate(x, gate, gate_ld, dv):
     T, heads, x_pad = x.shape
     out = torch.empty(T, heads * dv, dtype=x.dtype, device=x.device)
     _check(lib().ortb200_head_gate(ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(gate.data_ptr()), ctypes.c_void_p(out.data_ptr()), T, heads, dv, x_pad,
-                                   ctypes.c_int64(gate_ld), dtype_code(x.dtype), 0, ctypes.c_void_p(stream_ptr())), "ortb200_head_gate")
+                                   ctypes.c_int64(gate_ld), ctypes.c_int64(heads * dv), dtype_code(x.dtype), 0, ctypes.c_void_p(stream_ptr())), "ortb200_head_gate")
     return out
