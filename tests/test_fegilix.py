@@ -8,68 +8,26 @@ import pytest
 import torch
 
 import fegilix_oracle as oracle
+import packed_decoder
 import onnxruntime_b200 as ort
 from onnxruntime_b200 import onnx_lite as ol
+from packed_decoder import CPU, GPU, KINDS, ONNX, PROVIDERS, close, decoder, feed, i32, logits_close, run_op, tokens_of
 from onnxruntime_b200.models.decoder_cache import CacheFull, CachePool, CacheTensor
 from onnxruntime_b200.models.fegilix import FegilixConfig, random_weights, rotary_tables
 from onnxruntime_b200.models.generation import GenerationConfig, generate, generate_requests
 from onnxruntime_b200.models.registry import create_decoder, load_decoder
 from onnxruntime_b200.safetensors_lite import load_file, save_file
 
-CPU, GPU = "CPUExecutionProvider", "CUDAExecutionProvider"
-PROVIDERS = [pytest.param(CPU, id="cpu"), pytest.param(GPU, marks=pytest.mark.gpu, id="gpu")]
-# (provider, type of activations)
-KINDS = [pytest.param((CPU, torch.float32), id="cpu-fp32"), pytest.param((GPU, torch.float32), marks=pytest.mark.gpu, id="gpu-fp32"),
-         pytest.param((GPU, torch.bfloat16), marks=pytest.mark.gpu, id="gpu-bf16")]
-T = ol.TensorProto
-ONNX = {torch.float32: T.FLOAT, torch.bfloat16: T.BFLOAT16, torch.int32: T.INT32, torch.int64: T.INT64}
+
+def Reference(*args):
+    return packed_decoder.Reference(oracle, *args)
+
+
+def greedy_reference(*args):
+    return packed_decoder.greedy_reference(oracle, *args)
 
 
 # ---------------------------------------------------------------------------------------------------- one operator alone
-def run_op(provider, op, inputs, outputs, domain="com.ortb200", **attrs):
-    """One node over torch inputs (None = absent).  ``outputs``: tensors that receive the results; an output that is one of the
-    inputs is updated in place.  Returns the outputs on the CPU."""
-    dev = "cuda" if provider == GPU else "cpu"
-    moved = {}
-    def put(t):
-        if id(t) not in moved:
-            moved[id(t)] = t.to(dev)
-        return moved[id(t)]
-    names = [f"i{k}" if t is not None else "" for k, t in enumerate(inputs)]
-    while names and not names[-1]:
-        names.pop()
-    info = [ol.make_tensor_value_info(f"i{k}", ONNX[t.dtype], list(t.shape)) for k, t in enumerate(inputs) if t is not None]
-    outs = [ol.make_tensor_value_info(f"o{k}", ONNX[t.dtype], list(t.shape)) for k, t in enumerate(outputs)]
-    graph = ol.make_graph([ol.make_node(op, names, [f"o{k}" for k in range(len(outputs))], name="n", domain=domain, **attrs)], "g", info, outs, [])
-    sess = ort.InferenceSession(ol.make_model(graph, opset=17, extra_opsets={"com.ortb200": 1}).serialize(), providers=[provider],
-                                **({"enable_fallback": False} if provider == GPU else {}))
-    binding = sess.io_binding()
-    for k, t in enumerate(inputs):
-        if t is not None:
-            binding.bind_torch_input(f"i{k}", put(t))
-    results = [put(t) for t in outputs]
-    for k, t in enumerate(results):
-        binding.bind_torch_output(f"o{k}", t)
-    sess.run_with_iobinding(binding)
-    if provider == GPU:
-        sess.check_device_status()
-    for t in outputs:                       # in-place operands keep their identity for the next call of a test
-        t.copy_(put(t).cpu())
-    return list(outputs)
-
-
-def close(got, want, dtype, tol=None):
-    got, want = got.double(), want.double()
-    tol = tol or (2e-5 if dtype == torch.float32 else 2e-2)
-    scale = want.abs().max().clamp_min(1e-3)
-    assert torch.isfinite(got).all()
-    assert (got - want).abs().max() <= tol * scale, float((got - want).abs().max() / scale)
-
-
-def i32(*v):
-    return torch.tensor(v, dtype=torch.int32)
-
-
 @pytest.mark.parametrize("kind", KINDS)
 @pytest.mark.parametrize("streams,width", [(1, 40), (2, 64), (3, 30), (5, 136), (8, 16)])
 def test_hyper_connections(kind, streams, width):
@@ -430,63 +388,6 @@ def model_pair(name, seed=0):
     return cfg, random_weights(FegilixConfig.from_json(cfg), seed=seed, low_rank=6, gain=1.5)
 
 
-def tokens_of(cfg, n, seed):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def decoder(cfg, w, kind, **kw):
-    provider, dt = kind
-    kw.setdefault("batch", 4)
-    kw.setdefault("max_len", 96)
-    kw.setdefault("block_size", 16 if provider == CPU else 128)
-    return create_decoder(cfg, w, "bfloat16" if dt == torch.bfloat16 else "float32", provider=provider, **kw)
-
-
-class Reference:
-    """Logits of a token sequence, and what 16-bit projections alone would change at every place (its conditioning)."""
-
-    def __init__(self, cfg, w, tokens, logits=None, noise=None):
-        self.args, self.logits, self._noise = (cfg, w, tokens), oracle.forward(cfg, w, tokens) if logits is None else logits, noise
-
-    @property
-    def noise(self):
-        if self._noise is None:
-            self._noise = oracle.rounding_noise(*self.args)
-        return self._noise
-
-    def __getitem__(self, rows):
-        part = Reference(*self.args, logits=self.logits[rows])
-        part._noise, part.rows, part.whole = None, rows, self
-        return part
-
-
-def relative_error(diff, logits):
-    diff = diff - diff.mean(-1, keepdim=True)
-    return diff.pow(2).mean(-1).sqrt() / logits.pow(2).mean().sqrt()
-
-
-def logits_close(got, want, dtype):
-    got = got.double().cpu()
-    assert got.shape == want.logits.shape and torch.isfinite(got).all()
-    rel = relative_error(got - want.logits, want.logits)
-    if dtype == torch.float32:
-        assert rel.max() < 1e-4, float(rel.max())
-    else:
-        noise = want.whole.noise[want.rows] if hasattr(want, "whole") else want.noise
-        limit = 0.06 + 2.5 * relative_error(noise, want.logits)
-        assert (rel < limit).all(), float((rel / limit).max())
-
-
-def feed(runner, seq, tokens, cuts):
-    """The tokens of one sequence in portions; logits of every place."""
-    out, at = [], 0
-    for n in cuts:
-        out.append(runner.step([(seq, tokens[at:at + n], list(range(n)))]))
-        at += n
-    assert at == len(tokens)
-    return torch.cat(out)
-
-
 @pytest.mark.parametrize("kind", KINDS)
 @pytest.mark.parametrize("name", ["mixed", "attention", "recurrent", "plain", "odd"])
 def test_model_matches_the_restatement(kind, name):
@@ -606,13 +507,6 @@ def test_capacity_errors_leave_the_pool_usable():
     runner.release("b")
     assert runner.step([("c", toks[:1], [0])]).shape == (1, cfg["vocab"])
     assert runner.step([("c", toks[1:3], [])]).shape == (0, cfg["vocab"])
-
-
-def greedy_reference(cfg, w, prompt, n):
-    toks = list(prompt)
-    for _ in range(n):
-        toks.append(int(oracle.forward(cfg, w, toks)[-1].argmax()))
-    return toks[len(prompt):]
 
 
 @pytest.mark.parametrize("provider", PROVIDERS)
