@@ -108,11 +108,12 @@ def reference_arm(args):
     return 0
 
 
-def fegilix_workload(args):
-    from onnxruntime_b200.benchmarks import fegilix
+def decoder_workload(args):
+    import importlib
+    module = importlib.import_module("onnxruntime_b200.benchmarks." + args.workload)
     sampler = ClockSampler(0)
     sampler.start()
-    out = fegilix.run([int(s) for s in args.sizes.split(",")], batch=args.batch, prompt=args.prompt, steps=args.steps, warmup=args.warmup)
+    out = module.run([int(s) for s in args.sizes.split(",")], batch=args.batch, prompt=args.prompt, steps=args.steps, warmup=args.warmup)
     out["clocks"] = sampler.stop()
     print(json.dumps(out))
     return 0
@@ -126,10 +127,10 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "library"],
                     help="ours: this package; reference: the unmodified reference (when installed); library: the same model on cuBLAS / "
                          "FlashAttention / NCCL library kernels under PyTorch (the decomposition the reference executes)")
-    ap.add_argument("--workload", default="llama", choices=["llama", "fegilix"],
-                    help="llama: the headline workload; fegilix: prompt, decode and kernel numbers of the Fegilix decoder beside the paged Llama "
+    ap.add_argument("--workload", default="llama", choices=["llama", "fegilix", "rovurax"],
+                    help="llama: the headline workload; fegilix, rovurax: prompt, decode and kernel numbers of that decoder beside the paged Llama "
                          "decoder of equal size (one GPU)")
-    ap.add_argument("--sizes", default="2048,4096", help="fegilix workload: model widths")
+    ap.add_argument("--sizes", default="2048,4096", help="fegilix and rovurax workloads: model widths")
     ap.add_argument("--repeats", type=int, default=5, help="the timed K-step loop is run this many times; value = median")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--prompt", type=int, default=1024)
@@ -148,8 +149,8 @@ def main():
     nvls_active = False
     if args.impl == "reference":
         return reference_arm(args)
-    if args.workload == "fegilix":
-        return fegilix_workload(args)
+    if args.workload != "llama":
+        return decoder_workload(args)
 
     import torch
     import torch.distributed as dist

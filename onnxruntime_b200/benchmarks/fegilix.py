@@ -10,26 +10,12 @@ launches over rotating buffers larger than the L2.
 """
 from __future__ import annotations
 
-import json
-import os
-from typing import Callable, Dict, List
+from typing import Dict, List
 
 import torch
 
-from ..models.registry import create_decoder
 from ..ops import _kernels as K
-
-FP32_CORE_TFLOPS = 148 * 128 * 2 * 1.965e-3   # nominal: SMs x lanes x 2 x GHz
-
-
-def _peaks() -> Dict[str, float]:
-    path = os.path.join(os.path.dirname(os.path.abspath(__file__)), "..", "..", "MEASURED_PEAKS.json")
-    try:
-        with open(path) as f:
-            d = json.load(f)
-        return {"hbm_gbs": d["hbm_gbs"], "bf16_tflops": d["bf16_tflops"], "source": "measured"}
-    except OSError:
-        return {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+from .packed import KernelRows, graph_us, run_pair
 
 
 def configs(width: int, layers: int = 8, vocab: int = 32000):
@@ -47,67 +33,13 @@ def configs(width: int, layers: int = 8, vocab: int = 32000):
     return fegilix, llama
 
 
-def _event_ms(fn: Callable[[], None]) -> float:
-    torch.cuda.synchronize()
-    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    a.record()
-    fn()
-    b.record()
-    torch.cuda.synchronize()
-    return a.elapsed_time(b)
-
-
-def model_numbers(config, batch: int, prompt: int, steps: int, warmup: int) -> Dict[str, float]:
-    runner = create_decoder(config, None, "bfloat16", batch=batch, max_len=prompt + steps + warmup + 8)
-    ids = torch.randint(0, runner.cfg.vocab_size, (batch, prompt), generator=torch.Generator().manual_seed(1))
-    for _ in range(3):
-        runner.prefill(ids)
-    prefill = sorted(_event_ms(lambda: runner.prefill(ids)) for _ in range(5))[2]
-    for _ in range(warmup):
-        runner.decode_step(None)
-    launches = runner.sess.last_run_launch_count()
-
-    def loop():
-        for _ in range(steps):
-            runner.decode_step(None)
-    start = runner.cur_len
-    times = []
-    for _ in range(3):
-        runner.cur_len = start
-        times.append(_event_ms(loop) / steps)
-    runner.sess.check_device_status()
-    decode = sorted(times)[1]
-    return {"prefill_ms": round(prefill, 3), "prefill_tokens_per_s": round(batch * prompt / prefill * 1e3, 1), "decode_ms": round(decode, 4),
-            "decode_tokens_per_s": round(batch / decode * 1e3, 1), "decode_launches": launches}
-
-
-def _graph_us(calls: List[Callable[[], object]], rounds: int = 4) -> float:
-    """Microseconds per call of ``calls`` (the same kernel over different buffers) replayed as one CUDA graph."""
-    for c in calls[:3]:
-        c()
-    torch.cuda.synchronize()
-    keep, graph = [], torch.cuda.CUDAGraph()
-    with torch.cuda.graph(graph):
-        for c in calls:
-            keep.append(c())
-    for _ in range(3):
-        graph.replay()
-    t = sorted(_event_ms(graph.replay) for _ in range(rounds))[rounds // 2]
-    return t * 1e3 / len(calls)
-
-
 def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: int = 4) -> List[Dict]:
     dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
-    peaks, rows = _peaks(), []
     heads, kv, H = width // 128, width // 512, 128
     torch.manual_seed(0)
 
-    def row(name, design, us, bytes_=0, tflop=0.0, core_tflop=0.0):
-        r = {"kernel": name, "design": design, "us": round(us, 2)}
-        best = max((bytes_ / peaks["hbm_gbs"] * 1e-3, "hbm"), (tflop / peaks["bf16_tflops"] * 1e6, "bf16 tensor"),
-                   (core_tflop / FP32_CORE_TFLOPS * 1e6, "fp32 cores (nominal)"))
-        r.update(roofline_us=round(best[0], 2), of=best[1], fraction=round(best[0] / us, 3))
-        rows.append(r)
+    rows = KernelRows()
+    row = rows.add
 
     for phase, T in (("decode", batch), ("prefill", batch * prompt)):
         n_buf = max(2, min(64, int(400e6 / (T * width * 4)))) if phase == "prefill" else 64
@@ -120,12 +52,12 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: i
         xs = [torch.randn(T, streams, width, dtype=f32, device=dev) for _ in range(n_buf)]
         mix, wo, wi, gam = torch.eye(streams, device=dev), torch.ones(streams, device=dev), torch.full((streams,), 1 / streams, device=dev), \
             torch.ones(width, device=dev)
-        us = _graph_us([lambda x=x, y=y: K.hyper_norm(x, y, mix, wo, wi, gam, 1e-6) for x, y in zip(xs, ys)])
+        us = graph_us([lambda x=x, y=y: K.hyper_norm(x, y, mix, wo, wi, gam, 1e-6) for x, y in zip(xs, ys)])
         row(f"hyper_norm {phase}", "fegilix", us, T * width * (8 * streams + 4))
         del xs
         g16 = torch.ones(width, dtype=bf, device=dev)
         rs = [torch.randn(T, width, dtype=bf, device=dev) for _ in range(n_buf)]
-        us = _graph_us([lambda x=x, y=y: K.norm(x, g16, skip=y, simplified=True, want_sum=True) for x, y in zip(rs, ys)])
+        us = graph_us([lambda x=x, y=y: K.norm(x, g16, skip=y, simplified=True, want_sum=True) for x, y in zip(rs, ys)])
         row(f"skip rms norm {phase}", "llama", us, T * width * 8)
         del rs, ys
         # ---- step 1 of attention
@@ -137,27 +69,27 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: i
         cos16, sin16 = cos32.to(bf), sin32.to(bf)
         qn = torch.ones(H, device=dev)
         pk = [torch.randn(T, (2 * heads + 2 * kv) * H, dtype=bf, device=dev) for _ in range(n_buf)]
-        us = _graph_us([lambda x=x: K.qk_norm_rope(x, kc, vc, qn, qn, cos32, sin32, cu, past0, table, heads, H, H) for x in pk])
+        us = graph_us([lambda x=x: K.qk_norm_rope(x, kc, vc, qn, qn, cos32, sin32, cu, past0, table, heads, H, H) for x in pk])
         row(f"qk_norm_rope {phase}", "fegilix", us, T * (heads + 2 * kv) * H * 4)
         qk = [p[:, :(heads + 2 * kv) * H].contiguous() for p in pk]
-        us = _graph_us([lambda x=x: K.paged_prep(x, kc, vc, cu, past0, table, heads, kv, cos16, sin16) for x in qk])
+        us = graph_us([lambda x=x: K.paged_prep(x, kc, vc, cu, past0, table, heads, kv, cos16, sin16) for x in qk])
         row(f"paged_prep {phase}", "llama", us, T * (heads + 2 * kv) * H * 4)
         q = torch.randn(T, heads, H, dtype=bf, device=dev)
         sink = torch.zeros(heads, dtype=bf, device=dev)
         if phase == "prefill":
             fl = 4 * B * heads * H * prompt * (prompt + 1) / 2 * 1e-12
             calls = lambda split: [lambda: K.attn_prefill_paged(q, kc, vc, cu, past0, table, head_sink=sink if split else None, split_weights=split)] * 8
-            row("attention prefill (split weights)", "fegilix", _graph_us(calls(True)), tflop=fl)
-            row("attention prefill", "llama", _graph_us(calls(False)), tflop=fl)
+            row("attention prefill (split weights)", "fegilix", graph_us(calls(True)), tflop=fl)
+            row("attention prefill", "llama", graph_us(calls(False)), tflop=fl)
         else:
             caches = [(torch.randn_like(kc), torch.randn_like(vc)) for _ in range(max(2, int(300e6 / (kc.numel() * 4))))]
             by = B * (context + 1) * kv * H * 4
-            us = _graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, head_sink=sink, block_table=table, algo=1) for c in caches] * 2)
+            us = graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, head_sink=sink, block_table=table, algo=1) for c in caches] * 2)
             row("attention decode (fp32 weights)", "fegilix", us, by)
-            us = _graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, block_table=table, algo=2) for c in caches] * 2)
+            us = graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, block_table=table, algo=2) for c in caches] * 2)
             row("attention decode", "llama", us, by)
             del caches
-        us = _graph_us([lambda x=x: K.head_gate(q, x[:, (heads + 2 * kv) * H:], x.shape[1], H) for x in pk])
+        us = graph_us([lambda x=x: K.head_gate(q, x[:, (heads + 2 * kv) * H:], x.shape[1], H) for x in pk])
         row(f"head_gate {phase}", "fegilix", us, T * heads * H * 6)
         del pk, qk, kc, vc
         # ---- recurrences
@@ -170,7 +102,7 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: i
         states = [torch.zeros(B, heads, dk, dv, device=dev) for _ in range(nst)]
         x = torch.randn(T, C + heads, dtype=bf, device=dev)
         low = torch.randn(T, heads * (dk + dv), dtype=bf, device=dev)
-        us = _graph_us([lambda s=s: K.gated_delta(x, low, conv, a_log, dtb, nrm, ring, s, cu, past0, slots, G) for s in states])
+        us = graph_us([lambda s=s: K.gated_delta(x, low, conv, a_log, dtb, nrm, ring, s, cu, past0, slots, G) for s in states])
         io = T * (C + heads + heads * (dk + dv) + heads * dv) * 2
         row(f"gated delta {phase}", "fegilix", us, 2 * B * heads * dk * dv * 4 + io, core_tflop=T * heads * dk * dv * 7e-12)
         hm, dvm = heads // 2, 256
@@ -178,27 +110,13 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: i
         aux = torch.zeros(B, hm, dk + 1, device=dev)
         xm = torch.randn(T, hm * (2 * dk + 2 * dvm + 2), dtype=bf, device=dev)
         zb, nm = torch.zeros(hm, device=dev), torch.ones(hm * dvm, device=dev)
-        us = _graph_us([lambda s=s: K.mlstm(xm, zb, zb, nm, s, aux, cu, past0, slots, 15.0) for s in states])
+        us = graph_us([lambda s=s: K.mlstm(xm, zb, zb, nm, s, aux, cu, past0, slots, 15.0) for s in states])
         io = T * hm * (2 * dk + 3 * dvm) * 2
         row(f"mlstm {phase}", "fegilix", us, 2 * B * hm * dk * dvm * 4 + io, core_tflop=T * hm * dk * dvm * 5e-12)
         del states, x, low, xm
         torch.cuda.empty_cache()
-    return rows
+    return rows.rows
 
 
-def run(sizes, batch: int = 8, prompt: int = 1024, steps: int = 64, warmup: int = 4, kernels: bool = True, sampler=None) -> Dict:
-    out = {"metric": "fegilix_prefill_decode_tokens_per_s", "unit": "tokens/s", "dtype": "bf16", "n_gpus": 1, "data": "synthetic, random weights",
-           "config": {"layers": 8, "global_batch": batch, "seq_len": prompt, "decode_tokens": steps, "peaks": _peaks(),
-                      "l2": "weights larger than L2; kernels over rotating buffers"}, "sizes": {}}
-    for width in sizes:
-        fg, ll = configs(width)
-        entry = {}
-        for name, c in (("fegilix", fg), ("llama", ll)):
-            entry[name] = model_numbers(c, batch, prompt, steps, max(warmup, 3))
-            torch.cuda.empty_cache()
-        if kernels:
-            entry["kernels"] = kernel_numbers(width, batch, prompt, prompt)
-        out["sizes"][str(width)] = entry
-    first = out["sizes"][str(sizes[-1])]["fegilix"]
-    out.update(value=first["decode_tokens_per_s"], ms_per_step=first["decode_ms"], steps=steps, warmup=max(warmup, 3), higher_is_better=True)
-    return out
+def run(sizes, batch: int = 8, prompt: int = 1024, steps: int = 64, warmup: int = 4) -> Dict:
+    return run_pair("fegilix", configs, kernel_numbers, sizes, batch, prompt, steps, warmup)

@@ -254,7 +254,7 @@ _ATTN_WS = {}
 
 
 def gqa_decode(q, k_cache, v_cache, seqlens_k, splits=0, window=-1, scale=0.0, softcap=0.0, head_sink=None, block_table=None,
-               qkv=None, num_heads=0, cos=None, sin=None, interleaved=False, algo=0, prefetch=None):
+               qkv=None, num_heads=0, cos=None, sin=None, interleaved=False, algo=0, prefetch=None, chunk=0):
     """Dense cache [B,Nk,Smax,H]; or, with block_table [B,max_blocks] int32, a paged cache [num_blocks,block_size,Nk,H].
     With ``qkv`` (packed [B,(N+2Nk)H], ``num_heads`` = N) the kernel also rotates q / k and appends k / v itself.
     ``algo``: 0 = pick, 1 = CUDA-core split-KV kernel, 2 = tcgen05 kernel (head size 128, 16-bit types)."""
@@ -284,7 +284,7 @@ def gqa_decode(q, k_cache, v_cache, seqlens_k, splits=0, window=-1, scale=0.0, s
                       _ptr(block_table), block_size, max_blocks, _ptr(qkv), _ptr(cos), _ptr(sin), 0 if cos is None else 1,
                       1 if interleaved else 0, num_blocks, algo, _ptr(prefetch),
                       prefetch.numel() * prefetch.element_size() if prefetch is not None else 0,
-                      0 if cos is None else cos.shape[0])
+                      0 if cos is None else cos.shape[0], chunk, 0, 0)
     _check(lib().ortb200_gqa_decode(ctypes.byref(a), ctypes.c_void_p(stream_ptr())), "ortb200_gqa_decode")
     return out
 
@@ -322,7 +322,7 @@ def attn_prefill(q, k, v, seqlens_k=None, first_prompt=True, causal=True, window
 
 
 def attn_prefill_paged(q, k_cache, v_cache, cu_seqlens, past_seqlens, block_table, scale=0.0, head_sink=None, split_weights=False, status=None,
-                       window=-1):
+                       window=-1, chunk=0):
     """Packed queries q [T,N,H] of several sequences over a paged cache [num_blocks,block_size,Nk,H].  Returns [T,N,H]."""
     T, N, H = q.shape
     nb, bs, Nk, _ = k_cache.shape
@@ -330,7 +330,7 @@ def attn_prefill_paged(q, k_cache, v_cache, cu_seqlens, past_seqlens, block_tabl
     st = (ctypes.c_int64 * 3)(0, N * H, H)
     a = AttnPrefillArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), None, _ptr(head_sink), _ptr(out), past_seqlens.numel(), 0, N, Nk, H, 0, st, st,
                         (ctypes.c_int64 * 3)(0, 0, 0), 0, 1, window, scale, 0.0, dtype_code(q.dtype), _ptr(status), None, _ptr(block_table),
-                        _ptr(cu_seqlens), _ptr(past_seqlens), T, bs, block_table.shape[1], nb, 1 if split_weights else 0)
+                        _ptr(cu_seqlens), _ptr(past_seqlens), T, bs, block_table.shape[1], nb, 1 if split_weights else 0, chunk)
     _check(lib().ortb200_attn_prefill(ctypes.byref(a), ctypes.c_void_p(stream_ptr())), "ortb200_attn_prefill(paged)")
     return out
 
@@ -544,15 +544,18 @@ def hyper_norm(x, y, mix, w_out, w_in, gamma, eps, keep=True):
     return out, xo
 
 
-def qk_norm_rope(packed, k_cache, v_cache, q_norm, k_norm, cos, sin, cu, past, table, N, dk, dv, eps=1e-6):
-    """Packed q | k | v rows; caches [num_blocks, block_size, Nk, padded head] updated in place.  Returns q [T, N, padded head]."""
+def qk_norm_rope(packed, k_cache, v_cache, q_norm, k_norm, cos, sin, cu, past, table, N, dk, dv, eps=1e-6, keep_q=False, first_values=None,
+                 v_mix=None):
+    """Packed q | k | v rows; caches [num_blocks, block_size, Nk, padded head] updated in place.  Returns q [T, N, padded head], None
+    with ``keep_q`` (queries stay where they are).  ``first_values`` [T, >= Nk * dv] are mixed into the stored values by ``v_mix``."""
     T = packed.shape[0]
     nb, bs, Nk, dkp = k_cache.shape
-    q = torch.empty(T, N, dkp, dtype=packed.dtype, device=packed.device)
+    q = None if keep_q else torch.empty(T, N, dkp, dtype=packed.dtype, device=packed.device)
+    rot, rows = (0, 1 << 30) if cos is None else (cos.shape[1] * 2, cos.shape[0])
     _call("ortb200_qk_norm_rope", QkNormRopeArgs(_ptr(packed), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin),
                                                  _ptr(cu), _ptr(past), _ptr(table), T, past.numel(), packed.shape[1], N, Nk, dk, dv, dkp,
-                                                 v_cache.shape[3], cos.shape[1] * 2, cos.shape[0], bs, table.shape[1], nb, 0, eps,
-                                                 dtype_code(packed.dtype), 0, None))
+                                                 v_cache.shape[3], rot, rows, bs, table.shape[1], nb, 0, eps, dtype_code(packed.dtype), 0, None,
+                                                 _ptr(first_values), first_values.stride(0) if first_values is not None else 0, _ptr(v_mix)))
     return q
 
 
@@ -562,4 +565,110 @@ def head_gate(x, gate, gate_ld, dv):
     out = torch.empty(T, heads * dv, dtype=x.dtype, device=x.device)
     _check(lib().ortb200_head_gate(ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(gate.data_ptr()), ctypes.c_void_p(out.data_ptr()), T, heads, dv, x_pad,
                                    ctypes.c_int64(gate_ld), ctypes.c_int64(heads * dv), dtype_code(x.dtype), 0, ctypes.c_void_p(stream_ptr())), "ortb200_head_gate")
+    return out
+
+
+def swiglu(x):
+    """silu(gate) * up of x [rows, gate | up]."""
+    rows, cols = x.shape[0], x.shape[1] // 2
+    y = torch.empty(rows, cols, dtype=x.dtype, device=x.device)
+    _check(lib().ortb200_swiglu(_P(x.data_ptr()), _P(y.data_ptr()), _L(rows), cols, dtype_code(x.dtype), _P(stream_ptr())), "ortb200_swiglu")
+    return y
+
+
+def gated_unit(gate, up, act, limit=float("inf"), alpha=1.0, offset=0.0, out=None):
+    """Gated unit of two [rows, cols] inputs with one row stride; ``out`` may be columns of a wider tensor."""
+    rows, cols = gate.shape
+    assert gate.stride(0) == up.stride(0)
+    out = torch.empty(rows, cols, dtype=gate.dtype, device=gate.device) if out is None else out
+    _check(lib().ortb200_gated_unit(_P(gate.data_ptr()), _P(up.data_ptr()), _P(out.data_ptr()), _L(rows), cols, _L(gate.stride(0)), _L(out.stride(0)),
+                                    ACT[act], _F(limit), _F(alpha), _F(offset), dtype_code(gate.dtype), 0, _P(stream_ptr())), "ortb200_gated_unit")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------------- latent attention
+class LatentPrepArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("packed", "cache", "norm", "cos_table", "sin_table", "cu_seqlens", "past_seqlens", "block_table")] + \
+               [(n, _I) for n in ("T", "B", "ld", "N", "dk", "dr", "rank", "wide", "width", "rot_dim", "table_rows", "block_size", "max_blocks",
+                                  "num_blocks")] + [("eps", _F), ("dtype", _I), ("use_pdl", _I), ("status", _P), ("up", _P), ("q_abs", _P),
+                                                    ("q_abs_f32", _I), ("q_rot", _P), ("c_out", _P), ("k_rot_out", _P)]
+
+
+class LatentDecodeArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("q_abs", "cache", "cu_seqlens", "past_seqlens", "block_table", "o", "ml")] + \
+               [(n, _I) for n in ("T", "B", "N", "rank", "wide", "width", "parts", "block_size", "max_blocks", "num_blocks")] + \
+               [("scale", _F), ("dtype", _I), ("tensor_cores", _I), ("use_pdl", _I), ("status", _P)]
+
+
+class LatentOutArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("o", "ml", "sink", "up_v", "gate", "out")] + [("gate_ld", _L), ("out_ld", _L)] + \
+               [(n, _I) for n in ("T", "N", "dv", "rank", "wide", "parts", "dtype", "use_pdl")]
+
+
+class LatentPrefillArgs(ctypes.Structure):
+    _fields_ = [(n, _P) for n in ("q", "q_rot", "kv", "k_rot", "head_sink", "gate", "out", "cu_seqlens", "past_seqlens")] + \
+               [(n, _L) for n in ("q_ld", "kv_ld", "k_rot_ld", "gate_ld", "out_ld")] + \
+               [(n, _I) for n in ("T", "B", "N", "dk", "dr", "dv", "key_rows")] + [("scale", _F), ("dtype", _I), ("status", _P)]
+
+
+def _latent_prep(packed, cache, norm, cos, sin, cu, past, table, N, dk, dr, rank, wide, eps):
+    nb, bs, width = cache.shape
+    rot, rows = (0, 0) if cos is None else (cos.shape[1] * 2, cos.shape[0])
+    return LatentPrepArgs(_ptr(packed), _ptr(cache), _ptr(norm), _ptr(cos), _ptr(sin), _ptr(cu), _ptr(past), _ptr(table), packed.shape[0],
+                          past.numel(), packed.shape[1], N, dk, dr, rank, wide, width, rot, rows, bs, table.shape[1], nb, eps,
+                          dtype_code(packed.dtype), 0, None)
+
+
+def latent_prep(packed, cache, norm, cos, sin, cu, past, table, N, dk, dr, rank, eps=1e-6):
+    """Rotates the queries and appends the new entries (cache [num_blocks, block_size, width], latents not padded).  Returns
+    (q_rot [T, N, dr], c [T, rank], k_rot [T, width - rank])."""
+    T, dt, dev = packed.shape[0], packed.dtype, packed.device
+    q_rot, c, kr = [torch.empty(*s, dtype=dt, device=dev) for s in ((T, N, dr), (T, rank), (T, cache.shape[2] - rank))]
+    a = _latent_prep(packed, cache, norm, cos, sin, cu, past, table, N, dk, dr, rank, rank, eps)
+    a.q_rot, a.c_out, a.k_rot_out = _ptr(q_rot), _ptr(c), _ptr(kr)
+    _call("ortb200_latent_prep", a)
+    return q_rot, c, kr
+
+
+def latent_absorb(packed, cache, norm, cos, sin, cu, past, table, up, N, dk, dr, rank, eps=1e-6):
+    """Appends the new entries and returns the absorbed queries [T, N, width] in the type of the cache (latents not padded)."""
+    q = torch.empty(packed.shape[0], N, cache.shape[2], dtype=packed.dtype, device=packed.device)
+    a = _latent_prep(packed, cache, norm, cos, sin, cu, past, table, N, dk, dr, rank, rank, eps)
+    a.up, a.q_abs = _ptr(up), _ptr(q)
+    _call("ortb200_latent_absorb", a)
+    return q
+
+
+def latent_decode(q_abs, cache, cu, past, table, rank, scale, status=None):
+    """Tensor-core attention of absorbed queries over the cache.  Returns (o [T, N, parts, rank], ml [T, N, parts, 2])."""
+    T, N, width = q_abs.shape
+    nb, bs, _ = cache.shape
+    parts = ctypes.c_int(1)
+    if not lib().ortb200_latent_decode_plan(T, N, rank, width, bs, table.shape[1], dtype_code(cache.dtype), ctypes.byref(parts)):
+        raise ValueError("the tensor-core kernel does not take these sizes")
+    o = torch.empty(T, N, parts.value, rank, dtype=torch.float32, device=cache.device)
+    ml = torch.empty(T, N, parts.value, 2, dtype=torch.float32, device=cache.device)
+    _call("ortb200_latent_decode", LatentDecodeArgs(_ptr(q_abs), _ptr(cache), _ptr(cu), _ptr(past), _ptr(table), _ptr(o), _ptr(ml), T, past.numel(), N,
+                                                    rank, rank, width, parts.value, bs, table.shape[1], nb, scale, dtype_code(cache.dtype), 1, 0,
+                                                    _ptr(status)))
+    return o, ml
+
+
+def latent_out(o, ml, sink, up_v, gate, gate_ld, dv):
+    """Merged, divided, mapped to values and gated: [T, N * dv] of the type of ``up_v``."""
+    T, N, parts, rank = o.shape
+    out = torch.empty(T, N * dv, dtype=up_v.dtype, device=o.device)
+    _call("ortb200_latent_out", LatentOutArgs(_ptr(o), _ptr(ml), _ptr(sink), _ptr(up_v), _ptr(gate), _ptr(out), gate_ld, N * dv, T, N, dv, rank, rank,
+                                              parts, dtype_code(up_v.dtype), 0))
+    return out
+
+
+def latent_prefill(packed, q_rot, kv, k_rot, sink, gate, cu, past, N, dk, dr, dv, scale, status=None):
+    """Flash attention over expanded keys and values kv [key rows, N * (dk + dv)].  ``packed`` rows start with the query heads,
+    ``gate`` points at the first gate column of them.  Returns [T, N * dv]."""
+    T = packed.shape[0]
+    out = torch.empty(T, N * dv, dtype=packed.dtype, device=packed.device)
+    _call("ortb200_latent_prefill", LatentPrefillArgs(_ptr(packed), _ptr(q_rot), _ptr(kv), _ptr(k_rot), _ptr(sink), _ptr(gate), _ptr(out), _ptr(cu),
+                                                      _ptr(past), packed.shape[1], kv.shape[1], k_rot.shape[1], packed.shape[1], N * dv, T,
+                                                      past.numel(), N, dk, dr, dv, kv.shape[0], scale, dtype_code(packed.dtype), _ptr(status)))
     return out
