@@ -10,11 +10,7 @@
 //   the same threads fold O_tile into their fp32 register accumulator.
 // K/V tiles are double-buffered by a TMA producer warp; MMA 1 of the next tile is
 // issued as soon as P is published, so it overlaps the accumulator update.
-//
-// With split weights P is the sum of two 16-bit terms that lie in tensor memory, where MMA 2 takes them as its A operand:
-// no shared memory, so the latent form (query / key heads of an unrotated part and a rotated part that all heads share,
-// e.g. 128 + 64, values of 128) fits with both stages.  That form reads keys and values expanded from their latents, packed
-// sequence behind sequence; the tensor maps zero-fill heads that are narrower than a box.
+// (attn_split.cu holds the form whose softmax weights stay 32-bit up to the product with V.)
 //
 // Replaces, for prompt processing and encoder self-attention, the FlashAttention-2
 // (mma.sync) and CUTLASS FMHA kernels the reference dispatches to
@@ -24,6 +20,7 @@
 #include <cuda.h>
 #include <cuda_runtime.h>
 #include <math.h>
+#include "attn_internal.h"
 #include "ortb200_kernels.h"
 #include "ptx_sm100.cuh"
 #include "tensor_map.h"
@@ -34,46 +31,20 @@ constexpr int kQT = 128;   // query rows per CTA
 constexpr int kKT = 128;   // keys per tile
 constexpr int kAttnThreads = 192;
 
-struct AttnParams {
-  const int* seqlens_k;
-  const int* key_mask;
-  const void* head_sink;
-  void* out;
-  int B, S, N, Nk, kv_len;
-  long long o_strides[3];
-  int first_prompt, causal, window;
-  float scale_log2, softcap, scale;
-  int bf16;
-  int* status;
-  // packed queries over a paged cache (block_table given)
-  const int* block_table;
-  const int* cu_seqlens;
-  const int* past_seqlens;
-  int block_size, max_blocks, num_blocks;
-  int chunk;             // > 0: keys of the query's own chunk only
-  // latent form: keys of sequence b are the rows behind those of the sequences in front of it
-  int plain_boxes;       // leading boxes of a query / key tile that hold the unrotated part
-  int dv;                // value head size (columns of a head that are stored)
-  const void* gate;      // optional [T, gate_ld]: sigmoid factor per token and head
-  long long gate_ld;
-};
-
-// KB / VB: 64-element boxes of a query / key tile and of a value tile.  SPLIT: P is held as the sum of two 16-bit terms
-// (leading part and remainder) in tensor memory, both multiplied with V; else as one term in shared memory.
-template <int KB, int VB, bool SPLIT>
+template <int HD>
 struct AttnSmem {
   static constexpr int kBoxBytes = 128 * 128;          // [128 rows][64 elems] of 16-bit data
-  static constexpr int kQBytes = kBoxBytes * KB;
-  static constexpr int kKBytes = kBoxBytes * KB;
-  static constexpr int kStageBytes = kKBytes + kBoxBytes * VB;
+  static constexpr int kBoxes = HD / 64;                // boxes per Q / K / V tile
+  static constexpr int kQBytes = kBoxBytes * kBoxes;
+  static constexpr int kKVBytes = kBoxBytes * kBoxes;   // each of K and V
+  static constexpr int kPBytes = kBoxBytes * 2;         // P [128 q][128 keys]
+  static constexpr int kStageBytes = 2 * kKVBytes;
   static constexpr int kOffQ = 0;
   static constexpr int kOffKV = kQBytes;
   static constexpr int kOffP = kOffKV + 2 * kStageBytes;
-  static constexpr int kPBytes = SPLIT ? 0 : kBoxBytes * 2;   // P [128 q][128 keys]
   static constexpr int kOffBar = kOffP + kPBytes;
   static constexpr int kTotal = kOffBar + 128 + 1024;
-  // two score buffers (2 x 128 columns), O (up to 128), P as packed pairs (2 x 64)
-  static constexpr int kTmemCols = 512;
+  static constexpr int kTmemCols = 512;                // two score buffers (2 x 128 columns) + O (HD columns)
 };
 
 // Bit j of the result = key (key0 + j) of batch b may be attended to.  Called by all 32 lanes of a warp.
@@ -84,36 +55,22 @@ __device__ __forceinline__ unsigned key_keep_bits(const int* key_mask, int b, in
   return __ballot_sync(0xffffffffu, keep);
 }
 
-__device__ __forceinline__ float fmax3(float a, float b, float c) {
-  float r;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
-  return r;
-}
-__device__ __forceinline__ float ex2_approx(float x) {
-  float r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-
 // barrier indices
 enum { BAR_Q = 0, BAR_KV_FULL0, BAR_KV_FULL1, BAR_KV_EMPTY0, BAR_KV_EMPTY1, BAR_S_FULL0, BAR_S_FULL1, BAR_P_READY, BAR_O_FULL, BAR_COUNT };
 
-template <int KB, int VB, bool SPLIT, bool LATENT>
+template <int HD>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
-                    const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_qr,
-                    const __grid_constant__ CUtensorMap tm_kr, const AttnParams p) {
-  using L = AttnSmem<KB, VB, SPLIT>;
-  constexpr int HD = VB * 64;   // columns of O
+                    const __grid_constant__ CUtensorMap tm_v, const AttnParams p) {
+  using L = AttnSmem<HD>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::kOffBar);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + BAR_COUNT);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  int q0 = blockIdx.x * kQT, b = blockIdx.z, q_row0 = 0, S = p.S, k_row0 = 0;
-  const bool packed_queries = LATENT || p.block_table != nullptr;
-  if (packed_queries) {
+  int q0 = blockIdx.x * kQT, b = blockIdx.z, q_row0 = 0, S = p.S;
+  if (p.block_table != nullptr) {
     // query tiles of all sequences are numbered consecutively; the grid is an upper bound of their count
     pdl_wait_prior_grids();
     int tile = blockIdx.x;
@@ -123,7 +80,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       const int tiles = (S + kQT - 1) / kQT;
       if (tile < tiles) break;
       tile -= tiles;
-      if (LATENT) k_row0 += p.past_seqlens[b] + S;
     }
     if (b == p.B) return;
     q0 = tile * kQT;
@@ -135,10 +91,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     tma_prefetch_desc(&tm_q);
     tma_prefetch_desc(&tm_k);
     tma_prefetch_desc(&tm_v);
-    if (LATENT) {
-      tma_prefetch_desc(&tm_qr);
-      tma_prefetch_desc(&tm_kr);
-    }
     for (int i = 0; i < BAR_COUNT; ++i) mbar_init(&bars[i], i == BAR_P_READY ? 128 : 1);
     fence_mbar_init();
   }
@@ -152,12 +104,11 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   const uint32_t tmem_base = *tmem_slot;
   const uint32_t tmem_s = tmem_base;          // S: two buffers, columns [0, 128) and [128, 256)
   const uint32_t tmem_o = tmem_base + 256;    // O: columns [256, 256 + HD), accumulated over all key tiles
-  const uint32_t tmem_p = tmem_base + 384;    // SPLIT: leading terms of P (64 columns of pairs), then remainders
 
   pdl_wait_prior_grids();
-  const bool paged = !LATENT && p.block_table != nullptr;
-  const int total = packed_queries ? p.past_seqlens[b] + S : (p.seqlens_k ? p.seqlens_k[b] + 1 : p.kv_len);
-  const int past = packed_queries ? total - S : (p.first_prompt ? 0 : total - S);
+  const bool paged = p.block_table != nullptr;
+  const int total = paged ? p.past_seqlens[b] + S : (p.seqlens_k ? p.seqlens_k[b] + 1 : p.kv_len);
+  const int past = paged ? total - S : (p.first_prompt ? 0 : total - S);
   // key range needed by this query tile
   int kv_end = total;
   if (p.causal) kv_end = min(kv_end, past + q0 + kQT);
@@ -170,12 +121,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   if (warp == 0) {
     if (lane == 0 && n_tiles > 0) {
       mbar_expect_tx(&bars[BAR_Q], L::kQBytes);
-      for (int bx = 0; bx < KB; ++bx) {
-        if (LATENT && bx >= p.plain_boxes)
-          tma_load_4d(smem + L::kOffQ + bx * L::kBoxBytes, &tm_qr, &bars[BAR_Q], (bx - p.plain_boxes) * 64, q_row0 + q0, head, 0);
-        else
-          tma_load_4d(smem + L::kOffQ + bx * L::kBoxBytes, &tm_q, &bars[BAR_Q], bx * 64, q_row0 + q0, head, packed_queries ? 0 : b);
-      }
+      for (int bx = 0; bx < L::kBoxes; ++bx)
+        tma_load_4d(smem + L::kOffQ + bx * L::kBoxBytes, &tm_q, &bars[BAR_Q], bx * 64, q_row0 + q0, head, paged ? 0 : b);
       for (int t = 0; t < n_tiles; ++t) {
         const int s = t & 1;
         if (t >= 2) {
@@ -194,18 +141,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           c1 = key0 % p.block_size;
           c3 = min(max(p.block_table[static_cast<long long>(b) * p.max_blocks + bi], 0), p.num_blocks - 1);
         }
-        if (LATENT) {
-          c1 = k_row0 + key0;
-          c3 = 0;
+        for (int bx = 0; bx < L::kBoxes; ++bx) {
+          tma_load_4d(st + bx * L::kBoxBytes, &tm_k, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
+          tma_load_4d(st + L::kKVBytes + bx * L::kBoxBytes, &tm_v, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
         }
-        for (int bx = 0; bx < KB; ++bx) {
-          if (LATENT && bx >= p.plain_boxes)   // one rotated part for all heads
-            tma_load_4d(st + bx * L::kBoxBytes, &tm_kr, &bars[BAR_KV_FULL0 + s], (bx - p.plain_boxes) * 64, c1, 0, 0);
-          else
-            tma_load_4d(st + bx * L::kBoxBytes, &tm_k, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
-        }
-        for (int bx = 0; bx < VB; ++bx)
-          tma_load_4d(st + L::kKBytes + bx * L::kBoxBytes, &tm_v, &bars[BAR_KV_FULL0 + s], bx * 64, c1, kvh, c3);
       }
     }
   } else if (warp == 1) {
@@ -219,7 +158,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         const int s = t & 1;
         const uint32_t k_addr = smem_u32(smem + L::kOffKV + s * L::kStageBytes);
 #pragma unroll
-        for (int kk = 0; kk < KB * 4; ++kk) {
+        for (int kk = 0; kk < HD / 16; ++kk) {
           const uint32_t off = (kk / 4) * L::kBoxBytes + (kk % 4) * 32;
           umma_f16(tmem_s + s * kKT, umma_desc_sw128(q_addr + off), umma_desc_sw128(k_addr + off), idesc_s, kk > 0 ? 1u : 0u);
         }
@@ -242,17 +181,12 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         // P of tile t published (O rescaled if the row maxima moved)
         if (!mbar_wait(&bars[BAR_P_READY], t & 1)) { ok = false; break; }
         tcgen05_fence_after();
-        const uint32_t v_addr = smem_u32(smem + L::kOffKV + s * L::kStageBytes + L::kKBytes);
+        const uint32_t v_addr = smem_u32(smem + L::kOffKV + s * L::kStageBytes + L::kKVBytes);
 #pragma unroll
         for (int kk = 0; kk < kKT / 16; ++kk) {
+          const uint64_t pdesc = umma_desc_sw128(p_addr + (kk / 4) * L::kBoxBytes + (kk % 4) * 32);
           const uint64_t vdesc = umma_desc_mn_sw128(v_addr + kk * 2048, L::kBoxBytes, 1024);
-          if (SPLIT) {
-            umma_f16_ts(tmem_o, tmem_p + kk * 8, vdesc, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
-            umma_f16_ts(tmem_o, tmem_p + 64 + kk * 8, vdesc, idesc_o, 1u);
-          } else {
-            const uint64_t pdesc = umma_desc_sw128(p_addr + (kk / 4) * L::kBoxBytes + (kk % 4) * 32);
-            umma_f16(tmem_o, pdesc, vdesc, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
-          }
+          umma_f16(tmem_o, pdesc, vdesc, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
         }
         umma_commit(&bars[BAR_O_FULL]);
         umma_commit(&bars[BAR_KV_EMPTY0 + s]);
@@ -349,7 +283,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       float row_sum = 0.f, row_sum1 = 0.f;
 #pragma unroll
       for (int c = 0; c < kKT; c += 32) {
-        uint32_t packed[16], rest[SPLIT ? 16 : 1];
+        uint32_t packed[16];
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
           const float p0 = ex2_approx(fmaf(sv[c + j], fs, neg_m));
@@ -359,23 +293,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           if (p.bf16) {
             __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
             packed[j / 2] = *reinterpret_cast<uint32_t*>(&h);
-            if (SPLIT) {
-              __nv_bfloat162 e = __floats2bfloat162_rn(p0 - __bfloat162float(h.x), p1 - __bfloat162float(h.y));
-              rest[SPLIT ? j / 2 : 0] = *reinterpret_cast<uint32_t*>(&e);
-            }
           } else {
             __half2 h = __floats2half2_rn(p0, p1);
             packed[j / 2] = *reinterpret_cast<uint32_t*>(&h);
-            if (SPLIT) {
-              __half2 e = __floats2half2_rn(p0 - __half2float(h.x), p1 - __half2float(h.y));
-              rest[SPLIT ? j / 2 : 0] = *reinterpret_cast<uint32_t*>(&e);
-            }
           }
-        }
-        if (SPLIT) {
-          tmem_st_x16_u32(tmem_p + lane_addr + c / 2, packed);
-          tmem_st_x16_u32(tmem_p + 64 + lane_addr + c / 2, rest);
-          continue;
         }
         // 32 keys = 4 chunks of 16 bytes; column c lives in box c / 64
         const int box = c / 64;
@@ -387,9 +308,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         }
       }
       l += row_sum + row_sum1;
-      // make the writes of P visible to the tensor core, then publish
-      if (SPLIT) tmem_st_wait();
-      else fence_proxy_async();
+      // make the generic-proxy writes of P visible to the tensor core, then publish
+      fence_proxy_async();
       tcgen05_fence_before();
       mbar_arrive(&bars[BAR_P_READY]);
     }
@@ -406,13 +326,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       rescale = m == -INFINITY ? 0.f : exp2f(m - mm);
       denom = l * rescale + exp2f(sink - mm);
     }
-    float inv = (denom > 0.f && n_tiles > 0) ? rescale / denom : 0.f;
-    if (LATENT && p.gate != nullptr && s_idx < S) {
-      const long long gi = (q_row0 + s_idx) * p.gate_ld + head;
-      const float g = p.bf16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]) : __half2float(static_cast<const __half*>(p.gate)[gi]);
-      inv *= 1.f / (1.f + __expf(-g));
-    }
-    uint8_t* orow = static_cast<uint8_t*>(p.out) + 2 * ((packed_queries ? 0 : b * p.o_strides[0]) + (q_row0 + s_idx) * p.o_strides[1] + head * p.o_strides[2]);
+    const float inv = (denom > 0.f && n_tiles > 0) ? rescale / denom : 0.f;
+    uint8_t* orow = static_cast<uint8_t*>(p.out) + 2 * ((paged ? 0 : b * p.o_strides[0]) + (q_row0 + s_idx) * p.o_strides[1] + head * p.o_strides[2]);
 #pragma unroll 1
     for (int c0 = 0; c0 < HD; c0 += 32) {
       float v[32];
@@ -426,7 +341,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       if (ok && s_idx < S) {
 #pragma unroll
         for (int c = 0; c < 32; c += 8) {
-          if (LATENT && c0 + c >= p.dv) break;
           uint32_t w[4];
 #pragma unroll
           for (int j = 0; j < 8; j += 2) {
@@ -452,22 +366,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   }
 }
 
-template <int KB, int VB, bool SPLIT, bool LATENT>
-static int launch_attn_kernel(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tqr, const CUtensorMap& tkr,
-                              const AttnParams& p, dim3 grid, cudaStream_t stream) {
-  using L = AttnSmem<KB, VB, SPLIT>;
-  auto kern = attn_prefill_kernel<KB, VB, SPLIT, LATENT>;
-  static bool attr_set = false;
-  if (!attr_set) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal) != cudaSuccess) return -10;
-    attr_set = true;
-  }
-  kern<<<grid, kAttnThreads, L::kTotal, stream>>>(tq, tk, tv, tqr, tkr, p);
-  return cudaGetLastError() == cudaSuccess ? 0 : -11;
-}
-
-template <int HD, bool SPLIT>
+template <int HD>
 static int launch_attn(const ortb200_attn_prefill_args* a, cudaStream_t stream) {
+  using L = AttnSmem<HD>;
   const CUtensorMapDataType dt = a->dtype == ORTB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   const bool paged = a->block_table != nullptr;
   CUtensorMap tq, tk, tv;
@@ -485,7 +386,7 @@ static int launch_attn(const ortb200_attn_prefill_args* a, cudaStream_t stream) 
     if (make_tensor_map_4d(&tk, a->k, dt, 2, dims, strides, 64, kKT) != 0) return -6;
     if (make_tensor_map_4d(&tv, a->v, dt, 2, dims, strides, 64, kKT) != 0) return -6;
   }
-  AttnParams p;
+  AttnParams p{};
   p.seqlens_k = a->seqlens_k;
   p.key_mask = paged ? nullptr : a->key_mask;
   p.head_sink = a->head_sink;
@@ -501,48 +402,17 @@ static int launch_attn(const ortb200_attn_prefill_args* a, cudaStream_t stream) 
   p.block_table = a->block_table; p.cu_seqlens = a->cu_seqlens; p.past_seqlens = a->past_seqlens;
   p.block_size = a->block_size; p.max_blocks = a->max_blocks; p.num_blocks = a->num_blocks;
   p.chunk = a->chunk;
-  p.plain_boxes = HD / 64; p.dv = HD; p.gate = nullptr; p.gate_ld = 0;
+  auto kern = attn_prefill_kernel<HD>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal) != cudaSuccess) return -10;
+    attr_set = true;
+  }
   // packed form: every sequence has at most one partly filled query tile
   const int tiles = paged ? a->T / kQT + (a->B < a->T ? a->B : a->T) : (a->S + kQT - 1) / kQT;
   dim3 grid(tiles, a->N, paged ? 1 : a->B);
-  return launch_attn_kernel<HD / 64, HD / 64, SPLIT, false>(tq, tk, tv, tq, tk, p, grid, stream);
-}
-
-static int launch_latent(const ortb200_latent_prefill_args* a, cudaStream_t stream) {
-  const CUtensorMapDataType dt = a->dtype == ORTB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
-  CUtensorMap tq, tk, tv, tqr, tkr;
-  // [rows, heads, size] operands with `ld` elements between rows and `step` between heads
-  auto map = [&](CUtensorMap* m, const void* base, int64_t size, int64_t rows, int64_t heads, int64_t ld, int64_t step) {
-    const int64_t dims[4] = {size, rows, heads, 1};
-    const int64_t strides[3] = {ld * 2, step * 2, rows * ld * 2};
-    return make_tensor_map_4d(m, base, dt, 2, dims, strides, 64, kQT) == 0;
-  };
-  const char* kv = static_cast<const char*>(a->kv);
-  if (!map(&tq, a->q, a->dk, a->T, a->N, a->q_ld, a->dk + a->dr) || !map(&tqr, a->q_rot, a->dr, a->T, a->N, static_cast<int64_t>(a->N) * a->dr, a->dr) ||
-      !map(&tk, kv, a->dk, a->key_rows, a->N, a->kv_ld, a->dk) ||
-      !map(&tv, kv + static_cast<int64_t>(a->N) * a->dk * 2, a->dv, a->key_rows, a->N, a->kv_ld, a->dv) ||
-      !map(&tkr, a->k_rot, a->dr, a->key_rows, 1, a->k_rot_ld, a->k_rot_ld))
-    return -6;
-  AttnParams p{};
-  p.head_sink = a->head_sink;
-  p.out = a->out;
-  p.B = a->B; p.S = 0; p.N = a->N; p.Nk = a->N; p.kv_len = 1 << 30;
-  p.o_strides[0] = 0; p.o_strides[1] = a->out_ld; p.o_strides[2] = a->dv;
-  p.causal = 1;
-  p.scale = a->scale;
-  p.scale_log2 = p.scale * 1.4426950408889634f;
-  p.bf16 = a->dtype == ORTB200_BF16 ? 1 : 0;
-  p.status = a->status;
-  p.cu_seqlens = a->cu_seqlens; p.past_seqlens = a->past_seqlens;
-  p.plain_boxes = (a->dk + 63) / 64;
-  p.dv = a->dv; p.gate = a->gate; p.gate_ld = a->gate_ld;
-  const int kb = p.plain_boxes + (a->dr + 63) / 64, vb = (a->dv + 63) / 64;
-  dim3 grid(a->T / kQT + (a->B < a->T ? a->B : a->T), a->N, 1);
-  if (kb == 2 && vb == 1) return launch_attn_kernel<2, 1, true, true>(tq, tk, tv, tqr, tkr, p, grid, stream);
-  if (kb == 2 && vb == 2) return launch_attn_kernel<2, 2, true, true>(tq, tk, tv, tqr, tkr, p, grid, stream);
-  if (kb == 3 && vb == 1) return launch_attn_kernel<3, 1, true, true>(tq, tk, tv, tqr, tkr, p, grid, stream);
-  if (kb == 3 && vb == 2) return launch_attn_kernel<3, 2, true, true>(tq, tk, tv, tqr, tkr, p, grid, stream);
-  return -2;
+  kern<<<grid, kAttnThreads, L::kTotal, stream>>>(tq, tk, tv, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
 }  // namespace ortb200
@@ -566,27 +436,6 @@ extern "C" int ortb200_attn_prefill(const ortb200_attn_prefill_args* a, ortb200_
        reinterpret_cast<uintptr_t>(a->out)) & 15)
     return -3;
   if (a->chunk > 0 && !a->causal) return -2;
-  if (a->split_weights) return a->H == 128 ? launch_attn<128, true>(a, stream) : launch_attn<64, true>(a, stream);
-  return a->H == 128 ? launch_attn<128, false>(a, stream) : launch_attn<64, false>(a, stream);
-}
-
-extern "C" int ortb200_latent_prefill_supported(int dk, int dr, int dv, int dtype) {
-  if (dtype != ORTB200_BF16 && dtype != ORTB200_F16) return 0;
-  if (dk <= 0 || dr <= 0 || dv <= 0 || dk % 8 || dr % 8 || dv % 8 || dv > 128) return 0;
-  return (dk + 63) / 64 + (dr + 63) / 64 <= 3 ? 1 : 0;
-}
-
-extern "C" int ortb200_latent_prefill(const ortb200_latent_prefill_args* a, ortb200_stream_t stream_) {
-  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (!a || !a->q || !a->q_rot || !a->kv || !a->k_rot || !a->out || !a->cu_seqlens || !a->past_seqlens) return -1;
-  if (a->B <= 0 || a->T <= 0 || a->N <= 0 || a->N > 65535 || a->key_rows <= 0) return -1;
-  if (!ortb200_latent_prefill_supported(a->dk, a->dr, a->dv, a->dtype)) return -2;
-  if (a->q_ld < static_cast<int64_t>(a->N) * (a->dk + a->dr) || a->kv_ld < static_cast<int64_t>(a->N) * (a->dk + a->dv) || a->k_rot_ld < a->dr ||
-      a->out_ld < static_cast<int64_t>(a->N) * a->dv || (a->gate && a->gate_ld < a->N))
-    return -2;
-  if (a->q_ld % 8 || a->kv_ld % 8 || a->k_rot_ld % 8 || a->out_ld % 8) return -3;
-  if ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->q_rot) | reinterpret_cast<uintptr_t>(a->kv) |
-       reinterpret_cast<uintptr_t>(a->k_rot) | reinterpret_cast<uintptr_t>(a->out)) & 15)
-    return -3;
-  return launch_latent(a, stream);
+  if (a->split_weights) return paged ? launch_attn_split(a, stream) : -2;
+  return a->H == 128 ? launch_attn<128>(a, stream) : launch_attn<64>(a, stream);
 }

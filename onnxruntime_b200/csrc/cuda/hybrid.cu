@@ -190,22 +190,29 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kernel(const ortb200_qk_norm
     if (!is_q && !ok) continue;
     if (is_v) {
       const int h = u - a.N - a.Nk;
-      const T* src = row + (a.N + a.Nk) * a.dk + h * a.dv;
-      T* dst = static_cast<T*>(a.v_cache) + (entry * a.Nk + h) * a.dv_pad;
+      const T* __restrict__ src = row + (a.N + a.Nk) * a.dk + h * a.dv;
+      T* __restrict__ dst = static_cast<T*>(a.v_cache) + (entry * a.Nk + h) * a.dv_pad;
       if (a.first_values) {
-        const T* first = static_cast<const T*>(a.first_values) + t * a.first_ld + h * a.dv;
+        const T* __restrict__ first = static_cast<const T*>(a.first_values) + t * a.first_ld + h * a.dv;
         const float m = *a.v_mix;
+#pragma unroll 4
         for (int d = lane; d < a.dv_pad; d += 32)
           dst[d] = from_float<T>(d < a.dv ? fmaf(m, to_float<T>(first[d]), (1.f - m) * to_float<T>(src[d])) : 0.f);
         continue;
       }
+#pragma unroll 4
       for (int d = lane; d < a.dv_pad; d += 32) dst[d] = d < a.dv ? src[d] : from_float<T>(0.f);
       continue;
     }
-    const T* src = row + u * a.dk;
+    const T* __restrict__ src = row + u * a.dk;
     const float* w = is_q ? a.q_norm : a.k_norm;
-    T* dst = is_q ? static_cast<T*>(a.q_out) + (static_cast<long long>(t) * a.N + u) * a.dk_pad
-                  : static_cast<T*>(a.k_cache) + (entry * a.Nk + (u - a.N)) * a.dk_pad;
+    T* __restrict__ dst = is_q ? static_cast<T*>(a.q_out) + (static_cast<long long>(t) * a.N + u) * a.dk_pad
+                               : static_cast<T*>(a.k_cache) + (entry * a.Nk + (u - a.N)) * a.dk_pad;
+    if (!w && half == 0) {   // nothing to compute
+#pragma unroll 4
+      for (int d = lane; d < a.dk_pad; d += 32) dst[d] = d < a.dk ? src[d] : from_float<T>(0.f);
+      continue;
+    }
     float ss = 0.f;
     for (int d = lane; d < a.dk; d += 32) {
       const float x = to_float<T>(src[d]);

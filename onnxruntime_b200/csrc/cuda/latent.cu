@@ -39,13 +39,38 @@ __device__ __forceinline__ void load_vec(const T* p, float (&v)[E]) {
   }
 }
 
+// E entries as they lie in memory: converted where they are used, so that a group of loads goes out together
+template <typename T, int E>
+struct Raw {
+  static constexpr int kWords = E * sizeof(T) / 16;
+  uint4 q[kWords > 0 ? kWords : 1];
+  T one;
+  __device__ __forceinline__ void load(const T* p) {
+    if constexpr (E == 1) {
+      one = p[0];
+    } else {
+#pragma unroll
+      for (int i = 0; i < kWords; ++i) q[i] = reinterpret_cast<const uint4*>(p)[i];
+    }
+  }
+  __device__ __forceinline__ float at(int e) const {
+    if constexpr (E == 1) return to_float<T>(one);
+    else return to_float<T>(reinterpret_cast<const T*>(q)[e]);
+  }
+};
+
 struct TokenPlace {
   int pos;          // position in its sequence, clamped into the rotary tables
   long long entry;  // cache entry, -1 when the block table does not hold the position
 };
 __device__ __forceinline__ TokenPlace place_of(const ortb200_latent_prep_args& a, int t) {
-  const int b = sequence_of(a.cu_seqlens, a.B, t);
-  const int pos = a.past_seqlens[b] + (t - a.cu_seqlens[b]);
+  // one token per sequence: everything that does not depend on the search is loaded at once
+  const int guess = min(t, a.B - 1), c0 = a.cu_seqlens[guess], c1 = a.cu_seqlens[guess + 1], past = a.past_seqlens[guess];
+  int b = guess, pos = past;
+  if (c0 != t || c1 != t + 1) {
+    b = sequence_of(a.cu_seqlens, a.B, t);
+    pos = a.past_seqlens[b] + (t - a.cu_seqlens[b]);
+  }
   const int bi = pos / a.block_size;
   const int blk = pos >= 0 && bi < a.max_blocks ? a.block_table[static_cast<long long>(b) * a.max_blocks + bi] : -1;
   const bool ok = blk >= 0 && blk < a.num_blocks && (a.rot_dim == 0 || pos < a.table_rows);
@@ -68,19 +93,44 @@ __device__ __forceinline__ void append_entry(const ortb200_latent_prep_args& a, 
   const TokenPlace at = place_of(a, t);
   if (at.entry < 0 && lane == 0 && a.status) atomicExch(a.status, kStatusBadArgument);
   const T* c = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld + static_cast<long long>(a.N) * (a.dk + a.dr);
-  float ss = 0.f;
-  for (int d = lane; d < a.rank; d += 32) {
-    const float x = to_float<T>(c[d]);
-    ss = fmaf(x, x, ss);
-  }
-  const float r = 1.f / sqrtf(warp_sum(ss) / a.rank + a.eps);
   T* dst = at.entry >= 0 ? static_cast<T*>(a.cache) + at.entry * a.width : nullptr;
   T* co = a.c_out ? static_cast<T*>(a.c_out) + static_cast<long long>(t) * a.rank : nullptr;
   T* ko = a.k_rot_out ? static_cast<T*>(a.k_rot_out) + static_cast<long long>(t) * (a.width - a.wide) : nullptr;
-  for (int d = lane; d < a.wide; d += 32) {
-    const T y = from_float<T>(d < a.rank ? to_float<T>(c[d]) * r * a.norm[d] : 0.f);
-    if (dst) dst[d] = y;
-    if (co && d < a.rank) co[d] = y;
+  float ss = 0.f;
+  if (sizeof(T) == 2 && a.rank % 8 == 0 && a.wide == a.rank && (reinterpret_cast<uintptr_t>(c) & 15) == 0) {   // whole vectors, held in registers
+    constexpr int kVecs = kMaxLatent / 256;
+    float x[kVecs][8];
+#pragma unroll
+    for (int k = 0; k < kVecs; ++k) {
+      const int d = (k * 32 + lane) * 8;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[k][e] = 0.f;
+      if (d < a.rank) load_vec<T, 8>(c + d, x[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(x[k][e], x[k][e], ss);
+    }
+    const float r = 1.f / sqrtf(warp_sum(ss) / a.rank + a.eps);
+#pragma unroll
+    for (int k = 0; k < kVecs; ++k) {
+      const int d = (k * 32 + lane) * 8;
+      if (d >= a.rank) continue;
+      __align__(16) T y[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = from_float<T>(x[k][e] * r * a.norm[d + e]);
+      if (dst) *reinterpret_cast<uint4*>(dst + d) = *reinterpret_cast<const uint4*>(y);
+      if (co) *reinterpret_cast<uint4*>(co + d) = *reinterpret_cast<const uint4*>(y);
+    }
+  } else {
+    for (int d = lane; d < a.rank; d += 32) {
+      const float x = to_float<T>(c[d]);
+      ss = fmaf(x, x, ss);
+    }
+    const float r = 1.f / sqrtf(warp_sum(ss) / a.rank + a.eps);
+    for (int d = lane; d < a.wide; d += 32) {
+      const T y = from_float<T>(d < a.rank ? to_float<T>(c[d]) * r * a.norm[d] : 0.f);
+      if (dst) dst[d] = y;
+      if (co && d < a.rank) co[d] = y;
+    }
   }
   const T* kr = c + a.rank;
   for (int d = lane; d < a.width - a.wide; d += 32) {
@@ -97,24 +147,36 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const ortb200_latent_p
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp == 0) append_entry<T>(a, t, lane);
   const int pos = place_of(a, t).pos;
-  const T* q = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld + a.dk;
-  T* dst = static_cast<T*>(a.q_rot) + static_cast<long long>(t) * a.N * a.dr;
+  const T* __restrict__ q = static_cast<const T*>(a.packed) + static_cast<long long>(t) * a.ld + a.dk;
+  T* __restrict__ dst = static_cast<T*>(a.q_rot) + static_cast<long long>(t) * a.N * a.dr;
   const int n = a.N * a.dr;
   if (((a.dr | a.dk | a.ld) & 1) == 0) {   // whole pairs in one access
     struct __align__(2 * sizeof(T)) Pair {
       T u, v;
     };
     const int half = a.dr / 2;
-    for (int i = threadIdx.x; i < n / 2; i += 128) {
-      const int h = i / half, j = i - h * half;
-      Pair x = *reinterpret_cast<const Pair*>(q + static_cast<long long>(h) * (a.dk + a.dr) + 2 * j);
-      if (2 * j < a.rot_dim) {
-        const long long at = static_cast<long long>(pos) * (a.rot_dim / 2) + j;
-        const float c = a.cos_table[at], s = a.sin_table[at], u = to_float<T>(x.u), v = to_float<T>(x.v);
-        x.u = from_float<T>(fmaf(u, c, -(v * s)));
-        x.v = from_float<T>(fmaf(v, c, u * s));
+    const float* __restrict__ cs = a.cos_table + static_cast<long long>(pos) * (a.rot_dim / 2);
+    const float* __restrict__ sn = a.sin_table + static_cast<long long>(pos) * (a.rot_dim / 2);
+    constexpr int kBatch = 4;
+    for (int i0 = threadIdx.x; i0 < n / 2; i0 += kBatch * 128) {
+      Pair x[kBatch];
+      float c[kBatch], s[kBatch];
+#pragma unroll
+      for (int k = 0; k < kBatch; ++k) {
+        const int i = min(i0 + k * 128, n / 2 - 1), h = i / half, j = i - h * half;
+        x[k] = *reinterpret_cast<const Pair*>(q + static_cast<long long>(h) * (a.dk + a.dr) + 2 * j);
+        c[k] = 2 * j < a.rot_dim ? cs[j] : 1.f;
+        s[k] = 2 * j < a.rot_dim ? sn[j] : 0.f;
       }
-      *reinterpret_cast<Pair*>(dst + 2 * i) = x;
+#pragma unroll
+      for (int k = 0; k < kBatch; ++k) {
+        const int i = i0 + k * 128;
+        if (i >= n / 2) break;
+        const float u = to_float<T>(x[k].u), v = to_float<T>(x[k].v);
+        x[k].u = from_float<T>(fmaf(u, c[k], -(v * s[k])));
+        x[k].v = from_float<T>(fmaf(v, c[k], u * s[k]));
+        *reinterpret_cast<Pair*>(dst + 2 * i) = x[k];
+      }
     }
   } else {
     for (int i = threadIdx.x; i < n; i += 128) {
@@ -125,56 +187,79 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const ortb200_latent_p
   pdl_launch_dependents();
 }
 
-// Blocks (h, slice of 16 E latent entries, group of kTok tokens); thread = (E entries, one of 16 shares of the head's dk
-// rows).  The last block of the x axis appends the new entries.
+// The x axis holds blocks (h, slice of 16 E latent entries), whose threads are (E entries, one of 16 shares of the head's dk
+// rows); then blocks that rotate the queries' parts of eight heads each; then one that appends the new entries.  The y axis
+// holds groups of kTok tokens.
+constexpr int kRows = 8;           // rows of the key map that a thread has in flight
+
 template <typename T, typename QT, int E>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const ortb200_latent_prep_args a, const int slices) {
   extern __shared__ __align__(16) float q_s[];           // [dk][kTok], then [8 warps][kTok][16 E]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.y * kTok, nt = min(kTok, a.T - t0);
-  pdl_wait_prior_grids();
-  if (blockIdx.x == static_cast<unsigned>(a.N * slices)) {
-    if (warp < nt) append_entry<T>(a, t0 + warp, lane);
+  const int maps = a.N * slices, bx = blockIdx.x;
+  if (bx >= maps) {
+    pdl_wait_prior_grids();
+    if (bx == static_cast<int>(gridDim.x) - 1) {
+      if (warp < nt) append_entry<T>(a, t0 + warp, lane);
+    } else {
+      const int h = (bx - maps) * 8 + warp;
+      const int mine = lane < nt ? place_of(a, t0 + lane).pos : 0;
+      if (h < a.N) {
+        const T* q = static_cast<const T*>(a.packed) + static_cast<long long>(h) * (a.dk + a.dr) + a.dk;
+        QT* out = static_cast<QT*>(a.q_abs) + (static_cast<long long>(t0) * a.N + h) * a.width;
+        int pos[kTok];
+#pragma unroll
+        for (int tk = 0; tk < kTok; ++tk) pos[tk] = __shfl_sync(0xffffffffu, mine, tk);
+        for (int d = lane; d < a.width - a.wide; d += 32) {
+          float v[kTok];   // all tokens are read before the first is stored
+#pragma unroll
+          for (int tk = 0; tk < kTok; ++tk) v[tk] = tk < nt && d < a.dr ? rotated<T>(a, q + static_cast<long long>(t0 + tk) * a.ld, d, pos[tk]) : 0.f;
+#pragma unroll
+          for (int tk = 0; tk < kTok; ++tk)
+            if (tk < nt) out[static_cast<long long>(tk) * a.N * a.width + a.wide + d] = from_float<QT>(v[tk]);
+        }
+        for (int d = a.rank + lane; d < a.wide; d += 32)
+          for (int tk = 0; tk < nt; ++tk) out[static_cast<long long>(tk) * a.N * a.width + d] = from_float<QT>(0.f);
+      }
+    }
     pdl_launch_dependents();
     return;
   }
-  const int h = blockIdx.x / slices, slice = blockIdx.x % slices;
-  const T* q = static_cast<const T*>(a.packed) + static_cast<long long>(h) * (a.dk + a.dr);
-  QT* out = static_cast<QT*>(a.q_abs) + static_cast<long long>(h) * a.width;
-  const long long q_row = static_cast<long long>(a.N) * a.width;
-  for (int i = threadIdx.x; i < a.dk * kTok; i += 256) {
-    const int tk = i / a.dk, d = i - tk * a.dk;
-    q_s[d * kTok + tk] = tk < nt ? to_float<T>(q[static_cast<long long>(t0 + tk) * a.ld + d]) : 0.f;
-  }
-  if (slice == 0) {
-    for (int tk = warp; tk < nt; tk += 8) {
-      const int pos = place_of(a, t0 + tk).pos;
-      const T* qr = q + static_cast<long long>(t0 + tk) * a.ld + a.dk;
-      for (int d = lane; d < a.width - a.wide; d += 32)
-        out[(t0 + tk) * q_row + a.wide + d] = from_float<QT>(d < a.dr ? rotated<T>(a, qr, d, pos) : 0.f);
-      for (int d = a.rank + lane; d < a.wide; d += 32) out[(t0 + tk) * q_row + d] = from_float<QT>(0.f);
-    }
-  }
-  __syncthreads();
+  const int h = bx / slices, slice = bx % slices;
   const int cg = threadIdx.x & 15, share = threadIdx.x >> 4;
   const int c = (slice * 16 + cg) * E;
+  const bool in = c < a.rank;   // E divides rank
+  const T* w = static_cast<const T*>(a.up) + static_cast<long long>(h) * a.dk * a.rank + (in ? c : 0);
+  Raw<T, E> wv[kRows];          // the first rows are constants: fetched before the kernel in front has finished
+#pragma unroll
+  for (int k = 0; k < kRows; ++k) wv[k].load(w + static_cast<long long>(min(share + 16 * k, a.dk - 1)) * a.rank);
+  pdl_wait_prior_grids();
+  const T* q = static_cast<const T*>(a.packed) + static_cast<long long>(t0) * a.ld + static_cast<long long>(h) * (a.dk + a.dr);
+#pragma unroll
+  for (int tk = 0; tk < kTok; ++tk)
+    for (int d = threadIdx.x; d < a.dk; d += 256) q_s[d * kTok + tk] = tk < nt ? to_float<T>(q[static_cast<long long>(tk) * a.ld + d]) : 0.f;
+  __syncthreads();
   float acc[kTok][E];
 #pragma unroll
   for (int tk = 0; tk < kTok; ++tk)
 #pragma unroll
     for (int e = 0; e < E; ++e) acc[tk][e] = 0.f;
-  if (c < a.rank) {   // E divides rank
-    const T* w = static_cast<const T*>(a.up) + static_cast<long long>(h) * a.dk * a.rank + c;
-#pragma unroll 4
-    for (int d = share; d < a.dk; d += 16) {
-      float wv[E];
-      load_vec<T, E>(w + static_cast<long long>(d) * a.rank, wv);
+  for (int d0 = share; d0 < a.dk; d0 += 16 * kRows) {
+#pragma unroll
+    for (int k = 0; k < kRows; ++k) {
+      const int d = d0 + 16 * k;
+      if (d >= a.dk) break;
       const float4 qa = *reinterpret_cast<const float4*>(q_s + d * kTok), qb = *reinterpret_cast<const float4*>(q_s + d * kTok + 4);
       const float qv[kTok] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
 #pragma unroll
       for (int tk = 0; tk < kTok; ++tk)
 #pragma unroll
-        for (int e = 0; e < E; ++e) acc[tk][e] = fmaf(qv[tk], wv[e], acc[tk][e]);
+        for (int e = 0; e < E; ++e) acc[tk][e] = fmaf(qv[tk], wv[k].at(e), acc[tk][e]);
+    }
+    if (d0 + 16 * kRows < a.dk) {
+#pragma unroll
+      for (int k = 0; k < kRows; ++k) wv[k].load(w + static_cast<long long>(min(d0 + 16 * (kRows + k), a.dk - 1)) * a.rank);
     }
   }
   float* red = q_s + a.dk * kTok;
@@ -186,13 +271,14 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const ortb200_latent
       if (lane < 16) red[(warp * kTok + tk) * 16 * E + cg * E + e] = acc[tk][e];
     }
   __syncthreads();
+  QT* out = static_cast<QT*>(a.q_abs) + (static_cast<long long>(t0) * a.N + h) * a.width;
   for (int i = threadIdx.x; i < nt * 16 * E; i += 256) {
     const int tk = i / (16 * E), j = i % (16 * E), col = slice * 16 * E + j;
     if (col >= a.rank) continue;
     float v = 0.f;
 #pragma unroll
     for (int k = 0; k < 8; ++k) v += red[(k * kTok + tk) * 16 * E + j];
-    out[(t0 + tk) * q_row + col] = from_float<QT>(v);
+    out[static_cast<long long>(tk) * a.N * a.width + col] = from_float<QT>(v);
   }
   pdl_launch_dependents();
 }
@@ -339,6 +425,17 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const ortb200_latent_ou
   const int h = blockIdx.x / slices, j0 = (blockIdx.x % slices) * kOutRows;
   const int t0 = blockIdx.y * kTok, nt = min(kTok, a.T - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j = j0 + warp * 4;
+  const T* w = static_cast<const T*>(a.up_v) + (static_cast<long long>(h) * a.dv + min(j, a.dv - 1)) * a.rank;
+  // the lane's first two shares of its four rows are constants: fetched before the kernel in front has finished
+  constexpr int kAhead = 2;
+  Raw<T, E> wv[kAhead][4];
+  auto fetch = [&](int c, Raw<T, E> (&v)[4]) {
+#pragma unroll
+    for (int r = 0; r < 4; ++r) v[r].load(w + static_cast<long long>(j + r < a.dv ? r : 0) * a.rank + (c < a.rank ? c : 0));
+  };
+#pragma unroll
+  for (int k = 0; k < kAhead; ++k) fetch((k * 32 + lane) * E, wv[k]);
   pdl_wait_prior_grids();
   if (warp < nt) {   // factor of every part of token t0 + warp (parts <= 32)
     const float* ml = a.ml + (static_cast<long long>(t0 + warp) * a.N + h) * a.parts * 2;
@@ -350,37 +447,59 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const ortb200_latent_ou
     coef[warp][lane] = den > 0.f ? w / den : 0.f;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < kTok * a.rank; i += 256) {
-    const int tk = i / a.rank, c = i - tk * a.rank;
-    float v = 0.f;
-    if (tk < nt) {
-      const float* o = a.o + (static_cast<long long>(t0 + tk) * a.N + h) * a.parts * a.wide + c;
-      for (int p = 0; p < a.parts; ++p) {
-        const float f = coef[tk][p];
-        if (f != 0.f) v = fmaf(f, o[static_cast<long long>(p) * a.wide], v);   // a part without keys is not read
+  if constexpr (E == 8) {   // rank and wide are multiples of four then
+    const int vecs = a.rank / 4;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < kTok * vecs; i += 256) {
+      const int tk = i / vecs, c = (i - tk * vecs) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (tk < nt) {
+        const float* o = a.o + (static_cast<long long>(t0 + tk) * a.N + h) * a.parts * a.wide + c;
+        for (int p0 = 0; p0 < a.parts; p0 += 4) {   // factors of absent parts are 0
+          float4 x[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) x[k] = *reinterpret_cast<const float4*>(o + static_cast<long long>(min(p0 + k, a.parts - 1)) * a.wide);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float f = coef[tk][p0 + k];
+            v.x = fmaf(f, x[k].x, v.x); v.y = fmaf(f, x[k].y, v.y); v.z = fmaf(f, x[k].z, v.z); v.w = fmaf(f, x[k].w, v.w);
+          }
+        }
       }
+      *reinterpret_cast<float4*>(o_s + tk * a.rank + c) = v;
     }
-    o_s[i] = v;
+  } else {
+    for (int i = threadIdx.x; i < kTok * a.rank; i += 256) {
+      const int tk = i / a.rank, c = i - tk * a.rank;
+      float v = 0.f;
+      if (tk < nt) {
+        const float* o = a.o + (static_cast<long long>(t0 + tk) * a.N + h) * a.parts * a.wide + c;
+        for (int p = 0; p < a.parts; ++p) v = fmaf(coef[tk][p], o[static_cast<long long>(p) * a.wide], v);
+      }
+      o_s[i] = v;
+    }
   }
   __syncthreads();
   float acc[4 * kTok];
 #pragma unroll
   for (int i = 0; i < 4 * kTok; ++i) acc[i] = 0.f;
-  const int j = j0 + warp * 4;
   if (j < a.dv) {
-    const T* w = static_cast<const T*>(a.up_v) + (static_cast<long long>(h) * a.dv + j) * a.rank;
-    for (int c = lane * E; c < a.rank; c += 32 * E) {
-      float wv[4][E];
+    for (int c0 = 0; c0 < a.rank; c0 += kAhead * 32 * E) {
 #pragma unroll
-      for (int r = 0; r < 4; ++r) load_vec<T, E>(w + static_cast<long long>(j + r < a.dv ? r : 0) * a.rank + c, wv[r]);
+      for (int k = 0; k < kAhead; ++k) {
+        const int c = c0 + (k * 32 + lane) * E;
+        if (c < a.rank) {
 #pragma unroll
-      for (int tk = 0; tk < kTok; ++tk) {
-        float ov[E];
-        load_vec<float, E>(o_s + tk * a.rank + c, ov);
+          for (int tk = 0; tk < kTok; ++tk) {
+            float ov[E];
+            load_vec<float, E>(o_s + tk * a.rank + c, ov);
 #pragma unroll
-        for (int r = 0; r < 4; ++r)
+            for (int r = 0; r < 4; ++r)
 #pragma unroll
-          for (int e = 0; e < E; ++e) acc[r * kTok + tk] = fmaf(wv[r][e], ov[e], acc[r * kTok + tk]);
+              for (int e = 0; e < E; ++e) acc[r * kTok + tk] = fmaf(wv[k][r].at(e), ov[e], acc[r * kTok + tk]);
+          }
+        }
+        if (c0 + kAhead * 32 * E < a.rank) fetch(c + kAhead * 32 * E, wv[k]);
       }
     }
     // after the step of distance o, a lane holds the sums whose index has bit o equal to the lane's
@@ -415,7 +534,7 @@ int launch_absorb(const ortb200_latent_prep_args& a, cudaStream_t stream) {
   const int smem = (a.dk * kTok + 8 * kTok * 16 * E) * 4;
   auto kern = latent_absorb_kernel<T, QT, E>;
   if (int rc = opt_in_smem(kern, smem)) return rc;
-  return launch_kernel(kern, dim3(a.N * slices + 1, (a.T + kTok - 1) / kTok), 256, smem, stream, a.use_pdl != 0, a, slices);
+  return launch_kernel(kern, dim3(a.N * slices + (a.N + 7) / 8 + 1, (a.T + kTok - 1) / kTok), 256, smem, stream, a.use_pdl != 0, a, slices);
 }
 template <typename T>
 int dispatch_absorb(const ortb200_latent_prep_args& a, cudaStream_t stream) {

@@ -1,13 +1,15 @@
 // Attention of absorbed latent queries over the paged latent cache on the tcgen05 tensor cores: every query head of a token
 // reads the same cache rows, so the heads are the N columns of both products and the cache streams once per group of heads.
 //   MMA 1  S^T[128 keys, G]     = C_tile[128 keys, wide + rot] . Q[G heads, wide + rot]^T          (both K-major)
-//   MMA 2  O^T[128 dims, G] (m) += C_tile[:, 128 dims of block m]^T . (P_hi + P_lo)[G heads, 128 keys]^T   (C MN-major)
+//   MMA 2  O^T[128 dims, 2 G] (m) += C_tile[:, 128 dims of block m]^T . [P_hi; P_lo][2 G, 128 keys]^T   (C MN-major)
 // The value of a key is its latent, so one tile in shared memory serves both.  Softmax weights stay 32-bit: they enter MMA 2
-// as the sum of two 16-bit terms.
+// as two 16-bit terms, whose sums lie in separate columns and are added at the end (the product is bound by reading the
+// tile, so twice the columns cost nothing).
 //
-// A cluster of C CTAs shares one (token, group of heads, part); each CTA takes a contiguous range of 128-key tiles, keeps its
+// A cluster of C CTAs shares one (token, group of heads, part); each CTA takes a contiguous range of keys, keeps its
 // accumulator in tensor memory, and after one cluster barrier the CTAs merge their heads through distributed shared memory.
-// A tile (up to 147 KB) has one buffer; ranges are short because the tiles are dealt to all SMs.
+// Ranges are dealt in granules of 32 keys over all SMs.  A tile (up to 147 KB) has one buffer, but MMA 1 starts on each box
+// of 64 entries as it arrives, and the boxes of a block of entries are refilled as soon as MMA 2 has read that block.
 #include <cuda.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -27,14 +29,13 @@ constexpr int kBox = 128 * 128;           // [128 keys][64 entries] of 16-bit da
 constexpr int kThreads = 160;             // 4 softmax warps + 1 TMA / MMA warp
 constexpr int kMaxBoxes = 9;              // e.g. a latent of 512 and a rotated part of 64
 constexpr int kMaxWideBoxes = 8;
-constexpr int kTmemCols = 256;            // S^T (G), then up to four blocks of O^T (G each)
+constexpr int kGranule = 32;              // keys: unit of the ranges and of what is fetched and multiplied
 constexpr float kNegBig = -1.0e30f;
 constexpr float kRaise = 8.f;             // the reference maximum is raised only past 2^8
-// At most two CTAs per SM, so that their tensor-memory allocations always fit: a CTA that waits for an allocation while its
-// cluster waits for it must not depend on other clusters.
-constexpr int kMinSmem = 100 * 1024;
+constexpr int kMaxCluster = 4;
+constexpr int kMaxBlocks = kMaxWideBoxes / 2;
 
-enum { BAR_Q = 0, BAR_FULL, BAR_S, BAR_P, BAR_O, BAR_COUNT };
+enum { BAR_Q = 0, BAR_S, BAR_P, BAR_FULL0, BAR_O0 = BAR_FULL0 + kMaxBoxes, BAR_COUNT = BAR_O0 + kMaxBlocks };
 
 struct LatentTcParams {
   const int* cu_seqlens;
@@ -68,7 +69,7 @@ __device__ __forceinline__ float ld_dsmem(uint32_t addr) {
 }
 __device__ __forceinline__ float4 ld_dsmem4(uint32_t addr) {
   float4 v;
-  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr));
   return v;
 }
 __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const float* v) {
@@ -81,8 +82,14 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const float* v) {
 template <int G>
 struct Layout {
   static constexpr int kHeadBox = G * 128;               // [G heads][64 entries]
-  static constexpr int kPBytes = 4 * kHeadBox;           // two key boxes of leading terms, two of remainders
-  static constexpr int kSmall = 2 * 4 * G * 4 + 2 * G * 4 + 128;   // maxima, sums, (max, sum) per head, barriers
+  static constexpr int kPBox = 2 * G * 128;              // [G leading terms, G remainders][64 keys]
+  static constexpr int kPBytes = 2 * kPBox;
+  // maxima, sums, (max, sum) per head, merge factors, barriers
+  static constexpr int kSmall = 2 * 4 * G * 4 + 2 * G * 4 + G * kMaxCluster * 4 + 256;
+  static constexpr int kTmemCols = G == 32 ? 512 : 256;   // S^T (G of the first 2 G columns), then up to four blocks of O^T (2 G each)
+  // Shared memory is asked for so that the allocations of the CTAs on an SM always fit together: a CTA that waits for
+  // tensor memory while its cluster waits for it must not depend on other clusters.
+  static constexpr int kMinSmem = (G == 32 ? 120 : 100) * 1024;
   static int bytes(int boxes) { return boxes * (kBox + kHeadBox) + kPBytes + kSmall + 1024; }
 };
 
@@ -99,7 +106,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   float* sm_max = reinterpret_cast<float*>(sm_p + L::kPBytes);   // [4][G]
   float* sm_sum = sm_max + 4 * G;                                // [4][G]
   float* sm_ml = sm_sum + 4 * G;                                 // [G][2]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sm_ml + 2 * G);
+  float* sm_coef = sm_ml + 2 * G;                                // [heads merged here][kMaxCluster]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sm_coef + G * kMaxCluster);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + BAR_COUNT);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -116,13 +124,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     fence_mbar_init();
   }
   if (warp == 4) {
-    tmem_alloc(tmem_slot, kTmemCols);
+    tmem_alloc(tmem_slot, L::kTmemCols);
     tmem_relinquish();
   }
   tcgen05_fence_before();
   __syncthreads();
   tcgen05_fence_after();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + G;
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * G;
 
   pdl_wait_prior_grids();
   const int b = sequence_of(p.cu_seqlens, p.B, t);
@@ -131,18 +139,18 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (tid == 0 && p.status) atomicExch(p.status, kStatusBadLength);
     len = len < 0 ? 0 : p.max_blocks * p.block_size;
   }
-  const int all_tiles = (len + kTile - 1) / kTile;
-  const int per_cta = (all_tiles + p.parts * p.cluster - 1) / (p.parts * p.cluster);
-  const int tile0 = static_cast<int>(blockIdx.x) * per_cta;
-  const int n_tiles = max(0, min(all_tiles - tile0, per_cta));
+  const int ctas = p.parts * p.cluster, granules = (len + kGranule - 1) / kGranule;
+  const int range = (granules + ctas - 1) / ctas * kGranule;
+  const int k_begin = static_cast<int>(blockIdx.x) * range, k_end = min(len, k_begin + range);
+  const int n_tiles = k_end > k_begin ? (k_end - k_begin + kTile - 1) / kTile : 0;
   const int o_blocks = (p.wide_boxes + 1) / 2;
 
   if (warp == 4) {
     // ---------------------------------------------------------- TMA producer + MMA issuer (lane i fetches piece i of a tile)
     const uint32_t idesc_s = umma_idesc_f16(kBf16, kTile, G);
-    const uint32_t idesc_o = umma_idesc_f16(kBf16, 128, G) | (1u << 15);   // A (the tile read along its entries) is MN-major
+    const uint32_t idesc_o = umma_idesc_f16(kBf16, 128, 2 * G) | (1u << 15);   // A (the tile read along its entries) is MN-major
     const uint32_t c_addr = smem_u32(smem), q_addr = smem_u32(sm_q), p_addr = smem_u32(sm_p);
-    const int pieces = kTile / p.piece_rows;
+    const int granule_pieces = kGranule / p.piece_rows;
     bool ok = true;
     if (n_tiles > 0 && lane == 0) {
       mbar_expect_tx(&bars[BAR_Q], static_cast<uint32_t>(p.boxes) * L::kHeadBox);
@@ -152,32 +160,42 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       }
     }
     for (int i = 0; i < n_tiles && ok; ++i) {
-      if (i > 0 && !mbar_wait(&bars[BAR_O], (i - 1) & 1)) { ok = false; break; }   // the tile before has been read
-      if (lane == 0) mbar_expect_tx(&bars[BAR_FULL], static_cast<uint32_t>(p.boxes) * kBox);
-      __syncwarp();
-      if (lane < pieces) {
-        // blocks outside the sequence or the pool are clamped: masked keys only have to be finite
-        const int key = (tile0 + i) * kTile + lane * p.piece_rows;
-        const int bi = min(key / p.block_size, p.max_blocks - 1);
-        const int blk = min(max(p.block_table[static_cast<long long>(b) * p.max_blocks + bi], 0), p.num_blocks - 1);
-        const int row = blk * p.block_size + key % p.block_size;
-        uint8_t* dst = smem + lane * p.piece_rows * 128;
-        for (int bx = 0; bx < p.boxes; ++bx) {
-          if (bx < p.wide_boxes) tma_load_2d(dst + bx * kBox, &tm_c, &bars[BAR_FULL], bx * 64, row);
-          else tma_load_2d(dst + bx * kBox, &tm_cr, &bars[BAR_FULL], (bx - p.wide_boxes) * 64, row);
+      const int key0 = k_begin + i * kTile;
+      const int live = (min(kTile, k_end - key0) + kGranule - 1) / kGranule;   // granules
+      const int pieces = live * granule_pieces;   // at most 16: lanes take a piece of one of two boxes each
+      const int sub = lane / pieces, piece = lane - sub * pieces, key = key0 + piece * p.piece_rows;
+      // blocks outside the sequence or the pool are clamped: masked keys only have to be finite
+      const int bi = min(key / p.block_size, p.max_blocks - 1);
+      const int blk = min(max(p.block_table[static_cast<long long>(b) * p.max_blocks + bi], 0), p.num_blocks - 1);
+      const int row = blk * p.block_size + key % p.block_size;
+      for (int bx0 = 0; bx0 < p.boxes && ok; bx0 += 2) {
+        if (i > 0 && bx0 / 2 < o_blocks && !mbar_wait(&bars[BAR_O0 + bx0 / 2], (i - 1) & 1)) { ok = false; break; }
+        const int n = min(2, p.boxes - bx0);
+        if (lane < n) mbar_expect_tx(&bars[BAR_FULL0 + bx0 + lane], static_cast<uint32_t>(live) * (kGranule * 128));
+        __syncwarp();
+        if (sub < n) {
+          const int bx = bx0 + sub;
+          uint8_t* dst = smem + bx * kBox + piece * p.piece_rows * 128;
+          if (bx < p.wide_boxes) tma_load_2d(dst, &tm_c, &bars[BAR_FULL0 + bx], bx * 64, row);
+          else tma_load_2d(dst, &tm_cr, &bars[BAR_FULL0 + bx], (bx - p.wide_boxes) * 64, row);
         }
+        __syncwarp();
       }
-      __syncwarp();
+      if (!ok) break;
       if (i == 0 && !mbar_wait(&bars[BAR_Q], 0)) { ok = false; break; }
-      if (!mbar_wait(&bars[BAR_FULL], i & 1)) { ok = false; break; }
-      if (lane == 0) {
-        tcgen05_fence_after();
-        for (int bx = 0; bx < p.boxes; ++bx) {
+      for (int bx = 0; bx < p.boxes && ok; ++bx) {
+        if (!mbar_wait(&bars[BAR_FULL0 + bx], i & 1)) { ok = false; break; }
+        if (lane == 0) {
+          tcgen05_fence_after();
 #pragma unroll
           for (int kk = 0; kk < 4; ++kk)
             umma_f16(tmem_s, umma_desc_sw128(c_addr + bx * kBox + kk * 32), umma_desc_sw128(q_addr + bx * L::kHeadBox + kk * 32), idesc_s,
                      bx > 0 || kk > 0 ? 1u : 0u);
         }
+        __syncwarp();
+      }
+      if (!ok) break;
+      if (lane == 0) {
         umma_commit(&bars[BAR_S]);
       }
       __syncwarp();
@@ -185,15 +203,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (lane == 0) {
         tcgen05_fence_after();
         for (int m = 0; m < o_blocks; ++m) {
-#pragma unroll
-          for (int kk = 0; kk < kTile / 16; ++kk) {
-            const uint64_t cdesc = umma_desc_mn_sw128(c_addr + 2 * m * kBox + kk * 2048, kBox, 1024);
-            const uint32_t po = p_addr + (kk / 4) * L::kHeadBox + (kk % 4) * 32;
-            umma_f16(tmem_o + m * G, cdesc, umma_desc_sw128(po), idesc_o, i > 0 || kk > 0 ? 1u : 0u);
-            umma_f16(tmem_o + m * G, cdesc, umma_desc_sw128(po + 2 * L::kHeadBox), idesc_o, 1u);
-          }
+          for (int kk = 0; kk < live * (kGranule / 16); ++kk)
+            umma_f16(tmem_o + m * 2 * G, umma_desc_mn_sw128(c_addr + 2 * m * kBox + kk * 2048, kBox, 1024),
+                     umma_desc_sw128(p_addr + (kk / 4) * L::kPBox + (kk % 4) * 32), idesc_o, i > 0 || kk > 0 ? 1u : 0u);
+          umma_commit(&bars[BAR_O0 + m]);
         }
-        umma_commit(&bars[BAR_O]);
       }
       __syncwarp();
     }
@@ -219,7 +233,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
       for (int c = 0; c < G; c += 16) tmem_ld_x16(tmem_s + lane_addr + c, sv + c);
       tmem_ld_wait();
-      const bool valid = (tile0 + i) * kTile + tid < len;
+      const bool valid = k_begin + i * kTile + tid < k_end;
 #pragma unroll
       for (int g = 0; g < G; ++g) {
         sv[g] = valid ? sv[g] * p.scale_log2 : kNegBig;
@@ -243,24 +257,24 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
         for (int g = 0; g < G; ++g) l_part[g] *= corr[g];
         if (i > 0) {
-          if (ok && !mbar_wait(&bars[BAR_O], (i - 1) & 1)) ok = false;
+          if (ok && !mbar_wait(&bars[BAR_O0 + o_blocks - 1], (i - 1) & 1)) ok = false;
           tcgen05_fence_after();
           for (int m = 0; m < o_blocks; ++m) {
 #pragma unroll
-            for (int c = 0; c < G; c += 16) {
+            for (int c = 0; c < 2 * G; c += 16) {
               float ov[16];
-              tmem_ld_x16(tmem_o + m * G + lane_addr + c, ov);
+              tmem_ld_x16(tmem_o + m * 2 * G + lane_addr + c, ov);
               tmem_ld_wait();
 #pragma unroll
-              for (int j = 0; j < 16; ++j) ov[j] *= corr[c + j];
-              tmem_st_x16(tmem_o + m * G + lane_addr + c, ov);
+              for (int j = 0; j < 16; ++j) ov[j] *= corr[(c + j) % G];
+              tmem_st_x16(tmem_o + m * 2 * G + lane_addr + c, ov);
             }
           }
           tmem_st_wait();
         }
       }
       // weights of this key for every head, as leading term + remainder in the swizzled K-major layout MMA 2 reads
-      uint8_t* pb = sm_p + (tid >> 6) * L::kHeadBox;
+      uint8_t* pb = sm_p + (tid >> 6) * L::kPBox;
       const int col = tid & 63;
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -269,36 +283,46 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         l_part[g] += pr;
         uint8_t* dst = pb + g * 128 + (((col >> 3) ^ (g & 7)) << 4) + (col & 7) * 2;
         *reinterpret_cast<T*>(dst) = hi;
-        *reinterpret_cast<T*>(dst + 2 * L::kHeadBox) = from_float<T>(pr - to_float<T>(hi));
+        *reinterpret_cast<T*>(dst + L::kHeadBox) = from_float<T>(pr - to_float<T>(hi));
       }
       fence_proxy_async();
       tcgen05_fence_before();
       mbar_arrive(&bars[BAR_P]);
       asm volatile("bar.sync 1, 128;" ::: "memory");   // sm_max is free again
     }
-    if (n_tiles > 0 && ok && !mbar_wait(&bars[BAR_O], (n_tiles - 1) & 1)) ok = false;
+    // sums over the warp's keys: halving exchanges leave lane j with head j % G
+    float acc[G];
+#pragma unroll
+    for (int g = 0; g < G; ++g) acc[g] = l_part[g];
+#pragma unroll
+    for (int o = G / 2; o >= 1; o >>= 1) {
+#pragma unroll
+      for (int g = 0; g < o; ++g) {
+        const float send = lane & o ? acc[g] : acc[g + o], keep = lane & o ? acc[g + o] : acc[g];
+        acc[g] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      }
+    }
+    if (G == 16) acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 16);
+    if (lane < G) sm_sum[warp * G + lane] = acc[0];
+    if (tid == 0) {
+#pragma unroll
+      for (int g = 0; g < G; ++g) sm_ml[2 * g] = m_ref[g];
+    }
+    if (n_tiles > 0 && ok && !mbar_wait(&bars[BAR_O0 + o_blocks - 1], (n_tiles - 1) & 1)) ok = false;
     tcgen05_fence_after();
     if (!ok && p.status) atomicExch(p.status, kStatusTimeoutEpilogue);
-#pragma unroll
-    for (int g = 0; g < G; ++g) {
-      const float s = warp_sum(l_part[g]);
-      if (lane == 0) sm_sum[warp * G + g] = s;
-      if (tid == 0) sm_ml[2 * g] = m_ref[g];
-    }
     // O^T -> [G][wide_boxes * 64] fp32 in the tile's place
     const int pitch = p.wide_boxes * 64;
     if (n_tiles > 0) {
       float* stage = reinterpret_cast<float*>(smem);
       for (int m = 0; m < o_blocks; ++m) {
+        float ov[2 * G];
 #pragma unroll
-        for (int c = 0; c < G; c += 16) {
-          float ov[16];
-          tmem_ld_x16(tmem_o + m * G + lane_addr + c, ov);
-          tmem_ld_wait();
-          if (m * 128 + tid < pitch) {
+        for (int c = 0; c < 2 * G; c += 16) tmem_ld_x16(tmem_o + m * 2 * G + lane_addr + c, ov + c);
+        tmem_ld_wait();
+        if (m * 128 + tid < pitch) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) stage[(c + j) * pitch + m * 128 + tid] = ov[j];
-          }
+          for (int g = 0; g < G; ++g) stage[g * pitch + m * 128 + tid] = ov[g] + ov[G + g];
         }
       }
     }
@@ -309,51 +333,67 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   if (p.cluster > 1) cluster_sync_all();
   else __syncthreads();
   pdl_launch_dependents();
-  // ------------------------------------------------------------ merge: the CTAs of a cluster take every C-th head each
-  if (warp < 4) {
-    const int pitch = p.wide_boxes * 64;
-    const uint32_t stage = smem_u32(smem), ml = smem_u32(sm_ml);
-    for (int g = rank; g < n_heads; g += p.cluster) {
-      float mc[8], w[8];
-      float mm = kNegBig, sum = 0.f;
+  // ------------------------------------------------------------ merge: CTA r of C takes heads r, r + C, ...
+  const int mine = n_heads > rank ? (n_heads - rank + p.cluster - 1) / p.cluster : 0;
+  const int pitch = p.wide_boxes * 64, vecs = p.wide / 4;   // wide is a multiple of eight
+  const uint32_t stage_addr = smem_u32(smem), ml_addr = smem_u32(sm_ml);
+  const long long at0 = static_cast<long long>(t) * p.N + head0;
+  if (tid < mine) {
+    const int g = rank + tid * p.cluster;
+    float mc[kMaxCluster], lc[kMaxCluster], mm = kNegBig, sum = 0.f;
 #pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        mc[c] = c < p.cluster ? ld_dsmem(map_to_cta(ml + g * 8, c)) : kNegBig;
-        mm = fmaxf(mm, mc[c]);
-      }
+    for (int c = 0; c < kMaxCluster; ++c) {
+      mc[c] = c < p.cluster ? ld_dsmem(map_to_cta(ml_addr + g * 8, c)) : kNegBig;
+      lc[c] = c < p.cluster ? ld_dsmem(map_to_cta(ml_addr + g * 8 + 4, c)) : 0.f;
+    }
 #pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        w[c] = mc[c] <= kNegBig ? 0.f : exp2f(mc[c] - mm);
-        if (c < p.cluster) sum = fmaf(w[c], ld_dsmem(map_to_cta(ml + g * 8 + 4, c)), sum);
-      }
-      const long long at = (static_cast<long long>(t) * p.N + head0 + g) * p.parts + part;
-      for (int d = tid * 4; d < p.wide; d += 512) {   // wide is a multiple of eight
-        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c = 0; c < kMaxCluster; ++c) mm = fmaxf(mm, mc[c]);
 #pragma unroll
-        for (int c = 0; c < 8; ++c) {
-          if (w[c] == 0.f) continue;                  // no keys: nothing was staged
-          const float4 v = ld_dsmem4(map_to_cta(stage + (g * pitch + d) * 4, c));
-          o.x = fmaf(w[c], v.x, o.x); o.y = fmaf(w[c], v.y, o.y); o.z = fmaf(w[c], v.z, o.z); o.w = fmaf(w[c], v.w, o.w);
-        }
-        *reinterpret_cast<float4*>(p.o + at * p.wide + d) = o;
+    for (int c = 0; c < kMaxCluster; ++c) {
+      const float w = mc[c] <= kNegBig ? 0.f : exp2f(mc[c] - mm);
+      sum = fmaf(w, lc[c], sum);
+      sm_coef[tid * kMaxCluster + c] = w;
+    }
+    p.ml[((at0 + g) * p.parts + part) * 2] = mm;
+    p.ml[((at0 + g) * p.parts + part) * 2 + 1] = sum;
+  }
+  // a thread has four vectors of all CTAs in flight; what a CTA without keys has not staged is not used
+  constexpr int kBatch = 4;
+  for (int j0 = tid; j0 < mine * vecs || j0 == tid; j0 += kBatch * kThreads) {
+    float4 v[kBatch][kMaxCluster];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int j = j0 + i * kThreads, k = j / vecs, d = (j - k * vecs) * 4, g = rank + k * p.cluster;
+#pragma unroll
+      for (int c = 0; c < kMaxCluster; ++c)
+        if (j < mine * vecs && c < p.cluster) v[i][c] = ld_dsmem4(map_to_cta(stage_addr + (g * pitch + d) * 4, c));
+    }
+    if (j0 == tid) __syncthreads();   // every thread comes by once: the factors are complete
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int j = j0 + i * kThreads, k = j / vecs, d = (j - k * vecs) * 4, g = rank + k * p.cluster;
+      if (j >= mine * vecs) continue;
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int c = 0; c < kMaxCluster; ++c) {
+        const float w = c < p.cluster ? sm_coef[k * kMaxCluster + c] : 0.f;
+        if (w == 0.f) continue;
+        o.x = fmaf(w, v[i][c].x, o.x); o.y = fmaf(w, v[i][c].y, o.y); o.z = fmaf(w, v[i][c].z, o.z); o.w = fmaf(w, v[i][c].w, o.w);
       }
-      if (tid == 0) {
-        p.ml[at * 2] = mm;
-        p.ml[at * 2 + 1] = sum;
-      }
+      *reinterpret_cast<float4*>(p.o + ((at0 + g) * p.parts + part) * p.wide + d) = o;
     }
   }
   if (p.cluster > 1) cluster_sync_all();   // staged accumulators stay until the others have read them
   else __syncthreads();
   if (warp == 4) {
     tcgen05_fence_after();
-    tmem_dealloc(tmem_s, kTmemCols);
+    tmem_dealloc(tmem_s, L::kTmemCols);
   }
 }
 
 int cluster_for(int max_blocks, int block_size) {
   const long long tiles = (static_cast<long long>(max_blocks) * block_size + kTile - 1) / kTile;
-  return tiles >= 8 ? 8 : (tiles >= 4 ? 4 : (tiles >= 2 ? 2 : 1));
+  return tiles >= 4 ? 4 : (tiles >= 2 ? 2 : 1);   // larger clusters leave too many SMs without a place for a whole one
 }
 
 template <typename T, int G>
@@ -368,7 +408,7 @@ int launch_tc(const ortb200_latent_decode_args& a, cudaStream_t stream) {
   p.boxes = p.wide_boxes + (a.width - a.wide + 63) / 64;
   p.cluster = cluster_for(a.max_blocks, a.block_size);
   p.block_size = a.block_size; p.max_blocks = a.max_blocks; p.num_blocks = a.num_blocks;
-  p.piece_rows = a.block_size < kTile ? a.block_size : kTile;
+  p.piece_rows = a.block_size < kGranule ? a.block_size : kGranule;
   p.scale_log2 = a.scale * 1.4426950408889634f;
   const int rot = a.width - a.wide;
   const int64_t rows = static_cast<int64_t>(a.num_blocks) * a.block_size, heads = static_cast<int64_t>(a.T) * a.N, pitch = static_cast<int64_t>(a.width) * 2;
@@ -381,7 +421,7 @@ int launch_tc(const ortb200_latent_decode_args& a, cudaStream_t stream) {
   if (rot > 0 && (make_tensor_map_2d(&tqr, q + static_cast<int64_t>(a.wide) * 2, dt, 2, rot, heads, pitch, 64, G) != 0 ||
                   make_tensor_map_2d(&tcr, c + static_cast<int64_t>(a.wide) * 2, dt, 2, rot, rows, pitch, 64, p.piece_rows) != 0))
     return -6;
-  const int need = L::bytes(p.boxes), smem = need > kMinSmem ? need : kMinSmem;
+  const int need = L::bytes(p.boxes), smem = need > L::kMinSmem ? need : L::kMinSmem;
   auto kern = latent_decode_tc_kernel<T, G>;
   static int attr_smem = 0;
   if (smem > attr_smem) {
@@ -417,13 +457,16 @@ bool sizes_fit(int N, int wide, int width, int block_size, int dtype) {
   return wide_boxes <= kMaxWideBoxes && boxes <= kMaxBoxes && (wide_boxes % 2 == 0 || boxes > wide_boxes);
 }
 
-int heads_per_cta(int N) { return N > 16 ? 32 : 16; }
+// Sixteen heads per CTA as long as the groups of a token run side by side, else 32: the cache is then read half as often.
+int heads_per_cta(int T, int N, int max_blocks, int block_size) {
+  return N > 16 && static_cast<long long>(T) * ((N + 15) / 16) * cluster_for(max_blocks, block_size) > 148 ? 32 : 16;
+}
 
 }  // namespace
 
 int launch_latent_decode_tc(const ortb200_latent_decode_args* a, cudaStream_t stream) {
   if (!sizes_fit(a->N, a->wide, a->width, a->block_size, a->dtype) || a->T > 65535) return -2;
-  const bool wide_group = heads_per_cta(a->N) == 32;
+  const bool wide_group = heads_per_cta(a->T, a->N, a->max_blocks, a->block_size) == 32;
   if (a->dtype == ORTB200_BF16) return wide_group ? launch_tc<__nv_bfloat16, 32>(*a, stream) : launch_tc<__nv_bfloat16, 16>(*a, stream);
   return wide_group ? launch_tc<__half, 32>(*a, stream) : launch_tc<__half, 16>(*a, stream);
 }
@@ -435,13 +478,13 @@ using namespace ortb200;
 extern "C" int ortb200_latent_decode_plan(int T, int N, int wide, int width, int block_size, int max_blocks, int dtype, int* parts) {
   if (parts) *parts = 1;
   if (T <= 0 || T > 65535 || max_blocks <= 0 || !sizes_fit(N, wide, width, block_size, dtype)) return 0;
-  // one resident CTA per SM; a part should have at least a tile per CTA when the cache is full
+  // one resident CTA per SM; a part should have at least half a tile per CTA when the cache is full
   const int cluster = cluster_for(max_blocks, block_size);
-  const int G = heads_per_cta(N);
+  const int G = heads_per_cta(T, N, max_blocks, block_size);
   const long long ctas = static_cast<long long>(T) * ((N + G - 1) / G) * cluster;
   long long n = 148 / ctas;
   const long long tiles = (static_cast<long long>(max_blocks) * block_size + kTile - 1) / kTile;
-  if (n > tiles / cluster) n = tiles / cluster;
+  if (n > 2 * tiles / cluster) n = 2 * tiles / cluster;
   if (n > 16) n = 16;
   if (parts && n > 1) *parts = static_cast<int>(n);
   return 1;

@@ -25,6 +25,7 @@ inline int launch_kernel(K kern, dim3 grid, int threads, int smem, cudaStream_t 
 
 // sequence of packed token t: the last b with cu_seqlens[b] <= t (empty sequences own no token)
 __device__ __forceinline__ int sequence_of(const int* cu, int B, int t) {
+  if (t < B && cu[t] == t && cu[t + 1] == t + 1) return t;   // one token per sequence: no chain of dependent loads
   int lo = 0, hi = B;
   while (hi - lo > 1) {
     const int mid = (lo + hi) >> 1;

@@ -387,8 +387,8 @@ typedef struct {
   const int* cu_seqlens;
   const int* past_seqlens;
   int T, block_size, max_blocks, num_blocks;
-  // Softmax weights enter the second product as the sum of two 16-bit terms instead of one (fp32-like weights for 1.5x
-  // the tensor-core work).
+  // Paged form: softmax weights enter the second product as the sum of two 16-bit terms instead of one (fp32-like weights
+  // for 1.5x the tensor-core work); no key_mask, no softcap.
   int split_weights;
   int chunk;               // > 0: a query sees only keys of its own chunk of this many positions (positions count from 0)
 } ortb200_attn_prefill_args;
