@@ -84,7 +84,7 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int, streams: i
         else:
             caches = [(torch.randn_like(kc), torch.randn_like(vc)) for _ in range(max(2, int(300e6 / (kc.numel() * 4))))]
             by = B * (context + 1) * kv * H * 4
-            us = graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, head_sink=sink, block_table=table, algo=1) for c in caches] * 2)
+            us = graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, head_sink=sink, block_table=table, split_weights=True) for c in caches] * 2)
             row("attention decode (fp32 weights)", "fegilix", us, by)
             us = graph_us([lambda c=c: K.gqa_decode(q.view(B, heads, H), c[0], c[1], past0, block_table=table, algo=2) for c in caches] * 2)
             row("attention decode", "llama", us, by)

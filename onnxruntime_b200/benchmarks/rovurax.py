@@ -86,7 +86,7 @@ def kernel_numbers(width: int, batch: int, prompt: int, context: int) -> List[Di
             caches = [(torch.randn_like(kc), torch.randn_like(vc)) for _ in range(max(2, int(300e6 / (kc.numel() * 4))))]
             for chunk in (CHUNK, 1 << 20):
                 seen = (context - 1) % chunk + 1
-                us = graph_us([lambda c=c: K.gqa_decode(q.view(B, N, H), c[0], c[1], past, block_table=table, algo=1, chunk=chunk) for c in caches] * 2)
+                us = graph_us([lambda c=c: K.gqa_decode(q.view(B, N, H), c[0], c[1], past, block_table=table, split_weights=True, chunk=chunk) for c in caches] * 2)
                 row(f"attention decode, {seen} keys", "rovurax", us, B * seen * kv * H * 4)
             us = graph_us([lambda c=c: K.gqa_decode(q.view(B, N, H), c[0], c[1], past, block_table=table, algo=2) for c in caches] * 2)
             row("attention decode", "llama", us, B * context * kv * H * 4)

@@ -389,7 +389,7 @@ class GatedPagedAttentionKernel final : public OpKernel {
         d.block_size = p.block_size;
         d.max_blocks = p.max_blocks;
         d.num_blocks = p.num_blocks;
-        d.algo = 1;  // softmax weights stay fp32 up to the product with V
+        d.split_weights = 1;
         d.chunk = static_cast<int>(chunk_);
         d.q_ld = q_ld;
         d.out_ld = o_ld;

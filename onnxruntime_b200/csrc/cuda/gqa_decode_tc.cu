@@ -13,6 +13,9 @@
 // every tile.  O^T stays in TMEM for the whole key range; at the end thread t reads dim t.  Splits are merged by the
 // last CTA to arrive, as in the CUDA-core kernel.
 //
+// SPLIT: the softmax weights stay 32-bit up to the product: 16 more rows of P hold what rounding leaves, their sums lie in 16
+// more columns of O^T and are added at the end (MMA 2 is bound by reading V, the columns are free).
+//
 // A paged cache is read through a tensor map over [slots, kv heads, dims]: a tile is fetched in pieces of
 // min(128, block_size) rows, one TMA per piece, each landing at its row offset inside the swizzled tile.
 //
@@ -38,7 +41,7 @@ constexpr int kBox = 128 * 128;            // [128 rows][64 elems] of 16-bit dat
 constexpr int kTileBytes = 2 * kBox;       // K or V tile: two boxes (dims 0-63, 64-127)
 constexpr int kStageBytes = 2 * kTileBytes;
 constexpr int kQBox = 16 * 128;            // [16 heads][64 dims]
-constexpr int kPBox = 16 * 128;            // [16 heads][64 keys]
+constexpr int kPBox = 32 * 128;            // [16 heads, 16 remainders (SPLIT)][64 keys]
 constexpr int kOffQ = kStages * kStageBytes;
 constexpr int kOffP = kOffQ + 2 * kQBox;
 constexpr int kOffMax = kOffP + 2 * 2 * kPBox;      // float [2][4][16]
@@ -48,7 +51,7 @@ constexpr int kOffNew = kOffXch + 17 * 128 * 4;      // float [16]: scores of th
 constexpr int kOffBar = kOffNew + 16 * 4;
 constexpr int kSmemBytes = kOffBar + 256 + 1024;
 constexpr int kThreads = 160;              // 4 softmax warps + 1 TMA / MMA warp
-constexpr int kTmemCols = 64;              // S^T buffers at columns 0 and 16, O^T at 32
+constexpr int kTmemCols = 64;              // S^T buffers at columns 0 and 16, O^T at 32, its remainders at 48
 constexpr float kRaise = 8.f;              // raise the reference maximum only past 2^8
 
 enum { BAR_Q = 0, BAR_FULL0, BAR_EMPTY0 = BAR_FULL0 + kStages, BAR_S0 = BAR_EMPTY0 + kStages, BAR_S1, BAR_P0, BAR_P1, BAR_O,
@@ -75,7 +78,7 @@ __device__ __forceinline__ void tmem_ld_heads(uint32_t taddr, float* v) {
   tmem_ld_wait();
 }
 
-template <typename T, int G, bool PAGED>
+template <typename T, int G, bool PAGED, bool SPLIT>
 __global__ void __launch_bounds__(kThreads, 1)
 gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_v, const DecodeParams p, const int piece_rows) {
@@ -126,10 +129,12 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (threadIdx.x == 0 && p.status) atomicExch(p.status, kStatusBadLength);
     total = total < 0 ? 0 : p.Smax;
   }
-  const int start0 = p.window > 0 ? max(0, total - p.window) : 0;
+  int first_key = p.window > 0 ? max(0, total - p.window) : 0;
+  if (p.chunk > 0) first_key = max(first_key, (total - 1) / p.chunk * p.chunk);
+  const int start0 = PAGED ? first_key / piece_rows * piece_rows : first_key;   // tiles start on piece boundaries
   const int len = max(total - start0, 0);
   int chunk = (len + p.splits - 1) / p.splits;
-  if (PAGED) chunk = (chunk + kTile - 1) / kTile * kTile;   // tiles start on piece boundaries (start0 is 0 when paged)
+  if (PAGED) chunk = (chunk + kTile - 1) / kTile * kTile;
   const int k_begin = start0 + split * chunk;
   // fused: the newest key (position total - 1) is not in the cache yet; the CTA whose range reaches it takes it
   const bool owns_new = fused && k_begin < total && k_begin + chunk >= total;
@@ -151,7 +156,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     // ------------------------------------------------------------ TMA producer + MMA issuer (lane 0 issues; with a
     // paged cache lane i fetches piece i of a tile)
     const uint32_t idesc_s = umma_idesc_f16(kBf16, kTile, 16);
-    const uint32_t idesc_o = umma_idesc_f16(kBf16, H, 16) | (1u << 15);   // A (= V^T) is MN-major
+    const uint32_t idesc_o = umma_idesc_f16(kBf16, H, SPLIT ? 32 : 16) | (1u << 15);   // A (= V^T) is MN-major
     const uint32_t q_addr = smem_u32(smem + kOffQ);
     const int pieces = PAGED ? kTile / piece_rows : 1;
     auto load_tile = [&](int t) {
@@ -203,8 +208,8 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (n_tiles > 0) {
       if (lane == 0 && !fused) {
         mbar_expect_tx(&bars[BAR_Q], 2 * kQBox);
-        tma_load_2d(smem + kOffQ, &tm_q, &bars[BAR_Q], 0, b * p.N + head0);
-        tma_load_2d(smem + kOffQ + kQBox, &tm_q, &bars[BAR_Q], 64, b * p.N + head0);
+        tma_load_3d(smem + kOffQ, &tm_q, &bars[BAR_Q], 0, head0, b);
+        tma_load_3d(smem + kOffQ + kQBox, &tm_q, &bars[BAR_Q], 64, head0, b);
       }
       const int pre = n_tiles < kStages ? n_tiles : kStages;
       for (int t = 0; t < pre; ++t) load_tile(t);
@@ -341,7 +346,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       float sv[GV];
       tmem_ld_heads<G>(tmem_base + lane_addr + (t & 1) * 16, sv);
       const int key = k_begin + t * kTile + tid;
-      const bool valid = key < k_end;
+      const bool valid = key < k_end && key >= first_key;
       float* mx = sm_max + (t & 1) * 64;
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -378,18 +383,27 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           for (int g = 0; g < G; ++g) ov[g] *= corr[g];
 #pragma unroll
           for (int c = 0; c < GV / 8; ++c) tmem_st_x8(tmem_o + lane_addr + c * 8, ov + c * 8);
+          if (SPLIT) {
+            tmem_ld_heads<G>(tmem_o + 16 + lane_addr, ov);
+#pragma unroll
+            for (int g = 0; g < G; ++g) ov[g] *= corr[g];
+#pragma unroll
+            for (int c = 0; c < GV / 8; ++c) tmem_st_x8(tmem_o + 16 + lane_addr + c * 8, ov + c * 8);
+          }
           tmem_st_wait();
         }
       }
-      // probabilities of this key for every head, rounded to the MMA input type (the sum uses the rounded values)
+      // probabilities of this key for every head, rounded to the MMA input type (the sum uses what enters MMA 2)
       uint8_t* pb = smem + kOffP + (t & 1) * 2 * kPBox + (tid >> 6) * kPBox;
       const int col = tid & 63;
 #pragma unroll
       for (int g = 0; g < G; ++g) {
         const float pr = valid ? exp2f(sv[g] - m_ref[g]) : 0.f;
         const T pt = from_float<T>(pr);
-        l_part[g] += to_float<T>(pt);
-        *reinterpret_cast<T*>(pb + g * 128 + (((col >> 3) ^ (g & 7)) << 4) + (col & 7) * 2) = pt;
+        l_part[g] += SPLIT ? pr : to_float<T>(pt);
+        uint8_t* dst = pb + g * 128 + (((col >> 3) ^ (g & 7)) << 4) + (col & 7) * 2;
+        *reinterpret_cast<T*>(dst) = pt;
+        if (SPLIT) *reinterpret_cast<T*>(dst + 16 * 128) = from_float<T>(pr - to_float<T>(pt));
       }
       if (k_begin + (t + 1) * kTile > k_end) {
         // last, partial tile: rows past the range hold whatever the cache (or an earlier tile) left there; a
@@ -431,7 +445,15 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   float ov[GV];
 #pragma unroll
   for (int g = 0; g < GV; ++g) ov[g] = 0.f;
-  if (warp < 4 && ok && n_tiles > 0) tmem_ld_heads<G>(tmem_o + (static_cast<uint32_t>(warp * 32) << 16), ov);
+  if (warp < 4 && ok && n_tiles > 0) {
+    tmem_ld_heads<G>(tmem_o + (static_cast<uint32_t>(warp * 32) << 16), ov);
+    if (SPLIT) {
+      float rest[GV];
+      tmem_ld_heads<G>(tmem_o + 16 + (static_cast<uint32_t>(warp * 32) << 16), rest);
+#pragma unroll
+      for (int g = 0; g < G; ++g) ov[g] += rest[g];
+    }
+  }
   tcgen05_fence_before();
   __syncthreads();
   if (warp < 4 && tid == 0) {
@@ -469,10 +491,10 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   decode_finish<T, H, G>(p, tile, split, b, head0, n_heads, tid, fm, fl, fa, &sm_last);
 }
 
-template <typename T, int G, bool PAGED>
+template <typename T, int G, bool PAGED, bool SPLIT>
 int launch_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const DecodeParams& p, int piece_rows,
               dim3 grid, cudaStream_t stream, bool use_pdl) {
-  auto kern = gqa_decode_tc_kernel<T, G, PAGED>;
+  auto kern = gqa_decode_tc_kernel<T, G, PAGED, SPLIT>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) != cudaSuccess) return -10;
@@ -493,12 +515,12 @@ int launch_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& t
   return cudaLaunchKernelEx(&cfg, kern, tq, tk, tv, p, piece_rows) == cudaSuccess ? 0 : -11;
 }
 
-template <typename T, bool PAGED>
+template <typename T, bool PAGED, bool SPLIT>
 int launch_tc_g(int group, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const DecodeParams& p,
                 int piece_rows, dim3 grid, cudaStream_t stream, bool use_pdl) {
-  if (group <= 4) return launch_tc<T, 4, PAGED>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
-  if (group <= 8) return launch_tc<T, 8, PAGED>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
-  return launch_tc<T, 16, PAGED>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
+  if (group <= 4) return launch_tc<T, 4, PAGED, SPLIT>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
+  if (group <= 8) return launch_tc<T, 8, PAGED, SPLIT>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
+  return launch_tc<T, 16, PAGED, SPLIT>(tq, tk, tv, p, piece_rows, grid, stream, use_pdl);
 }
 
 }  // namespace
@@ -506,7 +528,8 @@ int launch_tc_g(int group, const CUtensorMap& tq, const CUtensorMap& tk, const C
 bool gqa_decode_tc_supported(const ortb200_gqa_decode_args* a) {
   if (a->H != 128 || (a->dtype != ORTB200_BF16 && a->dtype != ORTB200_F16)) return false;
   if (a->qkv == nullptr && a->q == nullptr) return false;
-  if (a->chunk > 0 || a->q_ld > 0 || a->out_ld > 0) return false;
+  if ((a->split_weights || a->chunk > 0) && !a->block_table) return false;
+  if (a->qkv == nullptr && a->q_ld % 8) return false;
   if (a->qkv != nullptr && (reinterpret_cast<uintptr_t>(a->qkv) & 15)) return false;
   const int group = a->N / a->Nk;
   if (group > 16 || !a->workspace) return false;
@@ -528,7 +551,8 @@ int launch_gqa_decode_tc(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   if (splits <= 0) {
     // One CTA per SM at most.  Merging splits costs about as much as four tiles, so a grid that already covers a
     // good part of the machine with short key ranges is not split; otherwise at least two tiles per split.
-    const int tiles = (a->Smax + kTile - 1) / kTile;
+    // a chunk may begin within a tile
+    const int tiles = a->chunk > 0 && a->chunk < a->Smax - kTile ? (a->chunk + kTile - 1) / kTile + 1 : (a->Smax + kTile - 1) / kTile;
     if (base >= 32 && tiles <= 12) {
       splits = 1;
     } else {
@@ -546,7 +570,8 @@ int launch_gqa_decode_tc(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   CUtensorMap tq, tk, tv;
   // fused launches build the query tile themselves; the map then only has to be a valid one
   const void* q_base = a->qkv != nullptr ? a->k_cache : a->q;
-  if (make_tensor_map_2d(&tq, q_base, dt, 2, H, static_cast<int64_t>(a->B) * a->N, H * 2, 64, 16) != 0) return -5;
+  const int64_t q_ld = a->qkv == nullptr && a->q_ld > 0 ? a->q_ld : static_cast<int64_t>(a->N) * H;
+  if (make_tensor_map_3d(&tq, q_base, dt, 2, H, a->N, a->B, H * 2, q_ld * 2, 64, 16) != 0) return -5;
   int piece_rows = kTile;
   if (a->block_table) {
     piece_rows = a->block_size < kTile ? a->block_size : kTile;
@@ -574,7 +599,9 @@ int launch_gqa_decode_tc(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   p.qkv = a->qkv; p.cos_cache = a->cos_cache; p.sin_cache = a->sin_cache; p.cos_rows = a->cos_rows;
   p.do_rotary = a->do_rotary; p.interleaved = a->rotary_interleaved;
   dim3 grid(splits, a->Nk, a->B);
-  p.q_ld = p.out_ld = static_cast<long long>(a->N) * H;
+  p.chunk = a->chunk;
+  p.q_ld = q_ld;
+  p.out_ld = a->out_ld > 0 ? a->out_ld : static_cast<long long>(a->N) * H;
   p.prefetch = nullptr; p.prefetch_bytes = 0; p.prefetch_per_cta = 0;
   if (a->prefetch != nullptr && a->prefetch_bytes >= 16 && (reinterpret_cast<uintptr_t>(a->prefetch) & 15) == 0) {
     const long long bytes = (a->prefetch_bytes < (48LL << 20) ? a->prefetch_bytes : (48LL << 20)) & ~15LL;
@@ -585,11 +612,13 @@ int launch_gqa_decode_tc(const ortb200_gqa_decode_args* a, cudaStream_t stream) 
   }
   const bool pdl = a->use_pdl != 0;
   if (a->dtype == ORTB200_BF16) {
-    return a->block_table ? launch_tc_g<__nv_bfloat16, true>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl)
-                          : launch_tc_g<__nv_bfloat16, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
+    if (a->split_weights) return launch_tc_g<__nv_bfloat16, true, true>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
+    return a->block_table ? launch_tc_g<__nv_bfloat16, true, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl)
+                          : launch_tc_g<__nv_bfloat16, false, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
   }
-  return a->block_table ? launch_tc_g<__half, true>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl)
-                        : launch_tc_g<__half, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
+  if (a->split_weights) return launch_tc_g<__half, true, true>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
+  return a->block_table ? launch_tc_g<__half, true, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl)
+                        : launch_tc_g<__half, false, false>(group, tq, tk, tv, p, piece_rows, grid, stream, pdl);
 }
 
 }  // namespace ortb200

@@ -34,7 +34,7 @@ struct DecodeParams {
   const unsigned char* prefetch;
   long long prefetch_bytes;
   int prefetch_per_cta;
-  int chunk;               // CUDA-core kernel: > 0 = keys of the new token's own chunk only
+  int chunk;               // > 0: keys of the new token's own chunk only
   long long q_ld, out_ld;  // elements between the rows of q and of out
 };
 

@@ -344,10 +344,12 @@ typedef struct {
   const void* prefetch;
   int64_t prefetch_bytes;
   int cos_rows;           // rows of cos_cache / sin_cache; the rotary position is clamped to it (0 = not checked)
-  // CUDA-core kernel only: attend within chunks of this many positions (the new token sees its own chunk; <= 0: none), and
-  // elements between the rows of q and of out (0 = N H)
+  // Attend within chunks of this many positions (the new token sees its own chunk; <= 0: none); elements between the rows
+  // of q and of out (0 = N H); softmax weights that stay 32-bit up to the product with V (always so in the CUDA-core kernel).
+  // The tcgen05 kernel takes chunks and 32-bit weights over paged caches.
   int chunk;
   int64_t q_ld, out_ld;
+  int split_weights;
 } ortb200_gqa_decode_args;
 int ortb200_gqa_decode(const ortb200_gqa_decode_args* args, ortb200_stream_t stream);
 int64_t ortb200_gqa_decode_workspace_bytes(int B, int N, int H);

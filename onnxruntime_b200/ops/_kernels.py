@@ -247,14 +247,16 @@ class GqaDecodeArgs(ctypes.Structure):
                 ("block_size", ctypes.c_int), ("max_blocks", ctypes.c_int), ("qkv", ctypes.c_void_p), ("cos_cache", ctypes.c_void_p),
                 ("sin_cache", ctypes.c_void_p), ("do_rotary", ctypes.c_int), ("rotary_interleaved", ctypes.c_int),
                 ("num_blocks", ctypes.c_int), ("algo", ctypes.c_int), ("prefetch", ctypes.c_void_p), ("prefetch_bytes", ctypes.c_int64),
-                ("cos_rows", ctypes.c_int), ("chunk", ctypes.c_int), ("q_ld", ctypes.c_int64), ("out_ld", ctypes.c_int64)]
+                ("cos_rows", ctypes.c_int), ("chunk", ctypes.c_int), ("q_ld", ctypes.c_int64), ("out_ld", ctypes.c_int64),
+                ("split_weights", ctypes.c_int)]
 
 
 _ATTN_WS = {}
 
 
 def gqa_decode(q, k_cache, v_cache, seqlens_k, splits=0, window=-1, scale=0.0, softcap=0.0, head_sink=None, block_table=None,
-               qkv=None, num_heads=0, cos=None, sin=None, interleaved=False, algo=0, prefetch=None, chunk=0):
+               qkv=None, num_heads=0, cos=None, sin=None, interleaved=False, algo=0, prefetch=None, chunk=0,
+               split_weights=False):
     """Dense cache [B,Nk,Smax,H]; or, with block_table [B,max_blocks] int32, a paged cache [num_blocks,block_size,Nk,H].
     With ``qkv`` (packed [B,(N+2Nk)H], ``num_heads`` = N) the kernel also rotates q / k and appends k / v itself.
     ``algo``: 0 = pick, 1 = CUDA-core split-KV kernel, 2 = tcgen05 kernel (head size 128, 16-bit types)."""
@@ -284,7 +286,8 @@ def gqa_decode(q, k_cache, v_cache, seqlens_k, splits=0, window=-1, scale=0.0, s
                       _ptr(block_table), block_size, max_blocks, _ptr(qkv), _ptr(cos), _ptr(sin), 0 if cos is None else 1,
                       1 if interleaved else 0, num_blocks, algo, _ptr(prefetch),
                       prefetch.numel() * prefetch.element_size() if prefetch is not None else 0,
-                      0 if cos is None else cos.shape[0], chunk, 0, 0)
+                      0 if cos is None else cos.shape[0], chunk, 0, 0,
+                      1 if split_weights else 0)
     _check(lib().ortb200_gqa_decode(ctypes.byref(a), ctypes.c_void_p(stream_ptr())), "ortb200_gqa_decode")
     return out
 
