@@ -48,7 +48,7 @@ struct Smem {
 };
 
 enum { BAR_Q = 0, BAR_K_FULL, BAR_K_EMPTY = BAR_K_FULL + 2, BAR_V_FULL = BAR_K_EMPTY + 2, BAR_V_EMPTY = BAR_V_FULL + 2, BAR_S = BAR_V_EMPTY + 2,
-       BAR_P = BAR_S + 2, BAR_O = BAR_P + 2, BAR_COUNT };
+       BAR_P = BAR_S + 2, BAR_O = BAR_P + 2, BAR_END, BAR_COUNT };
 
 template <int KB, int VB, int STAGES, bool LATENT>
 __global__ void __launch_bounds__(kThreads, 2)
@@ -183,6 +183,7 @@ attn_split_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         }
         umma_commit(&bars[BAR_O]);
         umma_commit(&bars[BAR_V_EMPTY + s]);
+        if (t == n_tiles - 1) umma_commit(&bars[BAR_END]);
       }
       if (!ok && p.status) atomicExch(p.status, kStatusTimeoutMma);
     }
@@ -195,6 +196,7 @@ attn_split_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t) {
+      // S of this tile was issued after the product of tile t - 2 had finished: BAR_O is at most one phase back below
       if (ok && !mbar_wait(&bars[BAR_S + (t & 1)], (t >> 1) & 1)) ok = false;
       tcgen05_fence_after();
       const int key0 = kv_begin + t * kKT;
@@ -266,7 +268,8 @@ attn_split_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       tcgen05_fence_before();
       mbar_arrive(&bars[BAR_P + (t & 1)]);
     }
-    if (n_tiles > 0 && ok && !mbar_wait(&bars[BAR_O], (n_tiles - 1) & 1)) ok = false;
+    // (BAR_O may still be two phases back here, where its parity would already read as done)
+    if (n_tiles > 0 && ok && !mbar_wait(&bars[BAR_END], 0)) ok = false;
     tcgen05_fence_after();
     if (!ok && p.status) atomicExch(p.status, kStatusTimeoutEpilogue);
     pdl_launch_dependents();

@@ -55,7 +55,7 @@ constexpr int kTmemCols = 64;              // S^T buffers at columns 0 and 16, O
 constexpr float kRaise = 8.f;              // raise the reference maximum only past 2^8
 
 enum { BAR_Q = 0, BAR_FULL0, BAR_EMPTY0 = BAR_FULL0 + kStages, BAR_S0 = BAR_EMPTY0 + kStages, BAR_S1, BAR_P0, BAR_P1, BAR_O,
-       BAR_COUNT };
+       BAR_END, BAR_COUNT };
 
 __device__ __forceinline__ float redux_max(float v) {
   float r;
@@ -240,6 +240,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           }
           umma_commit(&bars[BAR_EMPTY0 + s]);
           umma_commit(&bars[BAR_O]);
+          if (t == n_tiles - 1) umma_commit(&bars[BAR_END]);
         }
         __syncwarp();
         if (t + kStages < n_tiles) {
@@ -436,7 +437,8 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (warp < 4 && lane == 0) sm_sum[warp * 16 + g] = ws;
   }
   if (warp < 4 && ok && n_tiles > 0) {
-    if (!mbar_wait(&bars[BAR_O], (n_tiles - 1) & 1)) {
+    // a barrier of its own: the product of tile n - 2 may still run, and BAR_O's parity would then read as done
+    if (!mbar_wait(&bars[BAR_END], 0)) {
       ok = false;
       if (p.status) atomicExch(p.status, kStatusTimeoutEpilogue);
     }
