@@ -107,10 +107,12 @@ def write_ninja(kernels_only: bool = False, c_api: bool = True) -> str:
             "  description = LINK $out",
         ]
         cobjs = []
+        # named here too: objects that came without the compiler's dependency records follow their headers all the same
+        core_hdrs = sorted(glob.glob(os.path.join(CSRC, "core", "*.h"))) + [os.path.join(CSRC, "cuda", "ortb200_kernels.h")]
         for src in cpp_srcs:
             obj = os.path.join(BUILD, "core_" + os.path.basename(src)[:-3] + ".o")
             cobjs.append(obj)
-            lines.append(f"build {obj}: cxx {src}")
+            lines.append(f"build {obj}: cxx {src} | " + " ".join(core_hdrs))
         core_so = os.path.join(HERE, core_ext_name())
         lines.append(f"build {core_so}: cxxlink " + " ".join(cobjs) + f" | {kern_so}")
         defaults.append(core_so)

@@ -41,15 +41,18 @@ constexpr int kBox = 128 * 128;            // [128 rows][64 elems] of 16-bit dat
 constexpr int kTileBytes = 2 * kBox;       // K or V tile: two boxes (dims 0-63, 64-127)
 constexpr int kStageBytes = 2 * kTileBytes;
 constexpr int kQBox = 16 * 128;            // [16 heads][64 dims]
-constexpr int kPBox = 32 * 128;            // [16 heads, 16 remainders (SPLIT)][64 keys]
 constexpr int kOffQ = kStages * kStageBytes;
 constexpr int kOffP = kOffQ + 2 * kQBox;
-constexpr int kOffMax = kOffP + 2 * 2 * kPBox;      // float [2][4][16]
-constexpr int kOffSum = kOffMax + 2 * 4 * 16 * 4;   // float [4][16]
-constexpr int kOffXch = kOffSum + 4 * 16 * 4;        // float [17][128]: q heads and the new key, for the rotary partner
-constexpr int kOffNew = kOffXch + 17 * 128 * 4;      // float [16]: scores of the new key
-constexpr int kOffBar = kOffNew + 16 * 4;
-constexpr int kSmemBytes = kOffBar + 256 + 1024;
+template <bool SPLIT>
+struct Smem {
+  static constexpr int kPBox = (SPLIT ? 32 : 16) * 128;       // [16 heads, 16 remainders (SPLIT)][64 keys]
+  static constexpr int kOffMax = kOffP + 2 * 2 * kPBox;       // float [2][4][16]
+  static constexpr int kOffSum = kOffMax + 2 * 4 * 16 * 4;    // float [4][16]
+  static constexpr int kOffXch = kOffSum + 4 * 16 * 4;        // float [17][128]: q heads and the new key, for the rotary partner
+  static constexpr int kOffNew = kOffXch + 17 * 128 * 4;      // float [16]: scores of the new key
+  static constexpr int kOffBar = kOffNew + 16 * 4;
+  static constexpr int kBytes = kOffBar + 256 + 1024;
+};
 constexpr int kThreads = 160;              // 4 softmax warps + 1 TMA / MMA warp
 constexpr int kTmemCols = 64;              // S^T buffers at columns 0 and 16, O^T at 32, its remainders at 48
 constexpr float kRaise = 8.f;              // raise the reference maximum only past 2^8
@@ -82,17 +85,18 @@ template <typename T, int G, bool PAGED, bool SPLIT>
 __global__ void __launch_bounds__(kThreads, 1)
 gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_v, const DecodeParams p, const int piece_rows) {
+  using L = Smem<SPLIT>;
   constexpr int H = 128;
   constexpr int GV = (G + 7) / 8 * 8;   // columns fetched from tensor memory
   constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kOffBar);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::kOffBar);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + BAR_COUNT);
-  float* sm_max = reinterpret_cast<float*>(smem + kOffMax);
-  float* sm_sum = reinterpret_cast<float*>(smem + kOffSum);
-  float* sm_xch = reinterpret_cast<float*>(smem + kOffXch);
-  float* sm_new = reinterpret_cast<float*>(smem + kOffNew);
+  float* sm_max = reinterpret_cast<float*>(smem + L::kOffMax);
+  float* sm_sum = reinterpret_cast<float*>(smem + L::kOffSum);
+  float* sm_xch = reinterpret_cast<float*>(smem + L::kOffXch);
+  float* sm_new = reinterpret_cast<float*>(smem + L::kOffNew);
   __shared__ unsigned int sm_last;
   // Fused step 1 (one new token per sequence): q, k and v come from the packed projection output; this kernel
   // rotates q and k, writes the query tile itself, appends k / v to the cache and attends to the new key from
@@ -232,11 +236,11 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         if (lane == 0) {
           tcgen05_fence_after();
           const uint32_t v_addr = smem_u32(smem + s * kStageBytes + kTileBytes);
-          const uint32_t p_addr = smem_u32(smem + kOffP + (t & 1) * 2 * kPBox);
+          const uint32_t p_addr = smem_u32(smem + kOffP + (t & 1) * 2 * L::kPBox);
 #pragma unroll
           for (int kk = 0; kk < kTile / 16; ++kk) {
             umma_f16(tmem_o, umma_desc_mn_sw128(v_addr + kk * 2048, kBox, 1024),
-                     umma_desc_sw128(p_addr + (kk / 4) * kPBox + (kk % 4) * 32), idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
+                     umma_desc_sw128(p_addr + (kk / 4) * L::kPBox + (kk % 4) * 32), idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
           }
           umma_commit(&bars[BAR_EMPTY0 + s]);
           umma_commit(&bars[BAR_O]);
@@ -395,7 +399,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         }
       }
       // probabilities of this key for every head, rounded to the MMA input type (the sum uses what enters MMA 2)
-      uint8_t* pb = smem + kOffP + (t & 1) * 2 * kPBox + (tid >> 6) * kPBox;
+      uint8_t* pb = smem + kOffP + (t & 1) * 2 * L::kPBox + (tid >> 6) * L::kPBox;
       const int col = tid & 63;
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -499,13 +503,13 @@ int launch_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& t
   auto kern = gqa_decode_tc_kernel<T, G, PAGED, SPLIT>;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) != cudaSuccess) return -10;
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<SPLIT>::kBytes) != cudaSuccess) return -10;
     attr_set = true;
   }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = dim3(kThreads, 1, 1);
-  cfg.dynamicSmemBytes = kSmemBytes;
+  cfg.dynamicSmemBytes = Smem<SPLIT>::kBytes;
   cfg.stream = stream;
   cudaLaunchAttribute attrs[1];
   if (use_pdl) {

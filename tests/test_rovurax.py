@@ -635,3 +635,108 @@ def test_the_cases_show_mistakes(mistake, monkeypatch):
         monkeypatch.setattr(oracle, "dense_ff", lambda h, w_, p, limit: 0.9 * h)
     wrong = oracle.forward(cfg, w, toks)
     assert packed_decoder.relative_error(wrong - right, right).max() > 1e-2
+
+
+# ------------------------------------------------------------------------------------------------------- kernels alone
+def rounded_close(got, want, tol=1e-4):
+    """Equal up to rounding the result to bfloat16 and ``tol``: softmax weights in 16 bits would be a hundred times further off."""
+    assert ((got.double() - want).abs() - 2.0 ** -8 * want.abs()).max() < tol
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("N,G,chunk", [(4, 4, 0), (8, 2, 0), (16, 1, 100), (6, 2, 1), (8, 1, 300), (12, 4, 128)])
+def test_decode_attention_keeps_its_weights(N, G, chunk):
+    """Tensor-core decode kernel over a scattered paged cache: 32-bit weights, chunks that begin inside a tile."""
+    from onnxruntime_b200.ops import _kernels as K
+    g = torch.Generator().manual_seed(N)
+    H, bs, lens = 128, 128, [1, 100, 101, 128, 129, 300, 301, 500, 777]
+    B, per = len(lens), 7
+    table = torch.randperm(B * per, generator=g).to(torch.int32).reshape(B, per)
+    kc, vc = [torch.randn(B * per, bs, G, H, generator=g).to(torch.bfloat16) for _ in range(2)]
+    q = torch.randn(B, N, H, generator=g).to(torch.bfloat16)
+    past = i32(*[n - 1 for n in lens])
+    out = [K.gqa_decode(q.cuda(), kc.cuda(), vc.cuda(), past.cuda(), block_table=table.cuda(), split_weights=True, chunk=chunk, scale=0.2, algo=2).cpu()
+           for _ in range(3)]
+    assert torch.equal(out[0], out[1]) and torch.equal(out[0], out[2])
+    for b, n in enumerate(lens):
+        lo = (n - 1) // chunk * chunk if chunk else 0
+        k, v = [c[table[b].long()].reshape(per * bs, G, H)[lo:n].double().repeat_interleave(N // G, 1) for c in (kc, vc)]
+        s = torch.einsum("hd,lhd->hl", q[b].double(), k)[:, None] * 0.2
+        w = oracle.visible_softmax(s, torch.ones(1, n - lo, dtype=torch.bool))
+        rounded_close(out[0][b].reshape(N, H), torch.einsum("htl,lhv->hv", w, v))
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,chunk", [(64, 0), (128, 0), (128, 100)])
+def test_prompt_attention_is_repeatable(H, chunk):
+    """The same launch many times, on a machine full of other blocks: bit-equal, and right."""
+    from onnxruntime_b200.ops import _kernels as K
+    g = torch.Generator().manual_seed(H)
+    N, G, bs, lens, past = 8, 2, 128, [700, 130, 1, 500], [0, 300, 77, 900]
+    per = max(-(-(p + n) // bs) for p, n in zip(past, lens))
+    table = torch.randperm(4 * per, generator=g).to(torch.int32).reshape(4, per)
+    kc, vc = [torch.randn(4 * per, bs, G, H, generator=g).to(torch.bfloat16) for _ in range(2)]
+    q = torch.randn(sum(lens), N, H, generator=g).to(torch.bfloat16)
+    cu = i32(0, *torch.tensor(lens).cumsum(0).tolist()).cuda()
+    args = [q.cuda(), kc.cuda(), vc.cuda(), cu, i32(*past).cuda(), table.cuda()]
+    out = K.attn_prefill_paged(*args, scale=0.2, split_weights=True, chunk=chunk)
+    for _ in range(40):
+        assert torch.equal(K.attn_prefill_paged(*args, scale=0.2, split_weights=True, chunk=chunk), out)
+    out, at = out.cpu(), 0
+    for b, n in enumerate(lens):
+        total = past[b] + n
+        k, v = [c[table[b].long()].reshape(per * bs, G, H)[:total].double().repeat_interleave(N // G, 1) for c in (kc, vc)]
+        mask = (oracle.chunk_mask(total, chunk) if chunk else oracle.causal_mask(total))[past[b]:]
+        w = oracle.visible_softmax(torch.einsum("thd,lhd->htl", q[at:at + n].double(), k) * 0.2, mask)
+        rounded_close(out[at:at + n], torch.einsum("htl,lhv->thv", w, v))
+        at += n
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dk,dr,dv", [(32, 16, 32), (128, 64, 128), (64, 64, 128), (72, 8, 40)])
+def test_latent_prompt_kernel_is_repeatable(dk, dr, dv):
+    from onnxruntime_b200.ops import _kernels as K
+    g = torch.Generator().manual_seed(dk)
+    N, lens, past = 6, [300, 1, 600], [200, 5, 0]
+    T, rows, cols = sum(lens), sum(lens) + sum(past), N * (dk + dr) + N
+    rand = lambda *s: torch.randn(*s, generator=g).to(torch.bfloat16)
+    x, q_rot, kv, kr, sink = rand(T, cols + -cols % 8), rand(T, N, dr), rand(rows, N * (dk + dv)), rand(rows, dr + -dr % 8), rand(N)
+    dev = [t.cuda() for t in (x, q_rot, kv, kr, sink)]
+    cu = i32(0, *torch.tensor(lens).cumsum(0).tolist()).cuda()
+    run = lambda: K.latent_prefill(dev[0], dev[1], dev[2], dev[3], dev[4], dev[0][:, cols - N:], cu, i32(*past).cuda(), N, dk, dr, dv, 0.15)
+    out = run()
+    for _ in range(40):
+        assert torch.equal(run(), out)
+    out, at, k0 = out.cpu(), 0, 0
+    for b, n in enumerate(lens):
+        total = past[b] + n
+        q = torch.cat([x[at:at + n, :N * (dk + dr)].reshape(n, N, dk + dr)[..., :dk], q_rot[at:at + n]], -1).double()
+        k = torch.cat([kv[k0:k0 + total, :N * dk].reshape(total, N, dk), kr[k0:k0 + total, None, :dr].expand(total, N, dr)], -1).double()
+        v = kv[k0:k0 + total, N * dk:].reshape(total, N, dv).double()
+        w = oracle.visible_softmax(torch.einsum("thd,lhd->htl", q, k) * 0.15, oracle.causal_mask(total)[past[b]:], sink.double())
+        ref = torch.einsum("htl,lhv->thv", w, v) * torch.sigmoid(x[at:at + n, cols - N:cols].double())[:, :, None]
+        rounded_close(out[at:at + n].reshape(n, N, dv), ref, 2e-4)
+        at, k0 = at + n, k0 + total
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("N,rank,dr,bs", [(16, 512, 64, 128), (40, 136, 16, 64), (3, 64, 8, 8)])
+def test_latent_decode_kernel_is_repeatable(N, rank, dr, bs):
+    from onnxruntime_b200.ops import _kernels as K
+    g = torch.Generator().manual_seed(N)
+    lens = [900, 33, 1, 129, 640]
+    B, per = len(lens), -(-900 // bs)
+    table = torch.randperm(B * per, generator=g).to(torch.int32).reshape(B, per)
+    cache = torch.randn(B * per, bs, rank + dr, generator=g).to(torch.bfloat16)
+    q = (0.3 * torch.randn(B, N, rank + dr, generator=g)).to(torch.bfloat16)
+    args = [q.cuda(), cache.cuda(), torch.arange(B + 1, dtype=torch.int32).cuda(), i32(*[n - 1 for n in lens]).cuda(), table.cuda(), rank, 0.3]
+    o, ml = K.latent_decode(*args)
+    for _ in range(40):
+        again = K.latent_decode(*args)
+        assert torch.equal(again[0], o) and torch.equal(again[1], ml)
+    for b, n in enumerate(lens):
+        c = cache[table[b].long()].reshape(per * bs, -1)[:n].double()
+        want = oracle.visible_softmax((q[b].double() @ c.T)[:, None] * 0.3, torch.ones(1, n, dtype=torch.bool))[:, 0] @ c[:, :rank]
+        f = torch.exp2(ml[b, :, :, 0] - ml[b, :, :, 0].max(1, keepdim=True).values)
+        got = (f[..., None] * o[b]).sum(1) / (f * ml[b, :, :, 1]).sum(1, keepdim=True)
+        assert (got.double().cpu() - want).abs().max() < 1e-4
