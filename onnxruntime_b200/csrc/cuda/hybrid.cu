@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(256) softcap_kernel(const T* __restrict__ x, f
 
 // -------------------------------------------------------------------------------------------- norm + rotary + append
 template <typename T>
-__global__ void __launch_bounds__(256) qk_norm_rope_kernel(const ortb200_qk_norm_rope_args a) {
+__global__ void __launch_bounds__(256, 6) qk_norm_rope_kernel(const ortb200_qk_norm_rope_args a) {
   __shared__ float head[8][kMaxHead];
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
