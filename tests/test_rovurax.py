@@ -306,7 +306,7 @@ def test_latent_kernels_take_the_tensor_cores():
     import ctypes
     from onnxruntime_b200.ops import _kernels as K
     f = K.lib().ortb200_latent_prefill_supported
-    assert f(128, 64, 128, 1) and f(32, 32, 32, 1) and not f(30, 32, 32, 1) and not f(192, 64, 128, 1) and not f(64, 64, 64, 2)
+    assert f(128, 64, 128, 1) and f(40, 24, 56, 1) and not f(30, 24, 56, 1) and not f(192, 64, 128, 1) and not f(64, 64, 64, 2)
     parts = ctypes.c_int(0)
     plan = K.lib().ortb200_latent_decode_plan
     assert plan(1, 16, 512, 576, 128, 256, 1, ctypes.byref(parts)) and parts.value > 4
